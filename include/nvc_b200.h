@@ -408,6 +408,14 @@ int nvc_head_gate(nvc_ctx* ctx, const float* o, int ldo, const float* gate, int 
 /* (cos, sin) of position * base^(-2 i / dims), i < dims / 2, for positions below max_pos: out fp32 [max_pos, dims / 2, 2] in
  * device memory, angles taken in double precision on the host.  Synchronous. */
 int nvc_rotary_table_init_sync(nvc_ctx* ctx, float base, int dims, int max_pos, float* out);
+/* The same with YaRN frequencies (factor > 0): with pair(t) = dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(pair(fast)), 0),
+ * hi = min(ceil(pair(slow)), dims - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), pair i turns with
+ * f_i / factor * ramp_i + f_i (1 - ramp_i), f_i = base^(-2 i / dims), and cos and sin are multiplied by 0.1 ln(factor) + 1.
+ * factor == 0: plain frequencies. */
+typedef struct nvc_rotary_scaling {
+  double factor, original, fast, slow;
+} nvc_rotary_scaling;
+int nvc_rotary_table_init_scaled_sync(nvc_ctx* ctx, double base, int dims, nvc_rotary_scaling scaling, int max_pos, float* out);
 /* Everything between a fused q / k / v projection (fp32 rows `in`) and the attention or recurrence behind it, in one pass:
  * bias; per-head RMS norm of q and k (weights of `dim` numbers shared by the heads); rotary positions on the first rot_dims
  * numbers of every q / k head - pairs (2i, 2i + 1), or (i, i + rot_dims / 2) when rot_half - with (cos, sin) from rot_table at
@@ -435,13 +443,16 @@ typedef struct nvc_qkv_prep {
 } nvc_qkv_prep;
 enum { NVC_PREP_ACT_NONE = 0, NVC_PREP_ACT_SILU = 1 };
 int nvc_qkv_prep_run(nvc_ctx* ctx, const nvc_qkv_prep* p, int N, void* stream);
-/* Grouped-query softmax attention over a paged cache with separate key and value widths:
+/* Grouped-query attention over a paged cache with separate key and value widths:
  *   out[i, h, :vdim] = out_scale * gate_i,h * sum_j p_j v_j,   p_j = exp(s_j) / (sum_j' exp(s_j') + exp(sink_h)),
- *   s_j = scale * q[i, h] . k[j, h / (heads / kv_heads)],  j over max(0, pos_i - window + 1) .. pos_i  (window == 0: from 0).
+ *   s_j = scale * key_scale[slot of j] * q[i, h] . k[j, h / (heads / kv_heads)],  j over max(0, pos_i - window + 1) .. pos_i
+ *   (window == 0: from 0; key_scale == NULL: 1); weights == NVC_ATTN_SIGMOID: p_j = sigmoid(s_j + bias_h), not normalised (no sink).
  * sink (fp32 [heads]) and gate (fp32 [rows, ldg], through a sigmoid) are optional.  Rows, block tables and context lengths
  * as in nvc_latent_attn_paged (cu_seqlens == NULL: one row per sequence); rows = total query rows, max_qlen the longest
- * portion.  dim, vdim <= 512.  bf16 storage with dim and vdim multiples of 16 up to 256 runs on the tensor pipe, everything
- * else on the FMA pipe. */
+ * portion.  dim, vdim <= 512.  bf16 storage with dim and vdim multiples of 16 up to 128 runs on the tensor pipe, everything
+ * else on the FMA pipe.  When the values are the keys' own leading numbers (v_cache == k_cache, ldv == ldk, and one key head or
+ * vdim == dim) the tensor-pipe kernel loads every row once. */
+enum { NVC_ATTN_SOFTMAX = 0, NVC_ATTN_SIGMOID = 1 };
 typedef struct nvc_attn_spec {
   int heads, kv_heads, dim, vdim;
   float scale;
@@ -452,6 +463,9 @@ typedef struct nvc_attn_spec {
   float softcap;             /* > 0: s_j <- softcap * tanh(s_j / softcap) */
   int chunk;                 /* > 0 (window must be 0): j over pos_i - pos_i % chunk .. pos_i - the keys of the row's own chunk */
   int gate_per_head;         /* the gate is fp32 [rows, ldg] with ONE number per head (column h) instead of one per output number */
+  int weights;               /* NVC_ATTN_SOFTMAX or NVC_ATTN_SIGMOID */
+  const float* bias;         /* NVC_ATTN_SIGMOID: fp32 [heads], added to the scores (NULL: 0) */
+  const float* key_scale;    /* fp32 per cache row (indexed by slot): a factor on the row's scores, not on its value (NULL: 1) */
 } nvc_attn_spec;
 int nvc_attn_paged_wide(nvc_ctx* ctx, const void* q, int ldq, const void* k_cache, int ldk, const void* v_cache, int ldv,
                         const int32_t* block_tables, int bt_stride, const int32_t* context_lens, const int32_t* cu_seqlens, int B,
@@ -469,7 +483,8 @@ int nvc_retention_scan(nvc_ctx* ctx, const float* q, int ldq, const float* k, in
  * (Fefozen) ---- */
 /* Norms in front of and behind a sublayer on an fp32 residual stream, in one pass over the row (all sums fp32):
  *   s = res_in[r] + y[r] / sqrt(mean(y[r]^2) + eps) * (wy + weight_offset)      (y == NULL: s = res_in[r]);
- *   res_out[r] = s (optional, may alias res_in);   out[i, :H] = s / sqrt(mean(s^2) + eps) * (w + weight_offset)   (w == NULL: none).
+ *   res_out[r] = s (optional, may alias res_in);   out[i, :H] = s / sqrt(mean(s^2) + eps) * (w + weight_offset)
+ *   (w == NULL: out[i, :H] = s, the sum itself in the storage format; out == NULL: none).
  * y is the sublayer's output (fp32 [*, ld]), wy the weight of the norm behind it, w the weight of the norm in front of the next
  * sublayer; weight_offset = 1 for weights stored around zero.  rows as in nvc_rms_norm_pair (gathers; res_out must be NULL). */
 int nvc_rms_norm_sandwich(nvc_ctx* ctx, const float* res_in, const float* y, const float* wy, float* res_out, int ld, const float* w,
@@ -598,6 +613,27 @@ int nvc_moe_scatter_scaled(nvc_ctx* ctx, const void* h, int dtype, int ldh, cons
                            int ldo, int N, int H, void* stream);
 /* NVC_ACT_SILU_MUL for nvc_act_mul_p: out[n, j] = silu(in[n, j]) * in[n, Fp + j]. */
 enum { NVC_ACT_SILU_MUL = 5 };
+
+/* ---- mechanisms of the models with sigmoid attention over shared keys and values, windowed latent attention with YaRN frequencies,
+ * norms behind the sublayers only and capped logits (Buzutar) ---- */
+/* Between the fused projection and an attention whose values are the keys as projected, with RMS norms over the WHOLE query and the
+ * whole key projection.  The key norm stays out of the cached row: with r_j = 1 / sqrt(mean(k_j^2) + eps) the score of key j is
+ * r_j ((q * wq * wk) . k_j), so a token leaves its projected key (which is its value too) and the one number r_j behind:
+ *   q_out[n] = q / sqrt(mean(q^2) + eps) * wqk * (1 + temp_coef ln(floor((positions[n] + 1) / temp_every) + 1)),
+ *   cache[slot_mapping[n]] = k,   key_scale[slot_mapping[n]] = 1 / sqrt(mean(k^2) + eps)       (a negative slot skips the token)
+ * in: fp32 rows [q: qw at q_off | k: kw at k_off]; wqk fp32 [qw]: query weight times the weight of the key number it meets. */
+int nvc_qk_norm_fold_store(nvc_ctx* ctx, const float* in, int ldi, int q_off, int qw, int k_off, int kw, const float* wqk, float eps,
+                           const int32_t* positions, float temp_coef, int temp_every, void* q_out, int ldq, void* cache, int ldc,
+                           float* key_scale, const int32_t* slot_mapping, int dtype, int N, void* stream);
+/* Prompt portions on tcgen05 over a paged cache whose rows are keys AND values (128 numbers per key / value head, bf16): every tile is
+ * loaded once and serves both products.  spec as in nvc_attn_paged_wide (dim = vdim = 128): window, scale, out_scale = 1; softmax with an
+ * optional sink, or NVC_ATTN_SIGMOID with bias, key_scale and an optional gate per output number.  Sequences, cu_seqlens and block sizes as
+ * in nvc_prefill_attn_paged. */
+int nvc_prefill_attn_shared(nvc_ctx* ctx, const nvc_bf16* q, int ldq, const nvc_bf16* cache, const int32_t* block_tables, int bt_stride,
+                            const int32_t* context_lens, const int32_t* cu_seqlens_q, int B, int total_q_tokens, int max_seqlen_q,
+                            int block_size, int num_blocks, const nvc_attn_spec* spec, nvc_bf16* out, int ldo, void* stream);
+/* x[n, j] = cap tanh(x[n, j] / cap), j < V, in place (fp32 rows). */
+int nvc_softcap_f32(nvc_ctx* ctx, float* x, int ld, float cap, int N, int V, void* stream);
 
 /* K8. Replaces Qwen3ModelRunner::argmax (src/engine/llm_engine.rs:135-142) on device:
  * idx[b] = LAST index of the maximum of logits[b, :] (Iterator::max_by tie rule);

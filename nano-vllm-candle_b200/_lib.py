@@ -46,6 +46,11 @@ def check(status: int, where: str, ctx=None) -> None:
         raise NvcError(status, where, detail)
 
 
+class RotaryScalingC(C.Structure):
+    """nvc_rotary_scaling of include/nvc_b200.h (passed by value)."""
+    _fields_ = [("factor", C.c_double), ("original", C.c_double), ("fast", C.c_double), ("slow", C.c_double)]
+
+
 _vp, _i, _f, _sz = C.c_void_p, C.c_int, C.c_float, C.c_size_t
 
 
@@ -113,6 +118,10 @@ def _declare(l: C.CDLL) -> None:
         "nvc_head_gate": [_vp, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _f, _i, _f, _i, _vp],
         "nvc_rotary_table_init_sync": [_vp, _f, _i, _i, _vp],
         "nvc_qkv_prep_run": [_vp, _vp, _i, _vp],
+        "nvc_rotary_table_init_scaled_sync": [_vp, C.c_double, _i, RotaryScalingC, _i, _vp],
+        "nvc_qk_norm_fold_store": [_vp, _vp, _i, _i, _i, _i, _i, _vp, _f, _vp, _f, _i, _vp, _i, _vp, _i, _vp, _vp, _i, _i, _vp],
+        "nvc_prefill_attn_shared": [_vp, _vp, _i, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp, _i, _vp],
+        "nvc_softcap_f32": [_vp, _vp, _i, _f, _i, _i, _vp],
         "nvc_attn_paged_wide": [_vp, _vp, _i, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _i, _i, _vp],
         "nvc_retention_scan": [_vp, _vp, _i, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
         "nvc_prefill_attn_paged_sink": [_vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _i, _vp],

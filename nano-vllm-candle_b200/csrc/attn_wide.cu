@@ -1,5 +1,5 @@
-// nvc_attn_paged_wide: grouped-query softmax attention over a paged cache whose keys and values have their own widths
-// (dim, vdim), with an optional sliding window or chunk mask, an optional cap on the scores (cap tanh(s / cap)), an optional sink
+// nvc_attn_paged_wide: grouped-query attention - softmax, or sigmoid weights with a bias per head - over a paged cache whose keys and
+// values have their own widths (dim, vdim), with an optional factor per cached key, an optional sliding window or chunk mask, an optional cap on the scores (cap tanh(s / cap)), an optional sink
 // term in the denominator, an optional sigmoid gate (per output number or per head) and a constant factor on the output.  Rows of
 // sequence b are the LAST q_len positions of its context; row at position i sees keys max(0, i - window + 1) .. i (window), the
 // keys of its own chunk i - i % chunk .. i (chunk), or 0 .. i (neither).
@@ -66,7 +66,9 @@ __global__ void __launch_bounds__(kSimtWarps * 32) attn_wide_simt_kernel(const W
   float acc[kMaxVPL];
 #pragma unroll
   for (int c = 0; c < kMaxVPL; ++c) acc[c] = 0.f;
-  float m = -INFINITY, l = 0.f;
+  const bool sig = s.weights == NVC_ATTN_SIGMOID;
+  const float bias = sig && s.bias ? __ldg(s.bias + h) : 0.f;
+  float m = sig ? 0.f : -INFINITY, l = 0.f;
   for (int t = lo + 32 * wid; t <= pos; t += 32 * kSimtWarps) {
     const int j = t + lane;
     const bool valid = j <= pos;
@@ -78,15 +80,21 @@ __global__ void __launch_bounds__(kSimtWarps * 32) attn_wide_simt_kernel(const W
       float dot = 0.f;
       for (int d = 0; d < s.dim; ++d) dot = fmaf(q_s[d], ld_f(kp + d), dot);
       sc = dot * s.scale;
+      if (s.key_scale) sc *= __ldg(s.key_scale + slot);
       if (s.softcap > 0.f) sc = s.softcap * tanhf(sc / s.softcap);
     }
-    const float mn = fmaxf(m, warp_max(sc));     // finite: the tile's first key is visible
-    const float p = valid ? expf(sc - mn) : 0.f;
-    const float corr = expf(m - mn);             // m == -inf: 0
-    l = l * corr + warp_sum(p);
-    m = mn;
+    float p;
+    if (sig) {
+      p = valid ? sigmoid_f32(sc + bias) : 0.f;    // no normalisation: weights of different keys never meet
+    } else {
+      const float mn = fmaxf(m, warp_max(sc));     // finite: the tile's first key is visible
+      p = valid ? expf(sc - mn) : 0.f;
+      const float corr = expf(m - mn);             // m == -inf: 0
+      l = l * corr + warp_sum(p);
+      m = mn;
 #pragma unroll
-    for (int c = 0; c < kMaxVPL; ++c) acc[c] *= corr;
+      for (int c = 0; c < kMaxVPL; ++c) acc[c] *= corr;
+    }
     const int nk = min(32, pos - t + 1);
     for (int jj = 0; jj < nk; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
@@ -112,7 +120,7 @@ __global__ void __launch_bounds__(kSimtWarps * 32) attn_wide_simt_kernel(const W
     f[w] = expf(ml_s[2 * w] - M);       // a warp without keys has m = -inf: factor 0
     L += ml_s[2 * w + 1] * f[w];
   }
-  const float inv = 1.0f / L;
+  const float inv = sig ? 1.0f : 1.0f / L;       // sigmoid: every m is 0, every factor 1
   T* op = reinterpret_cast<T*>(a.out) + (int64_t)row * a.ldo + (int64_t)h * s.vdim;
   for (int c = threadIdx.x; c < s.vdim; c += blockDim.x) {
     float o = 0.f;
@@ -139,6 +147,7 @@ extern "C" int nvc_attn_paged_wide(nvc_ctx* ctx, const void* q, int ldq, const v
   NVC_REQUIRE(ctx, s.window >= 0 && s.chunk >= 0 && !(s.window > 0 && s.chunk > 0) && s.softcap >= 0.f &&
                        (!s.gate || s.ldg >= (s.gate_per_head ? s.heads : s.heads * s.vdim)),
               NVC_EINVAL, "bad window / chunk / cap / gate");
+  NVC_REQUIRE(ctx, s.weights == NVC_ATTN_SOFTMAX || (s.weights == NVC_ATTN_SIGMOID && !s.sink), NVC_EINVAL, "unknown weights, or a sink beside sigmoid weights");
   NVC_REQUIRE(ctx, ldq >= s.heads * s.dim && ldk >= s.kv_heads * s.dim && ldv >= s.kv_heads * s.vdim && ldo >= s.heads * s.vdim, NVC_EINVAL,
               "bad strides");
   WideArgs a{q, k_cache, v_cache, out, ldq, ldk, ldv, ldo, block_tables, context_lens, cu_seqlens, bt_stride, B, block_size, s};

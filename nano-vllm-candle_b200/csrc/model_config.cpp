@@ -35,6 +35,16 @@ bool get_float(const JValue* o, const char* key, float& out, std::string& err) {
   return true;
 }
 
+bool get_double(const JValue* o, const char* key, double& out, std::string& err) {
+  const JValue* v = o ? o->get(key) : nullptr;
+  if (!v || v->kind != JValue::Num) {
+    err = std::string("missing or invalid number `") + key + "`";
+    return false;
+  }
+  out = v->num;
+  return true;
+}
+
 int parse_karuzen(const JValue& root, nvc_karuzen_config& c) {
   std::string err;
   if (!get_int(&root, "vocab", c.vocab, 1, err) || !get_int(&root, "width", c.width, 1, err)) return cfg_fail(err);
@@ -98,15 +108,26 @@ int parse_karuzen(const JValue& root, nvc_karuzen_config& c) {
   return NVC_OK;
 }
 
-bool parse_rotary(const JValue* m, nvc_rotary_spec& r, int dim, std::string& err) {
+// with_scaling: the family knows rot.scaling (YaRN frequencies); the others refuse it
+bool parse_rotary(const JValue* m, nvc_rotary_spec& r, int dim, std::string& err, bool with_scaling = false) {
   const JValue* rot = m->get("rot");
   if (!rot || rot->kind == JValue::Null) { r.dims = 0; return true; }
-  if (rot->kind != JValue::Obj || !get_int(rot, "dims", r.dims, 0, err) || !get_float(rot, "base", r.base, err)) {
+  if (rot->kind != JValue::Obj || !get_int(rot, "dims", r.dims, 0, err) || !get_double(rot, "base", r.base, err)) {
     if (err.empty()) err = "`rot` must be an object";
     return false;
   }
   if (r.dims % 2 != 0 || r.dims > dim) { err = "rot.dims must be even and at most dim"; return false; }
-  if (!(r.base > 0.f)) { err = "rot.base must be positive"; return false; }
+  if (!(r.base > 0.0)) { err = "rot.base must be positive"; return false; }
+  const JValue* sc = rot->get("scaling");
+  if (!sc || sc->kind == JValue::Null) return true;
+  if (!with_scaling) { err = "rot.scaling is not supported"; return false; }
+  if (sc->kind != JValue::Obj) { err = "rot.scaling must be an object or null"; return false; }
+  auto& y = r.scaling;
+  if (!get_double(sc, "factor", y.factor, err) || !get_double(sc, "original", y.original, err) || !get_double(sc, "fast", y.fast, err) ||
+      !get_double(sc, "slow", y.slow, err))
+    return false;
+  if (!(y.factor > 0.0) || !(y.original > 0.0) || !(y.fast > 0.0) || !(y.slow > 0.0)) { err = "rot.scaling: numbers must be positive"; return false; }
+  if (r.base == 1.0) { err = "rot.scaling needs a base other than 1"; return false; }
   return true;
 }
 
@@ -188,6 +209,28 @@ int parse_ranilix(const JValue& root, nvc_ranilix_config& c) {
   return NVC_OK;
 }
 
+// the keys that every kind of rotary latent attention has; layer `i` may name an earlier layer whose cache rows it reads
+// (`source(j)`: that layer's latent spec, NULL when it is something else)
+template <typename Source>
+bool parse_latent(const JValue* m, nvc_latent_attn_spec& a, size_t i, Source&& source, std::string& err, bool with_scaling) {
+  if (!get_int(m, "heads", a.heads, 1, err) || !get_int(m, "dim", a.dim, 1, err) || !get_int(m, "rot_dim", a.rot_dim, 0, err) ||
+      !get_int(m, "vdim", a.vdim, 1, err) || !get_int(m, "kv_rank", a.kv_rank, 1, err) || !get_int(m, "q_rank", a.q_rank, 1, err) ||
+      !get_float(m, "scale", a.scale, err) || !parse_rotary(m, a.rot, a.rot_dim, err, with_scaling)) {
+    err = "mixer: " + err;
+    return false;
+  }
+  const JValue* from = m->get("kv_from");
+  if (!from || from->kind == JValue::Null) return true;
+  if (!get_int(m, "kv_from", a.kv_from, 0, err)) { err = "mixer: " + err; return false; }
+  if (a.kv_from >= (int)i) { err = "mixer.kv_from must name an earlier layer"; return false; }
+  const nvc_latent_attn_spec* src = source(a.kv_from);
+  if (!src || src->kv_from >= 0) { err = "mixer.kv_from must name a latent-attention layer with a cache of its own"; return false; }
+  if (src->kv_rank != a.kv_rank || src->rot_dim != a.rot_dim || !src->rot.same(a.rot) || src->rot_half != a.rot_half) {
+    err = "mixer.kv_from: kv_rank, rot_dim and the rotation must equal the named layer's";
+    return false;
+  }
+  return true;
+}
 
 int parse_fefozen(const JValue& root, nvc_fefozen_config& c) {
   std::string err;
@@ -210,20 +253,9 @@ int parse_fefozen(const JValue& root, nvc_fefozen_config& c) {
       auto& a = L.lat;
       a.rot_half = type->str == "latent_attention_2";
       a.sink = !a.rot_half;
-      if (!get_int(m, "heads", a.heads, 1, err) || !get_int(m, "dim", a.dim, 1, err) || !get_int(m, "rot_dim", a.rot_dim, 0, err) ||
-          !get_int(m, "vdim", a.vdim, 1, err) || !get_int(m, "kv_rank", a.kv_rank, 1, err) || !get_int(m, "q_rank", a.q_rank, 1, err) ||
-          !get_float(m, "scale", a.scale, err) || !parse_rotary(m, a.rot, a.rot_dim, err))
-        return cfg_fail(where + "mixer: " + err);
-      const JValue* from = m->get("kv_from");
-      if (from && from->kind != JValue::Null) {
-        if (!get_int(m, "kv_from", a.kv_from, 0, err)) return cfg_fail(where + "mixer: " + err);
-        if (a.kv_from >= (int)i) return cfg_fail(where + "mixer.kv_from must name an earlier layer");
-        const auto& src = c.layers[a.kv_from];
-        if (src.kind != nvc_fefozen_layer::Latent || src.lat.kv_from >= 0) return cfg_fail(where + "mixer.kv_from must name a latent-attention layer with a cache of its own");
-        if (src.lat.kv_rank != a.kv_rank || src.lat.rot_dim != a.rot_dim || src.lat.rot.dims != a.rot.dims || src.lat.rot.base != a.rot.base ||
-            src.lat.rot_half != a.rot_half)
-          return cfg_fail(where + "mixer.kv_from: kv_rank, rot_dim and the rotation must equal the named layer's");
-      }
+      a.gate = true;
+      auto source = [&](int j) { return c.layers[j].kind == nvc_fefozen_layer::Latent ? &c.layers[j].lat : nullptr; };
+      if (!parse_latent(m, a, i, source, err, false)) return cfg_fail(where + err);
     } else if (type->str == "delta") {
       L.kind = nvc_fefozen_layer::Delta;
       auto& d = L.delta;
@@ -349,6 +381,65 @@ int parse_batatar(const JValue& root, nvc_batatar_config& c) {
   return NVC_OK;
 }
 
+int parse_buzutar(const JValue& root, nvc_buzutar_config& c) {
+  std::string err;
+  if (!get_int(&root, "vocab", c.vocab, 1, err) || !get_int(&root, "width", c.width, 1, err)) return cfg_fail(err);
+  const JValue* norm = root.get("norm");
+  if (!norm || norm->kind != JValue::Obj || !get_float(norm, "eps", c.eps, err)) return cfg_fail("norm.eps: " + err);
+  if (const JValue* emb = root.get("embedding"); emb && emb->kind != JValue::Null) {
+    if (emb->kind != JValue::Obj) return cfg_fail("`embedding` must be an object or null");
+    if (emb->get("scale") && !get_float(emb, "scale", c.embedding_scale, err)) return cfg_fail("embedding.scale: " + err);
+  }
+  if (const JValue* cap = root.get("logit_softcap"); cap && cap->kind != JValue::Null) {
+    if (!get_float(&root, "logit_softcap", c.logit_softcap, err) || !(c.logit_softcap > 0.f)) return cfg_fail("logit_softcap must be a positive number");
+  }
+  const JValue* layers = root.get("layers");
+  if (!layers || layers->kind != JValue::Arr || layers->arr.empty()) return cfg_fail("`layers` must be a non-empty list");
+  for (size_t i = 0; i < layers->arr.size(); ++i) {
+    const JValue& jl = layers->arr[i];
+    const std::string where = "layers[" + std::to_string(i) + "]: ";
+    if (jl.kind != JValue::Obj) return cfg_fail(where + "not an object");
+    nvc_buzutar_layer L;
+    const JValue* type = jl.get("type");
+    const JValue* m = jl.get("mixer");
+    if (!type || type->kind != JValue::Str) return cfg_fail(where + "missing `type`");
+    if (!m || m->kind != JValue::Obj) return cfg_fail(where + "missing `mixer`");
+    if (type->str == "attention") {
+      L.kind = nvc_buzutar_layer::Attention;
+      auto& a = L.attn;
+      int vdim = 0;
+      if (!get_int(m, "heads", a.heads, 1, err) || !get_int(m, "kv_heads", a.kv_heads, 1, err) || !get_int(m, "dim", a.dim, 1, err) ||
+          !get_int(m, "vdim", vdim, 1, err) || !get_float(m, "scale", a.scale, err))
+        return cfg_fail(where + "mixer: " + err);
+      if (a.heads % a.kv_heads != 0) return cfg_fail(where + "mixer: heads must be a multiple of kv_heads");
+      if (vdim != a.dim) return cfg_fail(where + "mixer: the values are the keys, vdim must equal dim");
+      if (const JValue* t = m->get("q_temp"); t && t->kind != JValue::Null) {
+        if (t->kind != JValue::Obj || !get_float(t, "coef", a.temp_coef, err) || !get_int(t, "every", a.temp_every, 1, err))
+          return cfg_fail(where + "mixer.q_temp: " + (err.empty() ? "must be an object or null" : err));
+      }
+    } else if (type->str == "latent_attention") {
+      L.kind = nvc_buzutar_layer::Latent;
+      auto source = [&](int j) { return c.layers[j].kind == nvc_buzutar_layer::Latent ? &c.layers[j].lat : nullptr; };
+      if (!parse_latent(m, L.lat, i, source, err, true)) return cfg_fail(where + err);
+      if (const JValue* mask = m->get("mask"); mask && mask->kind != JValue::Null) {
+        if (mask->kind != JValue::Obj || !get_int(mask, "size", L.lat.window, 1, err)) return cfg_fail(where + "mixer.mask: " + err);
+      }
+    } else {
+      return cfg_fail(where + "mixer type `" + type->str + "` is not supported");
+    }
+    const JValue* mlp = jl.get("mlp");
+    if (mlp && mlp->kind == JValue::Obj) {
+      const JValue* kind = mlp->get("kind");
+      if (!kind || kind->kind != JValue::Str || kind->str != "dense") return cfg_fail(where + "mlp: only kind `dense` is supported");
+      if (!get_int(mlp, "ff", L.ff, 1, err)) return cfg_fail(where + "mlp: " + err);
+    } else if (mlp && mlp->kind != JValue::Null) {
+      return cfg_fail(where + "`mlp` must be an object or null");
+    }
+    c.layers.push_back(L);
+  }
+  return NVC_OK;
+}
+
 }  // namespace
 
 std::vector<nvc_karuzen_config::Run> nvc_karuzen_config::runs() const {
@@ -402,10 +493,12 @@ int nvc_model_config_from_json(const char* text, nvc_model_config** out) {
     rc = parse_fefozen(root, c->fefozen);
   } else if (arch == "Batatar") {
     rc = parse_batatar(root, c->batatar);
+  } else if (arch == "Buzutar") {
+    rc = parse_buzutar(root, c->buzutar);
   } else if (arch == "Qwen3ForCausalLM") {
     // parsed by nvc_qwen3_config_from_hf_dir (hf_loader.cpp) when loaded from a directory
   } else {
-    rc = cfg_fail("architecture `" + arch + "` is not registered (known: Qwen3ForCausalLM, Karuzen, Ranilix, Fefozen, Batatar)");
+    rc = cfg_fail("architecture `" + arch + "` is not registered (known: Qwen3ForCausalLM, Karuzen, Ranilix, Fefozen, Batatar, Buzutar)");
   }
   if (rc) { delete c; return rc; }
   *out = c;
@@ -432,11 +525,13 @@ int nvc_model_config_vocab(const nvc_model_config* c) {
   if (c->architecture == "Ranilix") return c->ranilix.vocab;
   if (c->architecture == "Fefozen") return c->fefozen.vocab;
   if (c->architecture == "Batatar") return c->batatar.vocab;
+  if (c->architecture == "Buzutar") return c->buzutar.vocab;
   return c->architecture == "Karuzen" ? c->karuzen.vocab : c->qwen3.vocab_size;
 }
 int nvc_model_config_layer_runs(const nvc_model_config* c, int32_t* layers, int32_t* passes, int32_t* readd, int capacity) {
-  if (c && (c->architecture == "Ranilix" || c->architecture == "Fefozen")) {      // no looped block: every layer runs once
-    const int n = (int)(c->architecture == "Ranilix" ? c->ranilix.layers.size() : c->fefozen.layers.size());
+  if (c && (c->architecture == "Ranilix" || c->architecture == "Fefozen" || c->architecture == "Buzutar")) {      // no looped block: every layer runs once
+    const int n = (int)(c->architecture == "Ranilix" ? c->ranilix.layers.size()
+                                                     : (c->architecture == "Fefozen" ? c->fefozen.layers.size() : c->buzutar.layers.size()));
     for (int i = 0; i < n && i < capacity; ++i) {
       if (layers) layers[i] = i;
       if (passes) passes[i] = 0;

@@ -41,7 +41,12 @@ struct nvc_karuzen_config {
 // per-head recurrent state with a fixed decay - summed with two constant weights).
 struct nvc_rotary_spec {
   int dims = 0;              // leading numbers of a head that are rotated (0: none)
-  float base = 10000.f;
+  double base = 10000.0;
+  nvc_rotary_scaling scaling{0.0, 0.0, 0.0, 0.0};   // factor 0: plain frequencies
+  bool same(const nvc_rotary_spec& o) const {
+    return dims == o.dims && base == o.base && scaling.factor == o.scaling.factor && scaling.original == o.scaling.original &&
+           scaling.fast == o.scaling.fast && scaling.slow == o.scaling.slow;
+  }
 };
 struct nvc_softmax_attn_spec {     // grouped-query softmax attention
   int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
@@ -90,6 +95,8 @@ struct nvc_latent_attn_spec {
   nvc_rotary_spec rot;       // on the rot_dim part of queries and of the shared key part
   bool rot_half = false;     // pairs (i, i + dims / 2) instead of (2i, 2i + 1)
   bool sink = false;         // one more term exp(sink_h) in the softmax denominator
+  bool gate = false;         // the heads' outputs are gated with sigmoid(W_g h)
+  int window = 0;            // 0: every earlier token is visible; n: the token itself and the n - 1 before it
   int kv_from = -1;          // >= 0: no key / value down-projection of its own, reads that layer's cache rows
 };
 struct nvc_delta_spec {
@@ -158,12 +165,39 @@ struct nvc_batatar_config {
   bool has_state() const { return !layers.empty(); }     // every mixer of the design keeps a recurrent state
 };
 
+// Buzutar: a stack of sequential layers whose sublayers read the fp32 residual stream as it is; only their outputs are normed,
+// x <- x + n1(mixer(x)), x <- x + n2(ff(x)).  Mixers: "attention" - grouped-query attention without positions whose weights are
+// sigmoid(score + a bias per head), not normalised; one RMS norm over all query heads and one over all key heads; the values are the
+// keys in front of their norm; a temperature on the queries that grows with the position; a sigmoid gate - or "latent_attention" -
+// latent attention with a rotated key part (YaRN frequencies) over a sliding window; a layer may read another layer's rows.
+// Feed-forward: squared relu.  The embedding has a constant factor, the head its own matrix, the logits a cap.
+struct nvc_sigmoid_attn_spec {
+  int heads = 0, kv_heads = 0, dim = 0;
+  float scale = 0.f;
+  float temp_coef = 0.f;     // queries at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1)
+  int temp_every = 1;
+};
+struct nvc_buzutar_layer {
+  enum Kind { Attention, Latent } kind = Attention;
+  nvc_sigmoid_attn_spec attn;
+  nvc_latent_attn_spec lat;
+  int ff = 0;                // 0: no feed-forward
+};
+struct nvc_buzutar_config {
+  int vocab = 0, width = 0;
+  float eps = 1e-5f;
+  float embedding_scale = 1.f;
+  float logit_softcap = 0.f; // 0: logits are not capped
+  std::vector<nvc_buzutar_layer> layers;
+};
+
 struct nvc_model_config {
-  std::string architecture;   // "Qwen3ForCausalLM", "Karuzen", "Ranilix", "Fefozen" or "Batatar"
+  std::string architecture;   // "Qwen3ForCausalLM", "Karuzen", "Ranilix", "Fefozen", "Batatar" or "Buzutar"
   nvc_qwen3_config qwen3{};
   int qwen3_tied = 0;
   nvc_karuzen_config karuzen;
   nvc_ranilix_config ranilix;
   nvc_fefozen_config fefozen;
   nvc_batatar_config batatar;
+  nvc_buzutar_config buzutar;
 };

@@ -4,16 +4,8 @@
 //   nvc_rms_norm_sandwich     x += norm-behind(previous sublayer's output); h = norm-in-front(x): one pass over the row
 //   latent attention:
 //     linear w_in             ONE fused projection of everything the mixer reads from h, fp32 out: [dq | dkv | gate]
-//     nvc_latent_norm_store_rot  RMS norms of both latents; the token's cache row [normed latent | rotated shared key part] goes
-//                             into this layer's paged pool (a layer with kv_from reads the named layer's pool and stores nothing)
-//     linear uq (fp32 out) -> nvc_head_split_rot: unrotated query parts, rotated parts straight into the absorbed queries
-//     linear uk^T per head    unrotated query parts carried into the latent space (absorbed key up-projection)
-//     attention               softmax over the cached rows: in the absorbed form a layer is multi-query attention with ONE key /
-//                             value head - key = the whole row (kv_rank + rot_dim numbers), value = its first kv_rank numbers.
-//                             nvc_attn_paged_wide (sink in its epilogue), or the tcgen05 paged-prefill kernel for long portions
-//                             when the row has 128 numbers (the sink joins the denominator in its epilogue; the rotated part
-//                             rides along as value columns that the value up-projection never reads)
-//     linear uv per head (fp32 out) -> nvc_head_gate (sigmoid gate of h) -> linear o
+//     latent_run              (latent_mixer.h) latents, absorbed queries, attention over shared rows, value up-projection, gate
+//     linear o
 //   delta:
 //     linear w_in             [q | k | v | beta | a | gate], fp32 out
 //     nvc_delta_prep_run      short convolutions + silu, unit q / k, decay and beta;  nvc_delta_rule_scan: the recurrence over the
@@ -32,13 +24,10 @@
 #include <string>
 #include <vector>
 
-#include "body_common.h"
-#include "model_config.h"
+#include "latent_mixer.h"
 #include "runner.h"
 
 namespace {
-
-inline int pad8(int v) { return (v + 7) / 8 * 8; }
 
 constexpr float kGluAlpha = 1.702f;      // g * sigmoid(alpha g) of the experts' gated unit
 constexpr float kUnitEps = 1e-6f;        // inside the root of the delta rule's unit vectors
@@ -48,15 +37,7 @@ struct FLayerW {
   void* w_in = nullptr;                 // [np, Wp]
   int np = 0;
   int g_off = 0;
-  // latent attention
-  int kv_off = 0;                       // first column of the key / value down-projection in a projection row
-  float *dq_norm = nullptr, *dkv_norm = nullptr, *sink = nullptr;
-  void* w_uq = nullptr;                 // [uqn, qrp]
-  void* w_ukT = nullptr;                // [heads][kv_rank, dimp]
-  void* w_uv = nullptr;                 // [heads][vdim, kvp]
-  int qrp = 0, uqn = 0, dimp = 0, kvp = 0, Dk = 0, ldpool = 0, ldqa = 0, ldol = 0;
-  void* pool = nullptr;                 // [slots, ldpool]: [normed latent | rotated key part] per token (own layers)
-  const float* rot = nullptr;
+  nvc_latent_weights lat;
   // delta
   int q_off = 0, k_off = 0, v_off = 0, b_off = 0, a_off = 0;
   float *conv_w = nullptr, *conv_state = nullptr, *A_log = nullptr, *dt_bias = nullptr, *onorm = nullptr, *state = nullptr;
@@ -74,20 +55,18 @@ struct FLayerW {
   bool moe_tc = false;
 };
 
-struct FefozenBody : nvc_body_base {
+struct FefozenBody : nvc_latent_body {
   nvc_fefozen_config cfg;
   int Wp = 0, Vp = 0;
   int state_slots = 0;
-  bool use_flash = true, use_moe_tc = true;
+  bool use_moe_tc = true;
   std::vector<FLayerW> L;
   void* embed = nullptr;
   float* fw = nullptr;
-  std::map<std::string, bool> want;
-  std::map<std::pair<int, uint32_t>, float*> rot_tables;
   // activations
-  float *x0 = nullptr, *res = nullptr, *proj = nullptr, *mix = nullptr, *ffo = nullptr, *qf = nullptr, *hv = nullptr;
+  float *x0 = nullptr, *res = nullptr, *proj = nullptr, *mix = nullptr, *ffo = nullptr;
   float *rq = nullptr, *rk = nullptr, *rv = nullptr, *ro = nullptr, *gb = nullptr, *zlog = nullptr, *tk_w = nullptr, *y = nullptr;
-  void *h = nullptr, *cq = nullptr, *qn = nullptr, *qabs = nullptr, *olat = nullptr, *ao = nullptr, *act = nullptr, *hn = nullptr;
+  void *h = nullptr, *ao = nullptr, *act = nullptr, *hn = nullptr;
   void *hid2 = nullptr, *hid = nullptr, *xs = nullptr;
   int32_t *tk_idx = nullptr, *offsets = nullptr, *src_rows = nullptr, *pos = nullptr, *tile_group = nullptr;
   float* tap_host = nullptr;
@@ -101,7 +80,7 @@ struct FefozenBody : nvc_body_base {
   int64_t cache_bytes_per_token() const override {
     int64_t b = 0;
     for (size_t i = 0; i < cfg.layers.size(); ++i)
-      if (cfg.layers[i].kind == nvc_fefozen_layer::Latent && cfg.layers[i].lat.kv_from < 0) b += (int64_t)L[i].ldpool * (int64_t)esz;
+      if (cfg.layers[i].kind == nvc_fefozen_layer::Latent && cfg.layers[i].lat.kv_from < 0) b += (int64_t)L[i].lat.ldpool * (int64_t)esz;
     return b;
   }
   int set_residual_tap(float* host, size_t cap) override {
@@ -111,24 +90,6 @@ struct FefozenBody : nvc_body_base {
   }
 
   static int moe_tiles(int pairs, int experts) { return (pairs + experts * 127 + 127) / 128; }
-
-  int rotary_table(nvc_runner* r, const nvc_rotary_spec& rs, const float** out) {
-    *out = nullptr;
-    if (rs.dims == 0) return NVC_OK;
-    uint32_t bits;
-    memcpy(&bits, &rs.base, 4);
-    auto key = std::make_pair(rs.dims, bits);
-    auto it = rot_tables.find(key);
-    if (it == rot_tables.end()) {
-      float* t = nullptr;
-      int rc = zalloc(r, &t, (size_t)r->opt.max_model_len * rs.dims * sizeof(float));
-      if (rc) return rc;
-      if ((rc = nvc_rotary_table_init_sync(r->ctx, rs.base, rs.dims, r->opt.max_model_len, t))) return rc;
-      it = rot_tables.emplace(key, t).first;
-    }
-    *out = it->second;
-    return NVC_OK;
-  }
 
   int init(nvc_runner* r) {
     nvc_ctx* ctx = r->ctx;
@@ -144,7 +105,7 @@ struct FefozenBody : nvc_body_base {
     const size_t slots = (size_t)r->opt.num_kvcache_blocks * r->opt.kvcache_block_size;
     int rc;
     L.resize(cfg.layers.size());
-    size_t m_np = 0, m_qrp = 0, m_uqn = 0, m_qn = 0, m_qa = 0, m_ol = 0, m_hv = 0, m_ow = 0, m_ff = 0, m_dqk = 0, m_dv = 0, m_gb = 0;
+    size_t m_np = 0, m_ow = 0, m_ff = 0, m_dqk = 0, m_dv = 0, m_gb = 0;
     size_t m_Ep = 0, m_top = 0, m_E = 0, m_hid = 0, m_pairs_rows = 0, m_tiles = 0;
     int64_t wbytes = 0;
     const int W = cfg.width;
@@ -158,42 +119,14 @@ struct FefozenBody : nvc_body_base {
       int ow = 0;
       if (ly.kind == nvc_fefozen_layer::Latent) {
         const auto& a = ly.lat;
-        const bool own = a.kv_from < 0;
-        w.Dk = a.kv_rank + a.rot_dim;
-        NVC_REQUIRE(ctx, w.Dk <= 512, NVC_ESHAPE, "kv_rank + rot_dim above 512");
-        w.kv_off = a.q_rank;
-        w.g_off = a.q_rank + (own ? w.Dk : 0);
+        int cols = 0;
+        int64_t wn = 0;
+        if ((rc = latent_init(r, a, p, slots, 0, w.lat, &cols, &wn))) return rc;
+        w.g_off = cols;
         ow = a.heads * a.vdim;
         w.np = pad64(w.g_off + ow);
-        w.qrp = pad64(a.q_rank);
-        w.uqn = pad64(a.heads * (a.dim + a.rot_dim));
-        w.dimp = pad8(a.dim);
-        w.kvp = pad8(a.kv_rank);
-        w.ldpool = pad8(w.Dk);
-        w.ldqa = pad8(a.heads * w.Dk);
-        w.ldol = pad8(a.heads * w.Dk);          // room for value columns as wide as the key (the tcgen05 route)
-        if ((rc = zalloc(r, &w.dq_norm, a.q_rank * 4)) || (rc = zalloc(r, &w.w_uq, (size_t)w.uqn * w.qrp * esz)) ||
-            (rc = zalloc(r, &w.w_ukT, (size_t)a.heads * a.kv_rank * w.dimp * esz)) || (rc = zalloc(r, &w.w_uv, (size_t)a.heads * a.vdim * w.kvp * esz)))
-          return rc;
-        for (const char* n : {"mix.dq", "mix.dq.norm", "mix.uq", "mix.uk", "mix.uv", "mix.g", "mix.o"}) want[p + n] = false;
-        if (own) {
-          if ((rc = zalloc(r, &w.dkv_norm, a.kv_rank * 4)) || (rc = zalloc(r, &w.pool, slots * w.ldpool * esz))) return rc;
-          want[p + "mix.dkv"] = false;
-          want[p + "mix.dkv.norm"] = false;
-        }
-        if (a.sink) {
-          if ((rc = zalloc(r, &w.sink, a.heads * 4))) return rc;
-          want[p + "mix.sink"] = false;
-        }
-        if ((rc = rotary_table(r, a.rot, &w.rot))) return rc;
-        wbytes += (int64_t)esz * ((int64_t)(a.q_rank + (own ? w.Dk : 0) + ow) * W + (int64_t)a.heads * (a.dim + a.rot_dim) * a.q_rank +
-                                  (int64_t)a.heads * (a.dim + a.vdim) * a.kv_rank + (int64_t)W * ow);
-        m_qrp = std::max(m_qrp, (size_t)w.qrp);
-        m_uqn = std::max(m_uqn, (size_t)w.uqn);
-        m_qn = std::max(m_qn, (size_t)a.heads * w.dimp);
-        m_qa = std::max(m_qa, (size_t)w.ldqa);
-        m_ol = std::max(m_ol, (size_t)w.ldol);
-        m_hv = std::max(m_hv, (size_t)ow);
+        for (const char* n : {"mix.g", "mix.o"}) want[p + n] = false;
+        wbytes += (int64_t)esz * ((int64_t)(cols + ow) * W + wn + (int64_t)W * ow);
       } else {
         const auto& d = ly.delta;
         const int qk = d.kv_heads * d.dim, vw = d.heads * d.vdim, C = 2 * qk + vw;
@@ -261,9 +194,7 @@ struct FefozenBody : nvc_body_base {
         (rc = zalloc(r, &ffo, T * Wp * 4)) || (rc = zalloc(r, &proj, T * m_np * 4)) || (rc = zalloc(r, &h, T * Wp * esz)) ||
         (rc = zalloc(r, &ao, T * m_ow * esz)) || (rc = zalloc(r, &hn, (size_t)r->max_logit_rows * Wp * esz)))
       return rc;
-    if (m_uqn && ((rc = zalloc(r, &cq, T * m_qrp * esz)) || (rc = zalloc(r, &qf, T * m_uqn * 4)) || (rc = zalloc(r, &qn, T * m_qn * esz)) ||
-                  (rc = zalloc(r, &qabs, T * m_qa * esz)) || (rc = zalloc(r, &olat, T * m_ol * esz)) || (rc = zalloc(r, &hv, T * m_hv * 4))))
-      return rc;
+    if ((rc = latent_alloc(r, T))) return rc;
     if (m_dv && ((rc = zalloc(r, &rq, T * m_dqk * 4)) || (rc = zalloc(r, &rk, T * m_dqk * 4)) || (rc = zalloc(r, &rv, T * m_dv * 4)) ||
                  (rc = zalloc(r, &ro, T * m_dv * 4)) || (rc = zalloc(r, &gb, T * m_gb * 4))))
       return rc;
@@ -312,32 +243,20 @@ struct FefozenBody : nvc_body_base {
       auto in_rows = [&](int off, int rows) { return shape_is(rows, W) ? put_matrix(r, w.w_in, Wp, off, 0, v.data(), rows, W, W, 1) : bad(); };
       const int ow = latent ? a.heads * a.vdim : d.heads * d.vdim;
       const int qk = d.kv_heads * d.dim;
+      if (latent) {
+        bool taken = false;
+        rc = latent_load(r, a, w.lat, sub, v, d0, d1, in_rows, bad, &taken);
+        if (taken) {
+          it->second = rc == NVC_OK;
+          return rc;
+        }
+      }
       if (sub == "norm1") rc = vec(w.n1, W);
       else if (sub == "norm1b") rc = vec(w.n1b, W);
       else if (sub == "norm2") rc = vec(w.n2, W);
       else if (sub == "norm2b") rc = vec(w.n2b, W);
       else if (sub == "mix.g") rc = in_rows(w.g_off, ow);
       else if (sub == "mix.o") { if (!shape_is(W, ow)) return bad(); rc = put_matrix(r, w.w_o, w.owp, 0, 0, v.data(), W, ow, ow, 1); }
-      else if (latent && sub == "mix.dq") rc = in_rows(0, a.q_rank);
-      else if (latent && sub == "mix.dkv") rc = in_rows(w.kv_off, w.Dk);
-      else if (latent && sub == "mix.dq.norm") rc = vec(w.dq_norm, a.q_rank);
-      else if (latent && sub == "mix.dkv.norm") rc = vec(w.dkv_norm, a.kv_rank);
-      else if (latent && sub == "mix.sink") rc = vec(w.sink, a.heads);
-      else if (latent && sub == "mix.uq") {
-        if (!shape_is(a.heads * (a.dim + a.rot_dim), a.q_rank)) return bad();
-        rc = put_matrix(r, w.w_uq, w.qrp, 0, 0, v.data(), a.heads * (a.dim + a.rot_dim), a.q_rank, a.q_rank, 1);
-      } else if (latent && sub == "mix.uk") {
-        // [heads * dim, kv_rank] -> per head the transposed block [kv_rank, dimp]: q' = W_uk,h^T q
-        if (!shape_is(a.heads * a.dim, a.kv_rank)) return bad();
-        for (int hh = 0; hh < a.heads && rc == NVC_OK; ++hh)
-          rc = put_matrix(r, reinterpret_cast<uint8_t*>(w.w_ukT) + (size_t)hh * a.kv_rank * w.dimp * esz, w.dimp, 0, 0,
-                          v.data() + (size_t)hh * a.dim * a.kv_rank, a.kv_rank, a.dim, 1, a.kv_rank);
-      } else if (latent && sub == "mix.uv") {
-        if (!shape_is(a.heads * a.vdim, a.kv_rank)) return bad();
-        for (int hh = 0; hh < a.heads && rc == NVC_OK; ++hh)
-          rc = put_matrix(r, reinterpret_cast<uint8_t*>(w.w_uv) + (size_t)hh * a.vdim * w.kvp * esz, w.kvp, 0, 0,
-                          v.data() + (size_t)hh * a.vdim * a.kv_rank, a.vdim, a.kv_rank, a.kv_rank, 1);
-      }
       else if (!latent && sub == "mix.q") rc = in_rows(w.q_off, qk);
       else if (!latent && sub == "mix.k") rc = in_rows(w.k_off, qk);
       else if (!latent && sub == "mix.v") rc = in_rows(w.v_off, ow);
@@ -378,92 +297,15 @@ struct FefozenBody : nvc_body_base {
   }
 
   int finalize(nvc_runner* r) override {
-    std::string missing;
-    int n = 0;
-    for (auto& kv : want)
-      if (!kv.second && ++n <= 4) missing += kv.first + " ";
-    NVC_REQUIRE(r->ctx, n == 0, NVC_ESTATE, "missing " + std::to_string(n) + " tensors: " + missing);
-    return NVC_OK;
+    return require_all_tensors(r);
   }
 
-  int tap(nvc_runner* r, int run, int N) {
-    const size_t need = (size_t)(run + 1) * N * cfg.width;
-    NVC_REQUIRE(r->ctx, need <= tap_cap, NVC_ENOMEM, "residual tap buffer too small");
-    NVC_CUDA_CHECK(r->ctx, cudaMemcpy2DAsync(tap_host + (size_t)run * N * cfg.width, (size_t)cfg.width * 4, res, (size_t)Wp * 4,
-                                             (size_t)cfg.width * 4, N, cudaMemcpyDeviceToHost, r->stream));
-    return NVC_OK;
-  }
-
-  static constexpr int kFlashMinChunk = 64;
-  bool flash_portions(const nvc_runner* r, const nvc_step_shape& s, const FLayerW& w, const nvc_latent_attn_spec& a) const {
-    const int bs = r->opt.kvcache_block_size;
-    return use_flash && w.Dk == 128 && w.ldpool == 128 && !s.decode && s.num_decode < s.B && s.max_chunk >= kFlashMinChunk &&
-           (bs == 16 || bs == 32 || bs == 64 || bs % 128 == 0);
-  }
+  int tap(nvc_runner* r, int run, int N) { return copy_tap(r, res, Wp, tap_host, tap_cap, run, N, cfg.width); }
 
   int latent_mixer(nvc_runner* r, const nvc_step_shape& s, int li) {
-    nvc_ctx* ctx = r->ctx;
-    void* st = r->stream;
     const auto& a = cfg.layers[li].lat;
     FLayerW& w = L[li];
-    const int N = s.N;
-    const bool own = a.kv_from < 0;
-    const void* pool = own ? w.pool : L[a.kv_from].pool;
-    int rc;
-    if ((rc = nvc_latent_norm_store_rot(ctx, proj, w.np, a.q_rank, w.kv_off, own ? a.kv_rank : 0, w.dq_norm, w.dkv_norm, cfg.eps, cq, w.qrp, own ? w.pool : nullptr,
-                                        w.ldpool, r->d_slots, a.rot_dim, a.rot.dims, a.rot_half ? 1 : 0, w.rot, r->d_pos, dt, N, st)))
-      return rc;
-    mark(r, "latent_norm_store");
-    if ((rc = linear(r, cq, w.qrp, w.w_uq, qf, w.uqn, NVC_DT_F32, N, w.uqn, w.qrp))) return rc;
-    mark(r, "gemm_uq");
-    const int hd = a.heads * w.dimp;
-    if ((rc = nvc_head_split_rot(ctx, qf, w.uqn, a.heads, a.dim, a.rot_dim, a.rot.dims, a.rot_half ? 1 : 0, w.rot, r->d_pos, qn, hd, w.dimp, qabs, w.ldqa,
-                                 w.Dk, a.kv_rank, dt, N, st)))
-      return rc;
-    mark(r, "q_split_rot");
-    if ((rc = nvc_linear(ctx, qn, hd, w.dimp, w.w_ukT, w.dimp, (int64_t)a.kv_rank * w.dimp, qabs, w.ldqa, w.Dk, dt, dt, N, a.kv_rank, w.dimp, a.heads,
-                         NVC_ACT_NONE, st)))
-      return rc;
-    mark(r, "absorb_uk");
-    const int bs = r->opt.kvcache_block_size, cap = r->max_blocks_cap;
-    nvc_attn_spec sp{};
-    sp.heads = a.heads; sp.kv_heads = 1; sp.dim = w.Dk; sp.vdim = a.kv_rank;
-    sp.scale = a.scale;
-    sp.window = 0;
-    sp.sink = a.sink ? w.sink : nullptr;
-    sp.gate = nullptr; sp.ldg = 0;
-    sp.out_scale = 1.f;
-    int ohs = a.kv_rank;                 // numbers per head in olat
-    if (flash_portions(r, s, w, a)) {
-      // key = value = the whole 128-number row: the value columns behind the latent come out as a weighted sum of rotated key parts,
-      // which the value up-projection below never reads.  One-token sequences of a mixed step come first in the batch and keep the
-      // decode path of the wide kernel (same output layout: value width = key width).
-      const int nd = s.num_decode;
-      ohs = w.Dk;
-      sp.vdim = w.Dk;
-      if (nd > 0 && (rc = nvc_attn_paged_wide(ctx, qabs, w.ldqa, pool, w.ldpool, pool, w.ldpool, r->d_bt, cap, r->d_ctx, nullptr, nd, nd, 1, bs, &sp, olat,
-                                              w.ldol, dt, st)))
-        return rc;
-      const nvc_bf16* qb = reinterpret_cast<const nvc_bf16*>(qabs);
-      nvc_bf16* ob = reinterpret_cast<nvc_bf16*>(olat);
-      const nvc_bf16* pb = reinterpret_cast<const nvc_bf16*>(pool);
-      if ((rc = nvc_prefill_attn_paged_sink(ctx, qb + (size_t)nd * w.ldqa, w.ldqa, pb, pb, r->d_bt + (size_t)nd * cap, cap, r->d_ctx + nd,
-                                            nd ? r->d_cu2 : r->d_cu, s.B - nd, s.N - nd, s.max_chunk, a.heads, 1, w.Dk, bs, r->opt.num_kvcache_blocks,
-                                            a.scale, sp.sink, ob + (size_t)nd * w.ldol, w.ldol, st)))
-        return rc;
-    } else if ((rc = nvc_attn_paged_wide(ctx, qabs, w.ldqa, pool, w.ldpool, pool, w.ldpool, r->d_bt, cap, r->d_ctx, s.decode ? nullptr : r->d_cu, s.B,
-                                         s.N, s.decode ? 1 : s.max_seqlen, bs, &sp, olat, w.ldol, dt, st))) {
-      return rc;
-    }
-    mark(r, "attention");
-    const int vw = a.heads * a.vdim;
-    if ((rc = nvc_linear(ctx, olat, w.ldol, ohs, w.w_uv, w.kvp, (int64_t)a.vdim * w.kvp, hv, vw, a.vdim, dt, NVC_DT_F32, N, a.vdim,
-                         ohs % 8 == 0 ? w.kvp : a.kv_rank, a.heads, NVC_ACT_NONE, st)))
-      return rc;
-    mark(r, "absorb_uv");
-    if ((rc = nvc_head_gate(ctx, hv, vw, proj + w.g_off, w.np, ao, w.owp, dt, a.heads, a.vdim, 0, cfg.eps, NVC_GATE_SIGMOID, 1.f, N, st))) return rc;
-    mark(r, "head_gate");
-    return NVC_OK;
+    return latent_run(r, s, a, w.lat, a.kv_from < 0 ? w.lat : L[a.kv_from].lat, cfg.eps, proj, w.np, proj + w.g_off, ao, w.owp);
   }
 
   int delta_mixer(nvc_runner* r, const nvc_step_shape& s, int li) {

@@ -55,7 +55,7 @@ struct RanilixBody : nvc_body_base {
   void *embed = nullptr, *head = nullptr;
   float* fw = nullptr;
   std::map<std::string, bool> want;
-  std::map<std::pair<int, uint32_t>, float*> rot_tables;   // (dims, bits of base) -> [max_model_len, dims / 2, 2]
+  std::map<std::pair<int, double>, float*> rot_tables;   // (dims, bits of base) -> [max_model_len, dims / 2, 2]
   // activations
   float *x0 = nullptr, *res = nullptr, *proj = nullptr, *mix = nullptr, *ffo = nullptr, *v_first = nullptr;
   float *rq = nullptr, *rk = nullptr, *rv = nullptr, *ro = nullptr;
@@ -83,15 +83,13 @@ struct RanilixBody : nvc_body_base {
   int rotary_table(nvc_runner* r, const nvc_rotary_spec& rs, const float** out) {
     *out = nullptr;
     if (rs.dims == 0) return NVC_OK;
-    uint32_t bits;
-    memcpy(&bits, &rs.base, 4);
-    auto key = std::make_pair(rs.dims, bits);
+    const auto key = std::make_pair(rs.dims, rs.base);
     auto it = rot_tables.find(key);
     if (it == rot_tables.end()) {
       float* t = nullptr;
       int rc = zalloc(r, &t, (size_t)r->opt.max_model_len * rs.dims * sizeof(float));
       if (rc) return rc;
-      if ((rc = nvc_rotary_table_init_sync(r->ctx, rs.base, rs.dims, r->opt.max_model_len, t))) return rc;
+      if ((rc = nvc_rotary_table_init_scaled_sync(r->ctx, rs.base, rs.dims, rs.scaling, r->opt.max_model_len, t))) return rc;
       it = rot_tables.emplace(key, t).first;
     }
     *out = it->second;

@@ -3,6 +3,7 @@
 //   nvc_rms_norm_pair             the residual accumulation fused with up to two RMS norms of the same sum (a parallel layer
 //                                 whose mixer and feed-forward have a norm each), optional row gather for the head
 //   nvc_rms_norm_sandwich         the norm behind a sublayer, the residual sum and the norm in front of the next sublayer in one pass
+//   nvc_softcap_f32               cap tanh(x / cap) on fp32 rows (capped logits)
 //   nvc_head_gate                 per-head output stage of a mixer: optional division by the head's root mean square, times a
 //                                 sigmoid or silu gate, times a constant
 // Every kernel exists for bf16 and fp32 storage; arithmetic is fp32.
@@ -19,6 +20,21 @@ __global__ void embed_gather_scaled_kernel(const int32_t* __restrict__ ids, cons
   if (i >= (int64_t)N * H) return;
   const int n = (int)(i / H), j = (int)(i % H);
   out[(int64_t)n * ldo + j] = ld_f(table + (int64_t)ids[n] * ldt + j) * scale;
+}
+
+// cap tanh(x / cap) in place; CTA = (row, block of columns)
+__global__ void softcap_kernel(float* __restrict__ x, int ld, float cap, int V) {
+  pdl_trigger();
+  pdl_wait();
+  float* p = x + (int64_t)blockIdx.y * ld;
+  const int j = 4 * (blockIdx.x * blockDim.x + threadIdx.x);
+  if (j + 4 <= V && (ld & 3) == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0) {
+    float4 v = *reinterpret_cast<float4*>(p + j);
+    v.x = cap * tanh_f32(v.x / cap); v.y = cap * tanh_f32(v.y / cap); v.z = cap * tanh_f32(v.z / cap); v.w = cap * tanh_f32(v.w / cap);
+    *reinterpret_cast<float4*>(p + j) = v;
+  } else {
+    for (int k = j; k < min(j + 4, V); ++k) p[k] = cap * tanh_f32(p[k] / cap);
+  }
 }
 
 // one CTA per output row; the summed row stays in shared memory between the two passes
@@ -100,7 +116,11 @@ __global__ void rms_norm_sandwich_kernel(const float* __restrict__ res_in, const
     row[j] = s;
     ss += s * s;
   }
-  if (!w) return;
+  if (!out) return;
+  if (!w) {          // every thread stores the numbers it has just summed
+    for (int j = threadIdx.x; j < H; j += blockDim.x) st_f(out + (int64_t)blockIdx.x * ldo + j, row[j]);
+    return;
+  }
   ss = warp_sum(ss);
   if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = ss;
   __syncthreads();
@@ -179,6 +199,7 @@ __global__ void rms_norm_sandwich_vec_kernel(const float* __restrict__ res_in, c
     const int j = threadIdx.x + k * blockDim.x;
     if (j < H4) {
       if (res_out) *reinterpret_cast<float4*>(res_out + src * ld + 4 * j) = s[k];
+      if (out && !w) st4(out + (int64_t)blockIdx.x * ldo + 4 * j, s[k]);
       ss += s[k].x * s[k].x + s[k].y * s[k].y + s[k].z * s[k].z + s[k].w * s[k].w;
     }
   }
@@ -292,13 +313,13 @@ int nvc_rms_norm_sandwich(nvc_ctx* ctx, const float* res_in, const float* y, con
                           void* out, int out_dtype, int ldo, float eps, float weight_offset, const int32_t* rows, int N, int H,
                           void* stream) {
   NVC_REQUIRE(ctx, ctx && res_in, NVC_EINVAL, "null pointer");
-  NVC_REQUIRE(ctx, (y == nullptr) == (wy == nullptr) && (w == nullptr) == (out == nullptr), NVC_EINVAL,
+  NVC_REQUIRE(ctx, (y == nullptr) == (wy == nullptr) && (out || !w), NVC_EINVAL,
               "every norm needs its weight and its input or output");
-  NVC_REQUIRE(ctx, N >= 0 && H > 0 && H <= 12288 && ld >= H && (!w || ldo >= H), NVC_EINVAL, "bad sizes (rows of up to 12 288 numbers)");
+  NVC_REQUIRE(ctx, N >= 0 && H > 0 && H <= 12288 && ld >= H && (!out || ldo >= H), NVC_EINVAL, "bad sizes (rows of up to 12 288 numbers)");
   NVC_REQUIRE(ctx, !(rows && res_out), NVC_EINVAL, "a gathering call does not write the residual back");
   if (N == 0) return NVC_OK;
   auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
-  if (H % 4 == 0 && ld % 4 == 0 && (!w || ldo % 4 == 0) && H <= 8192 && al16(res_in) && al16(y) && al16(wy) && al16(res_out) && al16(w) && al16(out)) {
+  if (H % 4 == 0 && ld % 4 == 0 && (!out || ldo % 4 == 0) && H <= 8192 && al16(res_in) && al16(y) && al16(wy) && al16(res_out) && al16(w) && al16(out)) {
     // rows in registers, 16-byte accesses: one float4 per thread up to 1024 numbers, two up to 4096 (256 and 512 threads), then four
     const int H4 = H / 4;
     const int threads = H4 <= 64 ? 64 : (H4 <= 128 ? 128 : (H4 <= 256 ? 256 : 512));
@@ -318,6 +339,15 @@ int nvc_rms_norm_sandwich(nvc_ctx* ctx, const float* res_in, const float* y, con
                   NVC_CUDA_CHECK(ctx, nvc_launch(ctx, rms_norm_sandwich_kernel<T>, dim3(N), dim3(threads), (size_t)H * sizeof(float),
                                                  nvc_stream(stream), res_in, y, wy, res_out, ld, w, reinterpret_cast<T*>(out), ldo, eps,
                                                  weight_offset, rows, H)));
+  ctx->launches++;
+  return NVC_OK;
+}
+
+int nvc_softcap_f32(nvc_ctx* ctx, float* x, int ld, float cap, int N, int V, void* stream) {
+  NVC_REQUIRE(ctx, ctx && x, NVC_EINVAL, "null pointer");
+  NVC_REQUIRE(ctx, N >= 0 && N <= 65535 && V > 0 && ld >= V && cap > 0.f, NVC_EINVAL, "bad sizes");
+  if (N == 0) return NVC_OK;
+  NVC_CUDA_CHECK(ctx, nvc_launch(ctx, softcap_kernel, dim3((unsigned)((V + 1023) / 1024), (unsigned)N), dim3(256), 0, nvc_stream(stream), x, ld, cap, V));
   ctx->launches++;
   return NVC_OK;
 }

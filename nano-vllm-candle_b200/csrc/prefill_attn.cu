@@ -35,6 +35,12 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+__device__ __forceinline__ float fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 struct PagedKV {                              // kPaged only
   const int32_t* block_tables;                // [B, bt_stride], -1 padded
   const int32_t* context_lens;                // [B]
@@ -42,6 +48,12 @@ struct PagedKV {                              // kPaged only
   int block_size;
   int box_rows;                               // token rows per K / V TMA box = min(64, block_size)
   const float* sink;                          // optional [nh]: one more term exp(sink_h) in every row's denominator, no value
+  // shared key / value rows only
+  int window;                                 // > 0: a row sees itself and the window - 1 keys before it
+  const float* bias;                          // sigmoid weights: [nh], added to the scores
+  const float* key_scale;                     // sigmoid weights: [slots], a factor on the scores of a cached key
+  const float* gate;                          // sigmoid weights: fp32 [rows, ldg], a sigmoid gate on every output number
+  int ldg;
 };
 
 int make_tma_heads(nvc_ctx* ctx, CUtensorMap* map, const void* base, int heads, int64_t tokens, int ld, int box_rows = 128) {
@@ -63,22 +75,23 @@ int make_tma_heads(nvc_ctx* ctx, CUtensorMap* map, const void* base, int heads, 
 #include "prefill_attn_v2.cuh"
 
 // persistent grid of the second-generation kernel: two CTAs per SM, or one CTA per work item when there are fewer
-template <bool kPaged>
+template <bool kPaged, int kMode = v2::kPlain>
 cudaError_t launch_v2(nvc_ctx* ctx, int QT, int nh, int kv, int B, cudaStream_t st, const CUtensorMap& tq, const CUtensorMap& tk,
                       const CUtensorMap& tv, const int32_t* cu_seqlens, float scale_log2e, nvc_bf16* out, int ldo, const PagedKV& pk) {
   const long long items = (long long)QT * nh * B;
   if (items > 0x7fffffffLL) return cudaErrorInvalidValue;
   const int grid = (int)(items < 2LL * ctx->num_sms ? items : 2LL * ctx->num_sms);
   v2::Sched sc{v2::make_fastdiv(nh * B), v2::make_fastdiv(nh), v2::make_fastdiv(nh / kv), QT, (int)items};
-  return nvc_launch(ctx, v2::prefill_attn_v2_kernel<kPaged>, dim3(grid), dim3(v2::kThreads), v2::kSmemBytes, st, tq, tk, tv,
+  return nvc_launch(ctx, v2::prefill_attn_v2_kernel<kPaged, kMode>, dim3(grid), dim3(v2::kThreads), v2::kSmemBytes, st, tq, tk, tv,
                     cu_seqlens, sc, scale_log2e, out, ldo, pk);
 }
 
 }  // namespace
 
 extern "C" int nvc_prefill_attn_init(nvc_ctx* ctx) {
-  NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(v2::prefill_attn_v2_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, v2::kSmemBytes));
-  NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(v2::prefill_attn_v2_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, v2::kSmemBytes));
+  for (auto k : {v2::prefill_attn_v2_kernel<false, v2::kPlain>, v2::prefill_attn_v2_kernel<true, v2::kPlain>,
+                 v2::prefill_attn_v2_kernel<true, v2::kShared>, v2::prefill_attn_v2_kernel<true, v2::kSigmoid>})
+    NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, v2::kSmemBytes));
   return NVC_OK;
 }
 
@@ -157,10 +170,49 @@ extern "C" int nvc_prefill_attn_paged_sink(nvc_ctx* ctx, const nvc_bf16* q, int 
   if (rc) return rc;
   rc = make_tma_heads(ctx, &tv, v_cache, kv, (int64_t)num_blocks * block_size, kv * hd, box_rows);
   if (rc) return rc;
-  PagedKV pk{block_tables, context_lens, bt_stride, block_size, box_rows, sink};
+  PagedKV pk{};
+  pk.block_tables = block_tables; pk.context_lens = context_lens; pk.bt_stride = bt_stride; pk.block_size = block_size; pk.box_rows = box_rows;
+  pk.sink = sink;
   const int QT = (max_seqlen_q + 127) / 128;
   NVC_CUDA_CHECK(ctx, launch_v2<true>(ctx, QT, nh, kv, B, nvc_stream(stream), tq, tk, tv, cu_seqlens_q,
                                       scale * 1.4426950408889634f, out, ldo, pk));
+  NVC_CUDA_CHECK(ctx, cudaGetLastError());
+  ctx->launches++;
+  return NVC_OK;
+}
+
+extern "C" int nvc_prefill_attn_shared(nvc_ctx* ctx, const nvc_bf16* q, int ldq, const nvc_bf16* cache, const int32_t* block_tables, int bt_stride,
+                                       const int32_t* context_lens, const int32_t* cu_seqlens_q, int B, int total_q_tokens, int max_seqlen_q,
+                                       int block_size, int num_blocks, const nvc_attn_spec* spec, nvc_bf16* out, int ldo, void* stream) {
+  NVC_REQUIRE(ctx, ctx && q && cache && block_tables && context_lens && cu_seqlens_q && spec && out, NVC_EINVAL, "null pointer");
+  const nvc_attn_spec& s = *spec;
+  const int nh = s.heads, kv = s.kv_heads;
+  const bool sig = s.weights == NVC_ATTN_SIGMOID;
+  NVC_REQUIRE(ctx, B >= 0 && total_q_tokens >= 0 && max_seqlen_q >= 0 && nh > 0 && kv > 0 && bt_stride > 0 && num_blocks > 0, NVC_EINVAL, "bad sizes");
+  NVC_REQUIRE(ctx, s.dim == 128 && s.vdim == 128 && nh % kv == 0, NVC_ESHAPE, "rows of 128 numbers per head, nh a multiple of kv");
+  NVC_REQUIRE(ctx, s.window >= 0 && s.chunk == 0 && s.softcap == 0.f && s.out_scale == 1.f && !s.gate_per_head && (sig ? !s.sink : (!s.gate && !s.bias && !s.key_scale)),
+              NVC_EINVAL, "unsupported attention variant");
+  NVC_REQUIRE(ctx, block_size >= 16 && (block_size >= 128 ? block_size % 128 == 0 : 128 % block_size == 0), NVC_ESHAPE,
+              "paged prefill needs block_size in {16, 32, 64} or a multiple of 128");
+  NVC_REQUIRE(ctx, ldq % 8 == 0 && ldq >= nh * 128 && ldo % 8 == 0 && ldo >= nh * 128 && (!s.gate || (s.ldg % 4 == 0 && s.ldg >= nh * 128)), NVC_ESHAPE,
+              "row strides must cover the heads and be multiples of 8 (gate: 4)");
+  auto al16 = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
+  NVC_REQUIRE(ctx, al16(q) && al16(cache) && al16(out) && al16(s.gate) && al16(s.key_scale), NVC_EINVAL, "pointers must be 16-byte aligned");
+  NVC_REQUIRE(ctx, ctx->encode_tiled != nullptr, NVC_EDEVICE, "cuTensorMapEncodeTiled unavailable");
+  if (B == 0 || total_q_tokens == 0 || max_seqlen_q == 0) return NVC_OK;
+  const int box_rows = block_size < v2::kKT ? block_size : v2::kKT;
+  CUtensorMap tq, tk;
+  int rc = make_tma_heads(ctx, &tq, q, nh, total_q_tokens, ldq);
+  if (rc) return rc;
+  rc = make_tma_heads(ctx, &tk, cache, kv, (int64_t)num_blocks * block_size, kv * 128, box_rows);
+  if (rc) return rc;
+  PagedKV pk{block_tables, context_lens, bt_stride, block_size, box_rows, s.sink, s.window, s.bias, s.key_scale, s.gate, s.ldg};
+  const int QT = (max_seqlen_q + 127) / 128;
+  const float scale_log2e = s.scale * 1.4426950408889634f;
+  if (sig)
+    NVC_CUDA_CHECK(ctx, (launch_v2<true, v2::kSigmoid>(ctx, QT, nh, kv, B, nvc_stream(stream), tq, tk, tk, cu_seqlens_q, scale_log2e, out, ldo, pk)));
+  else
+    NVC_CUDA_CHECK(ctx, (launch_v2<true, v2::kShared>(ctx, QT, nh, kv, B, nvc_stream(stream), tq, tk, tk, cu_seqlens_q, scale_log2e, out, ldo, pk)));
   NVC_CUDA_CHECK(ctx, cudaGetLastError());
   ctx->launches++;
   return NVC_OK;

@@ -20,6 +20,12 @@
 //   * barrier init / TMEM allocation / descriptor prefetch run before the PDL dependency wait.
 // A share of the exponentials on the FMA pipe (degree-3 polynomial) was measured and is not used: no gain at 1/4,
 // a loss at 1/2 (same profile file) - the kernel is bound by dependent latency per tile, not by the MUFU unit.
+// kMode: kPlain = separate key and value tensors, causal softmax.  kShared = the cache rows are keys AND values (latent attention in its
+// absorbed form): one ring of four tiles serves both products - S reads a tile K-major, P V reads the same bytes MN-major - with an
+// optional sliding window (kv tiles in front of the q tile's first visible key are never loaded).  kSigmoid = the same shared tiles
+// with sigmoid(scale key_scale_j s + bias_h) weights: no maximum, no sum and no rescaling of O, so P V runs without any wait on the
+// softmax warps' side; the keys' factors ride behind their tile (bulk copy on the tile's barrier), the output gate is applied on the
+// way out.
 // Included by prefill_attn.cu (shares PagedKV, make_tma_heads, fast_exp2).
 #pragma once
 
@@ -36,13 +42,17 @@ constexpr int kOffK = kQBytes;
 constexpr int kOffV = kOffK + kKStages * kKBytes;
 constexpr int kOffStage = kOffV + kVStages * kKBytes;   // 4 softmax warps x 4 KB row staging for the output
 constexpr int kOffBar = kOffStage + 4 * 4096;           // 114688
-// q_full, q_empty, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full, o_full, o_free
-constexpr int kNumBars = 2 + 2 * kKStages + 2 * kVStages + 2 + 3;
+// q_full, q_empty, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full, o_full, o_free, a second p_full
+constexpr int kNumBars = 2 + 2 * kKStages + 2 * kVStages + 2 + 4;
 // two CTAs per SM: 2 x (request + 1 KB reserved) <= 228 KB; the dynamic shared memory is requested 1024-byte aligned
 // (no static shared memory in this kernel: the pad is 0 in practice), a pad of up to 768 B fits, beyond that the kernel traps
 constexpr int kSmemBytes = 115712;
 static_assert(kOffBar + kNumBars * 8 + 16 + 768 <= kSmemBytes, "shared memory budget for two CTAs per SM");
 constexpr int kTmemCols = 256;                 // S / P (double-buffered): columns [0, 64) and [64, 128); O: [128, 256)
+enum { kPlain = 0, kShared = 1, kSigmoid = 2 };
+// shared tiles: stages of the one ring; the key factors of a stage take the place of a fourth tile
+template <int kMode> struct SharedRing { static constexpr int kStages = kMode == kSigmoid ? 3 : 4; };
+constexpr int kOffScale = kOffK + 3 * kKBytes;
 constexpr float kRescaleLog2 = 8.0f;           // rescale O only when a row's maximum grew by more than 2^8
 
 // work item -> (q tile, head, sequence): q tiles in DESCENDING order (longest first), heads fastest (the heads of a GQA
@@ -75,7 +85,7 @@ __device__ __forceinline__ Item item_of(int it, const Sched& sc) {
   return x;
 }
 
-template <bool kPaged>
+template <bool kPaged, int kMode>
 __global__ void __launch_bounds__(192, 2)
 prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                        const __grid_constant__ CUtensorMap tma_v, const int32_t* __restrict__ cu_seqlens, const Sched sc,
@@ -95,21 +105,32 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
   auto v_full = [&](int s) { return bar0 + 8u * (2 + 2 * kKStages + s); };
   auto v_empty = [&](int s) { return bar0 + 8u * (2 + 2 * kKStages + kVStages + s); };
   auto s_full = [&](int s) { return bar0 + 8u * (2 + 2 * kKStages + 2 * kVStages + s); };
-  const uint32_t p_full = bar0 + 8u * (kNumBars - 3), o_full = bar0 + 8u * (kNumBars - 2), o_free = bar0 + 8u * (kNumBars - 1);
+  // shared tiles: one ring on the same eight barriers
+  constexpr int kKV = SharedRing<kMode>::kStages;
+  auto kv_full = [&](int s) { return bar0 + 8u * (2 + s); };
+  auto kv_empty = [&](int s) { return bar0 + 8u * (6 + s); };
+  // P of tile g: one barrier, its phase counts tiles - a softmax warp is at most one tile ahead of the MMA warp, since it waits for
+  // P V(g - 1) before it hands over P(g).  Sigmoid warps do not wait for P V and could complete two phases before the MMA warp looks:
+  // two barriers, one per S buffer.
+  auto p_full = [&](uint32_t g) { return bar0 + 8u * (kMode == kSigmoid && (g & 1) ? kNumBars - 1 : kNumBars - 4); };
+  auto p_phase = [&](uint32_t g) { return (kMode == kSigmoid ? g >> 1 : g) & 1; };
+  const uint32_t o_full = bar0 + 8u * (kNumBars - 3), o_free = bar0 + 8u * (kNumBars - 2);
   const uint32_t tmem_slot = bar0 + 8u * kNumBars;
   volatile uint32_t* tmem_slot_gen = reinterpret_cast<volatile uint32_t*>(gen + kOffBar + kNumBars * 8);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // geometry of one item (every role derives the same numbers): q row i of the tile is context position q0 + i and sees
-  // keys 0 .. q0 + i; n_tiles = 0 marks a q tile past the end of its sequence (skipped by every role)
-  struct Geo { int seq_start, seq_len, kv_len, q0, n_tiles; };
+  // n_tiles = 0 marks a q tile past the end of its sequence (skipped by every role)
+  // keys 0 .. q0 + i, or the last `window` of them; j0 = the first kv tile, n_tiles are counted from there
+  struct Geo { int seq_start, seq_len, kv_len, q0, j0, n_tiles; };
   auto geo_of = [&](const Item& x) {
     Geo g;
     g.seq_start = __ldg(cu_seqlens + x.b);
     g.seq_len = __ldg(cu_seqlens + x.b + 1) - g.seq_start;
     g.kv_len = kPaged ? __ldg(pk.context_lens + x.b) : g.seq_len;
     g.q0 = g.kv_len - g.seq_len + x.qt * 128;
-    g.n_tiles = x.qt * 128 >= g.seq_len ? 0 : (min(g.kv_len, g.q0 + 128) + kKT - 1) / kKT;
+    g.j0 = kMode != kPlain && pk.window > 0 ? max(g.q0 - pk.window + 1, 0) / kKT : 0;
+    g.n_tiles = x.qt * 128 >= g.seq_len ? 0 : (min(g.kv_len, g.q0 + 128) + kKT - 1) / kKT - g.j0;
     return g;
   };
 
@@ -117,14 +138,14 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     if (lane == 0) {
       ptx::tma_prefetch_desc(&tma_q);
       ptx::tma_prefetch_desc(&tma_k);
-      ptx::tma_prefetch_desc(&tma_v);
+      if (kMode == kPlain) ptx::tma_prefetch_desc(&tma_v);
       ptx::mbar_init(q_full, 1);
       ptx::mbar_init(q_empty, 1);
-      for (int s = 0; s < kKStages; ++s) { ptx::mbar_init(k_full(s), 1); ptx::mbar_init(k_empty(s), 1); }
-      for (int s = 0; s < kVStages; ++s) { ptx::mbar_init(v_full(s), 1); ptx::mbar_init(v_empty(s), 1); }
+      for (int s = 0; s < 2 * (kKStages + kVStages); ++s) ptx::mbar_init(bar0 + 8u * (2 + s), 1);     // the tiles' full / empty pairs
       ptx::mbar_init(s_full(0), 1);
       ptx::mbar_init(s_full(1), 1);
-      ptx::mbar_init(p_full, 128);
+      ptx::mbar_init(p_full(0), 128);
+      if (kMode == kSigmoid) ptx::mbar_init(p_full(1), 128);
       ptx::mbar_init(o_full, 1);
       ptx::mbar_init(o_free, 128);
       ptx::fence_barrier_init();
@@ -176,6 +197,28 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       }
       __syncwarp();
     };
+    // shared tiles: boxes of box_rows cache rows (keys and values at once) and the rows' factors, one barrier per tile
+    auto load_shared = [&](const Item& x, const Geo& ge, int j, uint32_t g) {
+      const int s = (int)(g % kKV);
+      ptx::mbar_wait(kv_empty(s), ((g / kKV) & 1) ^ 1u);
+      if (ptx::elect_one()) {
+        const uint32_t dst = base + kOffK + s * kKBytes, bar = kv_full(s);
+        const int rows = pk.box_rows, tok0 = (ge.j0 + j) * kKT;
+        const int nbox = min(kKT / rows, (ge.kv_len - tok0 + rows - 1) / rows);
+        const bool factors = kMode == kSigmoid && pk.key_scale != nullptr;
+        ptx::mbar_arrive_expect_tx(bar, (uint32_t)(nbox * rows * (factors ? 260 : 256)));
+        const int32_t* bt = pk.block_tables + (int64_t)x.b * pk.bt_stride;
+        for (int i = 0; i < nbox; ++i) {
+          const int tok = tok0 + i * rows;
+          const int slot = __ldg(bt + tok / pk.block_size) * pk.block_size + tok % pk.block_size;
+          const uint32_t o = (uint32_t)(i * rows * 128);
+          ptx::tma_load_3d(dst + o, &tma_k, bar, 0, x.kvh, slot);
+          ptx::tma_load_3d(dst + kHalfKV + o, &tma_k, bar, 64, x.kvh, slot);
+          if (factors) ptx::bulk_load(base + kOffScale + s * (kKT * 4) + i * rows * 4, pk.key_scale + slot, (uint32_t)(rows * 4), bar);
+        }
+      }
+      __syncwarp();
+    };
     uint32_t g = 0, n_done = 0;
     Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
     Geo gn = geo_of(xn);
@@ -195,10 +238,14 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         ptx::tma_load_3d(base + kOffQ + 16384, &tma_q, q_full, 64, x.h, ge.seq_start + x.qt * 128);
       }
       __syncwarp();
-      load_kv(x, ge, 0, g, false);
-      for (int j = 0; j < ge.n_tiles; ++j) {
-        if (j + 1 < ge.n_tiles) load_kv(x, ge, j + 1, g + j + 1, false);   // K runs one tile ahead of V, as S runs ahead of P V
-        load_kv(x, ge, j, g + j, true);
+      if constexpr (kMode == kPlain) {
+        load_kv(x, ge, 0, g, false);
+        for (int j = 0; j < ge.n_tiles; ++j) {
+          if (j + 1 < ge.n_tiles) load_kv(x, ge, j + 1, g + j + 1, false);   // K runs one tile ahead of V, as S runs ahead of P V
+          load_kv(x, ge, j, g + j, true);
+        }
+      } else {
+        for (int j = 0; j < ge.n_tiles; ++j) load_shared(x, ge, j, g + j);
       }
       g += ge.n_tiles;
       ++n_done;
@@ -212,8 +259,9 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     // S(g) = Q K^T into S buffer g & 1 : 8 k-steps of 16 over head_dim (two 64-wide swizzled halves).  The buffer last
     // held S / P of tile g - 2, whose P V MMA was issued earlier by this thread: tcgen05.mma executes in issue order.
     auto issue_s = [&](uint32_t g, bool last_of_item) {
-      const int s = (int)(g % kKStages);
-      ptx::mbar_wait(k_full(s), (g / kKStages) & 1);
+      constexpr int kStagesS = kMode == kPlain ? kKStages : kKV;
+      const int s = (int)(g % kStagesS);
+      ptx::mbar_wait(kMode == kPlain ? k_full(s) : kv_full(s), (g / kStagesS) & 1);
       ptx::tcgen05_fence_after();
       if (ptx::elect_one()) {
         const uint32_t k_lo = ptx::umma_desc_lo(base + kOffK + s * kKBytes, 16);
@@ -225,7 +273,7 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
                             ks != 0);
         }
         ptx::umma_commit(s_full(g & 1));
-        ptx::umma_commit(k_empty(s));          // the K slot is free as soon as these MMAs have read it
+        if (kMode == kPlain) ptx::umma_commit(k_empty(s));          // the K slot is free as soon as these MMAs have read it
         if (last_of_item) ptx::umma_commit(q_empty);   // ... and so is Q after the item's last S
       }
       __syncwarp();
@@ -248,22 +296,23 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         // S is double-buffered: S(j+1) is computed while the softmax threads work on S(j)
         if (j + 1 < n) issue_s(g + j + 1, j + 2 == n);
         // P(j) is in tensor memory, O has been rescaled for tile j (both by the softmax threads)
-        ptx::mbar_wait(p_full, (g + j) & 1);
-        const int vs = (int)((g + j) % kVStages);
-        ptx::mbar_wait(v_full(vs), ((g + j) / kVStages) & 1);
+        ptx::mbar_wait(p_full(g + j), p_phase(g + j));
+        const int vs = (int)((g + j) % (kMode == kPlain ? kVStages : kKV));
+        if (kMode == kPlain) ptx::mbar_wait(v_full(vs), ((g + j) / kVStages) & 1);     // shared: S has read the same tile
         // the first P V of an item overwrites O: the previous item's output rows have been read out of it
         if (j == 0 && n_done > 0) ptx::mbar_wait(o_free, (n_done - 1) & 1);
         ptx::tcgen05_fence_after();
         if (ptx::elect_one()) {
           // O += P V_j: A = P from tensor memory (8 columns per 16 kv tokens); B = V (MN-major: LBO = 8 KB between the
           // two 64-wide head-dim halves, SBO = 1 KB between groups of 8 token rows, 16 token rows = 2048 bytes per step)
-          const uint32_t v_lo = ptx::umma_desc_lo(base + kOffV + vs * kKBytes, (uint32_t)kHalfKV);
+          const uint32_t v_lo = ptx::umma_desc_lo(base + (kMode == kPlain ? kOffV : kOffK) + vs * kKBytes, (uint32_t)kHalfKV);
 #pragma unroll
           for (int ks = 0; ks < kKT / 16; ++ks)
             ptx::umma_bf16_ts(tmem_o, tmem_s + ((g + j) & 1) * kKT + ks * 8, ptx::umma_desc(v_lo + ks * (2048 >> 4), hi_k),
                               idesc_pv, (j | ks) != 0);
-          ptx::umma_commit(o_full);
-          ptx::umma_commit(v_empty(vs));
+          // sigmoid: nobody looks at O before the item's last tile, whose barrier phase counts items
+          if (kMode != kSigmoid || j + 1 == n) ptx::umma_commit(o_full);
+          ptx::umma_commit(kMode == kPlain ? v_empty(vs) : kv_empty(vs));
         }
         __syncwarp();
       }
@@ -275,7 +324,7 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     const int quad = warp & 3;
     const int r = quad * 32 + lane;                 // row in the q tile
     const uint32_t lane_addr = (uint32_t)(quad * 32) << 16;
-    uint32_t g = 0;
+    uint32_t g = 0, n_done = 0;
     Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
     Geo gn = geo_of(xn);
     for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
@@ -287,7 +336,9 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       }
       if (ge.n_tiles == 0) continue;
       const int n = ge.n_tiles;
-      float m = -INFINITY, l = 0.f;                 // m: the maximum the exponentials are taken against (may lag the true one)
+      const float bias = kMode == kSigmoid && pk.bias ? __ldg(pk.bias + x.h) * 1.4426950408889634f : 0.f;
+      // with a window a row's first tiles may hold none of its keys: a finite floor keeps every difference of maxima defined
+      float m = kMode == kShared ? -1e30f : -INFINITY, l = 0.f;                 // m: the maximum the exponentials are taken against (may lag the true one)
       for (int j = 0; j < n; ++j) {
         const uint32_t gi = g + j;
         const uint32_t s_addr = tmem_s + (gi & 1) * kKT + lane_addr;
@@ -299,11 +350,54 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         ptx::tmem_ld_wait();
         // diagonal tiles only (the tile holds keys past some row's position): columns past this row's position
         // become -inf, i.e. p = exp2(-inf) = 0; every other tile takes the mask-free path below
-        if (j * kKT + kKT - 1 > ge.q0) {
-          const int lim = ge.q0 + r - j * kKT;            // last visible column of this row
+        const int t0 = (ge.j0 + j) * kKT;                  // the tile's first key position
+        uint32_t pk2[kKT / 2];
+        bool move = false;
+        float alpha = 1.0f;
+        if constexpr (kMode == kSigmoid) {
+          if (pk.key_scale) {
+            ptx::mbar_wait(kv_full((int)(gi % kKV)), (gi / kKV) & 1);      // long complete (S was made of this tile): orders the reads below
+            const float4* f = reinterpret_cast<const float4*>(gen + kOffScale + (gi % kKV) * (kKT * 4));
+#pragma unroll
+            for (int i = 0; i < kKT; i += 4) {
+              const float4 v = f[i >> 2];
+              sv[i] = __float_as_uint(__uint_as_float(sv[i]) * v.x);
+              sv[i + 1] = __float_as_uint(__uint_as_float(sv[i + 1]) * v.y);
+              sv[i + 2] = __float_as_uint(__uint_as_float(sv[i + 2]) * v.z);
+              sv[i + 3] = __float_as_uint(__uint_as_float(sv[i + 3]) * v.w);
+            }
+          }
+          // e = 2^-(x log2e) for 64 keys, then p = 1 / (1 + e)
+#pragma unroll
+          for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fast_exp2(fmaf(__uint_as_float(sv[i]), -scale_log2e, -bias)));
+#pragma unroll
+          for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fast_rcp(1.0f + __uint_as_float(sv[i])));
+          if (t0 + kKT - 1 > ge.q0) {
+            const int lim = ge.q0 + r - t0;
+#pragma unroll
+            for (int i = 0; i < kKT; ++i)
+              if (i > lim) sv[i] = 0u;
+          }
+          if (pk.window > 0 && t0 <= ge.q0 + 127 - pk.window) {
+            const int first = ge.q0 + r - pk.window + 1 - t0;
+#pragma unroll
+            for (int i = 0; i < kKT; ++i)
+              if (i < first) sv[i] = 0u;
+          }
+#pragma unroll
+          for (int i = 0; i < kKT; i += 2) pk2[i >> 1] = pack_bf16(__uint_as_float(sv[i]), __uint_as_float(sv[i + 1]));
+        } else {
+        if (t0 + kKT - 1 > ge.q0) {
+          const int lim = ge.q0 + r - t0;                 // last visible column of this row
 #pragma unroll
           for (int i = 0; i < kKT; ++i)
             if (i > lim) sv[i] = 0xff800000u;
+        }
+        if (kMode == kShared && pk.window > 0 && t0 <= ge.q0 + 127 - pk.window) {
+          const int first = ge.q0 + r - pk.window + 1 - t0;      // first visible column of this row
+#pragma unroll
+          for (int i = 0; i < kKT; ++i)
+            if (i < first) sv[i] = 0xff800000u;
         }
         // row maximum over four independent chains
         float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
@@ -317,8 +411,7 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         const float mt = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * scale_log2e;   // finite on tile 0: key 0 is visible to every row
         // lazy rescale: move the reference maximum (and pay the O round trip) only when some row of this warp outgrew it
         // by more than 2^kRescaleLog2; m = -inf on the first tile, so that one always moves
-        const bool move = __any_sync(0xffffffffu, mt > m + kRescaleLog2);
-        float alpha = 1.0f;
+        move = __any_sync(0xffffffffu, mt > m + kRescaleLog2);
         if (move) {
           const float m_new = fmaxf(m, mt);
           alpha = fast_exp2(m - m_new);
@@ -330,7 +423,6 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
 #pragma unroll
         for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fast_exp2(__uint_as_float(sv[i])));
         float ps0 = 0.f, ps1 = 0.f, ps2 = 0.f, ps3 = 0.f;
-        uint32_t pk2[kKT / 2];
 #pragma unroll
         for (int i = 0; i < kKT; i += 4) {
           const float p0 = __uint_as_float(sv[i]), p1 = __uint_as_float(sv[i + 1]);
@@ -340,7 +432,8 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
           pk2[(i >> 1) + 1] = pack_bf16(p2, p3);
         }
         l = l * alpha + ((ps0 + ps1) + (ps2 + ps3));
-        if (j > 0) {
+        }
+        if (kMode != kSigmoid && j > 0) {
           // P V(j-1) has completed: O holds the sum over tiles < j.  Waited for on EVERY tile, moved or not: a parity
           // wait is only meaningful within one phase of the barrier, so the softmax threads must observe each o_full
           // phase in turn (skipping them let the final wait take an older phase for the last one).  The MMA was issued a
@@ -367,11 +460,12 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
           // V rows at / past the end of the context (last tile only): zero them (every P column there is 0,
           // but the cache bytes may be NaN) once the slot's TMA has landed; the proxy fence orders these
           // generic stores before the P V MMA.
-          if (j * kKT + kKT > ge.kv_len) {
-            const int vs = (int)(gi % kVStages);
-            ptx::mbar_wait(v_full(vs), (gi / kVStages) & 1);
-            if (r < kKT && j * kKT + r >= ge.kv_len) {
-              uint8_t* v_row = gen + kOffV + vs * kKBytes + r * 128;
+          if (t0 + kKT > ge.kv_len) {
+            constexpr int kStagesV = kMode == kPlain ? kVStages : kKV;
+            const int vs = (int)(gi % kStagesV);
+            ptx::mbar_wait(kMode == kPlain ? v_full(vs) : kv_full(vs), (gi / kStagesV) & 1);
+            if (r < kKT && t0 + r >= ge.kv_len) {
+              uint8_t* v_row = gen + (kMode == kPlain ? kOffV : kOffK) + vs * kKBytes + r * 128;
 #pragma unroll
               for (int k16 = 0; k16 < 8; ++k16) {
                 *reinterpret_cast<uint4*>(v_row + (k16 << 4)) = make_uint4(0, 0, 0, 0);
@@ -382,13 +476,16 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
           }
         }
         ptx::tcgen05_fence_before();
-        ptx::mbar_arrive(p_full);
+        ptx::mbar_arrive(p_full(gi));
       }
       // ---- O / l -> bf16 rows of the output
-      ptx::mbar_wait(o_full, (g + n - 1) & 1);
+      ptx::mbar_wait(o_full, kMode == kSigmoid ? (n_done & 1) : ((g + n - 1) & 1));
       ptx::tcgen05_fence_after();
-      if (kPaged && pk.sink) l += exp2f(__ldg(pk.sink + x.h) * 1.4426950408889634f - m);   // the sink: in the denominator, without a value
-      const float inv = 1.0f / l;
+      if (kPaged && kMode != kSigmoid && pk.sink) l += exp2f(__ldg(pk.sink + x.h) * 1.4426950408889634f - m);   // the sink: in the denominator, without a value
+      const float inv = kMode == kSigmoid ? 1.0f : 1.0f / l;
+      // rows past the sequence are not stored; their gate row is clamped to the last real one
+      const float* grow = kMode == kSigmoid && pk.gate
+                              ? pk.gate + (int64_t)(ge.seq_start + min(x.qt * 128 + r, ge.seq_len - 1)) * pk.ldg + x.h * 128 : nullptr;
       // this warp's 32 rows x 128 head dims leave through its staging buffer: 8 lanes per row, 128 contiguous bytes each
       RowStage st = make_row_stage(gen + kOffStage + quad * 4096, out, 0, NVC_EPI_NONE, (int64_t)ldo,
                                    ge.seq_start + x.qt * 128 + quad * 32, ge.seq_start + ge.seq_len, x.h * 128, 128, nh * 128);
@@ -400,12 +497,23 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         float f[32];
 #pragma unroll
         for (int i = 0; i < 32; ++i) f[i] = __uint_as_float(v[i]) * inv;
+        if (kMode == kSigmoid && grow) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 4) {
+            const float4 z = *reinterpret_cast<const float4*>(grow + c * 32 + i);
+            f[i] *= fast_rcp(1.0f + fast_exp2(-1.4426950408889634f * z.x));
+            f[i + 1] *= fast_rcp(1.0f + fast_exp2(-1.4426950408889634f * z.y));
+            f[i + 2] *= fast_rcp(1.0f + fast_exp2(-1.4426950408889634f * z.z));
+            f[i + 3] *= fast_rcp(1.0f + fast_exp2(-1.4426950408889634f * z.w));
+          }
+        }
         st.emit32(lane, 0, NVC_EPI_NONE, f);
       }
       st.finish(lane);
       ptx::tcgen05_fence_before();
       ptx::mbar_arrive(o_free);                      // the next item's first P V may overwrite O
       g += n;
+      ++n_done;
     }
   }
   ptx::tcgen05_fence_before();

@@ -13,6 +13,9 @@
 // element-wise case (bias and silu only, plain fp32 rows out) runs a flat kernel with 16-byte accesses instead.
 #include "typed.cuh"
 
+#include <algorithm>
+#include <cmath>
+
 namespace {
 
 struct PrepArgs {
@@ -147,6 +150,102 @@ __global__ void head_split_rot_kernel(const float* __restrict__ in, int ldi, int
   }
 }
 
+// four neighbouring numbers in the storage format with one store
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
+  uint2 u;
+  u.x = pack_bf16(v.x, v.y);
+  u.y = pack_bf16(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+
+// one CTA per token: the sums of squares of the whole query and the whole key projection in one pass (the key rows leave for the cache
+// on the way), then the queries.  VEC: every offset, width and stride is a multiple of 4 and the pointers are 16-byte aligned.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) qk_norm_fold_store_kernel(const float* __restrict__ in, int ldi, int q_off, int qw, int k_off, int kw,
+                                                                 const float* __restrict__ wqk, float eps, const int32_t* __restrict__ positions,
+                                                                 float temp_coef, int temp_every, T* __restrict__ q_out, int ldq,
+                                                                 T* __restrict__ cache, int ldc, float* __restrict__ key_scale,
+                                                                 const int32_t* __restrict__ slots) {
+  constexpr int P = VEC ? 4 : 1;
+  constexpr int KEEP = 8;                              // accesses per thread that stay in registers between the passes
+  __shared__ float part[2][8];
+  pdl_trigger();
+  const int64_t n = blockIdx.x;
+  const int slot = slots[n];
+  const float temp = 1.0f + temp_coef * logf((float)((positions[n] + 1) / temp_every) + 1.0f);
+  pdl_wait();
+  const float* q = in + n * ldi + q_off;
+  const float* k = in + n * ldi + k_off;
+  T* row = cache + (int64_t)slot * ldc;
+  float sq = 0.f, sk = 0.f;
+  float4 keep[KEEP];
+  const int step = P * blockDim.x;
+#pragma unroll
+  for (int c = 0; c < KEEP; ++c) {
+    const int j = P * threadIdx.x + c * step;
+    if (j < qw) {
+      if constexpr (VEC) {
+        const float4 v = *reinterpret_cast<const float4*>(q + j);
+        keep[c] = v;
+        sq += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      } else {
+        keep[c].x = q[j];
+        sq += keep[c].x * keep[c].x;
+      }
+    }
+  }
+  for (int j = P * threadIdx.x + KEEP * step; j < qw; j += step) {
+    if constexpr (VEC) {
+      const float4 v = *reinterpret_cast<const float4*>(q + j);
+      sq += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    } else {
+      sq += q[j] * q[j];
+    }
+  }
+  if (slot >= 0) {
+    for (int j = P * threadIdx.x; j < kw; j += step) {
+      if constexpr (VEC) {
+        const float4 v = *reinterpret_cast<const float4*>(k + j);
+        store4(row + j, v);
+        sk += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      } else {
+        st_f(row + j, k[j]);
+        sk += k[j] * k[j];
+      }
+    }
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) { part[0][threadIdx.x >> 5] = sq; part[1][threadIdx.x >> 5] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) { sq += part[0][w]; sk += part[1][w]; }
+  if (threadIdx.x == 0 && slot >= 0) key_scale[slot] = 1.0f / sqrtf(sk / (float)kw + eps);
+  const float r = temp / sqrtf(sq / (float)qw + eps);
+  T* o = q_out + n * ldq;
+#pragma unroll
+  for (int c = 0; c < KEEP; ++c) {
+    const int j = P * threadIdx.x + c * step;
+    if (j < qw) {
+      if constexpr (VEC) {
+        const float4 w = *reinterpret_cast<const float4*>(wqk + j);
+        store4(o + j, make_float4(keep[c].x * r * w.x, keep[c].y * r * w.y, keep[c].z * r * w.z, keep[c].w * r * w.w));
+      } else {
+        st_f(o + j, keep[c].x * r * wqk[j]);
+      }
+    }
+  }
+  for (int j = P * threadIdx.x + KEEP * step; j < qw; j += step) {
+    if constexpr (VEC) {
+      const float4 v = *reinterpret_cast<const float4*>(q + j), w = *reinterpret_cast<const float4*>(wqk + j);
+      store4(o + j, make_float4(v.x * r * w.x, v.y * r * w.y, v.z * r * w.z, v.w * r * w.w));
+    } else {
+      st_f(o + j, q[j] * r * wqk[j]);
+    }
+  }
+}
+
 template <typename TQ, typename TKV>
 int launch_prep(nvc_ctx* ctx, const nvc_qkv_prep* p, int N, void* stream) {
   PrepArgs a{*p, N};
@@ -213,21 +312,59 @@ extern "C" int nvc_head_split_rot(nvc_ctx* ctx, const float* in, int ldi, int he
   return NVC_OK;
 }
 
-// (cos, sin) of position * base^(-2 i / dims) for every position below max_pos and i < dims / 2, angles in double precision.
-// Synchronous (called once, when a model is built).
-extern "C" int nvc_rotary_table_init_sync(nvc_ctx* ctx, float base, int dims, int max_pos, float* out) {
-  NVC_REQUIRE(ctx, ctx && out && dims > 0 && dims % 2 == 0 && max_pos > 0 && base > 0.f, NVC_EINVAL, "bad arguments");
+// (cos, sin) of position * base^(-2 i / dims) for every position below max_pos and i < dims / 2, angles in double precision; with YaRN
+// scaling the slow pairs turn `factor` times slower, the fast ones as before and those between the two bounds in part, and cos and sin
+// carry one common factor.  Synchronous (called once, when a model is built).
+extern "C" int nvc_rotary_table_init_scaled_sync(nvc_ctx* ctx, double base, int dims, nvc_rotary_scaling sc, int max_pos, float* out) {
+  NVC_REQUIRE(ctx, ctx && out && dims > 0 && dims % 2 == 0 && max_pos > 0 && base > 0.0, NVC_EINVAL, "bad arguments");
+  const bool yarn = sc.factor != 0.0;
+  NVC_REQUIRE(ctx, !yarn || (sc.factor > 0.0 && sc.original > 0.0 && sc.fast > 0.0 && sc.slow > 0.0 && base != 1.0), NVC_EINVAL, "bad scaling");
+  constexpr double kPi = 3.14159265358979323846;
+  auto pair_of = [&](double turns) { return dims * log(sc.original / (2.0 * kPi * turns)) / (2.0 * log(base)); };
+  const double lo = yarn ? std::max(floor(pair_of(sc.fast)), 0.0) : 0.0, hi = yarn ? std::min(ceil(pair_of(sc.slow)), (double)(dims - 1)) : 0.0;
+  const double mag = yarn ? 0.1 * log(sc.factor) + 1.0 : 1.0;
   const int half = dims / 2;
   std::string buf((size_t)max_pos * half * 2 * sizeof(float), '\0');
   float* h = reinterpret_cast<float*>(&buf[0]);
   for (int i = 0; i < half; ++i) {
-    const double f = pow((double)base, -2.0 * (double)i / (double)dims);
+    double f = pow(base, -2.0 * (double)i / (double)dims);
+    if (yarn) {
+      const double ramp = std::min(std::max(((double)i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+      f = f / sc.factor * ramp + f * (1.0 - ramp);
+    }
     for (int p = 0; p < max_pos; ++p) {
       const double ang = (double)p * f;
-      h[((size_t)p * half + i) * 2] = (float)cos(ang);
-      h[((size_t)p * half + i) * 2 + 1] = (float)sin(ang);
+      h[((size_t)p * half + i) * 2] = (float)(cos(ang) * mag);
+      h[((size_t)p * half + i) * 2 + 1] = (float)(sin(ang) * mag);
     }
   }
   NVC_CUDA_CHECK(ctx, cudaMemcpy(out, h, buf.size(), cudaMemcpyHostToDevice));
+  return NVC_OK;
+}
+
+extern "C" int nvc_rotary_table_init_sync(nvc_ctx* ctx, float base, int dims, int max_pos, float* out) {
+  return nvc_rotary_table_init_scaled_sync(ctx, (double)base, dims, nvc_rotary_scaling{0.0, 0.0, 0.0, 0.0}, max_pos, out);
+}
+
+extern "C" int nvc_qk_norm_fold_store(nvc_ctx* ctx, const float* in, int ldi, int q_off, int qw, int k_off, int kw, const float* wqk, float eps,
+                                      const int32_t* positions, float temp_coef, int temp_every, void* q_out, int ldq, void* cache, int ldc,
+                                      float* key_scale, const int32_t* slot_mapping, int dtype, int N, void* stream) {
+  NVC_REQUIRE(ctx, ctx && in && wqk && positions && q_out && cache && key_scale && slot_mapping, NVC_EINVAL, "null pointer");
+  NVC_REQUIRE(ctx, N >= 0 && qw > 0 && kw > 0 && q_off >= 0 && k_off >= 0 && ldi >= q_off + qw && ldi >= k_off + kw && ldq >= qw && ldc >= kw &&
+                       temp_every > 0,
+              NVC_EINVAL, "bad sizes");
+  if (N == 0) return NVC_OK;
+  auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = ((ldi | q_off | qw | k_off | kw | ldq | ldc) & 3) == 0 && al16(in) && al16(wqk) && al16(q_out) && al16(cache);
+  const int units = (qw + kw) / (vec ? 4 : 1);
+  const int threads = units >= 512 ? 256 : (units >= 192 ? 128 : 64);
+  NVC_DISPATCH_DT(dtype, T, {
+    auto kv = qk_norm_fold_store_kernel<T, true>;
+    auto k1 = qk_norm_fold_store_kernel<T, false>;
+    NVC_CUDA_CHECK(ctx, nvc_launch(ctx, vec ? kv : k1, dim3((unsigned)N), dim3((unsigned)threads), 0, nvc_stream(stream), in, ldi, q_off, qw, k_off, kw, wqk,
+                                   eps, positions, temp_coef, temp_every, reinterpret_cast<T*>(q_out), ldq, reinterpret_cast<T*>(cache), ldc, key_scale,
+                                   slot_mapping));
+  });
+  ctx->launches++;
   return NVC_OK;
 }

@@ -514,7 +514,7 @@ class AttnSpecC(C.Structure):
     """nvc_attn_spec of include/nvc_b200.h."""
     _fields_ = [("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("scale", C.c_float), ("window", C.c_int),
                 ("sink", C.c_void_p), ("gate", C.c_void_p), ("ldg", C.c_int), ("out_scale", C.c_float), ("softcap", C.c_float),
-                ("chunk", C.c_int), ("gate_per_head", C.c_int)]
+                ("chunk", C.c_int), ("gate_per_head", C.c_int), ("weights", C.c_int), ("bias", C.c_void_p), ("key_scale", C.c_void_p)]
 
 
 def _a(t: Optional[torch.Tensor]):
@@ -569,12 +569,13 @@ def qkv_prep(ctx, x, q_off, k_off, v_off, q_heads, kv_heads, dim, vdim, q_out, k
 
 def attn_paged_wide(ctx, q, k_cache, v_cache, block_tables, context_lens, cu_seqlens, max_qlen: int, block_size: int, heads: int,
                     kv_heads: int, dim: int, vdim: int, scale: float, window: int = 0, sink=None, gate=None, out_scale: float = 1.0,
-                    softcap: float = 0.0, chunk: int = 0, gate_per_head: bool = False):
-    """q: [rows, heads * dim]; k_cache [slots, kv_heads * dim], v_cache [slots, kv_heads * vdim]; returns [rows, heads * vdim]."""
+                    softcap: float = 0.0, chunk: int = 0, gate_per_head: bool = False, sigmoid: bool = False, bias=None, key_scale=None):
+    """q: [rows, heads * dim]; k_cache [slots, kv_heads * dim], v_cache [slots, kv_heads * vdim]; returns [rows, heads * vdim].
+    sigmoid: weights sigmoid(score + bias[head]) instead of a softmax; key_scale: fp32 [slots], a factor on a key's scores."""
     rows = q.shape[0]
     out = torch.empty(rows, heads * vdim, dtype=q.dtype, device=q.device)
     sp = AttnSpecC(heads, kv_heads, dim, vdim, scale, window, _a(sink), _a(gate), gate.stride(0) if gate is not None else 0, out_scale,
-                   softcap, chunk, 1 if gate_per_head else 0)
+                   softcap, chunk, 1 if gate_per_head else 0, 1 if sigmoid else 0, _a(bias), _a(key_scale))
     check(ctx.l.nvc_attn_paged_wide(ctx.h, _ptr(q), q.stride(0), _ptr(k_cache), k_cache.stride(0), _ptr(v_cache), v_cache.stride(0),
                                     _ptr(block_tables), block_tables.stride(0), _ptr(context_lens), _ptr(cu_seqlens), context_lens.numel(),
                                     rows, max_qlen, block_size, C.byref(sp), _ptr(out), out.stride(0), _dt(q), _stream()),
@@ -785,3 +786,42 @@ def moe_scatter_scaled(ctx, h, pos, w, rows: int):
     check(ctx.l.nvc_moe_scatter_scaled(ctx.h, _ptr(h), _dt(h), h.stride(0), _ptr(pos), _ptr(w), top, _ptr(out), out.stride(0), N, h.shape[1],
                                        _stream()), "nvc_moe_scatter_scaled", ctx.h)
     return out
+
+
+# ---------------------------------------------------------------- sigmoid attention over shared rows, scaled rotary frequencies, capped logits
+def rotary_table_scaled(ctx, base: float, dims: int, scaling: Optional[dict], max_pos: int, device="cuda:0"):
+    """scaling: {"factor", "original", "fast", "slow"} (YaRN) or None."""
+    out = torch.empty(max_pos, dims // 2, 2, dtype=torch.float32, device=device)
+    s = scaling or {"factor": 0.0, "original": 0.0, "fast": 0.0, "slow": 0.0}
+    check(ctx.l.nvc_rotary_table_init_scaled_sync(ctx.h, base, dims, _lib.RotaryScalingC(s["factor"], s["original"], s["fast"], s["slow"]), max_pos,
+                                                  _ptr(out)), "nvc_rotary_table_init_scaled_sync", ctx.h)
+    return out
+
+
+def qk_norm_fold_store(ctx, x, q_off: int, qw: int, k_off: int, kw: int, wqk, eps: float, positions, cache, key_scale, slot_mapping,
+                       temp_coef: float = 0.0, temp_every: int = 1):
+    """x: fp32 [N, ld] rows of the fused projection; returns the queries [N, qw] in the cache's format; the key rows and their factors go
+    to cache[slot], key_scale[slot]."""
+    q = torch.empty(x.shape[0], qw, dtype=cache.dtype, device=x.device)
+    check(ctx.l.nvc_qk_norm_fold_store(ctx.h, _ptr(x), x.stride(0), q_off, qw, k_off, kw, _ptr(wqk), eps, _ptr(positions), temp_coef, temp_every,
+                                       _ptr(q), q.stride(0), _ptr(cache), cache.stride(0), _ptr(key_scale), _ptr(slot_mapping), _dt(cache), x.shape[0],
+                                       _stream()), "nvc_qk_norm_fold_store", ctx.h)
+    return q
+
+
+def prefill_attn_shared(ctx, q, cache, block_tables, context_lens, cu_seqlens, max_qlen: int, block_size: int, heads: int, kv_heads: int,
+                        scale: float, window: int = 0, sink=None, sigmoid: bool = False, bias=None, key_scale=None, gate=None):
+    """Prompt portions on tcgen05; q: bf16 [rows, heads * 128]; cache [slots, kv_heads * 128]: keys and values at once."""
+    out = torch.empty_like(q)
+    sp = AttnSpecC(heads, kv_heads, 128, 128, scale, window, _a(sink), _a(gate), gate.stride(0) if gate is not None else 0, 1.0, 0.0, 0, 0,
+                   1 if sigmoid else 0, _a(bias), _a(key_scale))
+    check(ctx.l.nvc_prefill_attn_shared(ctx.h, _ptr(q), q.stride(0), _ptr(cache), _ptr(block_tables), block_tables.stride(0), _ptr(context_lens),
+                                        _ptr(cu_seqlens), context_lens.numel(), q.shape[0], max_qlen, block_size, cache.shape[0] // block_size,
+                                        C.byref(sp), _ptr(out), out.stride(0), _stream()), "nvc_prefill_attn_shared", ctx.h)
+    return out
+
+
+def softcap_f32(ctx, x, cap: float):
+    """x: fp32 [N, V], capped in place."""
+    check(ctx.l.nvc_softcap_f32(ctx.h, _ptr(x), x.stride(0), cap, x.shape[0], x.shape[1], _stream()), "nvc_softcap_f32", ctx.h)
+    return x
