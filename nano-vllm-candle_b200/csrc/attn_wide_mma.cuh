@@ -230,6 +230,73 @@ __device__ __forceinline__ void softmax_step(uint32_t stK, uint32_t stV, uint32_
   }
 }
 
+// The closing merge of a CTA whose warps hold partial results of the same rows in shared memory - per warp and row the running maximum
+// and sum (sm_m, sm_l: [kWarps][16]) and DVM output numbers (sm_o: [kWarps][16][DVM]); cta_ml: 2 x 16 floats of scratch - and, with
+// splits > 1, of the cluster's CTAs through distributed shared memory.  Row r0 + rr of the sequence is token (r0 + rr) / hg of its portion
+// and head g hg + (r0 + rr) % hg.  Sink, gate and factor are applied on the way out.
+template <int DVM, bool kSig>
+__device__ __forceinline__ void merge_store(const Args& a, const float* sm_m, const float* sm_l, float* cta_ml, float* sm_o, int nrows, int r0, int hg,
+                                            int g, int row_begin) {
+  float* cta_m = cta_ml;
+  float* cta_l = cta_ml + 16;
+  const auto finish = [&](int rr, int d, float M, float L, float O) {     // one output number from the merged partials
+    const int row = r0 + rr, t = row / hg, h = g * hg + row - t * hg;
+    if (a.sink) {
+      const float sk = __ldg(a.sink + h) * kLog2e, M2 = fmaxf(M, sk);
+      const float f = M == -INFINITY ? 0.f : fast_exp2(M - M2);
+      L = L * f + fast_exp2(sk - M2);
+      O *= f;
+    }
+    float y = kSig ? O * a.out_scale : (L > 0.f ? O / L * a.out_scale : 0.f);
+    if (a.gate) y *= sigmoid_f32(a.gate[(int64_t)(row_begin + t) * a.ldg + (a.gate_per_head ? (int64_t)h : (int64_t)h * a.dv + d)]);
+    a.out[(int64_t)(row_begin + t) * a.ldo + (int64_t)h * a.dv + d] = __bfloat16_as_ushort(__float2bfloat16_rn(y));
+  };
+  for (int idx = threadIdx.x; idx < nrows * a.dv; idx += kWarps * 32) {
+    const int rr = idx / a.dv, d = idx - rr * a.dv;
+    float M = -INFINITY, L = 0.f, O = 0.f;
+    if constexpr (!kSig) {
+#pragma unroll
+      for (int w = 0; w < kWarps; ++w) M = fmaxf(M, sm_m[w * 16 + rr]);
+    }
+#pragma unroll
+    for (int w = 0; w < kWarps; ++w) {
+      const float mw = sm_m[w * 16 + rr];
+      const float wt = kSig ? 1.f : (mw == -INFINITY ? 0.f : fast_exp2(mw - M));
+      L += sm_l[w * 16 + rr] * wt;
+      O += sm_o[(w * 16 + rr) * DVM + d] * wt;
+    }
+    if (a.splits == 1) {
+      finish(rr, d, M, L, O);
+    } else {
+      sm_o[rr * DVM + d] = O;                         // warp 0's partial of the same number: this thread alone reads and writes it
+      if (d == 0) { cta_m[rr] = M; cta_l[rr] = L; }
+    }
+  }
+  if (a.splits == 1) return;
+  // ---- merge the CTAs of the cluster: each takes a share of the output numbers and reads the others' partials
+  ptx::cluster_sync_all();
+  const uint32_t rank = ptx::cluster_ctarank();
+  for (int idx = rank * (kWarps * 32) + threadIdx.x; idx < nrows * a.dv; idx += a.splits * kWarps * 32) {
+    const int rr = idx / a.dv, d = idx - rr * a.dv;
+    float M = -INFINITY, L = 0.f, O = 0.f;
+    for (int c = 0; c < a.splits; ++c) {
+      const float oc = ld_cluster_f(ptx::mapa_u32(smem_u32(sm_o + rr * DVM + d), c));
+      if constexpr (kSig) {
+        O += oc;
+      } else {
+        const float mc = ld_cluster_f(ptx::mapa_u32(smem_u32(cta_m + rr), c)), lc = ld_cluster_f(ptx::mapa_u32(smem_u32(cta_l + rr), c));
+        const float Mn = fmaxf(M, mc), Mb = Mn == -INFINITY ? 0.f : Mn;
+        const float f0 = fast_exp2(M - Mb), f1 = fast_exp2(mc - Mb);          // -inf: 0
+        L = L * f0 + lc * f1;
+        O = O * f0 + oc * f1;
+        M = Mn;
+      }
+    }
+    finish(rr, d, M, L, O);
+  }
+  ptx::cluster_sync_all();                            // no CTA leaves while another still reads its partials
+}
+
 template <int DKM, int DVM, bool kSig>
 __global__ void __launch_bounds__(kWarps * 32, 3) attn_wide_mma_kernel(const Args a) {
   constexpr int RBK = DKM * 2, KS = DKM / 16, NT = DVM / 8;
@@ -467,9 +534,8 @@ __global__ void __launch_bounds__(kWarps * 32, 3) attn_wide_mma_kernel(const Arg
   __syncthreads();
   float* sm_m = reinterpret_cast<float*>(smem);       // [kWarps][16]
   float* sm_l = sm_m + kWarps * 16;
-  float* cta_m = sm_l + kWarps * 16;                  // [16], [16]: the CTA's own merge (splits > 1)
-  float* cta_l = cta_m + 16;
-  float* sm_o = cta_l + 16;                           // [kWarps][16][DVM]
+  float* cta_m = sm_l + kWarps * 16;                  // [2][16]: the CTA's own merge (splits > 1)
+  float* sm_o = cta_m + 32;                           // [kWarps][16][DVM]
   if (tq == 0) {
     sm_m[warp * 16 + quad] = m0;
     sm_m[warp * 16 + quad + 8] = m1;
@@ -485,66 +551,12 @@ __global__ void __launch_bounds__(kWarps * 32, 3) attn_wide_mma_kernel(const Arg
     p1[0] = o[nt][2]; p1[1] = o[nt][3];
   }
   __syncthreads();
-  const int nrows = min(16, total - r0);
-  const auto finish = [&](int rr, int d, float M, float L, float O) {     // one output number from the merged partials
-    const int row = r0 + rr, t = row / hg, h = g * hg + row - t * hg;
-    if (a.sink) {
-      const float sk = __ldg(a.sink + h) * kLog2e, M2 = fmaxf(M, sk);
-      const float f = M == -INFINITY ? 0.f : fast_exp2(M - M2);
-      L = L * f + fast_exp2(sk - M2);
-      O *= f;
-    }
-    float y = kSig ? O * a.out_scale : (L > 0.f ? O / L * a.out_scale : 0.f);
-    if (a.gate) y *= sigmoid_f32(a.gate[(int64_t)(row_begin + t) * a.ldg + (a.gate_per_head ? (int64_t)h : (int64_t)h * a.dv + d)]);
-    a.out[(int64_t)(row_begin + t) * a.ldo + (int64_t)h * a.dv + d] = __bfloat16_as_ushort(__float2bfloat16_rn(y));
-  };
-  for (int idx = threadIdx.x; idx < nrows * a.dv; idx += kWarps * 32) {
-    const int rr = idx / a.dv, d = idx - rr * a.dv;
-    float M = -INFINITY, L = 0.f, O = 0.f;
-    if constexpr (!kSig) {
-#pragma unroll
-      for (int w = 0; w < kWarps; ++w) M = fmaxf(M, sm_m[w * 16 + rr]);
-    }
-#pragma unroll
-    for (int w = 0; w < kWarps; ++w) {
-      const float mw = sm_m[w * 16 + rr];
-      const float wt = kSig ? 1.f : (mw == -INFINITY ? 0.f : fast_exp2(mw - M));
-      L += sm_l[w * 16 + rr] * wt;
-      O += sm_o[(w * 16 + rr) * DVM + d] * wt;
-    }
-    if (a.splits == 1) {
-      finish(rr, d, M, L, O);
-    } else {
-      sm_o[rr * DVM + d] = O;                         // warp 0's partial of the same number: this thread alone reads and writes it
-      if (d == 0) { cta_m[rr] = M; cta_l[rr] = L; }
-    }
-  }
-  if (a.splits == 1) return;
-  // ---- merge the CTAs of the cluster: each takes a share of the output numbers and reads the others' partials
-  ptx::cluster_sync_all();
-  const uint32_t rank = ptx::cluster_ctarank();
-  for (int idx = rank * (kWarps * 32) + threadIdx.x; idx < nrows * a.dv; idx += a.splits * kWarps * 32) {
-    const int rr = idx / a.dv, d = idx - rr * a.dv;
-    float M = -INFINITY, L = 0.f, O = 0.f;
-    for (int c = 0; c < a.splits; ++c) {
-      const float oc = ld_cluster_f(ptx::mapa_u32(smem_u32(sm_o + rr * DVM + d), c));
-      if constexpr (kSig) {
-        O += oc;
-      } else {
-        const float mc = ld_cluster_f(ptx::mapa_u32(smem_u32(cta_m + rr), c)), lc = ld_cluster_f(ptx::mapa_u32(smem_u32(cta_l + rr), c));
-        const float Mn = fmaxf(M, mc), Mb = Mn == -INFINITY ? 0.f : Mn;
-        const float f0 = fast_exp2(M - Mb), f1 = fast_exp2(mc - Mb);          // -inf: 0
-        L = L * f0 + lc * f1;
-        O = O * f0 + oc * f1;
-        M = Mn;
-      }
-    }
-    finish(rr, d, M, L, O);
-  }
-  ptx::cluster_sync_all();                            // no CTA leaves while another still reads its partials
+  merge_store<DVM, kSig>(a, sm_m, sm_l, cta_m, sm_o, min(16, total - r0), r0, hg, g, row_begin);
 }
 
 }  // namespace widemma
+
+#include "attn_shared_decode.cuh"
 
 namespace {
 
@@ -598,6 +610,7 @@ inline int attn_wide_mma_launch(nvc_ctx* ctx, const void* q, const void* k_cache
                   s.heads, s.kv_heads, s.dim, s.vdim, s.softcap > 0.f ? s.scale / s.softcap : s.scale * widemma::kLog2e, s.window, s.sink, s.gate, s.ldg,
                   s.out_scale, s.chunk, s.softcap * widemma::kLog2e, s.gate_per_head, s.bias, s.key_scale, shared ? 1 : 0, splits};
   const dim3 grid(gx, B, s.kv_heads);
+  if (attn_shared_decode_takes(a, max_total / hg)) return attn_shared_decode_launch(ctx, a, hg, grid, s.weights == NVC_ATTN_SIGMOID, stream);
   return s.weights == NVC_ATTN_SIGMOID ? attn_wide_mma_launch_s<true>(ctx, a, grid, stream) : attn_wide_mma_launch_s<false>(ctx, a, grid, stream);
 }
 

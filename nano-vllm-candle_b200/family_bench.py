@@ -1,4 +1,4 @@
-"""Karuzen, Ranilix, Fefozen or Batatar beside the closest existing family (Qwen3, dense GQA) at equal layer sizes: prefill and decode throughput
+"""Karuzen, Ranilix, Fefozen, Batatar or Buzutar beside the closest existing family (Qwen3, dense GQA) at equal layer sizes: prefill and decode throughput
 through LLMEngine, plus per-op times and roofline fractions.  Random weights, synthetic prompts.  Used by
 `bench.py --compare-families`; the default benchmark does not touch this module.
 
@@ -459,6 +459,124 @@ def batatar_rooflines(cfg, prof: Dict[str, float], N: int, B: int, ctx_lens: Lis
     return out
 
 
+# ---- Buzutar at the same sizes: four layers - sigmoid attention over shared key / value rows (as many heads as the Qwen3 layer, 8 key
+# heads of 128), windowed latent attention with YaRN frequencies (cache rows of 96 + 32 numbers), a layer that reads the latent layer's
+# rows, sigmoid attention again - with a squared-relu feed-forward of 1.5 ff (two matrices: the gated one's parameter count).
+Z_WINDOW = 256
+
+
+def buzutar_config(sz: dict) -> dict:
+    H, W = sz["heads"], sz["width"]
+    rot = {"dims": F_ROT, "base": 10000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+
+    def latent(kv_from=None):
+        m = {"heads": H, "dim": F_DIM, "rot_dim": F_ROT, "vdim": 128, "kv_rank": F_KV_RANK, "q_rank": Q_RANK, "scale": (F_DIM + F_ROT) ** -0.5,
+             "rot": dict(rot), "mask": {"size": Z_WINDOW}}
+        if kv_from is not None:
+            m["kv_from"] = kv_from
+        return {"type": "latent_attention", "mixer": m}
+
+    att = {"type": "attention", "mixer": {"heads": H, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "q_temp": {"coef": 0.1, "every": 4096}}}
+    kinds = [att, latent(), latent(1), att]
+    mlp = {"kind": "dense", "ff": sz["ff"] * 3 // 2}
+    return {"architecture": "Buzutar", "vocab": sz["vocab"], "width": W, "norm": {"eps": 1e-5}, "embedding": {"scale": W ** 0.5}, "logit_softcap": 30.0,
+            "layers": [dict(kinds[i % 4], mlp=dict(mlp)) for i in range(sz["layers"])]}
+
+
+def buzutar_weights(cfg: dict, seed: int = 0):
+    """(name, bf16 CPU tensor) pairs, generated one at a time."""
+    import torch
+    g = torch.Generator().manual_seed(seed)
+    W = cfg["width"]
+
+    def mat(o, i):
+        return (torch.randn(o, i, generator=g) * i ** -0.5).bfloat16()
+
+    yield "embed", (torch.randn(cfg["vocab"], W, generator=g) * W ** -0.5).bfloat16()
+    yield "head", mat(cfg["vocab"], W)
+    yield "final.norm", torch.ones(W).bfloat16()
+    for i, ly in enumerate(cfg["layers"]):
+        m, p = ly["mixer"], f"l{i}."
+        yield p + "norm1", torch.ones(W).bfloat16()
+        yield p + "norm2", torch.ones(W).bfloat16()
+        H, d = m["heads"], m["dim"]
+        if ly["type"] == "attention":
+            G = m["kv_heads"]
+            yield p + "mix.q", mat(H * d, W)
+            yield p + "mix.k", mat(G * d, W)
+            yield p + "mix.q.norm", torch.ones(H * d).bfloat16()
+            yield p + "mix.k.norm", torch.ones(G * d).bfloat16()
+            yield p + "mix.pb", torch.full((H,), -6.0).bfloat16()
+            yield p + "mix.g", mat(H * d, W)
+            yield p + "mix.o", mat(W, H * d)
+        else:
+            rd, vd, kr, qr = m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
+            yield p + "mix.dq", mat(qr, W)
+            yield p + "mix.dq.norm", torch.ones(qr).bfloat16()
+            yield p + "mix.uq", mat(H * (d + rd), qr)
+            if m.get("kv_from") is None:
+                yield p + "mix.dkv", mat(kr + rd, W)
+                yield p + "mix.dkv.norm", torch.ones(kr).bfloat16()
+            yield p + "mix.uk", mat(H * d, kr)
+            yield p + "mix.uv", mat(H * vd, kr)
+            yield p + "mix.o", mat(W, H * vd)
+        yield p + "mlp.up", mat(ly["mlp"]["ff"], W)
+        yield p + "mlp.down", mat(W, ly["mlp"]["ff"])
+
+
+def buzutar_rooflines(cfg, prof: Dict[str, float], N: int, B: int, ctx_lens: List[int], q_lens: List[int], pk) -> dict:
+    """Per-op roofline of one profiled step: the times are sums over the layers, the work is summed the same way.  A shared key / value row
+    counts once; a window counts its visible pairs only."""
+    W = cfg["width"]
+    names = ("gemm_in", "gemm_uq", "absorb_uk", "attention", "absorb_uv", "sigmoid_attention", "gemm_o", "gemm_up", "gemm_down", "lm_head",
+             "norm", "qk_norm_store", "latent_norm_store", "q_split_rot", "softcap")
+    work = {k: [0.0, 0.0] for k in names}
+
+    def add(name, flops, nbytes):
+        work[name][0] += flops
+        work[name][1] += nbytes
+
+    def visible(window):
+        pairs, keys = 0, 0
+        for q, c in zip(q_lens, ctx_lens):
+            pairs += sum(min(t + 1, window) if window else t + 1 for t in range(c - q, c))
+            keys += min(c, q + window - 1) if window else c
+        return pairs, keys
+
+    for ly in cfg["layers"]:
+        m, ff = ly["mixer"], ly["mlp"]["ff"]
+        H, d = m["heads"], m["dim"]
+        if ly["type"] == "attention":
+            G = m["kv_heads"]
+            n_in, n_o = 2 * H * d + G * d, H * d
+            pairs, keys = visible(0)
+            add("sigmoid_attention", 4.0 * pairs * H * d, 2.0 * (keys * G * d + 2 * N * H * d) + 4.0 * (keys + N * H * d))
+            add("qk_norm_store", 0.0, 6.0 * N * (H + G) * d)
+        else:
+            rd, vd, kr, qr = m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
+            own = m.get("kv_from") is None
+            n_in, n_o = qr + (kr + rd if own else 0), H * vd
+            pairs, keys = visible(m["mask"]["size"])
+            add("gemm_uq", 2.0 * N * H * (d + rd) * qr, 2.0 * (H * (d + rd) * qr + N * qr) + 4.0 * N * H * (d + rd))
+            add("absorb_uk", 2.0 * N * H * d * kr, 2.0 * (H * d * kr + N * H * (d + kr)))
+            add("absorb_uv", 2.0 * N * H * vd * kr, 2.0 * (H * vd * kr + N * H * (kr + vd)))
+            add("attention", 2.0 * pairs * H * (2 * kr + rd), 2.0 * (keys * (kr + rd) + N * H * (2 * kr + rd)))
+            add("latent_norm_store", 0.0, 6.0 * N * n_in)
+            add("q_split_rot", 0.0, 6.0 * N * H * (d + rd))
+        add("gemm_in", 2.0 * N * n_in * W, 2.0 * n_in * W + 2.0 * N * W + 4.0 * N * n_in)
+        add("gemm_o", 2.0 * N * n_o * W, 2.0 * n_o * W + 2.0 * N * n_o + 4.0 * N * W)
+        add("gemm_up", 2.0 * N * ff * W, 2.0 * (ff * W + N * (ff + W)))
+        add("gemm_down", 2.0 * N * ff * W, 2.0 * (ff * W + N * ff) + 4.0 * N * W)
+        add("norm", 0.0, N * W * (2 * (4 + 4 + 4 + 2)))
+    add("lm_head", 2.0 * B * cfg["vocab"] * W, 2.0 * cfg["vocab"] * W + 2.0 * B * W + 4.0 * B * cfg["vocab"])
+    add("softcap", 0.0, 8.0 * B * cfg["vocab"])
+    out = {name: _roof(fl, by, prof[name], pk) for name, (fl, by) in work.items() if name in prof and by > 0}
+    for name in ("embed", "final_norm"):
+        if name in prof:
+            out[name] = {"us": round(prof[name], 2)}
+    return out
+
+
 def _prompts(n, length, vocab, seed):
     rng = np.random.default_rng(seed)
     return [rng.integers(0, vocab, length).tolist() for _ in range(n)]
@@ -539,13 +657,14 @@ def compare(ctx_ours, sizes=None, batch_p=16, batch_d=64, plen=512, K=32, W=4, p
     make_config, make_weights, rooflines = {"karuzen": (karuzen_config, karuzen_weights, karuzen_rooflines),
                                             "ranilix": (ranilix_config, ranilix_weights, ranilix_rooflines),
                                             "fefozen": (fefozen_config, fefozen_weights, fefozen_rooflines),
-                                            "batatar": (batatar_config, batatar_weights, batatar_rooflines)}[family]
+                                            "batatar": (batatar_config, batatar_weights, batatar_rooflines),
+                                            "buzutar": (buzutar_config, buzutar_weights, buzutar_rooflines)}[family]
     T = batch_p * plen
     nblocks = max(batch_p, batch_d) * (-(-(plen + W + K + 24) // BLOCK)) + 8
     results = []
     for sz in sizes or SIZES:
         rec = {"size": sz["name"]}
-        if family == "ranilix" and "moe" in sz:
+        if family in ("ranilix", "buzutar") and "moe" in sz:
             continue                                               # the design has no mixture of experts
         if family == "batatar" and "moe" in sz:
             continue                                               # every size of this family already has experts
