@@ -258,9 +258,9 @@ __global__ void __launch_bounds__(kWarps * 32, 4) attn_shared_decode_kernel(cons
 
 namespace {
 
-// qlen: the longest portion of the launch (1: decode)
-inline bool attn_shared_decode_takes(const widemma::Args& a, int qlen) {
-  return qlen == 1 && !a.cu_seqlens && a.shared && (a.dk == 64 || a.dk == 128) && a.block_size % 16 == 0 && a.cap_log2e == 0.f;
+// without cu_seqlens every sequence has one row
+inline bool attn_shared_decode_takes(const nvc_attn_spec& s, bool shared, const int32_t* cu_seqlens, int block_size) {
+  return !cu_seqlens && shared && (s.dim == 64 || s.dim == 128) && block_size % 16 == 0 && s.softcap == 0.f;
 }
 
 template <int DK, int NR, bool kSig>
@@ -269,6 +269,7 @@ inline int attn_shared_decode_launch_t(nvc_ctx* ctx, const widemma::Args& a, dim
   static bool attr_set = false;
   if (!attr_set) {
     NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(widemma::attn_shared_decode_kernel<DK, NR, kSig>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(widemma::attn_shared_decode_kernel<DK, NR, kSig>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
     attr_set = true;
   }
   NVC_CUDA_CHECK(ctx, nvc_launch_cluster(ctx, widemma::attn_shared_decode_kernel<DK, NR, kSig>, grid, dim3(widemma::kWarps * 32), (size_t)smem, stream,

@@ -1,13 +1,14 @@
 // nvc_attn_paged_wide: grouped-query attention - softmax, or sigmoid weights with a bias per head - over a paged cache whose keys and
-// values have their own widths (dim, vdim), with an optional factor per cached key, an optional sliding window or chunk mask, an optional cap on the scores (cap tanh(s / cap)), an optional sink
-// term in the denominator, an optional sigmoid gate (per output number or per head) and a constant factor on the output.  Rows of
-// sequence b are the LAST q_len positions of its context; row at position i sees keys max(0, i - window + 1) .. i (window), the
-// keys of its own chunk i - i % chunk .. i (chunk), or 0 .. i (neither).
+// values have their own widths (dim, vdim), with an optional factor per cached key, an optional sliding window or chunk mask, an
+// optional cap on the scores (cap tanh(s / cap)), an optional sink term in the denominator, an optional sigmoid gate (per output number
+// or per head) and a constant factor on the output.  Rows of sequence b are the LAST q_len positions of its context; row at position i
+// sees keys max(0, i - window + 1) .. i (window), the keys of its own chunk i - i % chunk .. i (chunk), or 0 .. i (neither).
 //
-// Two kernels:
+// Three kernels:
+//   attn_shared_decode_kernel (attn_shared_decode.cuh)  bf16, one row per sequence, values = leading numbers of 64- or 128-number key rows
 //   attn_wide_mma_kernel (attn_wide_mma.cuh)  bf16 storage, dim and vdim multiples of 16 up to 256: tensor pipe
 //   attn_wide_simt_kernel                      any sizes, both storage formats, plain fp32 FMA: the exact mode
-// Both take the keys of a row in tiles that start at the row's own first visible key, so the order of every sum depends on
+// The last takes the keys of a row in tiles that start at the row's own first visible key, so the order of every sum depends on
 // the row's position alone - not on how the prompt was cut, on the batch or on the pages.
 #include "typed.cuh"
 #include "attn_wide_mma.cuh"

@@ -98,7 +98,8 @@ __device__ __forceinline__ float2 ld_shared_f2(uint32_t addr) {
 // stK / stV: shared-memory addresses of the tile's first key / value row; rows of DKM / DVM numbers, chunks swizzled by row & 7.
 // stS: the tile's key factors (0: none); bias0 / bias1 (log2 domain): the two rows' heads' (kSig).
 template <int DKM, int DVM, int NSUB, bool kSig>
-__device__ __forceinline__ void softmax_step(uint32_t stK, uint32_t stV, uint32_t rbv, uint32_t stS, float bias0, float bias1, int tok0, int nsub, int ks_n, int nt_n, const uint32_t (*qa)[4],
+__device__ __forceinline__ void softmax_step(uint32_t stK, uint32_t stV, uint32_t rbv, uint32_t stS, float bias0, float bias1, int tok0, int nsub,
+                                             int ks_n, int nt_n, const uint32_t (*qa)[4],
                                              float (*o)[4], float& m0, float& m1, float& l0, float& l1, int lo_a, int hi_a, int lo_b, int hi_b,
                                              float scale_log2e, float cap_log2e, bool all_visible, int lane) {
   constexpr int RBK = DKM * 2, KS = DKM / 16, NT = DVM / 8;
@@ -160,54 +161,54 @@ __device__ __forceinline__ void softmax_step(uint32_t stK, uint32_t stV, uint32_
       pa[jn >> 1][2 * (jn & 1) + 1] = pack_bf16(p2, p3);
     }
   } else {
-  if (all_visible) {
+    if (all_visible) {
+#pragma unroll
+      for (int jn = 0; jn < 2 * NSUB; ++jn) {
+        s[jn][0] *= scale_log2e; s[jn][1] *= scale_log2e; s[jn][2] *= scale_log2e; s[jn][3] *= scale_log2e;
+        mx0 = fmaxf(mx0, fmaxf(s[jn][0], s[jn][1]));
+        mx1 = fmaxf(mx1, fmaxf(s[jn][2], s[jn][3]));
+      }
+    } else {
+#pragma unroll
+      for (int jn = 0; jn < 2 * NSUB; ++jn) {
+        const int t0 = tok0 + 8 * jn + 2 * tq;
+        s[jn][0] = (t0 >= lo_a && t0 <= hi_a) ? s[jn][0] * scale_log2e : -INFINITY;
+        s[jn][1] = (t0 + 1 >= lo_a && t0 + 1 <= hi_a) ? s[jn][1] * scale_log2e : -INFINITY;
+        s[jn][2] = (t0 >= lo_b && t0 <= hi_b) ? s[jn][2] * scale_log2e : -INFINITY;
+        s[jn][3] = (t0 + 1 >= lo_b && t0 + 1 <= hi_b) ? s[jn][3] * scale_log2e : -INFINITY;
+        mx0 = fmaxf(mx0, fmaxf(s[jn][0], s[jn][1]));
+        mx1 = fmaxf(mx1, fmaxf(s[jn][2], s[jn][3]));
+      }
+    }
+    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
+    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
+    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+    const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
+    // a row that has seen no key yet keeps m = -inf: subtract 0 instead, every exponential below is then exp2(-inf) = 0
+    const float mb0 = mn0 == -INFINITY ? 0.f : mn0, mb1 = mn1 == -INFINITY ? 0.f : mn1;
+    const float al0 = fast_exp2(m0 - mb0), al1 = fast_exp2(m1 - mb1);
+    m0 = mn0;
+    m1 = mn1;
+    float ps0 = 0.f, ps1 = 0.f;
 #pragma unroll
     for (int jn = 0; jn < 2 * NSUB; ++jn) {
-      s[jn][0] *= scale_log2e; s[jn][1] *= scale_log2e; s[jn][2] *= scale_log2e; s[jn][3] *= scale_log2e;
-      mx0 = fmaxf(mx0, fmaxf(s[jn][0], s[jn][1]));
-      mx1 = fmaxf(mx1, fmaxf(s[jn][2], s[jn][3]));
+      const float p0 = fast_exp2(s[jn][0] - mb0), p1 = fast_exp2(s[jn][1] - mb0);
+      const float p2 = fast_exp2(s[jn][2] - mb1), p3 = fast_exp2(s[jn][3] - mb1);
+      ps0 += p0 + p1;
+      ps1 += p2 + p3;
+      pa[jn >> 1][2 * (jn & 1)] = pack_bf16(p0, p1);
+      pa[jn >> 1][2 * (jn & 1) + 1] = pack_bf16(p2, p3);
     }
-  } else {
+    l0 = l0 * al0 + ps0;
+    l1 = l1 * al1 + ps1;
+    if (__any_sync(0xffffffffu, al0 != 1.f || al1 != 1.f)) {      // a running maximum moved: rare after the first tiles
 #pragma unroll
-    for (int jn = 0; jn < 2 * NSUB; ++jn) {
-      const int t0 = tok0 + 8 * jn + 2 * tq;
-      s[jn][0] = (t0 >= lo_a && t0 <= hi_a) ? s[jn][0] * scale_log2e : -INFINITY;
-      s[jn][1] = (t0 + 1 >= lo_a && t0 + 1 <= hi_a) ? s[jn][1] * scale_log2e : -INFINITY;
-      s[jn][2] = (t0 >= lo_b && t0 <= hi_b) ? s[jn][2] * scale_log2e : -INFINITY;
-      s[jn][3] = (t0 + 1 >= lo_b && t0 + 1 <= hi_b) ? s[jn][3] * scale_log2e : -INFINITY;
-      mx0 = fmaxf(mx0, fmaxf(s[jn][0], s[jn][1]));
-      mx1 = fmaxf(mx1, fmaxf(s[jn][2], s[jn][3]));
+      for (int nt = 0; nt < NT; ++nt) {
+        o[nt][0] *= al0; o[nt][1] *= al0;
+        o[nt][2] *= al1; o[nt][3] *= al1;
+      }
     }
-  }
-  mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
-  mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
-  mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
-  mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-  const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
-  // a row that has seen no key yet keeps m = -inf: subtract 0 instead, every exponential below is then exp2(-inf) = 0
-  const float mb0 = mn0 == -INFINITY ? 0.f : mn0, mb1 = mn1 == -INFINITY ? 0.f : mn1;
-  const float al0 = fast_exp2(m0 - mb0), al1 = fast_exp2(m1 - mb1);
-  m0 = mn0;
-  m1 = mn1;
-  float ps0 = 0.f, ps1 = 0.f;
-#pragma unroll
-  for (int jn = 0; jn < 2 * NSUB; ++jn) {
-    const float p0 = fast_exp2(s[jn][0] - mb0), p1 = fast_exp2(s[jn][1] - mb0);
-    const float p2 = fast_exp2(s[jn][2] - mb1), p3 = fast_exp2(s[jn][3] - mb1);
-    ps0 += p0 + p1;
-    ps1 += p2 + p3;
-    pa[jn >> 1][2 * (jn & 1)] = pack_bf16(p0, p1);
-    pa[jn >> 1][2 * (jn & 1) + 1] = pack_bf16(p2, p3);
-  }
-  l0 = l0 * al0 + ps0;
-  l1 = l1 * al1 + ps1;
-  if (__any_sync(0xffffffffu, al0 != 1.f || al1 != 1.f)) {      // a running maximum moved: rare after the first tiles
-#pragma unroll
-    for (int nt = 0; nt < NT; ++nt) {
-      o[nt][0] *= al0; o[nt][1] *= al0;
-      o[nt][2] *= al1; o[nt][3] *= al1;
-    }
-  }
   }
   {
     const int r = (lane & 7) + (((lane >> 3) & 1) << 3);
@@ -451,8 +452,8 @@ __global__ void __launch_bounds__(kWarps * 32, 3) attn_wide_mma_kernel(const Arg
       const uint32_t st = ring + (i % kStages) * kTileBytes;
       const int nsub = min(kCtaTok / 16, (kmax_w - tok0) / 16 + 1);
       const bool all_visible = tok0 >= lo_last && tok0 + kCtaTok - 1 <= first_w;     // (rows past the end have q = 0: finite, never stored)
-      softmax_step<DKM, DVM, kCtaTok / 16, kSig>(st, st + kTileK, RBV, a.key_scale ? st + kCtaTok * row_bytes : 0u, bias0, bias1, tok0, nsub, ks_n, nt_n, qa, o, m0, m1, l0, l1, lo_a, hi_a, lo_b, hi_b, a.scale_log2e,
-                                           a.cap_log2e, all_visible, lane);
+      softmax_step<DKM, DVM, kCtaTok / 16, kSig>(st, st + kTileK, RBV, a.key_scale ? st + kCtaTok * row_bytes : 0u, bias0, bias1, tok0, nsub, ks_n,
+                                                 nt_n, qa, o, m0, m1, l0, l1, lo_a, hi_a, lo_b, hi_b, a.scale_log2e, a.cap_log2e, all_visible, lane);
     }
     cp_async_wait<0>();
   } else {
@@ -483,8 +484,8 @@ __global__ void __launch_bounds__(kWarps * 32, 3) attn_wide_mma_kernel(const Arg
       __syncwarp();
       const uint32_t st = ring + (i % kStages) * kWarpStage;
       const int tok0 = first + i * stride;
-      softmax_step<DKM, DVM, 1, kSig>(st, st + off_v, RBV, a.key_scale ? st + off_s : 0u, bias0, bias1, tok0, 1, ks_n, nt_n, qa, o, m0, m1, l0, l1, lo_a, hi_a, lo_b, hi_b, a.scale_log2e,
-                                a.cap_log2e, tok0 >= lo_last && tok0 + 15 <= hi_first, lane);
+      softmax_step<DKM, DVM, 1, kSig>(st, st + off_v, RBV, a.key_scale ? st + off_s : 0u, bias0, bias1, tok0, 1, ks_n, nt_n, qa, o, m0, m1, l0, l1,
+                                      lo_a, hi_a, lo_b, hi_b, a.scale_log2e, a.cap_log2e, tok0 >= lo_last && tok0 + 15 <= hi_first, lane);
       __syncwarp();
     }
     cp_async_wait<0>();
@@ -598,11 +599,13 @@ inline int attn_wide_mma_launch(nvc_ctx* ctx, const void* q, const void* k_cache
   int gx = max_total >= 64 ? std::max((max_total + 63) / 64, 4) : (max_total + 15) / 16;
   if (s.kv_heads > 65535 || B > 65535) return NVC_ENOTIMPL;
   const bool shared = k_cache == v_cache && ldk == ldv && s.vdim <= s.dim && (s.kv_heads == 1 || s.vdim == s.dim);
-  // few rows and few CTAs: clusters of up to 8 share the keys of a chunk, as long as a CTA keeps at least 128 of them
+  // few rows and few CTAs: clusters of up to 8 (16 for decode over shared rows) share the keys of a chunk, as long as a CTA keeps at least
+  // 128 of them
   int splits = 1;
+  const int max_splits = attn_shared_decode_takes(s, shared, cu_seqlens, block_size) ? 16 : 8;
   if (max_total < 64) {
     const int64_t keys = s.window > 0 ? s.window : (s.chunk > 0 ? s.chunk : (int64_t)bt_stride * block_size);
-    while (splits < 8 && (int64_t)gx * B * s.kv_heads * splits * 2 <= 3 * ctx->num_sms && keys >= 256 * splits) splits *= 2;
+    while (splits < max_splits && (int64_t)gx * B * s.kv_heads * splits * 2 <= 3 * ctx->num_sms && keys >= 256 * splits) splits *= 2;
     gx *= splits;
   }
   widemma::Args a{reinterpret_cast<const nvc_bf16*>(q), reinterpret_cast<const nvc_bf16*>(k_cache), reinterpret_cast<const nvc_bf16*>(v_cache),
@@ -610,7 +613,7 @@ inline int attn_wide_mma_launch(nvc_ctx* ctx, const void* q, const void* k_cache
                   s.heads, s.kv_heads, s.dim, s.vdim, s.softcap > 0.f ? s.scale / s.softcap : s.scale * widemma::kLog2e, s.window, s.sink, s.gate, s.ldg,
                   s.out_scale, s.chunk, s.softcap * widemma::kLog2e, s.gate_per_head, s.bias, s.key_scale, shared ? 1 : 0, splits};
   const dim3 grid(gx, B, s.kv_heads);
-  if (attn_shared_decode_takes(a, max_total / hg)) return attn_shared_decode_launch(ctx, a, hg, grid, s.weights == NVC_ATTN_SIGMOID, stream);
+  if (attn_shared_decode_takes(s, shared, cu_seqlens, block_size)) return attn_shared_decode_launch(ctx, a, hg, grid, s.weights == NVC_ATTN_SIGMOID, stream);
   return s.weights == NVC_ATTN_SIGMOID ? attn_wide_mma_launch_s<true>(ctx, a, grid, stream) : attn_wide_mma_launch_s<false>(ctx, a, grid, stream);
 }
 

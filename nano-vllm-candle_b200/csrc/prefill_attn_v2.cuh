@@ -189,249 +189,249 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
             ptx::tma_load_3d(dst + kHalfKV + o, map, bar, 64, kvh, slot);
           }
         } else {
-          ptx::mbar_arrive_expect_tx(bar, kKBytes);
-          const int row = ge.seq_start + j * kKT;
-          ptx::tma_load_3d(dst, map, bar, 0, kvh, row);
-          ptx::tma_load_3d(dst + kHalfKV, map, bar, 64, kvh, row);
-        }
-      }
-      __syncwarp();
-    };
-    // shared tiles: boxes of box_rows cache rows (keys and values at once) and the rows' factors, one barrier per tile
-    auto load_shared = [&](const Item& x, const Geo& ge, int j, uint32_t g) {
-      const int s = (int)(g % kKV);
-      ptx::mbar_wait(kv_empty(s), ((g / kKV) & 1) ^ 1u);
-      if (ptx::elect_one()) {
-        const uint32_t dst = base + kOffK + s * kKBytes, bar = kv_full(s);
-        const int rows = pk.box_rows, tok0 = (ge.j0 + j) * kKT;
-        const int nbox = min(kKT / rows, (ge.kv_len - tok0 + rows - 1) / rows);
-        const bool factors = kMode == kSigmoid && pk.key_scale != nullptr;
-        ptx::mbar_arrive_expect_tx(bar, (uint32_t)(nbox * rows * (factors ? 260 : 256)));
-        const int32_t* bt = pk.block_tables + (int64_t)x.b * pk.bt_stride;
-        for (int i = 0; i < nbox; ++i) {
-          const int tok = tok0 + i * rows;
-          const int slot = __ldg(bt + tok / pk.block_size) * pk.block_size + tok % pk.block_size;
-          const uint32_t o = (uint32_t)(i * rows * 128);
-          ptx::tma_load_3d(dst + o, &tma_k, bar, 0, x.kvh, slot);
-          ptx::tma_load_3d(dst + kHalfKV + o, &tma_k, bar, 64, x.kvh, slot);
-          if (factors) ptx::bulk_load(base + kOffScale + s * (kKT * 4) + i * rows * 4, pk.key_scale + slot, (uint32_t)(rows * 4), bar);
-        }
-      }
-      __syncwarp();
-    };
-    uint32_t g = 0, n_done = 0;
-    Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
-    Geo gn = geo_of(xn);
-    for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
-      const Item x = xn;
-      const Geo ge = gn;
-      if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
-        xn = item_of(it + gridDim.x, sc);
-        gn = geo_of(xn);
-      }
-      if (ge.n_tiles == 0) continue;
-      // Q: the previous item's last S MMA has read it (first item: the barrier is fresh, the wait falls through)
-      ptx::mbar_wait(q_empty, (n_done & 1) ^ 1u);
-      if (ptx::elect_one()) {
-        ptx::mbar_arrive_expect_tx(q_full, kQBytes);
-        ptx::tma_load_3d(base + kOffQ, &tma_q, q_full, 0, x.h, ge.seq_start + x.qt * 128);
-        ptx::tma_load_3d(base + kOffQ + 16384, &tma_q, q_full, 64, x.h, ge.seq_start + x.qt * 128);
-      }
-      __syncwarp();
-      if constexpr (kMode == kPlain) {
-        load_kv(x, ge, 0, g, false);
-        for (int j = 0; j < ge.n_tiles; ++j) {
-          if (j + 1 < ge.n_tiles) load_kv(x, ge, j + 1, g + j + 1, false);   // K runs one tile ahead of V, as S runs ahead of P V
-          load_kv(x, ge, j, g + j, true);
-        }
-      } else {
-        for (int j = 0; j < ge.n_tiles; ++j) load_shared(x, ge, j, g + j);
-      }
-      g += ge.n_tiles;
-      ++n_done;
-    }
-  } else if (warp == 1) {
-    // ------------------------------------------------------------ MMA issuer (whole warp loops, one lane issues)
-    constexpr uint32_t idesc_qk = ptx::umma_idesc_bf16(128, kKT, 0, 0);
-    constexpr uint32_t idesc_pv = ptx::umma_idesc_bf16(128, 128, 0, 1);   // B = V is MN-major
-    constexpr uint32_t hi_k = ptx::umma_desc_hi_sw128(1024);
-    const uint32_t q_lo = ptx::umma_desc_lo(base + kOffQ, 16);
-    // S(g) = Q K^T into S buffer g & 1 : 8 k-steps of 16 over head_dim (two 64-wide swizzled halves).  The buffer last
-    // held S / P of tile g - 2, whose P V MMA was issued earlier by this thread: tcgen05.mma executes in issue order.
-    auto issue_s = [&](uint32_t g, bool last_of_item) {
-      constexpr int kStagesS = kMode == kPlain ? kKStages : kKV;
-      const int s = (int)(g % kStagesS);
-      ptx::mbar_wait(kMode == kPlain ? k_full(s) : kv_full(s), (g / kStagesS) & 1);
-      ptx::tcgen05_fence_after();
-      if (ptx::elect_one()) {
-        const uint32_t k_lo = ptx::umma_desc_lo(base + kOffK + s * kKBytes, 16);
-#pragma unroll
-        for (int ks = 0; ks < 8; ++ks) {
-          const uint32_t qoff = ((ks >> 2) * 16384 + (ks & 3) * 32) >> 4;
-          const uint32_t koff = ((ks >> 2) * kHalfKV + (ks & 3) * 32) >> 4;
-          ptx::umma_bf16_ss(tmem_s + (g & 1) * kKT, ptx::umma_desc(q_lo + qoff, hi_k), ptx::umma_desc(k_lo + koff, hi_k), idesc_qk,
-                            ks != 0);
-        }
-        ptx::umma_commit(s_full(g & 1));
-        if (kMode == kPlain) ptx::umma_commit(k_empty(s));          // the K slot is free as soon as these MMAs have read it
-        if (last_of_item) ptx::umma_commit(q_empty);   // ... and so is Q after the item's last S
-      }
-      __syncwarp();
-    };
-    uint32_t g = 0, n_done = 0;
-    Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
-    Geo gn = geo_of(xn);
-    for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
-      const Item x = xn;
-      const Geo ge = gn;
-      if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
-        xn = item_of(it + gridDim.x, sc);
-        gn = geo_of(xn);
-      }
-      if (ge.n_tiles == 0) continue;
-      const int n = ge.n_tiles;
-      ptx::mbar_wait(q_full, n_done & 1);
-      issue_s(g, n == 1);
-      for (int j = 0; j < n; ++j) {
-        // S is double-buffered: S(j+1) is computed while the softmax threads work on S(j)
-        if (j + 1 < n) issue_s(g + j + 1, j + 2 == n);
-        // P(j) is in tensor memory, O has been rescaled for tile j (both by the softmax threads)
-        ptx::mbar_wait(p_full(g + j), p_phase(g + j));
-        const int vs = (int)((g + j) % (kMode == kPlain ? kVStages : kKV));
-        if (kMode == kPlain) ptx::mbar_wait(v_full(vs), ((g + j) / kVStages) & 1);     // shared: S has read the same tile
-        // the first P V of an item overwrites O: the previous item's output rows have been read out of it
-        if (j == 0 && n_done > 0) ptx::mbar_wait(o_free, (n_done - 1) & 1);
-        ptx::tcgen05_fence_after();
-        if (ptx::elect_one()) {
-          // O += P V_j: A = P from tensor memory (8 columns per 16 kv tokens); B = V (MN-major: LBO = 8 KB between the
-          // two 64-wide head-dim halves, SBO = 1 KB between groups of 8 token rows, 16 token rows = 2048 bytes per step)
-          const uint32_t v_lo = ptx::umma_desc_lo(base + (kMode == kPlain ? kOffV : kOffK) + vs * kKBytes, (uint32_t)kHalfKV);
-#pragma unroll
-          for (int ks = 0; ks < kKT / 16; ++ks)
-            ptx::umma_bf16_ts(tmem_o, tmem_s + ((g + j) & 1) * kKT + ks * 8, ptx::umma_desc(v_lo + ks * (2048 >> 4), hi_k),
-                              idesc_pv, (j | ks) != 0);
-          // sigmoid: nobody looks at O before the item's last tile, whose barrier phase counts items
-          if (kMode != kSigmoid || j + 1 == n) ptx::umma_commit(o_full);
-          ptx::umma_commit(kMode == kPlain ? v_empty(vs) : kv_empty(vs));
+            ptx::mbar_arrive_expect_tx(bar, kKBytes);
+            const int row = ge.seq_start + j * kKT;
+            ptx::tma_load_3d(dst, map, bar, 0, kvh, row);
+            ptx::tma_load_3d(dst + kHalfKV, map, bar, 64, kvh, row);
+          }
         }
         __syncwarp();
-      }
-      g += n;
-      ++n_done;
-    }
-  } else {
-    // ------------------------------------------------------------ softmax / correction / output warps
-    const int quad = warp & 3;
-    const int r = quad * 32 + lane;                 // row in the q tile
-    const uint32_t lane_addr = (uint32_t)(quad * 32) << 16;
-    uint32_t g = 0, n_done = 0;
-    Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
-    Geo gn = geo_of(xn);
-    for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
-      const Item x = xn;
-      const Geo ge = gn;
-      if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
-        xn = item_of(it + gridDim.x, sc);
-        gn = geo_of(xn);
-      }
-      if (ge.n_tiles == 0) continue;
-      const int n = ge.n_tiles;
-      const float bias = kMode == kSigmoid && pk.bias ? __ldg(pk.bias + x.h) * 1.4426950408889634f : 0.f;
-      // with a window a row's first tiles may hold none of its keys: a finite floor keeps every difference of maxima defined
-      float m = kMode == kShared ? -1e30f : -INFINITY, l = 0.f;                 // m: the maximum the exponentials are taken against (may lag the true one)
-      for (int j = 0; j < n; ++j) {
-        const uint32_t gi = g + j;
-        const uint32_t s_addr = tmem_s + (gi & 1) * kKT + lane_addr;
-        ptx::mbar_wait(s_full(gi & 1), (gi >> 1) & 1);
-        ptx::tcgen05_fence_after();
-        uint32_t sv[kKT];
-        ptx::tmem_ld_32x32b_x32(s_addr, sv);
-        ptx::tmem_ld_32x32b_x32(s_addr + 32, sv + 32);
-        ptx::tmem_ld_wait();
-        // diagonal tiles only (the tile holds keys past some row's position): columns past this row's position
-        // become -inf, i.e. p = exp2(-inf) = 0; every other tile takes the mask-free path below
-        const int t0 = (ge.j0 + j) * kKT;                  // the tile's first key position
-        uint32_t pk2[kKT / 2];
-        bool move = false;
-        float alpha = 1.0f;
-        if constexpr (kMode == kSigmoid) {
-          if (pk.key_scale) {
-            ptx::mbar_wait(kv_full((int)(gi % kKV)), (gi / kKV) & 1);      // long complete (S was made of this tile): orders the reads below
-            const float4* f = reinterpret_cast<const float4*>(gen + kOffScale + (gi % kKV) * (kKT * 4));
-#pragma unroll
-            for (int i = 0; i < kKT; i += 4) {
-              const float4 v = f[i >> 2];
-              sv[i] = __float_as_uint(__uint_as_float(sv[i]) * v.x);
-              sv[i + 1] = __float_as_uint(__uint_as_float(sv[i + 1]) * v.y);
-              sv[i + 2] = __float_as_uint(__uint_as_float(sv[i + 2]) * v.z);
-              sv[i + 3] = __float_as_uint(__uint_as_float(sv[i + 3]) * v.w);
-            }
+      };
+      // shared tiles: boxes of box_rows cache rows (keys and values at once) and the rows' factors, one barrier per tile
+      auto load_shared = [&](const Item& x, const Geo& ge, int j, uint32_t g) {
+        const int s = (int)(g % kKV);
+        ptx::mbar_wait(kv_empty(s), ((g / kKV) & 1) ^ 1u);
+        if (ptx::elect_one()) {
+          const uint32_t dst = base + kOffK + s * kKBytes, bar = kv_full(s);
+          const int rows = pk.box_rows, tok0 = (ge.j0 + j) * kKT;
+          const int nbox = min(kKT / rows, (ge.kv_len - tok0 + rows - 1) / rows);
+          const bool factors = kMode == kSigmoid && pk.key_scale != nullptr;
+          ptx::mbar_arrive_expect_tx(bar, (uint32_t)(nbox * rows * (factors ? 260 : 256)));
+          const int32_t* bt = pk.block_tables + (int64_t)x.b * pk.bt_stride;
+          for (int i = 0; i < nbox; ++i) {
+            const int tok = tok0 + i * rows;
+            const int slot = __ldg(bt + tok / pk.block_size) * pk.block_size + tok % pk.block_size;
+            const uint32_t o = (uint32_t)(i * rows * 128);
+            ptx::tma_load_3d(dst + o, &tma_k, bar, 0, x.kvh, slot);
+            ptx::tma_load_3d(dst + kHalfKV + o, &tma_k, bar, 64, x.kvh, slot);
+            if (factors) ptx::bulk_load(base + kOffScale + s * (kKT * 4) + i * rows * 4, pk.key_scale + slot, (uint32_t)(rows * 4), bar);
           }
-          // e = 2^-(x log2e) for 64 keys, then p = 1 / (1 + e)
-#pragma unroll
-          for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fast_exp2(fmaf(__uint_as_float(sv[i]), -scale_log2e, -bias)));
-#pragma unroll
-          for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fast_rcp(1.0f + __uint_as_float(sv[i])));
-          if (t0 + kKT - 1 > ge.q0) {
-            const int lim = ge.q0 + r - t0;
-#pragma unroll
-            for (int i = 0; i < kKT; ++i)
-              if (i > lim) sv[i] = 0u;
+        }
+        __syncwarp();
+      };
+      uint32_t g = 0, n_done = 0;
+      Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
+      Geo gn = geo_of(xn);
+      for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
+        const Item x = xn;
+        const Geo ge = gn;
+        if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
+          xn = item_of(it + gridDim.x, sc);
+          gn = geo_of(xn);
+        }
+        if (ge.n_tiles == 0) continue;
+        // Q: the previous item's last S MMA has read it (first item: the barrier is fresh, the wait falls through)
+        ptx::mbar_wait(q_empty, (n_done & 1) ^ 1u);
+        if (ptx::elect_one()) {
+          ptx::mbar_arrive_expect_tx(q_full, kQBytes);
+          ptx::tma_load_3d(base + kOffQ, &tma_q, q_full, 0, x.h, ge.seq_start + x.qt * 128);
+          ptx::tma_load_3d(base + kOffQ + 16384, &tma_q, q_full, 64, x.h, ge.seq_start + x.qt * 128);
+        }
+        __syncwarp();
+        if constexpr (kMode == kPlain) {
+          load_kv(x, ge, 0, g, false);
+          for (int j = 0; j < ge.n_tiles; ++j) {
+            if (j + 1 < ge.n_tiles) load_kv(x, ge, j + 1, g + j + 1, false);   // K runs one tile ahead of V, as S runs ahead of P V
+            load_kv(x, ge, j, g + j, true);
           }
-          if (pk.window > 0 && t0 <= ge.q0 + 127 - pk.window) {
-            const int first = ge.q0 + r - pk.window + 1 - t0;
-#pragma unroll
-            for (int i = 0; i < kKT; ++i)
-              if (i < first) sv[i] = 0u;
-          }
-#pragma unroll
-          for (int i = 0; i < kKT; i += 2) pk2[i >> 1] = pack_bf16(__uint_as_float(sv[i]), __uint_as_float(sv[i + 1]));
         } else {
-        if (t0 + kKT - 1 > ge.q0) {
-          const int lim = ge.q0 + r - t0;                 // last visible column of this row
-#pragma unroll
-          for (int i = 0; i < kKT; ++i)
-            if (i > lim) sv[i] = 0xff800000u;
+          for (int j = 0; j < ge.n_tiles; ++j) load_shared(x, ge, j, g + j);
         }
-        if (kMode == kShared && pk.window > 0 && t0 <= ge.q0 + 127 - pk.window) {
-          const int first = ge.q0 + r - pk.window + 1 - t0;      // first visible column of this row
+        g += ge.n_tiles;
+        ++n_done;
+      }
+    } else if (warp == 1) {
+      // ------------------------------------------------------------ MMA issuer (whole warp loops, one lane issues)
+      constexpr uint32_t idesc_qk = ptx::umma_idesc_bf16(128, kKT, 0, 0);
+      constexpr uint32_t idesc_pv = ptx::umma_idesc_bf16(128, 128, 0, 1);   // B = V is MN-major
+      constexpr uint32_t hi_k = ptx::umma_desc_hi_sw128(1024);
+      const uint32_t q_lo = ptx::umma_desc_lo(base + kOffQ, 16);
+      // S(g) = Q K^T into S buffer g & 1 : 8 k-steps of 16 over head_dim (two 64-wide swizzled halves).  The buffer last
+      // held S / P of tile g - 2, whose P V MMA was issued earlier by this thread: tcgen05.mma executes in issue order.
+      auto issue_s = [&](uint32_t g, bool last_of_item) {
+        constexpr int kStagesS = kMode == kPlain ? kKStages : kKV;
+        const int s = (int)(g % kStagesS);
+        ptx::mbar_wait(kMode == kPlain ? k_full(s) : kv_full(s), (g / kStagesS) & 1);
+        ptx::tcgen05_fence_after();
+        if (ptx::elect_one()) {
+          const uint32_t k_lo = ptx::umma_desc_lo(base + kOffK + s * kKBytes, 16);
 #pragma unroll
-          for (int i = 0; i < kKT; ++i)
-            if (i < first) sv[i] = 0xff800000u;
+          for (int ks = 0; ks < 8; ++ks) {
+            const uint32_t qoff = ((ks >> 2) * 16384 + (ks & 3) * 32) >> 4;
+            const uint32_t koff = ((ks >> 2) * kHalfKV + (ks & 3) * 32) >> 4;
+            ptx::umma_bf16_ss(tmem_s + (g & 1) * kKT, ptx::umma_desc(q_lo + qoff, hi_k), ptx::umma_desc(k_lo + koff, hi_k), idesc_qk,
+                              ks != 0);
+          }
+          ptx::umma_commit(s_full(g & 1));
+          if (kMode == kPlain) ptx::umma_commit(k_empty(s));          // the K slot is free as soon as these MMAs have read it
+          if (last_of_item) ptx::umma_commit(q_empty);   // ... and so is Q after the item's last S
         }
-        // row maximum over four independent chains
-        float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
-#pragma unroll
-        for (int i = 0; i < kKT; i += 4) {
-          mx0 = fmaxf(mx0, __uint_as_float(sv[i]));
-          mx1 = fmaxf(mx1, __uint_as_float(sv[i + 1]));
-          mx2 = fmaxf(mx2, __uint_as_float(sv[i + 2]));
-          mx3 = fmaxf(mx3, __uint_as_float(sv[i + 3]));
+        __syncwarp();
+      };
+      uint32_t g = 0, n_done = 0;
+      Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
+      Geo gn = geo_of(xn);
+      for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
+        const Item x = xn;
+        const Geo ge = gn;
+        if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
+          xn = item_of(it + gridDim.x, sc);
+          gn = geo_of(xn);
         }
-        const float mt = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * scale_log2e;   // finite on tile 0: key 0 is visible to every row
-        // lazy rescale: move the reference maximum (and pay the O round trip) only when some row of this warp outgrew it
-        // by more than 2^kRescaleLog2; m = -inf on the first tile, so that one always moves
-        move = __any_sync(0xffffffffu, mt > m + kRescaleLog2);
-        if (move) {
-          const float m_new = fmaxf(m, mt);
-          alpha = fast_exp2(m - m_new);
-          m = m_new;
+        if (ge.n_tiles == 0) continue;
+        const int n = ge.n_tiles;
+        ptx::mbar_wait(q_full, n_done & 1);
+        issue_s(g, n == 1);
+        for (int j = 0; j < n; ++j) {
+          // S is double-buffered: S(j+1) is computed while the softmax threads work on S(j)
+          if (j + 1 < n) issue_s(g + j + 1, j + 2 == n);
+          // P(j) is in tensor memory, O has been rescaled for tile j (both by the softmax threads)
+          ptx::mbar_wait(p_full(g + j), p_phase(g + j));
+          const int vs = (int)((g + j) % (kMode == kPlain ? kVStages : kKV));
+          if (kMode == kPlain) ptx::mbar_wait(v_full(vs), ((g + j) / kVStages) & 1);     // shared: S has read the same tile
+          // the first P V of an item overwrites O: the previous item's output rows have been read out of it
+          if (j == 0 && n_done > 0) ptx::mbar_wait(o_free, (n_done - 1) & 1);
+          ptx::tcgen05_fence_after();
+          if (ptx::elect_one()) {
+            // O += P V_j: A = P from tensor memory (8 columns per 16 kv tokens); B = V (MN-major: LBO = 8 KB between the
+            // two 64-wide head-dim halves, SBO = 1 KB between groups of 8 token rows, 16 token rows = 2048 bytes per step)
+            const uint32_t v_lo = ptx::umma_desc_lo(base + (kMode == kPlain ? kOffV : kOffK) + vs * kKBytes, (uint32_t)kHalfKV);
+#pragma unroll
+            for (int ks = 0; ks < kKT / 16; ++ks)
+              ptx::umma_bf16_ts(tmem_o, tmem_s + ((g + j) & 1) * kKT + ks * 8, ptx::umma_desc(v_lo + ks * (2048 >> 4), hi_k),
+                                idesc_pv, (j | ks) != 0);
+            // sigmoid: nobody looks at O before the item's last tile, whose barrier phase counts items
+            if (kMode != kSigmoid || j + 1 == n) ptx::umma_commit(o_full);
+            ptx::umma_commit(kMode == kPlain ? v_empty(vs) : kv_empty(vs));
+          }
+          __syncwarp();
         }
-        // exponentials: 64 independent FFMA, then 64 independent MUFU, in place
-#pragma unroll
-        for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fmaf(__uint_as_float(sv[i]), scale_log2e, -m));
-#pragma unroll
-        for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fast_exp2(__uint_as_float(sv[i])));
-        float ps0 = 0.f, ps1 = 0.f, ps2 = 0.f, ps3 = 0.f;
-#pragma unroll
-        for (int i = 0; i < kKT; i += 4) {
-          const float p0 = __uint_as_float(sv[i]), p1 = __uint_as_float(sv[i + 1]);
-          const float p2 = __uint_as_float(sv[i + 2]), p3 = __uint_as_float(sv[i + 3]);
-          ps0 += p0; ps1 += p1; ps2 += p2; ps3 += p3;
-          pk2[i >> 1] = pack_bf16(p0, p1);
-          pk2[(i >> 1) + 1] = pack_bf16(p2, p3);
+        g += n;
+        ++n_done;
+      }
+    } else {
+      // ------------------------------------------------------------ softmax / correction / output warps
+      const int quad = warp & 3;
+      const int r = quad * 32 + lane;                 // row in the q tile
+      const uint32_t lane_addr = (uint32_t)(quad * 32) << 16;
+      uint32_t g = 0, n_done = 0;
+      Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
+      Geo gn = geo_of(xn);
+      for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
+        const Item x = xn;
+        const Geo ge = gn;
+        if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
+          xn = item_of(it + gridDim.x, sc);
+          gn = geo_of(xn);
         }
-        l = l * alpha + ((ps0 + ps1) + (ps2 + ps3));
+        if (ge.n_tiles == 0) continue;
+        const int n = ge.n_tiles;
+        const float bias = kMode == kSigmoid && pk.bias ? __ldg(pk.bias + x.h) * 1.4426950408889634f : 0.f;
+        // with a window a row's first tiles may hold none of its keys: a finite floor keeps every difference of maxima defined
+        float m = kMode == kShared ? -1e30f : -INFINITY, l = 0.f;                 // m: the maximum the exponentials are taken against (may lag the true one)
+        for (int j = 0; j < n; ++j) {
+          const uint32_t gi = g + j;
+          const uint32_t s_addr = tmem_s + (gi & 1) * kKT + lane_addr;
+          ptx::mbar_wait(s_full(gi & 1), (gi >> 1) & 1);
+          ptx::tcgen05_fence_after();
+          uint32_t sv[kKT];
+          ptx::tmem_ld_32x32b_x32(s_addr, sv);
+          ptx::tmem_ld_32x32b_x32(s_addr + 32, sv + 32);
+          ptx::tmem_ld_wait();
+          // diagonal tiles only (the tile holds keys past some row's position): columns past this row's position
+          // become -inf, i.e. p = exp2(-inf) = 0; every other tile takes the mask-free path below
+          const int t0 = (ge.j0 + j) * kKT;                  // the tile's first key position
+          uint32_t pk2[kKT / 2];
+          bool move = false;
+          float alpha = 1.0f;
+          if constexpr (kMode == kSigmoid) {
+            if (pk.key_scale) {
+              ptx::mbar_wait(kv_full((int)(gi % kKV)), (gi / kKV) & 1);      // long complete (S was made of this tile): orders the reads below
+              const float4* f = reinterpret_cast<const float4*>(gen + kOffScale + (gi % kKV) * (kKT * 4));
+#pragma unroll
+              for (int i = 0; i < kKT; i += 4) {
+                const float4 v = f[i >> 2];
+                sv[i] = __float_as_uint(__uint_as_float(sv[i]) * v.x);
+                sv[i + 1] = __float_as_uint(__uint_as_float(sv[i + 1]) * v.y);
+                sv[i + 2] = __float_as_uint(__uint_as_float(sv[i + 2]) * v.z);
+                sv[i + 3] = __float_as_uint(__uint_as_float(sv[i + 3]) * v.w);
+              }
+            }
+            // e = 2^-(x log2e) for 64 keys, then p = 1 / (1 + e)
+#pragma unroll
+            for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fast_exp2(fmaf(__uint_as_float(sv[i]), -scale_log2e, -bias)));
+#pragma unroll
+            for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fast_rcp(1.0f + __uint_as_float(sv[i])));
+            if (t0 + kKT - 1 > ge.q0) {
+              const int lim = ge.q0 + r - t0;
+#pragma unroll
+              for (int i = 0; i < kKT; ++i)
+                if (i > lim) sv[i] = 0u;
+            }
+            if (pk.window > 0 && t0 <= ge.q0 + 127 - pk.window) {
+              const int first = ge.q0 + r - pk.window + 1 - t0;
+#pragma unroll
+              for (int i = 0; i < kKT; ++i)
+                if (i < first) sv[i] = 0u;
+            }
+#pragma unroll
+            for (int i = 0; i < kKT; i += 2) pk2[i >> 1] = pack_bf16(__uint_as_float(sv[i]), __uint_as_float(sv[i + 1]));
+          } else {
+          if (t0 + kKT - 1 > ge.q0) {
+            const int lim = ge.q0 + r - t0;                 // last visible column of this row
+#pragma unroll
+            for (int i = 0; i < kKT; ++i)
+              if (i > lim) sv[i] = 0xff800000u;
+          }
+          if (kMode == kShared && pk.window > 0 && t0 <= ge.q0 + 127 - pk.window) {
+            const int first = ge.q0 + r - pk.window + 1 - t0;      // first visible column of this row
+#pragma unroll
+            for (int i = 0; i < kKT; ++i)
+              if (i < first) sv[i] = 0xff800000u;
+          }
+          // row maximum over four independent chains
+          float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
+#pragma unroll
+          for (int i = 0; i < kKT; i += 4) {
+            mx0 = fmaxf(mx0, __uint_as_float(sv[i]));
+            mx1 = fmaxf(mx1, __uint_as_float(sv[i + 1]));
+            mx2 = fmaxf(mx2, __uint_as_float(sv[i + 2]));
+            mx3 = fmaxf(mx3, __uint_as_float(sv[i + 3]));
+          }
+          const float mt = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * scale_log2e;   // finite on tile 0: key 0 is visible to every row
+          // lazy rescale: move the reference maximum (and pay the O round trip) only when some row of this warp outgrew it
+          // by more than 2^kRescaleLog2; m = -inf on the first tile, so that one always moves
+          move = __any_sync(0xffffffffu, mt > m + kRescaleLog2);
+          if (move) {
+            const float m_new = fmaxf(m, mt);
+            alpha = fast_exp2(m - m_new);
+            m = m_new;
+          }
+          // exponentials: 64 independent FFMA, then 64 independent MUFU, in place
+#pragma unroll
+          for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fmaf(__uint_as_float(sv[i]), scale_log2e, -m));
+#pragma unroll
+          for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fast_exp2(__uint_as_float(sv[i])));
+          float ps0 = 0.f, ps1 = 0.f, ps2 = 0.f, ps3 = 0.f;
+#pragma unroll
+          for (int i = 0; i < kKT; i += 4) {
+            const float p0 = __uint_as_float(sv[i]), p1 = __uint_as_float(sv[i + 1]);
+            const float p2 = __uint_as_float(sv[i + 2]), p3 = __uint_as_float(sv[i + 3]);
+            ps0 += p0; ps1 += p1; ps2 += p2; ps3 += p3;
+            pk2[i >> 1] = pack_bf16(p0, p1);
+            pk2[(i >> 1) + 1] = pack_bf16(p2, p3);
+          }
+          l = l * alpha + ((ps0 + ps1) + (ps2 + ps3));
         }
         if (kMode != kSigmoid && j > 0) {
           // P V(j-1) has completed: O holds the sum over tiles < j.  Waited for on EVERY tile, moved or not: a parity

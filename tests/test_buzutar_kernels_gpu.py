@@ -241,6 +241,19 @@ def test_windowed_softmax_over_shared_rows(ctx, ops, dt, batch, G, d, vd, window
     assert close(b.wide(ctx, ops, 0.25, window), b.want(0.25, window), dt)
 
 
+@pytest.mark.parametrize("H,G,d,vd,sigmoid", [(16, 1, 128, 96, False), (20, 1, 64, 48, False), (7, 1, 128, 128, False), (40, 2, 64, 64, True),
+                                                (16, 1, 128, 128, True), (9, 3, 64, 64, True), (32, 4, 128, 128, True)])
+@pytest.mark.parametrize("bs,window", [(16, 0), (64, 0), (48, 37), (64, 16), (16, 1)])
+def test_decode_rows_in_the_transposed_form(ctx, ops, H, G, d, vd, sigmoid, bs, window):
+    """Key rows of 64 and 128 numbers, up to 8, up to 16 and more query heads per key head (one or two n-tiles, several CTAs per key head)."""
+    b = Batch(H, G, d, vd, lens=[300, 1, 64, 65, 17, 40, 41, 16, 530], qlens=[1] * 9, bs=bs, dt=torch.bfloat16, seed=H + window, shared=True,
+              scaled=sigmoid, sigmoid=sigmoid, gate=sigmoid)
+    assert close(b.wide(ctx, ops, 0.15, window), b.want(0.15, window), torch.bfloat16)
+    if not sigmoid:
+        sink = torch.linspace(-2, 4, H)
+        assert close(b.wide(ctx, ops, 0.15, window, sink), b.want(0.15, window, sink), torch.bfloat16)
+
+
 @pytest.mark.parametrize("sigmoid,window", [(True, 0), (False, 0), (False, 600), (True, 600)])
 @pytest.mark.parametrize("lens", [[2100], [2047, 3], [1, 1500, 700]])
 def test_decode_keys_split_over_a_cluster(ctx, ops, sigmoid, window, lens):
