@@ -120,8 +120,8 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // geometry of one item (every role derives the same numbers): q row i of the tile is context position q0 + i and sees
-  // n_tiles = 0 marks a q tile past the end of its sequence (skipped by every role)
-  // keys 0 .. q0 + i, or the last `window` of them; j0 = the first kv tile, n_tiles are counted from there
+  // keys 0 .. q0 + i, or the last `window` of them; j0 = the first kv tile, n_tiles are counted from there; n_tiles = 0 marks
+  // a q tile past the end of its sequence (skipped by every role)
   struct Geo { int seq_start, seq_len, kv_len, q0, j0, n_tiles; };
   auto geo_of = [&](const Item& x) {
     Geo g;
@@ -189,204 +189,219 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
             ptx::tma_load_3d(dst + kHalfKV + o, map, bar, 64, kvh, slot);
           }
         } else {
-            ptx::mbar_arrive_expect_tx(bar, kKBytes);
-            const int row = ge.seq_start + j * kKT;
-            ptx::tma_load_3d(dst, map, bar, 0, kvh, row);
-            ptx::tma_load_3d(dst + kHalfKV, map, bar, 64, kvh, row);
-          }
+          ptx::mbar_arrive_expect_tx(bar, kKBytes);
+          const int row = ge.seq_start + j * kKT;
+          ptx::tma_load_3d(dst, map, bar, 0, kvh, row);
+          ptx::tma_load_3d(dst + kHalfKV, map, bar, 64, kvh, row);
         }
-        __syncwarp();
-      };
-      // shared tiles: boxes of box_rows cache rows (keys and values at once) and the rows' factors, one barrier per tile
-      auto load_shared = [&](const Item& x, const Geo& ge, int j, uint32_t g) {
-        const int s = (int)(g % kKV);
-        ptx::mbar_wait(kv_empty(s), ((g / kKV) & 1) ^ 1u);
-        if (ptx::elect_one()) {
-          const uint32_t dst = base + kOffK + s * kKBytes, bar = kv_full(s);
-          const int rows = pk.box_rows, tok0 = (ge.j0 + j) * kKT;
-          const int nbox = min(kKT / rows, (ge.kv_len - tok0 + rows - 1) / rows);
-          const bool factors = kMode == kSigmoid && pk.key_scale != nullptr;
-          ptx::mbar_arrive_expect_tx(bar, (uint32_t)(nbox * rows * (factors ? 260 : 256)));
-          const int32_t* bt = pk.block_tables + (int64_t)x.b * pk.bt_stride;
-          for (int i = 0; i < nbox; ++i) {
-            const int tok = tok0 + i * rows;
-            const int slot = __ldg(bt + tok / pk.block_size) * pk.block_size + tok % pk.block_size;
-            const uint32_t o = (uint32_t)(i * rows * 128);
-            ptx::tma_load_3d(dst + o, &tma_k, bar, 0, x.kvh, slot);
-            ptx::tma_load_3d(dst + kHalfKV + o, &tma_k, bar, 64, x.kvh, slot);
-            if (factors) ptx::bulk_load(base + kOffScale + s * (kKT * 4) + i * rows * 4, pk.key_scale + slot, (uint32_t)(rows * 4), bar);
-          }
-        }
-        __syncwarp();
-      };
-      uint32_t g = 0, n_done = 0;
-      Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
-      Geo gn = geo_of(xn);
-      for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
-        const Item x = xn;
-        const Geo ge = gn;
-        if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
-          xn = item_of(it + gridDim.x, sc);
-          gn = geo_of(xn);
-        }
-        if (ge.n_tiles == 0) continue;
-        // Q: the previous item's last S MMA has read it (first item: the barrier is fresh, the wait falls through)
-        ptx::mbar_wait(q_empty, (n_done & 1) ^ 1u);
-        if (ptx::elect_one()) {
-          ptx::mbar_arrive_expect_tx(q_full, kQBytes);
-          ptx::tma_load_3d(base + kOffQ, &tma_q, q_full, 0, x.h, ge.seq_start + x.qt * 128);
-          ptx::tma_load_3d(base + kOffQ + 16384, &tma_q, q_full, 64, x.h, ge.seq_start + x.qt * 128);
-        }
-        __syncwarp();
-        if constexpr (kMode == kPlain) {
-          load_kv(x, ge, 0, g, false);
-          for (int j = 0; j < ge.n_tiles; ++j) {
-            if (j + 1 < ge.n_tiles) load_kv(x, ge, j + 1, g + j + 1, false);   // K runs one tile ahead of V, as S runs ahead of P V
-            load_kv(x, ge, j, g + j, true);
-          }
-        } else {
-          for (int j = 0; j < ge.n_tiles; ++j) load_shared(x, ge, j, g + j);
-        }
-        g += ge.n_tiles;
-        ++n_done;
       }
-    } else if (warp == 1) {
-      // ------------------------------------------------------------ MMA issuer (whole warp loops, one lane issues)
-      constexpr uint32_t idesc_qk = ptx::umma_idesc_bf16(128, kKT, 0, 0);
-      constexpr uint32_t idesc_pv = ptx::umma_idesc_bf16(128, 128, 0, 1);   // B = V is MN-major
-      constexpr uint32_t hi_k = ptx::umma_desc_hi_sw128(1024);
-      const uint32_t q_lo = ptx::umma_desc_lo(base + kOffQ, 16);
-      // S(g) = Q K^T into S buffer g & 1 : 8 k-steps of 16 over head_dim (two 64-wide swizzled halves).  The buffer last
-      // held S / P of tile g - 2, whose P V MMA was issued earlier by this thread: tcgen05.mma executes in issue order.
-      auto issue_s = [&](uint32_t g, bool last_of_item) {
-        constexpr int kStagesS = kMode == kPlain ? kKStages : kKV;
-        const int s = (int)(g % kStagesS);
-        ptx::mbar_wait(kMode == kPlain ? k_full(s) : kv_full(s), (g / kStagesS) & 1);
+      __syncwarp();
+    };
+    // shared tiles: boxes of box_rows cache rows (keys and values at once) and the rows' factors, one barrier per tile
+    auto load_shared = [&](const Item& x, const Geo& ge, int j, uint32_t g) {
+      const int s = (int)(g % kKV);
+      ptx::mbar_wait(kv_empty(s), ((g / kKV) & 1) ^ 1u);
+      if (ptx::elect_one()) {
+        const uint32_t dst = base + kOffK + s * kKBytes, bar = kv_full(s);
+        const int rows = pk.box_rows, tok0 = (ge.j0 + j) * kKT;
+        const int nbox = min(kKT / rows, (ge.kv_len - tok0 + rows - 1) / rows);
+        const bool factors = kMode == kSigmoid && pk.key_scale != nullptr;
+        ptx::mbar_arrive_expect_tx(bar, (uint32_t)(nbox * rows * (factors ? 260 : 256)));
+        const int32_t* bt = pk.block_tables + (int64_t)x.b * pk.bt_stride;
+        for (int i = 0; i < nbox; ++i) {
+          const int tok = tok0 + i * rows;
+          const int slot = __ldg(bt + tok / pk.block_size) * pk.block_size + tok % pk.block_size;
+          const uint32_t o = (uint32_t)(i * rows * 128);
+          ptx::tma_load_3d(dst + o, &tma_k, bar, 0, x.kvh, slot);
+          ptx::tma_load_3d(dst + kHalfKV + o, &tma_k, bar, 64, x.kvh, slot);
+          if (factors) ptx::bulk_load(base + kOffScale + s * (kKT * 4) + i * rows * 4, pk.key_scale + slot, (uint32_t)(rows * 4), bar);
+        }
+      }
+      __syncwarp();
+    };
+    uint32_t g = 0, n_done = 0;
+    Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
+    Geo gn = geo_of(xn);
+    for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
+      const Item x = xn;
+      const Geo ge = gn;
+      if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
+        xn = item_of(it + gridDim.x, sc);
+        gn = geo_of(xn);
+      }
+      if (ge.n_tiles == 0) continue;
+      // Q: the previous item's last S MMA has read it (first item: the barrier is fresh, the wait falls through)
+      ptx::mbar_wait(q_empty, (n_done & 1) ^ 1u);
+      if (ptx::elect_one()) {
+        ptx::mbar_arrive_expect_tx(q_full, kQBytes);
+        ptx::tma_load_3d(base + kOffQ, &tma_q, q_full, 0, x.h, ge.seq_start + x.qt * 128);
+        ptx::tma_load_3d(base + kOffQ + 16384, &tma_q, q_full, 64, x.h, ge.seq_start + x.qt * 128);
+      }
+      __syncwarp();
+      if constexpr (kMode == kPlain) {
+        load_kv(x, ge, 0, g, false);
+        for (int j = 0; j < ge.n_tiles; ++j) {
+          if (j + 1 < ge.n_tiles) load_kv(x, ge, j + 1, g + j + 1, false);   // K runs one tile ahead of V, as S runs ahead of P V
+          load_kv(x, ge, j, g + j, true);
+        }
+      } else {
+        for (int j = 0; j < ge.n_tiles; ++j) load_shared(x, ge, j, g + j);
+      }
+      g += ge.n_tiles;
+      ++n_done;
+    }
+  } else if (warp == 1) {
+    // ------------------------------------------------------------ MMA issuer (whole warp loops, one lane issues)
+    constexpr uint32_t idesc_qk = ptx::umma_idesc_bf16(128, kKT, 0, 0);
+    constexpr uint32_t idesc_pv = ptx::umma_idesc_bf16(128, 128, 0, 1);   // B = V is MN-major
+    constexpr uint32_t hi_k = ptx::umma_desc_hi_sw128(1024);
+    const uint32_t q_lo = ptx::umma_desc_lo(base + kOffQ, 16);
+    // S(g) = Q K^T into S buffer g & 1 : 8 k-steps of 16 over head_dim (two 64-wide swizzled halves).  The buffer last
+    // held S / P of tile g - 2, whose P V MMA was issued earlier by this thread: tcgen05.mma executes in issue order.
+    auto issue_s = [&](uint32_t g, bool last_of_item) {
+      constexpr int kStagesS = kMode == kPlain ? kKStages : kKV;
+      const int s = (int)(g % kStagesS);
+      ptx::mbar_wait(kMode == kPlain ? k_full(s) : kv_full(s), (g / kStagesS) & 1);
+      ptx::tcgen05_fence_after();
+      if (ptx::elect_one()) {
+        const uint32_t k_lo = ptx::umma_desc_lo(base + kOffK + s * kKBytes, 16);
+#pragma unroll
+        for (int ks = 0; ks < 8; ++ks) {
+          const uint32_t qoff = ((ks >> 2) * 16384 + (ks & 3) * 32) >> 4;
+          const uint32_t koff = ((ks >> 2) * kHalfKV + (ks & 3) * 32) >> 4;
+          ptx::umma_bf16_ss(tmem_s + (g & 1) * kKT, ptx::umma_desc(q_lo + qoff, hi_k), ptx::umma_desc(k_lo + koff, hi_k), idesc_qk,
+                            ks != 0);
+        }
+        ptx::umma_commit(s_full(g & 1));
+        if (kMode == kPlain) ptx::umma_commit(k_empty(s));          // the K slot is free as soon as these MMAs have read it
+        if (last_of_item) ptx::umma_commit(q_empty);   // ... and so is Q after the item's last S
+      }
+      __syncwarp();
+    };
+    uint32_t g = 0, n_done = 0;
+    Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
+    Geo gn = geo_of(xn);
+    for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
+      const Item x = xn;
+      const Geo ge = gn;
+      if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
+        xn = item_of(it + gridDim.x, sc);
+        gn = geo_of(xn);
+      }
+      if (ge.n_tiles == 0) continue;
+      const int n = ge.n_tiles;
+      ptx::mbar_wait(q_full, n_done & 1);
+      issue_s(g, n == 1);
+      for (int j = 0; j < n; ++j) {
+        // S is double-buffered: S(j+1) is computed while the softmax threads work on S(j)
+        if (j + 1 < n) issue_s(g + j + 1, j + 2 == n);
+        // P(j) is in tensor memory, O has been rescaled for tile j (both by the softmax threads)
+        ptx::mbar_wait(p_full(g + j), p_phase(g + j));
+        const int vs = (int)((g + j) % (kMode == kPlain ? kVStages : kKV));
+        if (kMode == kPlain) ptx::mbar_wait(v_full(vs), ((g + j) / kVStages) & 1);     // shared: S has read the same tile
+        // the first P V of an item overwrites O: the previous item's output rows have been read out of it
+        if (j == 0 && n_done > 0) ptx::mbar_wait(o_free, (n_done - 1) & 1);
         ptx::tcgen05_fence_after();
         if (ptx::elect_one()) {
-          const uint32_t k_lo = ptx::umma_desc_lo(base + kOffK + s * kKBytes, 16);
+          // O += P V_j: A = P from tensor memory (8 columns per 16 kv tokens); B = V (MN-major: LBO = 8 KB between the
+          // two 64-wide head-dim halves, SBO = 1 KB between groups of 8 token rows, 16 token rows = 2048 bytes per step)
+          const uint32_t v_lo = ptx::umma_desc_lo(base + (kMode == kPlain ? kOffV : kOffK) + vs * kKBytes, (uint32_t)kHalfKV);
 #pragma unroll
-          for (int ks = 0; ks < 8; ++ks) {
-            const uint32_t qoff = ((ks >> 2) * 16384 + (ks & 3) * 32) >> 4;
-            const uint32_t koff = ((ks >> 2) * kHalfKV + (ks & 3) * 32) >> 4;
-            ptx::umma_bf16_ss(tmem_s + (g & 1) * kKT, ptx::umma_desc(q_lo + qoff, hi_k), ptx::umma_desc(k_lo + koff, hi_k), idesc_qk,
-                              ks != 0);
-          }
-          ptx::umma_commit(s_full(g & 1));
-          if (kMode == kPlain) ptx::umma_commit(k_empty(s));          // the K slot is free as soon as these MMAs have read it
-          if (last_of_item) ptx::umma_commit(q_empty);   // ... and so is Q after the item's last S
+          for (int ks = 0; ks < kKT / 16; ++ks)
+            ptx::umma_bf16_ts(tmem_o, tmem_s + ((g + j) & 1) * kKT + ks * 8, ptx::umma_desc(v_lo + ks * (2048 >> 4), hi_k),
+                              idesc_pv, (j | ks) != 0);
+          // sigmoid: nobody looks at O before the item's last tile, whose barrier phase counts items
+          if (kMode != kSigmoid || j + 1 == n) ptx::umma_commit(o_full);
+          ptx::umma_commit(kMode == kPlain ? v_empty(vs) : kv_empty(vs));
         }
         __syncwarp();
-      };
-      uint32_t g = 0, n_done = 0;
-      Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
-      Geo gn = geo_of(xn);
-      for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
-        const Item x = xn;
-        const Geo ge = gn;
-        if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
-          xn = item_of(it + gridDim.x, sc);
-          gn = geo_of(xn);
-        }
-        if (ge.n_tiles == 0) continue;
-        const int n = ge.n_tiles;
-        ptx::mbar_wait(q_full, n_done & 1);
-        issue_s(g, n == 1);
-        for (int j = 0; j < n; ++j) {
-          // S is double-buffered: S(j+1) is computed while the softmax threads work on S(j)
-          if (j + 1 < n) issue_s(g + j + 1, j + 2 == n);
-          // P(j) is in tensor memory, O has been rescaled for tile j (both by the softmax threads)
-          ptx::mbar_wait(p_full(g + j), p_phase(g + j));
-          const int vs = (int)((g + j) % (kMode == kPlain ? kVStages : kKV));
-          if (kMode == kPlain) ptx::mbar_wait(v_full(vs), ((g + j) / kVStages) & 1);     // shared: S has read the same tile
-          // the first P V of an item overwrites O: the previous item's output rows have been read out of it
-          if (j == 0 && n_done > 0) ptx::mbar_wait(o_free, (n_done - 1) & 1);
-          ptx::tcgen05_fence_after();
-          if (ptx::elect_one()) {
-            // O += P V_j: A = P from tensor memory (8 columns per 16 kv tokens); B = V (MN-major: LBO = 8 KB between the
-            // two 64-wide head-dim halves, SBO = 1 KB between groups of 8 token rows, 16 token rows = 2048 bytes per step)
-            const uint32_t v_lo = ptx::umma_desc_lo(base + (kMode == kPlain ? kOffV : kOffK) + vs * kKBytes, (uint32_t)kHalfKV);
-#pragma unroll
-            for (int ks = 0; ks < kKT / 16; ++ks)
-              ptx::umma_bf16_ts(tmem_o, tmem_s + ((g + j) & 1) * kKT + ks * 8, ptx::umma_desc(v_lo + ks * (2048 >> 4), hi_k),
-                                idesc_pv, (j | ks) != 0);
-            // sigmoid: nobody looks at O before the item's last tile, whose barrier phase counts items
-            if (kMode != kSigmoid || j + 1 == n) ptx::umma_commit(o_full);
-            ptx::umma_commit(kMode == kPlain ? v_empty(vs) : kv_empty(vs));
-          }
-          __syncwarp();
-        }
-        g += n;
-        ++n_done;
       }
-    } else {
-      // ------------------------------------------------------------ softmax / correction / output warps
-      const int quad = warp & 3;
-      const int r = quad * 32 + lane;                 // row in the q tile
-      const uint32_t lane_addr = (uint32_t)(quad * 32) << 16;
-      uint32_t g = 0, n_done = 0;
-      Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
-      Geo gn = geo_of(xn);
-      for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
-        const Item x = xn;
-        const Geo ge = gn;
-        if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
-          xn = item_of(it + gridDim.x, sc);
-          gn = geo_of(xn);
-        }
-        if (ge.n_tiles == 0) continue;
-        const int n = ge.n_tiles;
-        const float bias = kMode == kSigmoid && pk.bias ? __ldg(pk.bias + x.h) * 1.4426950408889634f : 0.f;
-        // with a window a row's first tiles may hold none of its keys: a finite floor keeps every difference of maxima defined
-        float m = kMode == kShared ? -1e30f : -INFINITY, l = 0.f;                 // m: the maximum the exponentials are taken against (may lag the true one)
-        for (int j = 0; j < n; ++j) {
-          const uint32_t gi = g + j;
-          const uint32_t s_addr = tmem_s + (gi & 1) * kKT + lane_addr;
-          ptx::mbar_wait(s_full(gi & 1), (gi >> 1) & 1);
-          ptx::tcgen05_fence_after();
-          uint32_t sv[kKT];
-          ptx::tmem_ld_32x32b_x32(s_addr, sv);
-          ptx::tmem_ld_32x32b_x32(s_addr + 32, sv + 32);
-          ptx::tmem_ld_wait();
+      g += n;
+      ++n_done;
+    }
+  } else {
+    // ------------------------------------------------------------ softmax / correction / output warps
+    const int quad = warp & 3;
+    const int r = quad * 32 + lane;                 // row in the q tile
+    const uint32_t lane_addr = (uint32_t)(quad * 32) << 16;
+    uint32_t g = 0, n_done = 0;
+    Item xn = item_of(blockIdx.x, sc);               // gridDim.x <= num_items
+    Geo gn = geo_of(xn);
+    for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
+      const Item x = xn;
+      const Geo ge = gn;
+      if (it + (int)gridDim.x < num_items) {          // the next item's geometry: its loads fly under this item
+        xn = item_of(it + gridDim.x, sc);
+        gn = geo_of(xn);
+      }
+      if (ge.n_tiles == 0) continue;
+      const int n = ge.n_tiles;
+      const float bias = kMode == kSigmoid && pk.bias ? __ldg(pk.bias + x.h) * 1.4426950408889634f : 0.f;
+      // rows past the sequence are not stored; their gate row is clamped to the last real one
+      const float* grow = kMode == kSigmoid && pk.gate
+                              ? pk.gate + (int64_t)(ge.seq_start + min(x.qt * 128 + r, ge.seq_len - 1)) * pk.ldg + x.h * 128 : nullptr;
+      if (kMode == kSigmoid && grow) {               // the row's gate is needed behind the last tile: on its way to L2 until then
+#pragma unroll
+        for (int c = 0; c < 4; ++c) asm volatile("prefetch.global.L2 [%0];" ::"l"(grow + c * 32));
+      }
+      // with a window a row's first tiles may hold none of its keys: a finite floor keeps every difference of maxima defined
+      float m = kMode == kShared ? -1e30f : -INFINITY, l = 0.f;                 // m: the maximum the exponentials are taken against (may lag the true one)
+      for (int j = 0; j < n; ++j) {
+        const uint32_t gi = g + j;
+        const uint32_t s_addr = tmem_s + (gi & 1) * kKT + lane_addr;
+        ptx::mbar_wait(s_full(gi & 1), (gi >> 1) & 1);
+        ptx::tcgen05_fence_after();
+        uint32_t sv[kKT];
+        ptx::tmem_ld_32x32b_x32(s_addr, sv);
+        ptx::tmem_ld_32x32b_x32(s_addr + 32, sv + 32);
+        ptx::tmem_ld_wait();
+        const int t0 = (ge.j0 + j) * kKT;                  // the tile's first key position
+        uint32_t pk2[kKT / 2];
+        bool move = false;
+        float alpha = 1.0f;
+        if constexpr (kMode == kSigmoid) {
+          if (pk.key_scale) {
+            ptx::mbar_wait(kv_full((int)(gi % kKV)), (gi / kKV) & 1);      // long complete (S was made of this tile): orders the reads below
+            const float4* f = reinterpret_cast<const float4*>(gen + kOffScale + (gi % kKV) * (kKT * 4));
+#pragma unroll
+            for (int i = 0; i < kKT; i += 4) {
+              const float4 v = f[i >> 2];
+              sv[i] = __float_as_uint(__uint_as_float(sv[i]) * v.x);
+              sv[i + 1] = __float_as_uint(__uint_as_float(sv[i + 1]) * v.y);
+              sv[i + 2] = __float_as_uint(__uint_as_float(sv[i + 2]) * v.z);
+              sv[i + 3] = __float_as_uint(__uint_as_float(sv[i + 3]) * v.w);
+            }
+          }
+          // d = 1 + 2^-(x log2e) for 64 keys, then 1 / d for two keys from ONE reciprocal of their product: the MUFU unit is this kernel's
+          // bound.  The exponent stops at 2^60 - a weight of 2^-60 at least, the product of two far inside fp32 - which also keeps stale
+          // (NaN) columns behind the context from reaching their neighbour; those are set to 0 below.
+#pragma unroll
+          for (int i = 0; i < kKT; ++i)
+            sv[i] = __float_as_uint(1.0f + fast_exp2(fminf(fmaf(__uint_as_float(sv[i]), -scale_log2e, -bias), 60.0f)));
+#pragma unroll
+          for (int i = 0; i < kKT; i += 2) {
+            const float d0 = __uint_as_float(sv[i]), d1 = __uint_as_float(sv[i + 1]);
+            const float q = fast_rcp(d0 * d1);
+            sv[i] = __float_as_uint(q * d1);
+            sv[i + 1] = __float_as_uint(q * d0);
+          }
+          if (t0 + kKT - 1 > ge.q0) {
+            const int lim = ge.q0 + r - t0;
+#pragma unroll
+            for (int i = 0; i < kKT; ++i)
+              if (i > lim) sv[i] = 0u;
+          }
+          if (pk.window > 0 && t0 <= ge.q0 + 127 - pk.window) {
+            const int first = ge.q0 + r - pk.window + 1 - t0;
+#pragma unroll
+            for (int i = 0; i < kKT; ++i)
+              if (i < first) sv[i] = 0u;
+          }
+#pragma unroll
+          for (int i = 0; i < kKT; i += 2) pk2[i >> 1] = pack_bf16(__uint_as_float(sv[i]), __uint_as_float(sv[i + 1]));
+        } else {
           // diagonal tiles only (the tile holds keys past some row's position): columns past this row's position
           // become -inf, i.e. p = exp2(-inf) = 0; every other tile takes the mask-free path below
-          const int t0 = (ge.j0 + j) * kKT;                  // the tile's first key position
-          uint32_t pk2[kKT / 2];
-          bool move = false;
-          float alpha = 1.0f;
-          if constexpr (kMode == kSigmoid) {
-            if (pk.key_scale) {
-              ptx::mbar_wait(kv_full((int)(gi % kKV)), (gi / kKV) & 1);      // long complete (S was made of this tile): orders the reads below
-              const float4* f = reinterpret_cast<const float4*>(gen + kOffScale + (gi % kKV) * (kKT * 4));
-#pragma unroll
-              for (int i = 0; i < kKT; i += 4) {
-                const float4 v = f[i >> 2];
-                sv[i] = __float_as_uint(__uint_as_float(sv[i]) * v.x);
-                sv[i + 1] = __float_as_uint(__uint_as_float(sv[i + 1]) * v.y);
-                sv[i + 2] = __float_as_uint(__uint_as_float(sv[i + 2]) * v.z);
-                sv[i + 3] = __float_as_uint(__uint_as_float(sv[i + 3]) * v.w);
-              }
-            }
-            // e = 2^-(x log2e) for 64 keys, then p = 1 / (1 + e)
-#pragma unroll
-            for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fast_exp2(fmaf(__uint_as_float(sv[i]), -scale_log2e, -bias)));
-#pragma unroll
-            for (int i = 0; i < kKT; ++i) sv[i] = __float_as_uint(fast_rcp(1.0f + __uint_as_float(sv[i])));
-            if (t0 + kKT - 1 > ge.q0) {
-              const int lim = ge.q0 + r - t0;
-#pragma unroll
-              for (int i = 0; i < kKT; ++i)
-                if (i > lim) sv[i] = 0u;
-            }
-            if (pk.window > 0 && t0 <= ge.q0 + 127 - pk.window) {
-              const int first = ge.q0 + r - pk.window + 1 - t0;
-#pragma unroll
-              for (int i = 0; i < kKT; ++i)
-                if (i < first) sv[i] = 0u;
-            }
-#pragma unroll
-            for (int i = 0; i < kKT; i += 2) pk2[i >> 1] = pack_bf16(__uint_as_float(sv[i]), __uint_as_float(sv[i + 1]));
-          } else {
           if (t0 + kKT - 1 > ge.q0) {
             const int lim = ge.q0 + r - t0;                 // last visible column of this row
 #pragma unroll
@@ -483,9 +498,6 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       ptx::tcgen05_fence_after();
       if (kPaged && kMode != kSigmoid && pk.sink) l += exp2f(__ldg(pk.sink + x.h) * 1.4426950408889634f - m);   // the sink: in the denominator, without a value
       const float inv = kMode == kSigmoid ? 1.0f : 1.0f / l;
-      // rows past the sequence are not stored; their gate row is clamped to the last real one
-      const float* grow = kMode == kSigmoid && pk.gate
-                              ? pk.gate + (int64_t)(ge.seq_start + min(x.qt * 128 + r, ge.seq_len - 1)) * pk.ldg + x.h * 128 : nullptr;
       // this warp's 32 rows x 128 head dims leave through its staging buffer: 8 lanes per row, 128 contiguous bytes each
       RowStage st = make_row_stage(gen + kOffStage + quad * 4096, out, 0, NVC_EPI_NONE, (int64_t)ldo,
                                    ge.seq_start + x.qt * 128 + quad * 32, ge.seq_start + ge.seq_len, x.h * 128, 128, nh * 128);
