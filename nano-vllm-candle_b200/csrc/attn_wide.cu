@@ -6,7 +6,7 @@
 //
 // Three kernels:
 //   attn_shared_decode_kernel (attn_shared_decode.cuh)  bf16, one row per sequence, values = leading numbers of 64- or 128-number key rows
-//   attn_wide_mma_kernel (attn_wide_mma.cuh)  bf16 storage, dim and vdim multiples of 16 up to 256: tensor pipe
+//   attn_wide_mma_kernel (attn_wide_mma.cuh)  bf16 storage, dim and vdim multiples of 16 up to 128: tensor pipe
 //   attn_wide_simt_kernel                      any sizes, both storage formats, plain fp32 FMA: the exact mode
 // The last takes the keys of a row in tiles that start at the row's own first visible key, so the order of every sum depends on
 // the row's position alone - not on how the prompt was cut, on the batch or on the pages.
