@@ -423,6 +423,19 @@ int nvc_rotary_table_init_scaled_sync(nvc_ctx* ctx, double base, int dims, nvc_r
  * *lambda v_first[n]); v *= v_scale; q goes to q_out[n], k and v to row slot_mapping[n] of k_out / v_out (a paged cache; a negative slot
  * skips the token) or to row n when slot_mapping == NULL. */
 enum { NVC_BLEND_NONE = 0, NVC_BLEND_PROVIDE = 1, NVC_BLEND_MIX = 2 };
+/* A short causal convolution over time per channel of the step's rows: y_t = sum_j w[j, c] x_(t - taps + 1 + j).  The taps - 1 inputs in
+ * front of a portion come from the sequence's state slot, zeros when the portion starts at position 0. */
+typedef struct nvc_short_conv {
+  int taps;                               /* 1 .. 16 */
+  const float* w;                         /* [taps, channels], tap-major, last row = the current token */
+  float* state;                           /* [slots, taps - 1, channels] */
+  const int32_t* state_slots; const int32_t* cu_seqlens;   /* cu_seqlens NULL: one row per sequence */
+  int B;                                  /* sequences */
+} nvc_short_conv;
+/* Writes every sequence's last taps - 1 inputs (column off + c of a row, plus bias[c] when bias != NULL) into its state slot; runs behind
+ * the kernel that applies the convolution. */
+int nvc_short_conv_advance(nvc_ctx* ctx, const nvc_short_conv* cv, const float* in, int ldi, int off, const float* bias, int C,
+                           const int32_t* positions, void* stream);
 typedef struct nvc_qkv_prep {
   const float* in; int ldi;
   const float* bias;                      /* indexed like a row of `in`; NULL: none */
@@ -440,6 +453,10 @@ typedef struct nvc_qkv_prep {
   int unit_norm;                          /* q and k heads are divided by their root mean square (eps inside the root) without a weight;
                                            * q_norm and k_norm must be NULL */
   int act;                                /* NVC_PREP_ACT_SILU: q, k and v go through z sigmoid(z) right after the bias */
+  int wide_norm;                          /* q_norm and k_norm span the WHOLE query / key projection (q_heads * dim and kv_heads * dim numbers) */
+  const nvc_short_conv* conv;             /* optional (host pointer): right behind the bias; channels [q | k | v], which must be neighbours in a
+                                           * row (k_off = q_off + q_heads * dim, v_off = k_off + kv_heads * dim).  With cu_seqlens == NULL the call
+                                           * moves the convolution state on; with portions the caller does (nvc_short_conv_advance). */
 } nvc_qkv_prep;
 enum { NVC_PREP_ACT_NONE = 0, NVC_PREP_ACT_SILU = 1 };
 int nvc_qkv_prep_run(nvc_ctx* ctx, const nvc_qkv_prep* p, int N, void* stream);
@@ -514,7 +531,9 @@ int nvc_act_mul_p(nvc_ctx* ctx, const void* in, int ldi, void* out, int ldo, int
                   void* stream);
 /* nvc_moe_route_logits with a choice of score function and weights: score NVC_ROUTE_SIGMOID or NVC_ROUTE_SOFTMAX (over all E
  * columns); normalize != 0: topk_w = s_chosen / (sum of the chosen s + 1e-20) * scale, else topk_w = s_chosen * scale. */
-enum { NVC_ROUTE_SIGMOID = 0, NVC_ROUTE_SOFTMAX = 1 };
+/* NVC_ROUTE_CHOSEN: `correction` is a bias of the logits; the experts with the largest z + correction are chosen and their scores are
+ * exp(z + correction) (with normalize: the softmax over the chosen logits alone). */
+enum { NVC_ROUTE_SIGMOID = 0, NVC_ROUTE_SOFTMAX = 1, NVC_ROUTE_CHOSEN = 2 };
 int nvc_moe_route_logits_ex(nvc_ctx* ctx, const float* z, int ldz, const float* correction, int E, int top, float scale, int gate_col,
                             int score, int normalize, int32_t* topk_idx, float* topk_w, float* gate, int N, void* stream);
 /* nvc_moe_sort_padded for a router whose experts from E_real on have no product (identity experts): their tiles get
@@ -545,6 +564,10 @@ typedef struct nvc_delta_prep {
   float* q_out; float* k_out; float* v_out; int ldq, ldk, ldv;
   float* gb_out;
   int B;
+  /* a decay per head AND key channel: channel_a fp32 rows [N, ldca] (heads * dim) take the place of the columns at a_off, dt_bias holds
+   * heads * dim numbers, and the log decays go to channel_g [N, heads * dim] (the first numbers of gb_out's pairs are not written);
+   * the recurrence then multiplies row d of a head's state by that channel's decay.  NULL: one decay per head */
+  const float* channel_a; int ldca; float* channel_g;
 } nvc_delta_prep;
 int nvc_delta_prep_run(nvc_ctx* ctx, const nvc_delta_prep* p, int N, int max_qlen, void* stream);   /* max_qlen: the longest portion (a bound will do) */
 /* The recurrence, per (sequence, head) with state S [dim, vdim] fp32 in state [slots, heads, dim, vdim]:
@@ -634,6 +657,41 @@ int nvc_prefill_attn_shared(nvc_ctx* ctx, const nvc_bf16* q, int ldq, const nvc_
                             int block_size, int num_blocks, const nvc_attn_spec* spec, nvc_bf16* out, int ldo, void* stream);
 /* x[n, j] = cap tanh(x[n, j] / cap), j < V, in place (fp32 rows). */
 int nvc_softcap_f32(nvc_ctx* ctx, float* x, int ld, float cap, int N, int V, void* stream);
+
+/* ---- mechanisms of the models with several residual streams, window attention beside a matrix memory and channel-wise decays in the
+ * delta rule (Vizotar) ---- */
+/* Closes a sublayer and opens the next on `streams` fp32 residual streams (1 .. 16), one pass over a token's rows (all sums fp32):
+ *   y = c0 f(y0[r] + b0, w0) + c1 f(y1[r], w1)       f(v, w) = v (w == NULL) or v / sqrt(mean(v^2) + eps) * w; y0, b0, y1 optional
+ *   X_t <- sum_s mix[s * streams + t] X_s + out_w[t] y, all from the old streams (no y0, y1: the streams stay);  x_out optional
+ *   u = sum_t in_w[t] X_t (in_w == NULL: the plain sum);  out[i, :H] = u / sqrt(mean(u^2) + eps) * norm_w (norm_w == NULL: u; out optional)
+ * Stream s of row r is x[r * ldx + s * sx]; sx_in == 0 reads the same row as every stream (the embedding).  x_out may be x_in.
+ * rows as in nvc_rms_norm_pair (gathers; x_out must be NULL). */
+typedef struct nvc_streams_args {
+  const float* x_in; int ldx_in, sx_in;
+  float* x_out; int ldx_out, sx_out;
+  int streams;
+  const float* y0; const float* b0; const float* w0; float c0;
+  const float* y1; const float* w1; float c1;
+  int ldy;
+  const float* mix; const float* out_w; const float* in_w; const float* norm_w;
+  int ldo; float eps;
+  const int32_t* rows;
+} nvc_streams_args;
+int nvc_streams_norm(nvc_ctx* ctx, const nvc_streams_args* p, void* out, int out_dtype, int N, int H, void* stream);
+/* Matrix memory with an exponential input gate and a sigmoid forget gate, per (sequence, head), in its max-stabilised form.  With
+ *   c(z) = cap tanh(z / cap),  i_t = c(i_in[t, h] + i_bias[h]),  f_t = log sigmoid(c(f_in[t, h] + f_bias[h])):
+ *   m_t = max(f_t + m_(t-1), i_t);  S_t = exp(f_t + m_(t-1) - m_t) S_(t-1) + exp(i_t - m_t) k_t v_t^T;  n_t likewise with k_t alone;
+ *   o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + den_eps),   q_t = q_scale times the row's query
+ * S, n and m start at zero.  state: fp32 [slots, heads, dim, vdim]; nm_state: fp32 [slots, heads, ceil(vdim / 32), dim + 1] - n and m, a
+ * copy for every 32 value columns.  Rows, slots, start from zeros and max_qlen as in nvc_retention_scan. */
+typedef struct nvc_memory_scan_args {
+  const float* q; const float* k; const float* v; int ldq, ldk, ldv; float q_scale;
+  const float* i_in; const float* f_in; int ldg; const float* i_bias; const float* f_bias; float cap, den_eps;
+  float* o; int ldo;
+  float* state; float* nm_state; const int32_t* state_slots; const int32_t* cu_seqlens; const int32_t* positions;
+  int heads, dim, vdim;
+} nvc_memory_scan_args;
+int nvc_memory_scan(nvc_ctx* ctx, const nvc_memory_scan_args* p, int B, int max_qlen, void* stream);
 
 /* K8. Replaces Qwen3ModelRunner::argmax (src/engine/llm_engine.rs:135-142) on device:
  * idx[b] = LAST index of the maximum of logits[b, :] (Iterator::max_by tie rule);

@@ -1,12 +1,14 @@
 // What the model bodies behind the step executor share: number formats of checkpoint tensors, zeroed device allocations,
 // matrices written into padded device layouts, the plain product (tcgen05 GEMM when it takes the shape, the generic kernel
-// otherwise) and the per-op event profile of a step.
+// otherwise), rotary tables, the list of wanted tensors, the residual tap and the per-op event profile of a step.
 #pragma once
 #include <cstring>
 #include <map>
 #include <string>
+#include <tuple>
 #include <vector>
 
+#include "model_config.h"
 #include "runner.h"
 
 namespace {
@@ -59,6 +61,8 @@ struct nvc_body_base : nvc_model_body {
   bool prof_armed = false, prof_on = false;
   std::vector<std::pair<const char*, cudaEvent_t>> marks;
   std::string prof_json = "{}";
+  std::map<std::string, bool> want;     // tensors of the configuration: true once loaded
+  std::map<std::tuple<int, double, double, double, double, double>, float*> rot_tables;
 
   int arm_profile() override { prof_armed = true; return NVC_OK; }
   bool profile_armed() const override { return prof_armed; }
@@ -134,6 +138,40 @@ struct nvc_body_base : nvc_model_body {
       return nvc_gemm_bf16(r->ctx, reinterpret_cast<const nvc_bf16*>(A), lda, reinterpret_cast<const nvc_bf16*>(Wt), C, ldc, out_dt, M, N, K,
                            r->stream);
     return nvc_linear(r->ctx, A, lda, 0, Wt, K, 0, C, ldc, 0, dt, dt == NVC_DT_F32 ? NVC_DT_F32 : out_dt, M, N, K, 1, act, r->stream);
+  }
+
+  // (cos, sin) tables, one per rotation of the configuration
+  int rotary_table(nvc_runner* r, const nvc_rotary_spec& rs, const float** out) {
+    *out = nullptr;
+    if (rs.dims == 0) return NVC_OK;
+    const auto key = std::make_tuple(rs.dims, rs.base, rs.scaling.factor, rs.scaling.original, rs.scaling.fast, rs.scaling.slow);
+    auto it = rot_tables.find(key);
+    if (it == rot_tables.end()) {
+      float* t = nullptr;
+      int rc = zalloc(r, &t, (size_t)r->opt.max_model_len * rs.dims * sizeof(float));
+      if (rc) return rc;
+      if ((rc = nvc_rotary_table_init_scaled_sync(r->ctx, rs.base, rs.dims, rs.scaling, r->opt.max_model_len, t))) return rc;
+      it = rot_tables.emplace(key, t).first;
+    }
+    *out = it->second;
+    return NVC_OK;
+  }
+
+  // residual stream after layer `run` (stride ld) into the host buffer of the debug tap
+  int copy_tap(nvc_runner* r, const float* res, int ld, float* host, size_t cap, int run, int N, int W) {
+    const size_t need = (size_t)(run + 1) * N * W;
+    NVC_REQUIRE(r->ctx, need <= cap, NVC_ENOMEM, "residual tap buffer too small");
+    NVC_CUDA_CHECK(r->ctx, cudaMemcpy2DAsync(host + (size_t)run * N * W, (size_t)W * 4, res, (size_t)ld * 4, (size_t)W * 4, N, cudaMemcpyDeviceToHost, r->stream));
+    return NVC_OK;
+  }
+
+  int require_all_tensors(nvc_runner* r) {
+    std::string missing;
+    int n = 0;
+    for (auto& kv : want)
+      if (!kv.second && ++n <= 4) missing += kv.first + " ";
+    NVC_REQUIRE(r->ctx, n == 0, NVC_ESTATE, "missing " + std::to_string(n) + " tensors: " + missing);
+    return NVC_OK;
   }
 };
 

@@ -12,9 +12,14 @@
 //                       (the same sums as the four steps above, regrouped so that a token needs one reduction over row groups).
 //                       The CTAs of a sequence also advance its convolution state, a share of the channels each.
 //   delta_chunk_kernel  the same recurrence 32 tokens at a time for prompt portions (see there).
+// With a decay per head and key CHANNEL (g a vector, S <- diag(g) S) the token kernel scales every row of S first and then follows the
+// four steps, and the chunk kernel works with the running sums L_t of each channel: the token-by-token products take
+// exp(L_t - L_j) inside their sums, the keys and queries that meet the state carry exp(L_t), those that enter it exp(L_n - L_j).
 // Both states live in fp32 in pools of state slots; a sequence whose first new token sits at position 0 starts from zeros.
 // Everything here is plain fp32 FMA code.
 #include <cooperative_groups.h>
+
+#include <type_traits>
 
 #include "typed.cuh"
 
@@ -45,9 +50,23 @@ __global__ void __launch_bounds__(128, 8) delta_prep_kernel(const DeltaArgs a) {
   const int n = r0 + blockIdx.x * (blockDim.x >> 5) + wid;
   if (n >= r1) return;
   const float* in = p.in + (int64_t)n * p.ldi;
+  if (uu >= units) {
+    // ---- log decays of one head's key channels
+    const int h = uu - units;
+    const float* x = p.channel_a + (int64_t)n * p.ldca + h * p.dim;
+    const float* bias = p.dt_bias + h * p.dim;
+    float* g = p.channel_g + ((int64_t)n * p.heads + h) * p.dim;
+    const float na = -expf(__ldg(p.A_log + h));
+    for (int j = lane; j < p.dim; j += 32) g[j] = na * softplus_f32(x[j] + __ldg(bias + j));
+    return;
+  }
   if (uu == units - 1) {
     // ---- decay and beta of every head
     for (int h = lane; h < p.heads; h += 32) {
+      if (p.channel_a) {
+        p.gb_out[(int64_t)n * 2 * p.heads + 2 * h + 1] = sigmoid_f32(in[p.b_off + h]);
+        continue;
+      }
       const float dt = softplus_f32(in[p.a_off + h] + __ldg(p.dt_bias + h));
       p.gb_out[(int64_t)n * 2 * p.heads + 2 * h] = -expf(__ldg(p.A_log + h)) * dt;       // log of the decay
       p.gb_out[(int64_t)n * 2 * p.heads + 2 * h + 1] = sigmoid_f32(in[p.b_off + h]);
@@ -145,7 +164,8 @@ __device__ __forceinline__ void advance_conv_state(const nvc_delta_prep& p, int 
   }
 }
 
-template <int DPT>
+// CH: a decay per key channel
+template <int DPT, bool CH>
 __global__ void delta_scan_kernel(const DeltaArgs a) {
   extern __shared__ float sm[];
   pdl_trigger();
@@ -157,7 +177,8 @@ __global__ void delta_scan_kernel(const DeltaArgs a) {
   const int hk = h / (p.heads / p.kv_heads);
   float* q_s = sm;                    // [2][dim]
   float* k_s = sm + 2 * p.dim;        // [2][dim]
-  float* red = sm + 4 * p.dim;        // [3][groups][32]
+  float* g_s = sm + 4 * p.dim;        // [2][dim] (CH): decays
+  float* red = sm + (CH ? 6 : 4) * p.dim;        // [3][groups][32]
   pdl_wait();
   const int r0 = p.cu_seqlens ? p.cu_seqlens[b] : b;
   const int r1 = p.cu_seqlens ? p.cu_seqlens[b + 1] : b + 1;
@@ -172,9 +193,10 @@ __global__ void delta_scan_kernel(const DeltaArgs a) {
   for (int d = threadIdx.x; d < p.dim; d += blockDim.x) {
     q_s[d] = p.q_out[(int64_t)r0 * p.ldq + hk * p.dim + d];
     k_s[d] = p.k_out[(int64_t)r0 * p.ldk + hk * p.dim + d];
+    if (CH) g_s[d] = expf(p.channel_g[((int64_t)r0 * p.heads + h) * p.dim + d]);
   }
   float vt = vok ? p.v_out[(int64_t)r0 * p.ldv + h * p.vdim + v] : 0.f;
-  float gt = expf(p.gb_out[(int64_t)r0 * 2 * p.heads + 2 * h]), bt = p.gb_out[(int64_t)r0 * 2 * p.heads + 2 * h + 1];
+  float gt = CH ? 1.f : expf(p.gb_out[(int64_t)r0 * 2 * p.heads + 2 * h]), bt = p.gb_out[(int64_t)r0 * 2 * p.heads + 2 * h + 1];
   __syncthreads();
   for (int t = r0; t < r1; ++t) {
     const int cur = (t - r0) & 1;
@@ -185,9 +207,10 @@ __global__ void delta_scan_kernel(const DeltaArgs a) {
       for (int d = threadIdx.x; d < p.dim; d += blockDim.x) {
         q_s[(cur ^ 1) * p.dim + d] = p.q_out[(int64_t)(t + 1) * p.ldq + hk * p.dim + d];
         k_s[(cur ^ 1) * p.dim + d] = p.k_out[(int64_t)(t + 1) * p.ldk + hk * p.dim + d];
+        if (CH) g_s[(cur ^ 1) * p.dim + d] = expf(p.channel_g[((int64_t)(t + 1) * p.heads + h) * p.dim + d]);
       }
       vn = vok ? p.v_out[(int64_t)(t + 1) * p.ldv + h * p.vdim + v] : 0.f;
-      gn = expf(p.gb_out[(int64_t)(t + 1) * 2 * p.heads + 2 * h]);
+      if (!CH) gn = expf(p.gb_out[(int64_t)(t + 1) * 2 * p.heads + 2 * h]);
       bn = p.gb_out[(int64_t)(t + 1) * 2 * p.heads + 2 * h + 1];
     }
     float sk = 0.f, sq = 0.f, kq = 0.f;
@@ -195,6 +218,7 @@ __global__ void delta_scan_kernel(const DeltaArgs a) {
     for (int i = 0; i < DPT; ++i) {
       if (d0 + i < p.dim) {
         const float kv = kc[d0 + i], qv = qc[d0 + i];
+        if (CH) S[i] *= g_s[cur * p.dim + d0 + i];
         sk = fmaf(S[i], kv, sk);
         sq = fmaf(S[i], qv, sq);
         kq = fmaf(kv, qv, kq);
@@ -212,6 +236,7 @@ __global__ void delta_scan_kernel(const DeltaArgs a) {
         kq += red[(2 * groups + g) * 32 + lane];
       }
     }
+    if (CH) gt = 1.f;                 // the decay is in the rows already
     const float u = bt * (vt - gt * sk);
     if (vok && rg == 0) a.o[(int64_t)t * a.ldo + h * p.vdim + v] = fmaf(kq, u, gt * sq);
 #pragma unroll
@@ -242,8 +267,8 @@ constexpr int kDAs = kDC + 4;            // row stride of the token-by-token mat
 
 // staged key / query rows: 4 DPT numbers and more (zeros behind `dim`), 16-byte aligned, rows 4 banks apart
 __host__ __device__ inline int delta_chunk_row(int dim, int dpt) { return max((dim + 3) / 4 * 4, kDW * dpt) + 4; }
-__host__ __device__ inline size_t delta_chunk_smem_floats(int dim, int dpt) {
-  return (size_t)2 * kDC * delta_chunk_row(dim, dpt) + 2 * kDC * kDAs + 3 * kDC * 32 + (size_t)kDW * kDC * 32 + 2 * kDC + 8;
+__host__ __device__ inline size_t delta_chunk_smem_floats(int dim, int dpt, bool channels) {
+  return (size_t)(channels ? 3 : 2) * kDC * delta_chunk_row(dim, dpt) + 2 * kDC * kDAs + 3 * kDC * 32 + (size_t)kDW * kDC * 32 + 2 * kDC + 8;
 }
 
 __device__ __forceinline__ float fma4(const float4& x, const float4& y, float acc) {
@@ -251,6 +276,12 @@ __device__ __forceinline__ float fma4(const float4& x, const float4& y, float ac
   acc = fmaf(x.y, y.y, acc);
   acc = fmaf(x.z, y.z, acc);
   return fmaf(x.w, y.w, acc);
+}
+
+// x exp(min(a - b, 0)), number by number
+__device__ __forceinline__ float4 scaled_by_exp(const float4& x, const float4& a, const float4& b) {
+  return make_float4(x.x * expf(fminf(a.x - b.x, 0.f)), x.y * expf(fminf(a.y - b.y, 0.f)), x.z * expf(fminf(a.z - b.z, 0.f)),
+                     x.w * expf(fminf(a.w - b.w, 0.f)));
 }
 
 // Forward substitution of the chunk's triangular system, one value column per lane of one warp: Us holds v_t on entry and u_t on
@@ -278,7 +309,9 @@ __device__ __noinline__ void delta_chunk_solve(const float* Am, float* Us, const
 // kCluster: the CTAs of one (sequence, head) - its slices of 32 value columns - form a thread-block cluster, split the rows of the two
 // token-by-token matrices among themselves and write them into one another's shared memory: the products that do not depend on the
 // value column are computed once per (sequence, head), not once per slice.
-template <int DPT, bool kCluster>
+// CH: a decay per key channel; the running sums of the channels' log decays stand beside the keys and queries in shared memory, the
+// per-head ones (Ls) stay zero.
+template <int DPT, bool kCluster, bool CH>
 __global__ void __launch_bounds__(kDW * 32) delta_chunk_kernel(const DeltaArgs a) {
   namespace cg = cooperative_groups;
   extern __shared__ __align__(16) float sm[];
@@ -301,6 +334,7 @@ __global__ void __launch_bounds__(kDW * 32) delta_chunk_kernel(const DeltaArgs a
   float* Wp = W2 + kDC * 32;               // [kDW][kDC][32] partial sums of the row groups
   float* Ls = Wp + kDW * kDC * 32;         // [kDC]
   float* Bs = Ls + kDC;                    // [kDC]
+  float* Gs = Bs + kDC;                    // [kDC][ds] (CH) running sums of the log decays, channel by channel
   pdl_wait();
   const int r0 = p.cu_seqlens ? p.cu_seqlens[b] : b;
   const int r1 = p.cu_seqlens ? p.cu_seqlens[b + 1] : b + 1;
@@ -322,11 +356,12 @@ __global__ void __launch_bounds__(kDW * 32) delta_chunk_kernel(const DeltaArgs a
         const bool in = t < n && c < dim;
         Ks[t * ds + c] = in ? kg[c] : 0.f;
         Qs[t * ds + c] = in ? qg[c] : 0.f;
+        if (CH) Gs[t * ds + c] = in ? p.channel_g[((int64_t)(c0 + t) * p.heads + h) * dim + c] : 0.f;
       }
       Us[t * 32 + lane] = (t < n && vok) ? p.v_out[(int64_t)(c0 + t) * p.ldv + h * p.vdim + v] : 0.f;
     }
     if (w == 0) {
-      float lg = lane < n ? p.gb_out[(int64_t)(c0 + lane) * 2 * p.heads + 2 * h] : 0.f;
+      float lg = (!CH && lane < n) ? p.gb_out[(int64_t)(c0 + lane) * 2 * p.heads + 2 * h] : 0.f;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
         const float up = __shfl_up_sync(0xffffffffu, lg, o);
@@ -336,6 +371,13 @@ __global__ void __launch_bounds__(kDW * 32) delta_chunk_kernel(const DeltaArgs a
       Bs[lane] = lane < n ? p.gb_out[(int64_t)(c0 + lane) * 2 * p.heads + 2 * h + 1] : 0.f;
     }
     __syncthreads();
+    if constexpr (CH) {
+      for (int c = threadIdx.x; c < dz; c += kDW * 32) {
+        float l = 0.f;
+        for (int t = 0; t < kDC; ++t) { l += Gs[t * ds + c]; Gs[t * ds + c] = l; }
+      }
+      __syncthreads();
+    }
     // ---- products between the chunk's tokens: two rows t per warp and pass, column j per lane, 16-byte operands
     {
       const int Z = kCluster ? (int)gridDim.z : 1, zr = kCluster ? (int)blockIdx.z : 0;
@@ -347,6 +389,20 @@ __global__ void __launch_bounds__(kDW * 32) delta_chunk_kernel(const DeltaArgs a
           const float4* kt1 = reinterpret_cast<const float4*>(Ks + (t + 1) * ds);
           const float4* qt1 = reinterpret_cast<const float4*>(Qs + (t + 1) * ds);
           const float4* kj = reinterpret_cast<const float4*>(Ks + lane * ds);
+          if constexpr (CH) {
+            const float4* gt0 = reinterpret_cast<const float4*>(Gs + t * ds);
+            const float4* gt1 = reinterpret_cast<const float4*>(Gs + (t + 1) * ds);
+            const float4* gj = reinterpret_cast<const float4*>(Gs + lane * ds);
+#pragma unroll 1
+            for (int c = 0; c < dz / 4; ++c) {
+              const float4 x = kj[c], g = gj[c];
+              const float4 y0 = scaled_by_exp(x, gt0[c], g), y1 = scaled_by_exp(x, gt1[c], g);
+              kk0 = fma4(kt0[c], y0, kk0);
+              qk0 = fma4(qt0[c], y0, qk0);
+              kk1 = fma4(kt1[c], y1, kk1);
+              qk1 = fma4(qt1[c], y1, qk1);
+            }
+          } else
 #pragma unroll 2
           for (int c = 0; c < dz / 4; ++c) {
             const float4 x = kj[c];
@@ -381,10 +437,26 @@ __global__ void __launch_bounds__(kDW * 32) delta_chunk_kernel(const DeltaArgs a
       }
     }
     // ---- what the state before the chunk says to every key and query: partial sums over this warp's rows, then over the warps
+    if constexpr (CH) {
+      __syncthreads();                       // the products above have read the plain rows
+      for (int t = w; t < kDC; t += kDW)
+        for (int c = lane; c < dz; c += 32) Qs[t * ds + c] *= expf(Gs[t * ds + c]);
+      __syncthreads();
+    }
 #pragma unroll 1
     for (int pass = 0; pass < 2; ++pass) {
-      const float* X = pass == 0 ? Ks : Qs;
-      float* Wd = pass == 0 ? W1 : W2;
+      // CH: the queries first; their rows then hold the keys, scaled for the second pass, and the keys are scaled for the state update
+      const float* X = CH || pass == 1 ? Qs : Ks;
+      float* Wd = (pass == 0) != CH ? W1 : W2;
+      if (CH && pass == 1) {
+        for (int t = w; t < kDC; t += kDW)
+          for (int c = lane; c < dz; c += 32) {
+            const float k = Ks[t * ds + c], l = Gs[t * ds + c];
+            Qs[t * ds + c] = k * expf(l);
+            Ks[t * ds + c] = k * expf(Gs[(kDC - 1) * ds + c] - l);
+          }
+        __syncthreads();
+      }
 #pragma unroll 1
       for (int t0 = 0; t0 < kDC; t0 += 8) {
         float acc[8];
@@ -437,7 +509,7 @@ __global__ void __launch_bounds__(kDW * 32) delta_chunk_kernel(const DeltaArgs a
       const float Ln = Ls[kDC - 1];
       const float gn = expf(Ln);
 #pragma unroll
-      for (int i = 0; i < DPT; ++i) S[i] *= gn;
+      for (int i = 0; i < DPT; ++i) S[i] *= CH ? expf(Gs[(kDC - 1) * ds + min(d0 + i, dz - 1)]) : gn;
 #pragma unroll 4
       for (int j = 0; j < kDC; ++j) {             // a loop over the tokens around an unrolled pass over this thread's rows: short code
         const float uj = Us[j * 32 + lane] * expf(Ln - Ls[j]);
@@ -460,19 +532,19 @@ __global__ void __launch_bounds__(kDW * 32) delta_chunk_kernel(const DeltaArgs a
       if (d0 + i < dim) sp[(int64_t)(d0 + i) * p.vdim + v] = S[i];
 }
 
-template <int DPT>
+template <int DPT, bool CH>
 cudaError_t launch_delta_chunk(nvc_ctx* ctx, const DeltaArgs& a, dim3 grid, size_t smem, cudaStream_t st) {
   static bool attr_set = false;
   if (!attr_set && smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(delta_chunk_kernel<DPT, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_kernel<DPT, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(delta_chunk_kernel<DPT, false, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_kernel<DPT, true, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (e != cudaSuccess) return e;
     attr_set = true;
   }
   static const bool no_cluster = getenv("NVC_DELTA_CLUSTER") && atoi(getenv("NVC_DELTA_CLUSTER")) == 0;
   if (grid.z >= 2 && grid.z <= 8 && !no_cluster)       // the value slices of a (sequence, head) as one cluster
-    return nvc_launch_cluster3(ctx, delta_chunk_kernel<DPT, true>, grid, dim3(kDW * 32), smem, st, dim3(1, 1, grid.z), a);
-  return nvc_launch(ctx, delta_chunk_kernel<DPT, false>, grid, dim3(kDW * 32), smem, st, a);
+    return nvc_launch_cluster3(ctx, delta_chunk_kernel<DPT, true, CH>, grid, dim3(kDW * 32), smem, st, dim3(1, 1, grid.z), a);
+  return nvc_launch(ctx, delta_chunk_kernel<DPT, false, CH>, grid, dim3(kDW * 32), smem, st, a);
 }
 
 int check_prep(nvc_ctx* ctx, const nvc_delta_prep* p) {
@@ -481,6 +553,7 @@ int check_prep(nvc_ctx* ctx, const nvc_delta_prep* p) {
   NVC_REQUIRE(ctx, p->heads > 0 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->vdim > 0 && p->taps >= 1 && p->B > 0 &&
                        p->dim <= 1024 && p->heads <= 65535, NVC_EINVAL, "bad sizes");
   NVC_REQUIRE(ctx, p->ldq >= p->kv_heads * p->dim && p->ldk >= p->kv_heads * p->dim && p->ldv >= p->heads * p->vdim, NVC_EINVAL, "bad strides");
+  NVC_REQUIRE(ctx, !p->channel_a || (p->channel_g && p->ldca >= p->heads * p->dim), NVC_EINVAL, "decays per channel need their output rows");
   return NVC_OK;
 }
 
@@ -495,7 +568,7 @@ extern "C" int nvc_delta_prep_run(nvc_ctx* ctx, const nvc_delta_prep* p, int N, 
   const int vec = p->dim % 4 == 0 && p->vdim % 4 == 0 && p->ldi % 4 == 0 && p->q_off % 4 == 0 && p->k_off % 4 == 0 && p->v_off % 4 == 0 && p->ldq % 4 == 0 &&
                   p->ldk % 4 == 0 && p->ldv % 4 == 0 && al16(p->in) && al16(p->conv_state) && al16(p->conv_w) && al16(p->q_out) && al16(p->k_out) && al16(p->v_out);
   DeltaArgs a{*p, N, vec, nullptr, 0, nullptr};
-  const int units = 2 * p->kv_heads + p->heads + 1;
+  const int units = 2 * p->kv_heads + p->heads + 1 + (p->channel_a ? p->heads : 0);
   const int longest = p->cu_seqlens ? std::min(N, std::max(max_qlen, 1)) : 1;
   NVC_REQUIRE(ctx, units <= 65535 && p->B <= 65535, NVC_ESHAPE, "more than 65 535 heads or sequences");
   const int warps = longest >= 4 ? 4 : 1;
@@ -516,12 +589,17 @@ extern "C" int nvc_delta_rule_scan(nvc_ctx* ctx, const nvc_delta_prep* p, float*
     const int per = (dim + kDW - 1) / kDW;     // rows of the state per warp
     const int cd = per <= 8 ? 8 : (per <= 16 ? 16 : (per <= 32 ? 32 : 64));
     const dim3 grid(p->B, p->heads, (p->vdim + 31) / 32);
-    const size_t smem = delta_chunk_smem_floats(dim, cd) * sizeof(float);
+    const size_t smem = delta_chunk_smem_floats(dim, cd, p->channel_a != nullptr) * sizeof(float);
     cudaError_t ce;
-    if (cd == 8) ce = launch_delta_chunk<8>(ctx, a, grid, smem, nvc_stream(stream));
-    else if (cd == 16) ce = launch_delta_chunk<16>(ctx, a, grid, smem, nvc_stream(stream));
-    else if (cd == 32) ce = launch_delta_chunk<32>(ctx, a, grid, smem, nvc_stream(stream));
-    else ce = launch_delta_chunk<64>(ctx, a, grid, smem, nvc_stream(stream));
+    auto go = [&](auto ch) {
+      constexpr bool CH = decltype(ch)::value;
+      if (cd == 8) ce = launch_delta_chunk<8, CH>(ctx, a, grid, smem, nvc_stream(stream));
+      else if (cd == 16) ce = launch_delta_chunk<16, CH>(ctx, a, grid, smem, nvc_stream(stream));
+      else if (cd == 32) ce = launch_delta_chunk<32, CH>(ctx, a, grid, smem, nvc_stream(stream));
+      else ce = launch_delta_chunk<64, CH>(ctx, a, grid, smem, nvc_stream(stream));
+    };
+    if (p->channel_a) go(std::true_type());
+    else go(std::false_type());
     NVC_CUDA_CHECK(ctx, ce);
     ctx->launches++;
     return NVC_OK;
@@ -531,14 +609,19 @@ extern "C" int nvc_delta_rule_scan(nvc_ctx* ctx, const nvc_delta_prep* p, float*
   const int dpt = dim <= 64 ? 16 : (dim <= 128 ? 32 : (dim <= 256 ? 64 : 128));
   const int groups = (dim + dpt - 1) / dpt;
   const dim3 grid(p->B, p->heads, (p->vdim + 31) / 32), block(32 * groups);
-  const size_t smem = ((size_t)4 * dim + (size_t)3 * groups * 32) * sizeof(float);
+  const size_t smem = ((size_t)(p->channel_a ? 6 : 4) * dim + (size_t)3 * groups * 32) * sizeof(float);
   cudaError_t ce;
-  switch (dpt) {
-    case 16: ce = nvc_launch(ctx, delta_scan_kernel<16>, grid, block, smem, nvc_stream(stream), a); break;
-    case 32: ce = nvc_launch(ctx, delta_scan_kernel<32>, grid, block, smem, nvc_stream(stream), a); break;
-    case 64: ce = nvc_launch(ctx, delta_scan_kernel<64>, grid, block, smem, nvc_stream(stream), a); break;
-    default: ce = nvc_launch(ctx, delta_scan_kernel<128>, grid, block, smem, nvc_stream(stream), a); break;
-  }
+  auto go = [&](auto ch) {
+    constexpr bool CH = decltype(ch)::value;
+    switch (dpt) {
+      case 16: ce = nvc_launch(ctx, delta_scan_kernel<16, CH>, grid, block, smem, nvc_stream(stream), a); break;
+      case 32: ce = nvc_launch(ctx, delta_scan_kernel<32, CH>, grid, block, smem, nvc_stream(stream), a); break;
+      case 64: ce = nvc_launch(ctx, delta_scan_kernel<64, CH>, grid, block, smem, nvc_stream(stream), a); break;
+      default: ce = nvc_launch(ctx, delta_scan_kernel<128, CH>, grid, block, smem, nvc_stream(stream), a); break;
+    }
+  };
+  if (p->channel_a) go(std::true_type());
+  else go(std::false_type());
   NVC_CUDA_CHECK(ctx, ce);
   ctx->launches++;
   return NVC_OK;

@@ -38,28 +38,9 @@ struct nvc_latent_weights {
 
 struct nvc_latent_body : nvc_body_base {
   bool use_flash = true;
-  std::map<std::string, bool> want;     // tensors of the configuration: true once loaded
-  std::map<std::tuple<int, double, double, double, double, double>, float*> rot_tables;
   float *lat_qf = nullptr, *lat_hv = nullptr;
   void *lat_cq = nullptr, *lat_qn = nullptr, *lat_qabs = nullptr, *lat_olat = nullptr;
   size_t lat_qrp = 0, lat_uqn = 0, lat_qn_cols = 0, lat_qa = 0, lat_ol = 0, lat_hv_cols = 0;
-
-  // (cos, sin) tables, one per rotation of the configuration
-  int rotary_table(nvc_runner* r, const nvc_rotary_spec& rs, const float** out) {
-    *out = nullptr;
-    if (rs.dims == 0) return NVC_OK;
-    const auto key = std::make_tuple(rs.dims, rs.base, rs.scaling.factor, rs.scaling.original, rs.scaling.fast, rs.scaling.slow);
-    auto it = rot_tables.find(key);
-    if (it == rot_tables.end()) {
-      float* t = nullptr;
-      int rc = zalloc(r, &t, (size_t)r->opt.max_model_len * rs.dims * sizeof(float));
-      if (rc) return rc;
-      if ((rc = nvc_rotary_table_init_scaled_sync(r->ctx, rs.base, rs.dims, rs.scaling, r->opt.max_model_len, t))) return rc;
-      it = rot_tables.emplace(key, t).first;
-    }
-    *out = it->second;
-    return NVC_OK;
-  }
 
   // sizes, weights and pool of one layer; off = first free column of its projection row.  *columns = columns the layer reads there.
   int latent_init(nvc_runner* r, const nvc_latent_attn_spec& a, const std::string& p, size_t slots, int off, nvc_latent_weights& w, int* columns,
@@ -224,23 +205,6 @@ struct nvc_latent_body : nvc_body_base {
     mark(r, "absorb_uv");
     if ((rc = nvc_head_gate(ctx, lat_hv, vw, gate, np, ao, owp, dt, a.heads, a.vdim, 0, eps, NVC_GATE_SIGMOID, 1.f, N, st))) return rc;
     mark(r, "head_gate");
-    return NVC_OK;
-  }
-
-  // residual stream after layer `run` (stride ld) into the host buffer of the debug tap
-  int copy_tap(nvc_runner* r, const float* res, int ld, float* host, size_t cap, int run, int N, int W) {
-    const size_t need = (size_t)(run + 1) * N * W;
-    NVC_REQUIRE(r->ctx, need <= cap, NVC_ENOMEM, "residual tap buffer too small");
-    NVC_CUDA_CHECK(r->ctx, cudaMemcpy2DAsync(host + (size_t)run * N * W, (size_t)W * 4, res, (size_t)ld * 4, (size_t)W * 4, N, cudaMemcpyDeviceToHost, r->stream));
-    return NVC_OK;
-  }
-
-  int require_all_tensors(nvc_runner* r) {
-    std::string missing;
-    int n = 0;
-    for (auto& kv : want)
-      if (!kv.second && ++n <= 4) missing += kv.first + " ";
-    NVC_REQUIRE(r->ctx, n == 0, NVC_ESTATE, "missing " + std::to_string(n) + " tensors: " + missing);
     return NVC_OK;
   }
 };

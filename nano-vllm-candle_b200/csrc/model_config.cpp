@@ -232,6 +232,15 @@ bool parse_latent(const JValue* m, nvc_latent_attn_spec& a, size_t i, Source&& s
   return true;
 }
 
+// the sizes of a gated delta rule mixer
+bool parse_delta(const JValue* m, nvc_delta_spec& d, std::string& err) {
+  if (!get_int(m, "heads", d.heads, 1, err) || !get_int(m, "kv_heads", d.kv_heads, 1, err) || !get_int(m, "dim", d.dim, 1, err) ||
+      !get_int(m, "vdim", d.vdim, 1, err) || !get_int(m, "conv", d.taps, 1, err))
+    return false;
+  if (d.heads % d.kv_heads != 0) { err = "heads must be a multiple of kv_heads"; return false; }
+  return true;
+}
+
 int parse_fefozen(const JValue& root, nvc_fefozen_config& c) {
   std::string err;
   if (!get_int(&root, "vocab", c.vocab, 1, err) || !get_int(&root, "width", c.width, 1, err)) return cfg_fail(err);
@@ -258,11 +267,7 @@ int parse_fefozen(const JValue& root, nvc_fefozen_config& c) {
       if (!parse_latent(m, a, i, source, err, false)) return cfg_fail(where + err);
     } else if (type->str == "delta") {
       L.kind = nvc_fefozen_layer::Delta;
-      auto& d = L.delta;
-      if (!get_int(m, "heads", d.heads, 1, err) || !get_int(m, "kv_heads", d.kv_heads, 1, err) || !get_int(m, "dim", d.dim, 1, err) ||
-          !get_int(m, "vdim", d.vdim, 1, err) || !get_int(m, "conv", d.taps, 1, err))
-        return cfg_fail(where + "mixer: " + err);
-      if (d.heads % d.kv_heads != 0) return cfg_fail(where + "mixer: heads must be a multiple of kv_heads");
+      if (!parse_delta(m, L.delta, err)) return cfg_fail(where + "mixer: " + err);
     } else {
       return cfg_fail(where + "mixer type `" + type->str + "` is not supported");
     }
@@ -440,6 +445,95 @@ int parse_buzutar(const JValue& root, nvc_buzutar_config& c) {
   return NVC_OK;
 }
 
+int parse_vizotar(const JValue& root, nvc_vizotar_config& c) {
+  std::string err;
+  if (!get_int(&root, "vocab", c.vocab, 1, err) || !get_int(&root, "width", c.width, 1, err) || !get_int(&root, "streams", c.streams, 1, err))
+    return cfg_fail(err);
+  if (c.streams > 16) return cfg_fail("at most 16 streams");
+  const JValue* norm = root.get("norm");
+  if (!norm || norm->kind != JValue::Obj || !get_float(norm, "eps", c.eps, err)) return cfg_fail("norm.eps: " + err);
+  const JValue* layers = root.get("layers");
+  if (!layers || layers->kind != JValue::Arr || layers->arr.empty()) return cfg_fail("`layers` must be a non-empty list");
+  const int n = (int)layers->arr.size();
+  for (int i = 0; i < n; ++i) {
+    const JValue& jl = layers->arr[i];
+    const std::string where = "layers[" + std::to_string(i) + "]: ";
+    if (jl.kind != JValue::Obj) return cfg_fail(where + "not an object");
+    nvc_vizotar_layer L;
+    if (const JValue* of = jl.get("weights_of"); of && of->kind != JValue::Null) {
+      if (!get_int(&jl, "weights_of", L.weights_of, 0, err)) return cfg_fail(where + err);
+      if (L.weights_of >= n || L.weights_of == i) return cfg_fail(where + "weights_of must name another layer");
+      c.layers.push_back(L);            // the rest comes from the named layer, below
+      continue;
+    }
+    const JValue* type = jl.get("type");
+    const JValue* m = jl.get("mixer");
+    if (!type || type->kind != JValue::Str) return cfg_fail(where + "missing `type`");
+    if (!m || m->kind != JValue::Obj) return cfg_fail(where + "missing `mixer`");
+    if (type->str == "parallel") {
+      L.kind = nvc_vizotar_layer::Parallel;
+      const JValue* l = m->get("left");
+      const JValue* r = m->get("right");
+      if (!l || l->kind != JValue::Obj || !r || r->kind != JValue::Obj) return cfg_fail(where + "a parallel mixer needs `left` and `right`");
+      auto& a = L.attn;
+      if (!get_int(l, "heads", a.heads, 1, err) || !get_int(l, "kv_heads", a.kv_heads, 1, err) || !get_int(l, "dim", a.dim, 1, err) ||
+          !get_int(l, "vdim", a.vdim, 1, err) || !get_int(l, "conv", a.taps, 1, err) || !get_float(l, "scale", a.scale, err) ||
+          !parse_rotary(l, a.rot, a.dim, err, true))
+        return cfg_fail(where + "mixer.left: " + err);
+      if (a.heads % a.kv_heads != 0) return cfg_fail(where + "mixer.left: heads must be a multiple of kv_heads");
+      if (a.taps > 16) return cfg_fail(where + "mixer.left: at most 16 taps");
+      if (const JValue* mask = l->get("mask"); mask && mask->kind != JValue::Null) {
+        if (mask->kind != JValue::Obj || !get_int(mask, "size", a.window, 1, err)) return cfg_fail(where + "mixer.left.mask: " + err);
+      }
+      auto& d = L.mem;
+      if (!get_int(r, "heads", d.heads, 1, err) || !get_int(r, "dim", d.dim, 1, err) || !get_int(r, "vdim", d.vdim, 1, err) ||
+          !get_float(r, "gate_cap", d.gate_cap, err))
+        return cfg_fail(where + "mixer.right: " + err);
+      if (!(d.gate_cap > 0.f)) return cfg_fail(where + "mixer.right: gate_cap must be positive");
+    } else if (type->str == "channel_delta") {
+      L.kind = nvc_vizotar_layer::ChannelDelta;
+      if (!parse_delta(m, L.delta, err)) return cfg_fail(where + "mixer: " + err);
+    } else {
+      return cfg_fail(where + "mixer type `" + type->str + "` is not supported");
+    }
+    const JValue* mlp = jl.get("mlp");
+    if (mlp && mlp->kind == JValue::Obj) {
+      const JValue* kind = mlp->get("kind");
+      if (!kind || kind->kind != JValue::Str) return cfg_fail(where + "mlp: missing `kind`");
+      if (kind->str == "dense") {
+        L.mlp.kind = nvc_routed_mlp_spec::Dense;
+        if (!get_int(mlp, "ff", L.mlp.ff, 1, err) || !get_float(mlp, "limit", L.mlp.limit, err)) return cfg_fail(where + "mlp: " + err);
+      } else if (kind->str == "moe") {
+        L.mlp.kind = nvc_routed_mlp_spec::Moe;
+        const JValue* r = mlp->get("router");
+        const JValue* e = mlp->get("expert");
+        if (!r || !e) return cfg_fail(where + "mlp: a mixture of experts needs `router` and `expert`");
+        if (!get_int(r, "experts", L.mlp.experts, 1, err) || !get_int(r, "top", L.mlp.top, 1, err) || !get_int(e, "ff", L.mlp.expert_ff, 1, err))
+          return cfg_fail(where + "mlp: " + err);
+        if (L.mlp.top > L.mlp.experts) return cfg_fail(where + "mlp: top exceeds the experts");
+        if (L.mlp.experts > 256) return cfg_fail(where + "mlp: at most 256 experts");
+      } else {
+        return cfg_fail(where + "mlp kind `" + kind->str + "` is not supported");
+      }
+    } else if (mlp && mlp->kind != JValue::Null) {
+      return cfg_fail(where + "`mlp` must be an object or null");
+    }
+    c.layers.push_back(L);
+  }
+  for (int i = 0; i < n; ++i) {
+    int j = i;
+    for (int hops = 0; c.layers[j].weights_of >= 0; ++hops) {
+      if (hops > n) return cfg_fail("layers[" + std::to_string(i) + "]: weights_of goes round in a circle");
+      j = c.layers[j].weights_of;
+    }
+    if (j == i) continue;
+    nvc_vizotar_layer L = c.layers[j];
+    L.weights_of = j;
+    c.layers[i] = L;
+  }
+  return NVC_OK;
+}
+
 }  // namespace
 
 std::vector<nvc_karuzen_config::Run> nvc_karuzen_config::runs() const {
@@ -495,10 +589,12 @@ int nvc_model_config_from_json(const char* text, nvc_model_config** out) {
     rc = parse_batatar(root, c->batatar);
   } else if (arch == "Buzutar") {
     rc = parse_buzutar(root, c->buzutar);
+  } else if (arch == "Vizotar") {
+    rc = parse_vizotar(root, c->vizotar);
   } else if (arch == "Qwen3ForCausalLM") {
     // parsed by nvc_qwen3_config_from_hf_dir (hf_loader.cpp) when loaded from a directory
   } else {
-    rc = cfg_fail("architecture `" + arch + "` is not registered (known: Qwen3ForCausalLM, Karuzen, Ranilix, Fefozen, Batatar, Buzutar)");
+    rc = cfg_fail("architecture `" + arch + "` is not registered (known: Qwen3ForCausalLM, Karuzen, Ranilix, Fefozen, Batatar, Buzutar, Vizotar)");
   }
   if (rc) { delete c; return rc; }
   *out = c;
@@ -526,6 +622,7 @@ int nvc_model_config_vocab(const nvc_model_config* c) {
   if (c->architecture == "Fefozen") return c->fefozen.vocab;
   if (c->architecture == "Batatar") return c->batatar.vocab;
   if (c->architecture == "Buzutar") return c->buzutar.vocab;
+  if (c->architecture == "Vizotar") return c->vizotar.vocab;
   return c->architecture == "Karuzen" ? c->karuzen.vocab : c->qwen3.vocab_size;
 }
 int nvc_model_config_layer_runs(const nvc_model_config* c, int32_t* layers, int32_t* passes, int32_t* readd, int capacity) {
@@ -536,6 +633,20 @@ int nvc_model_config_layer_runs(const nvc_model_config* c, int32_t* layers, int3
       if (layers) layers[i] = i;
       if (passes) passes[i] = 0;
       if (readd) readd[i] = 0;
+    }
+    return n;
+  }
+  if (c && c->architecture == "Vizotar") {      // a layer that runs another one's weights names that layer, with the count of earlier runs
+    const int n = (int)c->vizotar.layers.size();
+    std::vector<int> seen(n, 0);
+    for (int i = 0; i < n; ++i) {
+      const int j = c->vizotar.owner(i);
+      if (i < capacity) {
+        if (layers) layers[i] = j;
+        if (passes) passes[i] = seen[j];
+        if (readd) readd[i] = 0;
+      }
+      ++seen[j];
     }
     return n;
   }

@@ -191,8 +191,40 @@ struct nvc_buzutar_config {
   std::vector<nvc_buzutar_layer> layers;
 };
 
+// Vizotar: a stack of sequential pre-normed layers on several fp32 residual streams (hyper-connections): a sublayer reads a weighted sum
+// of the streams, and every stream is rebuilt from all the old ones plus the sublayer's output.  Mixers: "parallel" - grouped-query
+// window attention (biases, short convolutions, one norm over the whole query / key projection, rotate-half positions with YaRN
+// frequencies, a learned sink) beside a matrix memory (mLSTM: exponential input gate, sigmoid forget gate, max-stabilised state), each
+// side normed over the width and averaged - or "channel_delta" (the gated delta rule with a decay per head and key channel).
+// Feed-forward: dense clamped gated units or experts chosen by biased logits with a softmax over the chosen.  A layer may run another
+// layer's weights again with a cache and state of its own.  Tied logits.
+struct nvc_window_attn_spec {
+  int heads = 0, kv_heads = 0, dim = 0, vdim = 0, taps = 1;
+  float scale = 0.f;
+  nvc_rotary_spec rot;       // rotate-half pairs (i, i + dims / 2), optional YaRN frequencies
+  int window = 0;            // 0: every earlier token is visible; n: the token itself and the n - 1 before it
+};
+struct nvc_memory_spec {
+  int heads = 0, dim = 0, vdim = 0;
+  float gate_cap = 0.f;
+};
+struct nvc_vizotar_layer {
+  enum Kind { Parallel, ChannelDelta } kind = Parallel;
+  nvc_window_attn_spec attn;       // left half of "parallel"
+  nvc_memory_spec mem;             // right half of "parallel"
+  nvc_delta_spec delta;
+  nvc_routed_mlp_spec mlp;         // no identity experts; `limit` belongs to the dense kind
+  int weights_of = -1;             // >= 0: this layer runs that layer's weights (never the name of a layer that borrows itself)
+};
+struct nvc_vizotar_config {
+  int vocab = 0, width = 0, streams = 1;
+  float eps = 1e-5f;
+  std::vector<nvc_vizotar_layer> layers;
+  int owner(int i) const { return layers[i].weights_of < 0 ? i : layers[i].weights_of; }
+};
+
 struct nvc_model_config {
-  std::string architecture;   // "Qwen3ForCausalLM", "Karuzen", "Ranilix", "Fefozen", "Batatar" or "Buzutar"
+  std::string architecture;   // "Qwen3ForCausalLM", "Karuzen", "Ranilix", "Fefozen", "Batatar", "Buzutar" or "Vizotar"
   nvc_qwen3_config qwen3{};
   int qwen3_tied = 0;
   nvc_karuzen_config karuzen;
@@ -200,4 +232,5 @@ struct nvc_model_config {
   nvc_fefozen_config fefozen;
   nvc_batatar_config batatar;
   nvc_buzutar_config buzutar;
+  nvc_vizotar_config vizotar;
 };

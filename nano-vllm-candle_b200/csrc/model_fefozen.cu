@@ -25,6 +25,7 @@
 #include <vector>
 
 #include "latent_mixer.h"
+#include "routed_experts.h"
 #include "runner.h"
 
 namespace {
@@ -47,28 +48,21 @@ struct FLayerW {
   // dense ff
   void *w_up = nullptr, *w_down = nullptr;
   int ffp = 0;
-  // moe
-  void* router = nullptr;               // [Ep, Wp]
-  float* corr = nullptr;
-  int Ep = 0, effp = 0;
-  void *w_egu = nullptr, *w_edown = nullptr;   // [E][2 effp, Wp] (gate rows, then up rows at effp), [E][Wp, effp]
-  bool moe_tc = false;
+  nvc_experts_weights moe;
 };
 
 struct FefozenBody : nvc_latent_body {
   nvc_fefozen_config cfg;
   int Wp = 0, Vp = 0;
   int state_slots = 0;
-  bool use_moe_tc = true;
+  nvc_experts experts{{"mlp.correction", NVC_ROUTE_SOFTMAX, 0, NVC_ACT_GLU_CLAMP, kGluAlpha}};
   std::vector<FLayerW> L;
   void* embed = nullptr;
   float* fw = nullptr;
   // activations
   float *x0 = nullptr, *res = nullptr, *proj = nullptr, *mix = nullptr, *ffo = nullptr;
-  float *rq = nullptr, *rk = nullptr, *rv = nullptr, *ro = nullptr, *gb = nullptr, *zlog = nullptr, *tk_w = nullptr, *y = nullptr;
+  float *rq = nullptr, *rk = nullptr, *rv = nullptr, *ro = nullptr, *gb = nullptr;
   void *h = nullptr, *ao = nullptr, *act = nullptr, *hn = nullptr;
-  void *hid2 = nullptr, *hid = nullptr, *xs = nullptr;
-  int32_t *tk_idx = nullptr, *offsets = nullptr, *src_rows = nullptr, *pos = nullptr, *tile_group = nullptr;
   float* tap_host = nullptr;
   size_t tap_cap = 0;
 
@@ -89,15 +83,13 @@ struct FefozenBody : nvc_latent_body {
     return NVC_OK;
   }
 
-  static int moe_tiles(int pairs, int experts) { return (pairs + experts * 127 + 127) / 128; }
-
   int init(nvc_runner* r) {
     nvc_ctx* ctx = r->ctx;
     dt = r->dtype;
     esz = dt == NVC_DT_F32 ? 4 : 2;
     use_tc = dt == NVC_DT_BF16 && !(getenv("NVC_FEFOZEN_TC") && atoi(getenv("NVC_FEFOZEN_TC")) == 0);
     use_flash = use_tc && !(getenv("NVC_FEFOZEN_FLASH") && atoi(getenv("NVC_FEFOZEN_FLASH")) == 0);
-    use_moe_tc = use_tc && !(getenv("NVC_FEFOZEN_MOE_TC") && atoi(getenv("NVC_FEFOZEN_MOE_TC")) == 0);
+    experts.use_tc = use_tc && !(getenv("NVC_FEFOZEN_MOE_TC") && atoi(getenv("NVC_FEFOZEN_MOE_TC")) == 0);
     Wp = pad64(cfg.width);
     Vp = pad64(cfg.vocab);
     state_slots = cfg.has_state() ? r->opt.max_num_seqs : 0;
@@ -106,7 +98,6 @@ struct FefozenBody : nvc_latent_body {
     int rc;
     L.resize(cfg.layers.size());
     size_t m_np = 0, m_ow = 0, m_ff = 0, m_dqk = 0, m_dv = 0, m_gb = 0;
-    size_t m_Ep = 0, m_top = 0, m_E = 0, m_hid = 0, m_pairs_rows = 0, m_tiles = 0;
     int64_t wbytes = 0;
     const int W = cfg.width;
     for (size_t i = 0; i < cfg.layers.size(); ++i) {
@@ -163,26 +154,7 @@ struct FefozenBody : nvc_latent_body {
         wbytes += (int64_t)esz * 2 * f.ff * W;
         m_ff = std::max(m_ff, (size_t)w.ffp);
       } else if (f.kind == nvc_routed_mlp_spec::Moe) {
-        const int Et = f.experts + f.identity;
-        w.Ep = pad64(Et);
-        w.effp = pad64(f.expert_ff);
-        w.moe_tc = use_moe_tc && f.experts > 0 && w.effp >= 128;
-        if ((rc = zalloc(r, &w.router, (size_t)w.Ep * Wp * esz)) || (rc = zalloc(r, &w.corr, Et * 4))) return rc;
-        want[p + "mlp.router"] = false;
-        want[p + "mlp.correction"] = false;
-        if (f.experts > 0 &&
-            ((rc = zalloc(r, &w.w_egu, (size_t)f.experts * 2 * w.effp * Wp * esz)) || (rc = zalloc(r, &w.w_edown, (size_t)f.experts * Wp * w.effp * esz))))
-          return rc;
-        for (int e = 0; e < f.experts; ++e)
-          for (const char* n : {"gate", "up", "down"}) want[p + "mlp.e" + std::to_string(e) + "." + n] = false;
-        wbytes += (int64_t)esz * ((int64_t)Et * W + (int64_t)f.experts * 3 * f.expert_ff * W);
-        m_Ep = std::max(m_Ep, (size_t)w.Ep);
-        m_top = std::max(m_top, (size_t)f.top);
-        m_E = std::max(m_E, (size_t)Et);
-        m_hid = std::max(m_hid, (size_t)w.effp);
-        const size_t rows = w.moe_tc ? (size_t)moe_tiles((int)T * f.top, Et) * 128 : T * f.top;
-        m_pairs_rows = std::max(m_pairs_rows, rows);
-        if (w.moe_tc) m_tiles = std::max(m_tiles, (size_t)moe_tiles((int)T * f.top, Et));
+        if ((rc = experts.init(*this, r, f, p, W, T, w.moe, &wbytes))) return rc;
       }
     }
     if ((rc = zalloc(r, &embed, (size_t)Vp * Wp * esz)) || (rc = zalloc(r, &fw, W * 4))) return rc;
@@ -199,14 +171,7 @@ struct FefozenBody : nvc_latent_body {
                  (rc = zalloc(r, &ro, T * m_dv * 4)) || (rc = zalloc(r, &gb, T * m_gb * 4))))
       return rc;
     if (m_ff && (rc = zalloc(r, &act, T * m_ff * esz))) return rc;
-    if (m_E) {
-      if ((rc = zalloc(r, &zlog, T * m_Ep * 4)) || (rc = zalloc(r, &tk_idx, T * m_top * 4)) || (rc = zalloc(r, &tk_w, T * m_top * 4)) ||
-          (rc = zalloc(r, &offsets, (m_E + 1) * 4)) || (rc = zalloc(r, &src_rows, m_pairs_rows * 4)) || (rc = zalloc(r, &pos, T * m_top * 4)) ||
-          (rc = zalloc(r, &hid2, m_pairs_rows * 2 * m_hid * esz)) || (rc = zalloc(r, &hid, m_pairs_rows * m_hid * esz)) ||
-          (rc = zalloc(r, &y, m_pairs_rows * Wp * 4)))
-        return rc;
-      if (m_tiles && ((rc = zalloc(r, &tile_group, m_tiles * 4)) || (rc = zalloc(r, &xs, m_pairs_rows * Wp * esz)))) return rc;
-    }
+    if ((rc = experts.alloc(*this, r, Wp, T))) return rc;
     return NVC_OK;
   }
 
@@ -251,6 +216,14 @@ struct FefozenBody : nvc_latent_body {
           return rc;
         }
       }
+      {
+        bool taken = false;
+        rc = experts.load(*this, r, f, W, w.moe, sub, v, d0, d1, bad, &taken);
+        if (taken) {
+          it->second = rc == NVC_OK;
+          return rc;
+        }
+      }
       if (sub == "norm1") rc = vec(w.n1, W);
       else if (sub == "norm1b") rc = vec(w.n1b, W);
       else if (sub == "norm2") rc = vec(w.n2, W);
@@ -277,20 +250,6 @@ struct FefozenBody : nvc_latent_body {
       else if (!latent && sub == "mix.norm") rc = vec(w.onorm, d.vdim);
       else if (sub == "mlp.up") { if (!shape_is(f.ff, W)) return bad(); rc = put_matrix(r, w.w_up, Wp, 0, 0, v.data(), f.ff, W, W, 1); }
       else if (sub == "mlp.down") { if (!shape_is(W, f.ff)) return bad(); rc = put_matrix(r, w.w_down, w.ffp, 0, 0, v.data(), W, f.ff, f.ff, 1); }
-      else if (sub == "mlp.router") { if (!shape_is(f.experts + f.identity, W)) return bad(); rc = put_matrix(r, w.router, Wp, 0, 0, v.data(), f.experts + f.identity, W, W, 1); }
-      else if (sub == "mlp.correction") rc = vec(w.corr, f.experts + f.identity);
-      else if (sub.rfind("mlp.e", 0) == 0) {
-        const size_t d2 = sub.find('.', 5);
-        const int e = atoi(sub.substr(5, d2 - 5).c_str());
-        const std::string part = sub.substr(d2 + 1);
-        uint8_t* gu = reinterpret_cast<uint8_t*>(w.w_egu) + (size_t)e * 2 * w.effp * Wp * esz;
-        if (part == "gate") { if (!shape_is(f.expert_ff, W)) return bad(); rc = put_matrix(r, gu, Wp, 0, 0, v.data(), f.expert_ff, W, W, 1); }
-        else if (part == "up") { if (!shape_is(f.expert_ff, W)) return bad(); rc = put_matrix(r, gu, Wp, w.effp, 0, v.data(), f.expert_ff, W, W, 1); }
-        else if (part == "down") {
-          if (!shape_is(W, f.expert_ff)) return bad();
-          rc = put_matrix(r, reinterpret_cast<uint8_t*>(w.w_edown) + (size_t)e * Wp * w.effp * esz, w.effp, 0, 0, v.data(), W, f.expert_ff, f.expert_ff, 1);
-        }
-      }
     }
     if (rc == NVC_OK) it->second = true;
     return rc;
@@ -331,59 +290,6 @@ struct FefozenBody : nvc_latent_body {
     mark(r, "delta_scan");
     rc = nvc_head_gate_w(ctx, ro, p.ldv, proj + w.g_off, w.np, w.onorm, ao, w.owp, dt, d.heads, d.vdim, 1, cfg.eps, NVC_GATE_SILU, 1.f, s.N, st);
     mark(r, "head_gate");
-    return rc;
-  }
-
-  int moe_ff(nvc_runner* r, const nvc_step_shape& s, int li) {
-    nvc_ctx* ctx = r->ctx;
-    void* st = r->stream;
-    const auto& f = cfg.layers[li].mlp;
-    FLayerW& w = L[li];
-    const int N = s.N, W = cfg.width, Et = f.experts + f.identity, P = N * f.top;
-    int rc;
-    if (use_tc) {
-      if ((rc = linear(r, h, Wp, w.router, zlog, w.Ep, NVC_DT_F32, N, w.Ep, Wp))) return rc;
-    } else if ((rc = nvc_linear(ctx, h, Wp, 0, w.router, Wp, 0, zlog, w.Ep, 0, dt, NVC_DT_F32, N, Et, Wp, 1, NVC_ACT_NONE, st))) {
-      return rc;
-    }
-    if ((rc = nvc_moe_route_logits_ex(ctx, zlog, w.Ep, w.corr, Et, f.top, 1.f, -1, NVC_ROUTE_SOFTMAX, 0, tk_idx, tk_w, nullptr, N, st))) return rc;
-    mark(r, "moe_route");
-    if (f.experts > 0 && w.moe_tc) {
-      const int tiles = moe_tiles(P, Et), mcap = tiles * 128;
-      if ((rc = nvc_moe_sort_padded_ex(ctx, tk_idx, N, f.top, Et, f.experts, 128, offsets, src_rows, pos, tile_group, tiles, st))) return rc;
-      mark(r, "moe_sort");
-      if ((rc = nvc_gather_rows_bf16(ctx, reinterpret_cast<const nvc_bf16*>(h), Wp, src_rows, offsets + f.experts, reinterpret_cast<nvc_bf16*>(xs), Wp,
-                                     mcap, Wp, st)))
-        return rc;
-      mark(r, "moe_gather");
-      if ((rc = nvc_gemm_bf16_grouped(ctx, reinterpret_cast<const nvc_bf16*>(xs), Wp, reinterpret_cast<const nvc_bf16*>(w.w_egu), hid2, 2 * w.effp,
-                                      NVC_DT_BF16, mcap, 2 * w.effp, Wp, tile_group, f.experts, NVC_ACT_NONE, st)))
-        return rc;
-      mark(r, "moe_gate_up");
-      if ((rc = nvc_act_mul_p(ctx, hid2, 2 * w.effp, hid, w.effp, dt, mcap, f.expert_ff, w.effp, NVC_ACT_GLU_CLAMP, f.limit, kGluAlpha, st))) return rc;
-      mark(r, "moe_glu");
-      if ((rc = nvc_gemm_bf16_grouped(ctx, reinterpret_cast<const nvc_bf16*>(hid), w.effp, reinterpret_cast<const nvc_bf16*>(w.w_edown), y, Wp, NVC_DT_F32,
-                                      mcap, Wp, w.effp, tile_group, f.experts, NVC_ACT_NONE, st)))
-        return rc;
-      mark(r, "moe_down");
-    } else {
-      if ((rc = nvc_moe_sort(ctx, tk_idx, N, f.top, Et, offsets, src_rows, pos, st))) return rc;
-      mark(r, "moe_sort");
-      if (f.experts > 0) {
-        if ((rc = nvc_linear_grouped(ctx, h, Wp, src_rows, w.w_egu, Wp, (int64_t)2 * w.effp * Wp, hid2, 2 * w.effp, offsets, f.experts, P, dt, dt,
-                                     2 * w.effp, Wp, NVC_ACT_NONE, st)))
-          return rc;
-        mark(r, "moe_gate_up");
-        if ((rc = nvc_act_mul_p(ctx, hid2, 2 * w.effp, hid, w.effp, dt, P, f.expert_ff, w.effp, NVC_ACT_GLU_CLAMP, f.limit, kGluAlpha, st))) return rc;
-        mark(r, "moe_glu");
-        if ((rc = nvc_linear_grouped(ctx, hid, w.effp, nullptr, w.w_edown, w.effp, (int64_t)Wp * w.effp, y, Wp, offsets, f.experts, P, dt, NVC_DT_F32, Wp,
-                                     w.effp, NVC_ACT_NONE, st)))
-          return rc;
-        mark(r, "moe_down");
-      }
-    }
-    rc = nvc_moe_combine_identity(ctx, y, NVC_DT_F32, Wp, pos, tk_w, tk_idx, f.top, f.experts, h, dt, Wp, ffo, Wp, N, W, st);
-    mark(r, "moe_combine");
     return rc;
   }
 
@@ -437,7 +343,7 @@ struct FefozenBody : nvc_latent_body {
         mark(r, "gemm_up");
         if ((rc = linear(r, act, w.ffp, w.w_down, ffo, Wp, NVC_DT_F32, N, Wp, w.ffp))) return rc;
         mark(r, "gemm_down");
-      } else if ((rc = moe_ff(r, s, (int)i))) {
+      } else if ((rc = experts.run(*this, r, f, w.moe, h, ffo, N, W))) {
         return rc;
       }
       pend = ffo;

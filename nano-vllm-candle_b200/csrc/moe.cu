@@ -81,14 +81,25 @@ __global__ void moe_topk_kernel(const float* __restrict__ z, int ldz, const floa
     den = warp_sum(den);
 #pragma unroll
     for (int i = 0; i < kMaxPerLane; ++i) s[i] = s[i] / den;
+  } else if (score == NVC_ROUTE_CHOSEN) { // choice by biased logits; the scores are their exponentials (the largest logit is always chosen)
+    float mx = -INFINITY;
+#pragma unroll
+    for (int i = 0; i < kMaxPerLane; ++i)
+      if (lane + 32 * i < E) { c[i] = s[i] + __ldg(corr + lane + 32 * i); mx = fmaxf(mx, c[i]); }
+    mx = warp_max(mx);
+#pragma unroll
+    for (int i = 0; i < kMaxPerLane; ++i)
+      if (lane + 32 * i < E) s[i] = expf(c[i] - mx);
   } else {
 #pragma unroll
     for (int i = 0; i < kMaxPerLane; ++i)
       if (lane + 32 * i < E) s[i] = sigmoid_f32(s[i]);
   }
+  if (score != NVC_ROUTE_CHOSEN) {
 #pragma unroll
-  for (int i = 0; i < kMaxPerLane; ++i)
-    if (lane + 32 * i < E) c[i] = s[i] + __ldg(corr + lane + 32 * i);
+    for (int i = 0; i < kMaxPerLane; ++i)
+      if (lane + 32 * i < E) c[i] = s[i] + __ldg(corr + lane + 32 * i);
+  }
   if (gate_col >= 0 && gate && lane == 0) gate[n] = sigmoid_f32(zr[gate_col]);
   topk_write(s, c, lane, E, top, scale, idx, wout, n, normalize != 0);
 }
@@ -323,7 +334,7 @@ int nvc_moe_route_logits(nvc_ctx* ctx, const float* z, int ldz, const float* cor
 int nvc_moe_route_logits_ex(nvc_ctx* ctx, const float* z, int ldz, const float* correction, int E, int top, float scale, int gate_col,
                             int score, int normalize, int32_t* topk_idx, float* topk_w, float* gate, int N, void* stream) {
   NVC_REQUIRE(ctx, ctx && z && correction && topk_idx && topk_w, NVC_EINVAL, "null pointer");
-  NVC_REQUIRE(ctx, score == NVC_ROUTE_SIGMOID || score == NVC_ROUTE_SOFTMAX, NVC_EINVAL, "unknown score function");
+  NVC_REQUIRE(ctx, score >= NVC_ROUTE_SIGMOID && score <= NVC_ROUTE_CHOSEN, NVC_EINVAL, "unknown score function");
   NVC_REQUIRE(ctx, E > 0 && E <= 32 * kMaxPerLane && top > 0 && top <= E, NVC_ESHAPE, "experts must be in [1, 256], top in [1, experts]");
   NVC_REQUIRE(ctx, N >= 0 && ldz >= E && gate_col < ldz && (gate_col < 0 || gate), NVC_EINVAL, "bad sizes");
   if (N == 0) return NVC_OK;

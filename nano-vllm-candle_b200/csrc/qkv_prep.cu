@@ -10,7 +10,8 @@
 //   v *= v_scale                             (a constant weight of the mixer, so that every attention kernel can leave it out)
 //   stores                                   q to its buffer; k and v to rows of a paged cache (slot mapping) or to plain rows
 // One warp per (token, head) of q, k or v; a head is staged in shared memory so that any pairing reads its partner.  The purely
-// element-wise case (bias and silu only, plain fp32 rows out) runs a flat kernel with 16-byte accesses instead.
+// element-wise case (bias and silu only, plain fp32 rows out) runs a flat kernel with 16-byte accesses instead.  With a short causal
+// convolution behind the bias, or norms that span the whole query / key projection, one CTA takes a whole token (prep_token_kernel).
 #include "typed.cuh"
 
 #include <algorithm>
@@ -117,6 +118,167 @@ __global__ void __launch_bounds__(256) prep_flat_kernel(const PrepArgs a) {
   *reinterpret_cast<float4*>(out) = v;
 }
 
+// four neighbouring numbers in the storage format with one store
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
+  uint2 u;
+  u.x = pack_bf16(v.x, v.y);
+  u.y = pack_bf16(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+
+__device__ __forceinline__ int prep_find_seq(const int32_t* cu, int B, int row) {
+  int lo = 0, hi = B - 1;      // largest b with cu[b] <= row
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu[mid] <= row) lo = mid; else hi = mid - 1;
+  }
+  return lo;
+}
+
+// One CTA per token: bias, short causal convolution, activation (the whole row [q | k | v] waits in shared memory), the norms over the
+// whole query and key projection - or none - then rotation and stores.  P: numbers per access (4: every width, offset and stride is a
+// multiple of 4 and the pointers are 16-byte aligned).
+template <typename TQ, typename TKV, int P>
+__global__ void __launch_bounds__(256) prep_token_kernel(const PrepArgs a, const nvc_short_conv cv) {
+  extern __shared__ __align__(16) float row[];          // [qw + kw + vw]
+  __shared__ float part[2][8];
+  __shared__ int s_r0, s_fresh, s_slot;
+  pdl_trigger();
+  const nvc_qkv_prep& p = a.p;
+  const int qw = p.q_heads * p.dim, kw = p.kv_heads * p.dim, vw = p.kv_heads * p.vdim, C = qw + kw + vw;
+  const int64_t n = blockIdx.x;
+  if (cv.w && threadIdx.x == 0) {
+    int b = (int)n, r0 = (int)n;
+    if (cv.cu_seqlens) {
+      b = prep_find_seq(cv.cu_seqlens, cv.B, (int)n);
+      r0 = cv.cu_seqlens[b];
+    }
+    s_r0 = r0;
+    s_fresh = p.positions[r0] == 0;
+    s_slot = cv.state_slots[b];
+  }
+  const int64_t orow = p.slot_mapping ? p.slot_mapping[n] : n;
+  pdl_wait();
+  __syncthreads();
+  const int step = P * blockDim.x;
+  float sq = 0.f, sk = 0.f;
+  for (int c = P * threadIdx.x; c < C; c += step) {
+    const int col = c < qw ? p.q_off + c : (c < qw + kw ? p.k_off + c - qw : p.v_off + c - qw - kw);
+    float b[P], y[P];
+    if constexpr (P == 4) {
+      const float4 t = p.bias ? *reinterpret_cast<const float4*>(p.bias + col) : make_float4(0.f, 0.f, 0.f, 0.f);
+      b[0] = t.x; b[1] = t.y; b[2] = t.z; b[3] = t.w;
+    } else {
+      b[0] = p.bias ? __ldg(p.bias + col) : 0.f;
+    }
+    if (cv.w) {
+      const int keep = cv.taps - 1, t = (int)n - s_r0;
+      float* st = cv.state + (int64_t)s_slot * keep * C + c;
+      const bool shift = cv.cu_seqlens == nullptr;      // one row per sequence: this CTA is the state's only reader
+#pragma unroll
+      for (int e = 0; e < P; ++e) y[e] = 0.f;
+      for (int i = 0; i < cv.taps; ++i) {
+        const int src = t - keep + i;                   // the input's index inside the portion; negative: in front of it
+        float x[P];
+        if (src >= 0) {
+          const float* xp = p.in + (s_r0 + src) * (int64_t)p.ldi + col;
+          if constexpr (P == 4) {
+            const float4 v = *reinterpret_cast<const float4*>(xp);
+            x[0] = v.x + b[0]; x[1] = v.y + b[1]; x[2] = v.z + b[2]; x[3] = v.w + b[3];
+          } else {
+            x[0] = *xp + b[0];
+          }
+        } else {
+          const float* sp = st + (int64_t)(keep + src) * C;
+#pragma unroll
+          for (int e = 0; e < P; ++e) x[e] = 0.f;
+          if (!s_fresh) {
+            if constexpr (P == 4) {
+              const float4 v = *reinterpret_cast<const float4*>(sp);
+              x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
+            } else {
+              x[0] = *sp;
+            }
+          }
+        }
+        const float* wp = cv.w + (int64_t)i * C + c;
+        if constexpr (P == 4) {
+          const float4 w = __ldg(reinterpret_cast<const float4*>(wp));
+          y[0] = fmaf(w.x, x[0], y[0]); y[1] = fmaf(w.y, x[1], y[1]); y[2] = fmaf(w.z, x[2], y[2]); y[3] = fmaf(w.w, x[3], y[3]);
+        } else {
+          y[0] = fmaf(__ldg(wp), x[0], y[0]);
+        }
+        if (shift && i > 0) {                           // input i becomes input i - 1 of the next step (read before, by this thread)
+          float* dp = st + (int64_t)(i - 1) * C;
+          if constexpr (P == 4) *reinterpret_cast<float4*>(dp) = make_float4(x[0], x[1], x[2], x[3]);
+          else *dp = x[0];
+        }
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < P; ++e) y[e] = p.in[n * p.ldi + col + e] + b[e];
+    }
+#pragma unroll
+    for (int e = 0; e < P; ++e) {
+      if (p.act == NVC_PREP_ACT_SILU) y[e] *= sigmoid_f32(y[e]);
+      row[c + e] = y[e];
+      if (c + e < qw) sq += y[e] * y[e];
+      else if (c + e < qw + kw) sk += y[e] * y[e];
+    }
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) { part[0][threadIdx.x >> 5] = sq; part[1][threadIdx.x >> 5] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) { sq += part[0][w]; sk += part[1][w]; }
+  const float rq = p.q_norm ? 1.0f / sqrtf(sq / (float)qw + p.eps) : 1.f, rk = p.k_norm ? 1.0f / sqrtf(sk / (float)kw + p.eps) : 1.f;
+  const int half = p.rot_dims >> 1;
+  const float2* tab = reinterpret_cast<const float2*>(p.rot_table) + (int64_t)(p.rot_dims ? p.positions[n] : 0) * half;
+  for (int c = P * threadIdx.x; c < C; c += step) {
+    float y[P];
+    if (c >= qw + kw) {
+      if (orow < 0) continue;
+#pragma unroll
+      for (int e = 0; e < P; ++e) y[e] = row[c + e] * p.v_scale;
+      TKV* o = reinterpret_cast<TKV*>(p.v_out) + orow * p.ldv + c - qw - kw;
+      if constexpr (P == 4) store4(o, make_float4(y[0], y[1], y[2], y[3]));
+      else st_f(o, y[0]);
+      continue;
+    }
+    const bool is_q = c < qw;
+    if (!is_q && orow < 0) continue;
+    const int c0 = is_q ? 0 : qw, cc = c - c0, j0 = cc % p.dim;
+    const float r = is_q ? rq : rk, post = is_q ? 1.f : p.k_scale;
+    const float* nw = is_q ? p.q_norm : p.k_norm;
+    const float* x = row + c0;
+#pragma unroll
+    for (int e = 0; e < P; ++e) {
+      const int j = j0 + e, k = cc + e;                 // number inside its head, number inside the projection
+      float z = x[k] * r * (nw ? __ldg(nw + k) : 1.f);
+      if (j < p.rot_dims) {
+        int i, kp;
+        float sign;
+        if (p.rot_half) { i = j < half ? j : j - half; kp = j < half ? k + half : k - half; sign = j < half ? -1.f : 1.f; }
+        else { i = j >> 1; kp = k - j + (j ^ 1); sign = (j & 1) ? 1.f : -1.f; }
+        const float2 cs = __ldg(tab + i);
+        z = z * cs.x + sign * (x[kp] * r * (nw ? __ldg(nw + kp) : 1.f)) * cs.y;
+      }
+      y[e] = z * post;
+    }
+    if (is_q) {
+      TQ* o = reinterpret_cast<TQ*>(p.q_out) + n * p.ldq + cc;
+      if constexpr (P == 4) store4(o, make_float4(y[0], y[1], y[2], y[3]));
+      else st_f(o, y[0]);
+    } else {
+      TKV* o = reinterpret_cast<TKV*>(p.k_out) + orow * p.ldk + cc;
+      if constexpr (P == 4) store4(o, make_float4(y[0], y[1], y[2], y[3]));
+      else st_f(o, y[0]);
+    }
+  }
+}
+
 // one warp per (token, head) of a query projection laid out [heads][dim | rot_dim]: the unrotated part goes to out_a, the rotated
 // part (turned by the token's position) to out_b
 template <typename T>
@@ -148,15 +310,6 @@ __global__ void head_split_rot_kernel(const float* __restrict__ in, int ldi, int
     }
     st_f(b + j, y);
   }
-}
-
-// four neighbouring numbers in the storage format with one store
-__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
-  uint2 u;
-  u.x = pack_bf16(v.x, v.y);
-  u.y = pack_bf16(v.z, v.w);
-  *reinterpret_cast<uint2*>(p) = u;
 }
 
 // one CTA per token: the sums of squares of the whole query and the whole key projection in one pass (the key rows leave for the cache
@@ -257,6 +410,28 @@ int launch_prep(nvc_ctx* ctx, const nvc_qkv_prep* p, int N, void* stream) {
   return NVC_OK;
 }
 
+template <typename TQ, typename TKV>
+int launch_prep_token(nvc_ctx* ctx, const nvc_qkv_prep* p, int N, void* stream) {
+  PrepArgs a{*p, N};
+  nvc_short_conv cv{};
+  if (p->conv) cv = *p->conv;
+  const int qw = p->q_heads * p->dim, kw = p->kv_heads * p->dim, vw = p->kv_heads * p->vdim;
+  auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = ((p->dim | kw | vw | p->q_off | p->k_off | p->v_off | p->ldi | p->ldq | p->ldk | p->ldv) & 3) == 0 && al16(p->in) && al16(p->bias) &&
+                   al16(cv.w) && al16(cv.state) && al16(p->q_out) && al16(p->k_out) && al16(p->v_out);
+  const size_t smem = (size_t)(qw + kw + vw) * sizeof(float);
+  static bool attr_set = false;
+  if (!attr_set && smem > 48 * 1024) {
+    NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(prep_token_kernel<TQ, TKV, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(prep_token_kernel<TQ, TKV, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    attr_set = true;
+  }
+  if (vec) NVC_CUDA_CHECK(ctx, nvc_launch(ctx, prep_token_kernel<TQ, TKV, 4>, dim3((unsigned)N), dim3(256), smem, nvc_stream(stream), a, cv));
+  else NVC_CUDA_CHECK(ctx, nvc_launch(ctx, prep_token_kernel<TQ, TKV, 1>, dim3((unsigned)N), dim3(256), smem, nvc_stream(stream), a, cv));
+  ctx->launches++;
+  return NVC_OK;
+}
+
 }  // namespace
 
 extern "C" int nvc_qkv_prep_run(nvc_ctx* ctx, const nvc_qkv_prep* p, int N, void* stream) {
@@ -271,7 +446,23 @@ extern "C" int nvc_qkv_prep_run(nvc_ctx* ctx, const nvc_qkv_prep* p, int N, void
               NVC_EINVAL, "value blending needs its buffer and weight");
   NVC_REQUIRE(ctx, p->ldq >= p->q_heads * p->dim && p->ldk >= p->kv_heads * p->dim && p->ldv >= p->kv_heads * p->vdim, NVC_EINVAL,
               "bad strides");
+  if (p->conv) {
+    const nvc_short_conv& cv = *p->conv;
+    NVC_REQUIRE(ctx, cv.w && cv.state && cv.state_slots && p->positions && cv.taps >= 1 && cv.taps <= 16 && cv.B > 0 && (cv.cu_seqlens || N == cv.B),
+                NVC_EINVAL, "bad convolution arguments");
+    NVC_REQUIRE(ctx, p->k_off == p->q_off + p->q_heads * p->dim && p->v_off == p->k_off + p->kv_heads * p->dim, NVC_EINVAL,
+                "a convolution reads neighbouring q, k and v columns");
+  }
   if (N == 0) return NVC_OK;
+  if (p->conv || p->wide_norm) {
+    NVC_REQUIRE(ctx, p->blend == NVC_BLEND_NONE && !p->unit_norm && (p->wide_norm || !p->q_norm), NVC_ENOTIMPL,
+                "a convolution goes with whole-projection norms or none, and without blending");
+    NVC_REQUIRE(ctx, (size_t)(p->q_heads * p->dim + p->kv_heads * (p->dim + p->vdim)) * sizeof(float) <= 200 * 1024, NVC_ESHAPE,
+                "q, k and v of one token above 200 KB");
+    if (p->q_dtype == NVC_DT_F32 && p->kv_dtype == NVC_DT_F32) return launch_prep_token<float, float>(ctx, p, N, stream);
+    if (p->q_dtype == NVC_DT_BF16 && p->kv_dtype == NVC_DT_BF16) return launch_prep_token<__nv_bfloat16, __nv_bfloat16>(ctx, p, N, stream);
+    return NVC_ENOTIMPL;
+  }
   {
     auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
     const int qw = p->q_heads * p->dim, kw = p->kv_heads * p->dim, vw = p->kv_heads * p->vdim;

@@ -1019,6 +1019,7 @@ nvc_model_body* nvc_make_ranilix_body(nvc_runner* r, const nvc_ranilix_config& c
 nvc_model_body* nvc_make_fefozen_body(nvc_runner* r, const nvc_fefozen_config& cfg, int* status);   // model_fefozen.cu
 nvc_model_body* nvc_make_batatar_body(nvc_runner* r, const nvc_batatar_config& cfg, int* status);   // model_batatar.cu
 nvc_model_body* nvc_make_buzutar_body(nvc_runner* r, const nvc_buzutar_config& cfg, int* status);   // model_buzutar.cu
+nvc_model_body* nvc_make_vizotar_body(nvc_runner* r, const nvc_vizotar_config& cfg, int* status);   // model_vizotar.cu
 
 extern "C" int nvc_runner_create_from_config(nvc_ctx* ctx, const nvc_model_config* mc, const nvc_runner_options* opt,
                                              nvc_runner** out) {
@@ -1029,7 +1030,7 @@ extern "C" int nvc_runner_create_from_config(nvc_ctx* ctx, const nvc_model_confi
     return nvc_runner_create(ctx, &mc->qwen3, opt, out);
   }
   NVC_REQUIRE(ctx, mc->architecture == "Karuzen" || mc->architecture == "Ranilix" || mc->architecture == "Fefozen" || mc->architecture == "Batatar" ||
-                       mc->architecture == "Buzutar",
+                       mc->architecture == "Buzutar" || mc->architecture == "Vizotar",
               NVC_ENOTIMPL,
               "architecture " + mc->architecture + " has no model body");
   NVC_REQUIRE(ctx, ctx->tp_size == 1, NVC_ENOTIMPL, mc->architecture + " runs on one GPU");
@@ -1052,6 +1053,7 @@ extern "C" int nvc_runner_create_from_config(nvc_ctx* ctx, const nvc_model_confi
   else if (mc->architecture == "Fefozen") r->body = nvc_make_fefozen_body(r, mc->fefozen, &rc);
   else if (mc->architecture == "Batatar") r->body = nvc_make_batatar_body(r, mc->batatar, &rc);
   else if (mc->architecture == "Buzutar") r->body = nvc_make_buzutar_body(r, mc->buzutar, &rc);
+  else if (mc->architecture == "Vizotar") r->body = nvc_make_vizotar_body(r, mc->vizotar, &rc);
   else r->body = nvc_make_karuzen_body(r, mc->karuzen, &rc);
   if (rc) return rc;
   r->V_l = r->body->vocab();

@@ -5,8 +5,8 @@
 //   dt_h                     softplus(projection + dt_bias_h), no clamp
 //   outputs                  x, v = dt x (what the recurrence adds to the state, with B as its key), B, C,
 //                            log decay = -exp(A_log_h) dt   (the recurrence multiplies the state by its exponential)
-// nvc_ssd_conv_advance then writes every sequence's last taps - 1 inputs into its state slot (a portion shorter than that keeps the
-// tail of what the slot held).  It runs behind the first kernel on the same stream, which still reads the old state.
+// nvc_ssd_conv_advance then moves the convolution state past the step (nvc_short_conv_advance, behind the first kernel on the same
+// stream, which still reads the old state).
 // The recurrence itself is nvc_decay_scan (retention.cu) with q = C, k = B, a decay per token and head and the skip term D x.
 #include "typed.cuh"
 
@@ -109,34 +109,6 @@ __global__ void __launch_bounds__(kPrepThreads) ssd_prep_kernel(const SsdArgs a)
   else out[0] = y[0];
 }
 
-// thread = (sequence, channel): reads the taps - 1 inputs that end the sequence so far, then writes them
-__global__ void ssd_conv_advance_kernel(const SsdArgs a) {
-  pdl_trigger();
-  pdl_wait();
-  const nvc_ssd_prep& p = a.p;
-  const int C = p.heads * p.vdim + 2 * p.groups * p.state, keep = p.taps - 1;
-  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= (int64_t)p.B * C) return;
-  const int b = (int)(i / C), c = (int)(i % C);
-  const int r0 = p.cu_seqlens ? p.cu_seqlens[b] : b;
-  const int r1 = p.cu_seqlens ? p.cu_seqlens[b + 1] : b + 1;
-  const int qlen = r1 - r0;
-  const bool fresh = p.positions[r0] == 0;
-  float* st = p.conv_state + (int64_t)p.state_slots[b] * keep * C;
-  float v[kMaxTaps];
-#pragma unroll
-  for (int j = 0; j < kMaxTaps; ++j) {
-    if (j < keep) {
-      const int idx = qlen - keep + j;
-      if (idx >= 0) v[j] = p.in[(int64_t)(r0 + idx) * p.ldi + p.xbc_off + c];
-      else v[j] = fresh ? 0.f : st[(int64_t)(keep + idx) * C + c];
-    }
-  }
-#pragma unroll
-  for (int j = 0; j < kMaxTaps; ++j)
-    if (j < keep) st[(int64_t)j * C + c] = v[j];
-}
-
 int check(nvc_ctx* ctx, const nvc_ssd_prep* p) {
   NVC_REQUIRE(ctx, ctx && p && p->in && p->conv_w && p->conv_b && p->conv_state && p->state_slots && p->positions, NVC_EINVAL, "null pointer");
   NVC_REQUIRE(ctx, p->heads > 0 && p->vdim > 0 && p->groups > 0 && p->heads % p->groups == 0 && p->state > 0 && p->taps >= 1 && p->taps <= kMaxTaps &&
@@ -175,11 +147,6 @@ extern "C" int nvc_ssd_prep_run(nvc_ctx* ctx, const nvc_ssd_prep* p, int N, void
 extern "C" int nvc_ssd_conv_advance(nvc_ctx* ctx, const nvc_ssd_prep* p, void* stream) {
   int rc = check(ctx, p);
   if (rc) return rc;
-  if (p->taps == 1) return NVC_OK;
-  const int C = p->heads * p->vdim + 2 * p->groups * p->state;
-  SsdArgs a{*p, 0};
-  const int64_t total = (int64_t)p->B * C;
-  NVC_CUDA_CHECK(ctx, nvc_launch(ctx, ssd_conv_advance_kernel, dim3((unsigned)((total + 127) / 128)), dim3(128), 0, nvc_stream(stream), a));
-  ctx->launches++;
-  return NVC_OK;
+  const nvc_short_conv cv{p->taps, p->conv_w, p->conv_state, p->state_slots, p->cu_seqlens, p->B};
+  return nvc_short_conv_advance(ctx, &cv, p->in, p->ldi, p->xbc_off, nullptr, p->heads * p->vdim + 2 * p->groups * p->state, p->positions, stream);
 }
