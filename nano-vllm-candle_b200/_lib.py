@@ -141,6 +141,9 @@ def _declare(l: C.CDLL) -> None:
         "nvc_ssd_prep_run": [_vp, _vp, _i, _vp],
         "nvc_ssd_conv_advance": [_vp, _vp, _vp],
         "nvc_moe_scatter_scaled": [_vp, _vp, _i, _i, _vp, _vp, _i, _vp, _i, _i, _i, _vp],
+        "nvc_streams_norm": [_vp, _vp, _vp, _i, _i, _i, _vp],
+        "nvc_short_conv_advance": [_vp, _vp, _vp, _i, _i, _vp, _i, _vp, _vp],
+        "nvc_memory_scan": [_vp, _vp, _i, _i, _vp],
         "nvc_debug_set": [_i, _i],
     }
     for name, args in sigs.items():

@@ -507,7 +507,12 @@ class QkvPrepC(C.Structure):
                 ("positions", C.c_void_p), ("k_scale", C.c_float), ("blend", C.c_int), ("lambda_", C.c_void_p), ("v_first", C.c_void_p),
                 ("ldvf", C.c_int), ("q_out", C.c_void_p), ("ldq", C.c_int), ("k_out", C.c_void_p), ("v_out", C.c_void_p), ("ldk", C.c_int),
                 ("ldv", C.c_int), ("slot_mapping", C.c_void_p), ("q_dtype", C.c_int), ("kv_dtype", C.c_int), ("v_scale", C.c_float),
-                ("unit_norm", C.c_int), ("act", C.c_int)]
+                ("unit_norm", C.c_int), ("act", C.c_int), ("wide_norm", C.c_int), ("conv", C.c_void_p)]
+
+
+class ShortConvC(C.Structure):
+    """nvc_short_conv of include/nvc_b200.h."""
+    _fields_ = [("taps", C.c_int), ("w", C.c_void_p), ("state", C.c_void_p), ("state_slots", C.c_void_p), ("cu_seqlens", C.c_void_p), ("B", C.c_int)]
 
 
 class AttnSpecC(C.Structure):
@@ -594,7 +599,7 @@ def retention_scan(ctx, q, k, v, state, state_slots, cu_seqlens, positions, deca
 
 # ---------------------------------------------------------------- sandwich norms, rotary latent rows, delta rule, softmax routing
 ACT_GELU_TANH, ACT_GLU_CLAMP = 3, 4
-ROUTE_SIGMOID, ROUTE_SOFTMAX = 0, 1
+ROUTE_SIGMOID, ROUTE_SOFTMAX, ROUTE_CHOSEN = 0, 1, 2
 
 
 class DeltaPrepC(C.Structure):
@@ -604,7 +609,7 @@ class DeltaPrepC(C.Structure):
                 ("conv_w", C.c_void_p), ("conv_state", C.c_void_p), ("state_slots", C.c_void_p), ("cu_seqlens", C.c_void_p),
                 ("positions", C.c_void_p), ("A_log", C.c_void_p), ("dt_bias", C.c_void_p), ("unit_eps", C.c_float), ("q_scale", C.c_float),
                 ("q_out", C.c_void_p), ("k_out", C.c_void_p), ("v_out", C.c_void_p), ("ldq", C.c_int), ("ldk", C.c_int), ("ldv", C.c_int),
-                ("gb_out", C.c_void_p), ("B", C.c_int)]
+                ("gb_out", C.c_void_p), ("B", C.c_int), ("channel_a", C.c_void_p), ("ldca", C.c_int), ("channel_g", C.c_void_p)]
 
 
 def rms_norm_sandwich(ctx, res, y, wy, w, eps: float = 1e-5, weight_offset: float = 1.0, out_dtype=torch.float32, rows=None,
@@ -685,9 +690,9 @@ def moe_combine_identity(ctx, y, pos, w, idx, E_real: int, x):
 
 
 def delta_rule(ctx, x, offs, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, conv_w, conv_state, state, state_slots, cu_seqlens,
-               positions, A_log, dt_bias, unit_eps: float = 1e-6, q_scale: Optional[float] = None, max_qlen: int = 1 << 20):
+               positions, A_log, dt_bias, unit_eps: float = 1e-6, q_scale: Optional[float] = None, max_qlen: int = 1 << 20, channel_a=None):
     """x: fp32 [N, ld] rows of the fused projection, offs = (q, k, v, beta, a) columns; conv_w: [taps, C] (tap-major).  Runs the
-    preparation and the recurrence;
+    preparation and the recurrence; channel_a (fp32 [N, heads * dim], dt_bias then too): a decay per head and key channel;
     conv_state [slots, taps - 1, C] and state [slots, heads, dim, vdim] are updated in place.  Returns (o [N, heads * vdim], q, k, v, gb)."""
     N = x.shape[0]
     dev = x.device
@@ -696,9 +701,11 @@ def delta_rule(ctx, x, offs, heads: int, kv_heads: int, dim: int, vdim: int, tap
     v = torch.empty(N, heads * vdim, dtype=torch.float32, device=dev)
     gb = torch.empty(N, 2 * heads, dtype=torch.float32, device=dev)
     o = torch.empty(N, heads * vdim, dtype=torch.float32, device=dev)
+    channel_g = torch.empty(N, heads * dim, dtype=torch.float32, device=dev) if channel_a is not None else None
     p = DeltaPrepC(_a(x), x.stride(0), offs[0], offs[1], offs[2], offs[3], offs[4], heads, kv_heads, dim, vdim, taps, _a(conv_w), _a(conv_state),
                    _a(state_slots), _a(cu_seqlens), _a(positions), _a(A_log), _a(dt_bias), unit_eps, dim ** -0.5 if q_scale is None else q_scale,
-                   _a(q), _a(k), _a(v), q.stride(0), k.stride(0), v.stride(0), _a(gb), state_slots.numel())
+                   _a(q), _a(k), _a(v), q.stride(0), k.stride(0), v.stride(0), _a(gb), state_slots.numel(), _a(channel_a),
+                   channel_a.stride(0) if channel_a is not None else 0, _a(channel_g))
     longest = int((cu_seqlens[1:] - cu_seqlens[:-1]).max().item()) if cu_seqlens is not None else 1
     check(ctx.l.nvc_delta_prep_run(ctx.h, C.byref(p), N, longest, _stream()), "nvc_delta_prep_run", ctx.h)
     check(ctx.l.nvc_delta_rule_scan(ctx.h, C.byref(p), _ptr(o), o.stride(0), _ptr(state), max_qlen, _stream()), "nvc_delta_rule_scan", ctx.h)
@@ -825,3 +832,69 @@ def softcap_f32(ctx, x, cap: float):
     """x: fp32 [N, V], capped in place."""
     check(ctx.l.nvc_softcap_f32(ctx.h, _ptr(x), x.stride(0), cap, x.shape[0], x.shape[1], _stream()), "nvc_softcap_f32", ctx.h)
     return x
+
+
+# ---------------------------------------------------------------- several residual streams, short convolutions, matrix memory
+class StreamsC(C.Structure):
+    """nvc_streams_args of include/nvc_b200.h."""
+    _fields_ = [("x_in", C.c_void_p), ("ldx_in", C.c_int), ("sx_in", C.c_int), ("x_out", C.c_void_p), ("ldx_out", C.c_int), ("sx_out", C.c_int),
+                ("streams", C.c_int), ("y0", C.c_void_p), ("b0", C.c_void_p), ("w0", C.c_void_p), ("c0", C.c_float), ("y1", C.c_void_p),
+                ("w1", C.c_void_p), ("c1", C.c_float), ("ldy", C.c_int), ("mix", C.c_void_p), ("out_w", C.c_void_p), ("in_w", C.c_void_p),
+                ("norm_w", C.c_void_p), ("ldo", C.c_int), ("eps", C.c_float), ("rows", C.c_void_p)]
+
+
+class MemoryScanC(C.Structure):
+    """nvc_memory_scan_args of include/nvc_b200.h."""
+    _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("ldq", C.c_int), ("ldk", C.c_int), ("ldv", C.c_int), ("q_scale", C.c_float),
+                ("i_in", C.c_void_p), ("f_in", C.c_void_p), ("ldg", C.c_int), ("i_bias", C.c_void_p), ("f_bias", C.c_void_p), ("cap", C.c_float),
+                ("den_eps", C.c_float), ("o", C.c_void_p), ("ldo", C.c_int), ("state", C.c_void_p), ("nm_state", C.c_void_p),
+                ("state_slots", C.c_void_p), ("cu_seqlens", C.c_void_p), ("positions", C.c_void_p), ("heads", C.c_int), ("dim", C.c_int),
+                ("vdim", C.c_int)]
+
+
+def streams_norm(ctx, x, streams: int, y0=None, b0=None, w0=None, c0: float = 1.0, y1=None, w1=None, c1: float = 1.0, mix=None, out_w=None,
+                 in_w=None, norm_w=None, eps: float = 1e-5, out_dtype=torch.float32, rows=None, x_out=None, want_out: bool = True):
+    """x: fp32 [N, streams, H], or [N, H] for streams that are all the same row; x_out (None: the streams are not written back) may be x.
+    Returns the normed (norm_w) or plain weighted sum of the streams."""
+    H = x.shape[-1]
+    same = x.dim() == 2
+    N = x.shape[0] if rows is None else rows.numel()
+    out = torch.empty(N, H, dtype=out_dtype, device=x.device) if want_out else None
+    ref = y0 if y0 is not None else y1
+    p = StreamsC(_a(x), x.stride(0), 0 if same else x.stride(1), _a(x_out), x_out.stride(0) if x_out is not None else 0,
+                 x_out.stride(1) if x_out is not None else 0, streams, _a(y0), _a(b0), _a(w0), c0, _a(y1), _a(w1), c1,
+                 ref.stride(0) if ref is not None else 0, _a(mix), _a(out_w), _a(in_w), _a(norm_w), H, eps, _a(rows))
+    check(ctx.l.nvc_streams_norm(ctx.h, C.byref(p), _ptr(out), 0 if out_dtype == torch.bfloat16 else 1, N, H, _stream()), "nvc_streams_norm", ctx.h)
+    return out
+
+
+def qkv_conv_prep(ctx, x, q_off: int, q_heads: int, kv_heads: int, dim: int, vdim: int, q_out, k_out, v_out, bias, conv_w, conv_state, state_slots,
+                  cu_seqlens, positions, q_norm=None, k_norm=None, eps: float = 1e-5, rot_dims: int = 0, rot_half: bool = True, rot_table=None,
+                  slot_mapping=None, silu: bool = False):
+    """Bias, short convolution (conv_w [taps, channels of q | k | v] tap-major; the state is moved on), whole-projection norms, rotation and
+    stores of neighbouring q | k | v columns that start at q_off."""
+    k_off = q_off + q_heads * dim
+    v_off = k_off + kv_heads * dim
+    taps, C_ = conv_w.shape
+    cv = ShortConvC(taps, _a(conv_w), _a(conv_state), _a(state_slots), _a(cu_seqlens), state_slots.numel())
+    dt = _dt(q_out)
+    p = QkvPrepC(_a(x), x.stride(0), _a(bias), q_off, k_off, v_off, q_heads, kv_heads, dim, vdim, _a(q_norm), _a(k_norm), eps, rot_dims,
+                 1 if rot_half else 0, _a(rot_table), _a(positions), 1.0, 0, None, None, 0, _a(q_out), q_out.stride(0), _a(k_out), _a(v_out),
+                 k_out.stride(0), v_out.stride(0), _a(slot_mapping), dt, dt, 1.0, 0, 1 if silu else 0, 1, C.addressof(cv))
+    check(ctx.l.nvc_qkv_prep_run(ctx.h, C.byref(p), x.shape[0], _stream()), "nvc_qkv_prep_run", ctx.h)
+    if cu_seqlens is not None:
+        b = None if bias is None else bias[q_off:].contiguous()
+        check(ctx.l.nvc_short_conv_advance(ctx.h, C.byref(cv), _ptr(x), x.stride(0), q_off, _ptr(b), C_, _ptr(positions), _stream()),
+              "nvc_short_conv_advance", ctx.h)
+
+
+def memory_scan(ctx, q, k, v, i_in, f_in, i_bias, f_bias, cap: float, state, nm_state, state_slots, cu_seqlens, positions, heads: int, dim: int,
+                vdim: int, q_scale: Optional[float] = None, den_eps: float = 1e-6, max_qlen: int = 1 << 20):
+    """q, k: fp32 [N, heads * dim]; v: fp32 [N, heads * vdim]; i_in, f_in: fp32 [N, heads] (equal strides); state [slots, heads, dim, vdim] and
+    nm_state [slots, heads, ceil(vdim / 32), dim + 1] are updated in place."""
+    o = torch.empty(q.shape[0], heads * vdim, dtype=torch.float32, device=q.device)
+    p = MemoryScanC(_a(q), _a(k), _a(v), q.stride(0), k.stride(0), v.stride(0), dim ** -0.5 if q_scale is None else q_scale, _a(i_in), _a(f_in),
+                    i_in.stride(0), _a(i_bias), _a(f_bias), cap, den_eps, _a(o), o.stride(0), _a(state), _a(nm_state), _a(state_slots),
+                    _a(cu_seqlens), _a(positions), heads, dim, vdim)
+    check(ctx.l.nvc_memory_scan(ctx.h, C.byref(p), state_slots.numel(), max_qlen, _stream()), "nvc_memory_scan", ctx.h)
+    return o

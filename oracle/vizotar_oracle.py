@@ -256,16 +256,23 @@ def sub(params: Dict[str, torch.Tensor], prefix: str) -> Dict[str, torch.Tensor]
 
 
 class Vizotar:
-    """The whole model over explicit per-request caches.  cfg: the dict of config.json; params: name -> tensor."""
+    """The whole model over explicit per-request caches.  cfg: the dict of config.json; params: name -> tensor.  rows: a dtype that the
+    rows in front of every sublayer are rounded to (None: not rounded) - how far rounding alone moves a position's logits; the first
+    outputs of a recurrence are a sign, sign(k . q) v / rms(v), and some prompts sit close to the jump."""
 
-    def __init__(self, cfg: dict, params: Dict[str, torch.Tensor]):
+    def __init__(self, cfg: dict, params: Dict[str, torch.Tensor], rows: Optional[torch.dtype] = None):
         self.cfg = cfg
+        self.rows = rows
         self.p = {k: v.float() for k, v in params.items()}
         self.eps = cfg["norm"]["eps"]
 
     def owner(self, i: int) -> int:
         j = self.cfg["layers"][i].get("weights_of")
         return i if j is None else j
+
+    def sublayer_row(self, X: torch.Tensor, w_in: torch.Tensor, norm: torch.Tensor) -> torch.Tensor:
+        h = rms_norm(read_streams(X, w_in), norm, self.eps)
+        return h if self.rows is None else h.to(self.rows).float()
 
     def new_cache(self) -> dict:
         return {"len": 0, "state": {}}
@@ -281,7 +288,7 @@ class Vizotar:
         for i, ly in enumerate(cfg["layers"]):
             lp = sub(self.p, f"l{self.owner(i)}.")
             mp, m = sub(lp, "mix."), ly["mixer"]
-            h = rms_norm(read_streams(X, lp["hc1.in"]), lp["norm1"], eps)
+            h = self.sublayer_row(X, lp["hc1.in"], lp["norm1"])
             if ly["type"] == "parallel":
                 y, state[i] = parallel_mixer(h, mp, m, eps, pos0, state.get(i))
             elif ly["type"] == "channel_delta":
@@ -290,7 +297,7 @@ class Vizotar:
                 raise ValueError(ly["type"])
             X = write_streams(X, lp["hc1.mix"], lp["hc1.out"], y)
             if ly.get("mlp"):
-                h = rms_norm(read_streams(X, lp["hc2.in"]), lp["norm2"], eps)
+                h = self.sublayer_row(X, lp["hc2.in"], lp["norm2"])
                 fp = sub(lp, "mlp.")
                 y = dense_ff(h, fp, ly["mlp"]["limit"]) if ly["mlp"]["kind"] == "dense" else moe_ff(h, fp, ly["mlp"])
                 X = write_streams(X, lp["hc2.mix"], lp["hc2.out"], y)
