@@ -1,4 +1,4 @@
-"""Karuzen, Ranilix, Fefozen, Batatar or Buzutar beside the closest existing family (Qwen3, dense GQA) at equal layer sizes: prefill and decode throughput
+"""Karuzen, Ranilix, Fefozen, Batatar, Buzutar or Vizotar beside the closest existing family (Qwen3, dense GQA) at equal layer sizes: prefill and decode throughput
 through LLMEngine, plus per-op times and roofline fractions.  Random weights, synthetic prompts.  Used by
 `bench.py --compare-families`; the default benchmark does not touch this module.
 
@@ -577,6 +577,168 @@ def buzutar_rooflines(cfg, prof: Dict[str, float], N: int, B: int, ctx_lens: Lis
     return out
 
 
+# ---- Vizotar at the same sizes: four layers - the delta rule with channel decays (heads of 128 x 128, two per query / key head, low ranks of
+# 128), window attention (as many heads as the Qwen3 layer, 8 key / value heads of 128, half of each rotated with YaRN frequencies) beside a
+# matrix memory (heads of 128 x 256, twice the width inside), and both again - on four residual streams, with clamped gated units of ff
+# hidden units or, in the mixture-of-experts size, 16 experts of which 2 are chosen.
+V_WINDOW, V_STREAMS, V_RANK = 256, 4, 128
+
+
+def vizotar_config(sz: dict) -> dict:
+    H, W = sz["heads"], sz["width"]
+    rot = {"dims": 64, "base": 10000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+    par = {"left": {"heads": H, "kv_heads": 8, "dim": 128, "vdim": 128, "conv": 4, "scale": 128 ** -0.5, "rot": rot, "mask": {"size": V_WINDOW}},
+           "right": {"heads": 2 * W // 256, "dim": 128, "vdim": 256, "gate_cap": 15.0}}
+    delta = {"heads": H, "kv_heads": H // 2, "dim": 128, "vdim": 128, "conv": 4}
+    if "moe" in sz:
+        m = sz["moe"]
+        mlp = {"kind": "moe", "router": {"experts": m["experts"], "top": m["top"]}, "expert": {"ff": m["expert_ff"]}}
+    else:
+        mlp = {"kind": "dense", "ff": sz["ff"], "limit": 7.0}
+    kinds = [{"type": "channel_delta", "mixer": delta, "mlp": mlp}, {"type": "parallel", "mixer": par, "mlp": mlp}]
+    return {"architecture": "Vizotar", "vocab": sz["vocab"], "width": W, "norm": {"eps": 1e-5}, "streams": V_STREAMS,
+            "layers": [kinds[i % 2] for i in range(sz["layers"])]}
+
+
+def vizotar_weights(cfg: dict, seed: int = 0):
+    """(name, bf16 CPU tensor) pairs, generated one at a time."""
+    import torch
+    g = torch.Generator().manual_seed(seed)
+    W, n = cfg["width"], cfg["streams"]
+
+    def mat(o, i):
+        return (torch.randn(o, i, generator=g) * i ** -0.5).bfloat16()
+
+    def full(k, v):
+        return torch.full((k,), v).bfloat16()
+
+    yield "embed", (torch.randn(cfg["vocab"], W, generator=g) * 0.05).bfloat16()
+    yield "final.norm", full(W, 1.0)
+    for i, ly in enumerate(cfg["layers"]):
+        m, p = ly["mixer"], f"l{i}."
+        for q in (1, 2):
+            yield p + f"norm{q}", full(W, 1.0)
+            yield p + f"hc{q}.in", full(n, 1.0 / n)
+            yield p + f"hc{q}.out", full(n, 1.0)
+            yield p + f"hc{q}.mix", torch.eye(n).bfloat16()
+        if ly["type"] == "channel_delta":
+            H, G, d, vd, taps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+            for t, rows in (("q", G * d), ("k", G * d), ("v", H * vd)):
+                yield p + "mix." + t, mat(rows, W)
+                yield p + "mix." + t + ".conv", (torch.randn(rows, taps, generator=g) * 0.5).bfloat16()
+            yield p + "mix.b", mat(H, W)
+            yield p + "mix.A_log", full(H, 0.0)
+            yield p + "mix.dt_bias", full(H * d, -3.0)
+            yield p + "mix.norm", full(vd, 1.0)
+            for t, rows in (("a", H * d), ("g", H * vd)):
+                yield p + f"mix.{t}1", mat(V_RANK, W)
+                yield p + f"mix.{t}2", mat(rows, V_RANK)
+            yield p + "mix.o", mat(W, H * vd)
+        else:
+            a, r = m["left"], m["right"]
+            H, G, d, vd, taps = a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["conv"]
+            for t, rows in (("q", H * d), ("k", G * d), ("v", G * vd)):
+                yield p + "mix.left." + t, mat(rows, W)
+                yield p + "mix.left." + t + ".b", full(rows, 0.0)
+                yield p + "mix.left." + t + ".conv", (torch.randn(rows, taps, generator=g) * 0.5).bfloat16()
+            yield p + "mix.left.q.norm", full(H * d, 1.0)
+            yield p + "mix.left.k.norm", full(G * d, 1.0)
+            yield p + "mix.left.sink", full(H, 0.0)
+            yield p + "mix.left.o", mat(W, H * vd)
+            yield p + "mix.left.o.b", full(W, 0.0)
+            yield p + "mix.left.out", full(W, 1.0)
+            yield p + "mix.right.out", full(W, 1.0)
+            H, d, vd = r["heads"], r["dim"], r["vdim"]
+            for t, rows in (("q", H * d), ("k", H * d), ("v", H * vd), ("g", H * vd), ("i", H), ("f", H)):
+                yield p + "mix.right." + t, mat(rows, W)
+            yield p + "mix.right.i.b", full(H, -1.0)
+            yield p + "mix.right.f.b", full(H, 3.0)
+            yield p + "mix.right.norm", full(H * vd, 1.0)
+            yield p + "mix.right.o", mat(W, H * vd)
+        f = ly["mlp"]
+        if f["kind"] == "dense":
+            yield p + "mlp.gate", mat(f["ff"], W)
+            yield p + "mlp.up", mat(f["ff"], W)
+            yield p + "mlp.down", mat(W, f["ff"])
+        else:
+            E, ef = f["router"]["experts"], f["expert"]["ff"]
+            yield p + "mlp.router", mat(E, W)
+            yield p + "mlp.router.b", full(E, 0.0)
+            for e in range(E):
+                yield p + f"mlp.e{e}.gate", mat(ef, W)
+                yield p + f"mlp.e{e}.up", mat(ef, W)
+                yield p + f"mlp.e{e}.down", mat(W, ef)
+
+
+def vizotar_rooflines(cfg, prof: Dict[str, float], N: int, B: int, ctx_lens: List[int], q_lens: List[int], pk) -> dict:
+    """Per-op roofline of one profiled step: the times are sums over the layers, the work is summed the same way.  The scans run on the
+    fp32 FMA pipe (their state is fp32): their fractions are against that pipe's peak (pk["fp32"]).  A window counts its visible pairs."""
+    W, n = cfg["width"], cfg["streams"]
+    work: Dict[str, List[float]] = {}
+
+    def add(name, flops, nbytes):
+        w = work.setdefault(name, [0.0, 0.0])
+        w[0] += flops
+        w[1] += nbytes
+
+    def gemm(name, o, i, rows=N, out_bytes=4):
+        add(name, 2.0 * rows * o * i, 2.0 * (o * i + rows * i) + out_bytes * rows * o)
+
+    for ly in cfg["layers"]:
+        m, f = ly["mixer"], ly["mlp"]
+        if ly["type"] == "channel_delta":
+            H, G, d, vd = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            C = 2 * G * d + H * vd
+            gemm("gemm_in", C + H + 2 * V_RANK, W)
+            add("low_rank_cast", 0.0, 6.0 * N * 2 * V_RANK)
+            add("gemm_low_rank", 2.0 * N * V_RANK * H * (d + vd), 2.0 * V_RANK * (H * (d + vd) + 2 * N) + 4.0 * N * H * (d + vd))
+            add("delta_prep", 0.0, 8.0 * N * (C + H * d))
+            add("delta_scan", 6.0 * N * H * d * vd, 4.0 * (N * (C + H * d + H * vd) + 2 * B * H * d * vd))
+            add("head_gate", 0.0, 10.0 * N * H * vd)
+            gemm("gemm_o", W, H * vd)
+            add("streams_norm", 0.0, N * W * (8.0 * n + 4.0 + 2.0))
+        else:
+            a, r = m["left"], m["right"]
+            H, G, d, vd = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            C, size = H * d + G * (d + vd), a["mask"]["size"]
+            pairs = sum(sum(min(t + 1, size) for t in range(c - q, c)) for q, c in zip(q_lens, ctx_lens))
+            keys = sum(min(c, q + size - 1) for q, c in zip(q_lens, ctx_lens))
+            add("qkv_prep", 0.0, 6.0 * N * C)
+            add("attention", 2.0 * pairs * H * (d + vd), 2.0 * (keys * G * (d + vd) + N * H * (d + vd)))
+            gemm("gemm_o", W, H * vd)
+            Hm, dm, vm = r["heads"], r["dim"], r["vdim"]
+            gemm("gemm_in", C + 2 * Hm * (dm + vm + 1), W)
+            add("memory_scan", 4.0 * N * Hm * dm * vm, 4.0 * (N * 2 * Hm * (dm + vm) + 2 * B * Hm * dm * vm))
+            add("memory_norm_gate", 0.0, 10.0 * N * Hm * vm)
+            gemm("gemm_o", W, Hm * vm)
+            add("streams_norm", 0.0, N * W * (8.0 * n + 8.0 + 2.0))
+        add("streams_norm", 0.0, N * W * (8.0 * n + 4.0 + 2.0))
+        if f["kind"] == "dense":
+            gemm("gemm_gate_up", 2 * f["ff"], W, out_bytes=2)
+            add("glu", 0.0, 6.0 * N * f["ff"])
+            gemm("gemm_down", W, f["ff"])
+        else:
+            E, top, ef = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+            touched = min(E, N * top)
+            add("moe_gate_up", 4.0 * N * top * ef * W, 2.0 * (2 * touched * ef * W + N * top * (2 * ef + W)))
+            add("moe_down", 2.0 * N * top * ef * W, 2.0 * (touched * ef * W + N * top * ef) + 4.0 * N * top * W)
+    add("lm_head", 2.0 * B * cfg["vocab"] * W, 2.0 * cfg["vocab"] * W + 2.0 * B * W + 4.0 * B * cfg["vocab"])
+    out = {}
+    for name, (fl, by) in work.items():
+        if name not in prof:
+            continue
+        if name in ("delta_scan", "memory_scan"):
+            tmin = max(fl / (pk.get("fp32", 70.0) * 1e12), by / (pk["hbm"] * 1e9)) * 1e6
+            out[name] = {"us": round(prof[name], 2), "fp32_tflops": round(fl / prof[name] / 1e6, 2), "gbs": round(by / prof[name] / 1e3, 1),
+                         "roofline_frac": round(tmin / prof[name], 3)}
+        else:
+            out[name] = _roof(fl, by, prof[name], pk)
+    for name in ("moe_route", "moe_sort", "moe_gather", "moe_glu", "moe_combine", "embed", "final_norm"):
+        if name in prof:
+            out[name] = {"us": round(prof[name], 2)}
+    return out
+
+
 def _prompts(n, length, vocab, seed):
     rng = np.random.default_rng(seed)
     return [rng.integers(0, vocab, length).tolist() for _ in range(n)]
@@ -658,7 +820,8 @@ def compare(ctx_ours, sizes=None, batch_p=16, batch_d=64, plen=512, K=32, W=4, p
                                             "ranilix": (ranilix_config, ranilix_weights, ranilix_rooflines),
                                             "fefozen": (fefozen_config, fefozen_weights, fefozen_rooflines),
                                             "batatar": (batatar_config, batatar_weights, batatar_rooflines),
-                                            "buzutar": (buzutar_config, buzutar_weights, buzutar_rooflines)}[family]
+                                            "buzutar": (buzutar_config, buzutar_weights, buzutar_rooflines),
+                                            "vizotar": (vizotar_config, vizotar_weights, vizotar_rooflines)}[family]
     T = batch_p * plen
     nblocks = max(batch_p, batch_d) * (-(-(plen + W + K + 24) // BLOCK)) + 8
     results = []
