@@ -17,8 +17,6 @@
 // exp(L_t - L_j) inside their sums, the keys and queries that meet the state carry exp(L_t), those that enter it exp(L_n - L_j).
 // Both states live in fp32 in pools of state slots; a sequence whose first new token sits at position 0 starts from zeros.
 // Everything here is plain fp32 FMA code.
-#include <cooperative_groups.h>
-
 #include <type_traits>
 
 #include "typed.cuh"
@@ -252,24 +250,43 @@ __global__ void delta_scan_kernel(const DeltaArgs a) {
 }
 
 
-// ---- prompt portions: 32 tokens at a time.  Within a chunk that starts from the state S0, with L_t the running sum of log g up to
-// token t (so exp(L_t - L_j) is the decay between tokens j and t),
-//   u_t = beta_t (v_t - exp(L_t) S0^T k_t - sum_{j<t} exp(L_t - L_j) (k_j . k_t) u_j)        a triangular system, solved forwards
-//   o_t = exp(L_t) S0^T q_t + sum_{j<=t} exp(L_t - L_j) (k_j . q_t) u_j
-//   S   = exp(L_n) S0 + sum_j exp(L_n - L_j) k_j u_j^T
+// ---- prompt portions: 16 tokens at a time.  Within a chunk that starts from the state S0, with L_t the running sum of log g up to
+// token t (so exp(L_t - L_j) is the decay between tokens j and t; a number, or one per key channel),
+//   u_t = beta_t (v_t - S0^T (exp(L_t) k_t) - sum_{j<t} (k_t . exp(L_t - L_j) k_j) u_j)      a unit lower triangular system
+//   o_t = S0^T (exp(L_t) q_t) + sum_{j<=t} (q_t . exp(L_t - L_j) k_j) u_j
+//   S   = exp(L_n) S0 + sum_j (exp(L_n - L_j) k_j) u_j^T
 // which are the four steps of the recurrence written out over the chunk; only differences L_t - L_j <= 0 are exponentiated, so a
-// decay that underflows over a chunk stays a plain zero.  One CTA of four warps per (sequence, head, 32 value columns); thread
-// (column v, warp w) keeps rows [w DPT, (w + 1) DPT) of column v of the state in registers.  Tokens behind a portion's end are
-// padded with g = 1, beta = 0, k = q = v = 0, which leaves state and outputs alone.
-constexpr int kDC = 32;
-constexpr int kDW = 4;
-constexpr int kDAs = kDC + 4;            // row stride of the token-by-token matrices (16-byte rows)
+// decay that underflows over a chunk stays a plain zero.  (A product of two one-sided factors would not do for the token-by-token
+// terms of a channel: exp(-L_j) overflows.  That, and the exponentials it costs, is why a chunk is no longer than 16 tokens.)
+// One CTA per (sequence, head, COLS = 32 C NW / 4 value columns); the state slice stays in shared memory.  Stages of a chunk:
+//   copy      k, q (and log decays) of the chunk, asynchronously; running sums by one thread per channel
+//   products  token against token, lanes along the channels, a warp takes whole rows t; A is kept transposed (AT)
+//   scale     (channels) the rows that meet the state get exp(L_t), those that enter it exp(L_n - L_t)
+//   state     a warp takes 8 of the 32 rows [k | q] against 32 C columns of the state: 8 C sums per thread
+//   solve     forward substitution, column by column of A (every step updates all later right sides: no long dependent sums)
+//   outputs by the warps that hold the query rows' sums, then the state update, 8 rows x C columns at a time
+// Tokens behind a portion's end are padded with g = 1, beta = 0, k = q = v = 0, which leaves state and outputs alone.
+constexpr int kDT = 16;                  // tokens per chunk
+constexpr int kDA = kDT + 4;             // row stride of the token-by-token matrices (16-byte rows)
 
-// staged key / query rows: 4 DPT numbers and more (zeros behind `dim`), 16-byte aligned, rows 4 banks apart
-__host__ __device__ inline int delta_chunk_row(int dim, int dpt) { return max((dim + 3) / 4 * 4, kDW * dpt) + 4; }
-__host__ __device__ inline size_t delta_chunk_smem_floats(int dim, int dpt, bool channels) {
-  return (size_t)(channels ? 3 : 2) * kDC * delta_chunk_row(dim, dpt) + 2 * kDC * kDAs + 3 * kDC * 32 + (size_t)kDW * kDC * 32 + 2 * kDC + 8;
+__host__ __device__ inline int delta_row(int dim) { return (dim + 7) / 8 * 8; }       // staged numbers of a row (zeros behind dim)
+__host__ __device__ inline size_t delta_chunk_smem_floats(int dim, int cols, bool channels) {
+  const int dz = delta_row(dim);
+  return (size_t)(channels ? 3 : 2) * kDT * (dz + 4) + 2 * kDT * kDA + (size_t)kDT * cols + (size_t)dz * cols + dz + 2 * kDT;
 }
+
+__device__ __forceinline__ float ex2(float x) {          // 2^x
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void copy_async16(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void copy_async4(float* dst, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
 __device__ __forceinline__ float fma4(const float4& x, const float4& y, float acc) {
   acc = fmaf(x.x, y.x, acc);
@@ -278,273 +295,347 @@ __device__ __forceinline__ float fma4(const float4& x, const float4& y, float ac
   return fmaf(x.w, y.w, acc);
 }
 
-// x exp(min(a - b, 0)), number by number
-__device__ __forceinline__ float4 scaled_by_exp(const float4& x, const float4& a, const float4& b) {
-  return make_float4(x.x * expf(fminf(a.x - b.x, 0.f)), x.y * expf(fminf(a.y - b.y, 0.f)), x.z * expf(fminf(a.z - b.z, 0.f)),
-                     x.w * expf(fminf(a.w - b.w, 0.f)));
+template <int C> __device__ __forceinline__ void ld_cols(float (&x)[C], const float* p) {
+  if constexpr (C == 2) { const float2 v = *reinterpret_cast<const float2*>(p); x[0] = v.x; x[1] = v.y; }
+  else x[0] = *p;
+}
+template <int C> __device__ __forceinline__ void st_cols(float* p, const float (&x)[C]) {
+  if constexpr (C == 2) *reinterpret_cast<float2*>(p) = make_float2(x[0], x[1]);
+  else *p = x[0];
 }
 
-// Forward substitution of the chunk's triangular system, one value column per lane of one warp: Us holds v_t on entry and u_t on
-// return.  Fully unrolled (the u_t live in registers); not inlined, so that it is compiled once and not once per kernel variant.
-__device__ __noinline__ void delta_chunk_solve(const float* Am, float* Us, const float* W1, const float* Ls, const float* Bs, int lane) {
-  constexpr int as = kDAs;
-  float u[kDC];
-#pragma unroll
-  for (int t = 0; t < kDC; ++t) {
-    float x = Bs[t] * (Us[t * 32 + lane] - expf(Ls[t]) * W1[t * 32 + lane]);
-#pragma unroll
-    for (int j4 = 0; j4 < t; j4 += 4) {       // entries at and behind the diagonal are zero
-      const float4 am = *reinterpret_cast<const float4*>(Am + t * as + j4);
-      x = fmaf(-am.x, u[j4], x);
-      if (j4 + 1 < t) x = fmaf(-am.y, u[j4 + 1], x);
-      if (j4 + 2 < t) x = fmaf(-am.z, u[j4 + 2], x);
-      if (j4 + 3 < t) x = fmaf(-am.w, u[j4 + 3], x);
-    }
-    u[t] = x;
-  }
-#pragma unroll
-  for (int t = 0; t < kDC; ++t) Us[t * 32 + lane] = u[t];
-}
-
-// kCluster: the CTAs of one (sequence, head) - its slices of 32 value columns - form a thread-block cluster, split the rows of the two
-// token-by-token matrices among themselves and write them into one another's shared memory: the products that do not depend on the
-// value column are computed once per (sequence, head), not once per slice.
-// CH: a decay per key channel; the running sums of the channels' log decays stand beside the keys and queries in shared memory, the
-// per-head ones (Ls) stay zero.
-template <int DPT, bool kCluster, bool CH>
-__global__ void __launch_bounds__(kDW * 32) delta_chunk_kernel(const DeltaArgs a) {
-  namespace cg = cooperative_groups;
+template <int C, int NW, bool CH>
+__global__ void __launch_bounds__(NW * 32, NW == 8 ? 2 : 3) delta_chunk_kernel(const DeltaArgs a) {
+  constexpr int COLS = 32 * C * (NW / 4), THREADS = NW * 32;
+  constexpr float kLog2e = 1.4426950408889634f;
   extern __shared__ __align__(16) float sm[];
   pdl_trigger();
   const nvc_delta_prep& p = a.p;
-  const int b = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * 32;
-  const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
-  const int v = v0 + lane;
-  const bool vok = v < p.vdim;
+  const int b = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * COLS;
+  const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, rg = w & 3;
   const int hk = h / (p.heads / p.kv_heads);
-  const int dim = p.dim, ds = delta_chunk_row(dim, DPT), dz = ds - 4;      // dz: numbers of a row that the products read
-  constexpr int as = kDAs;
-  float* Ks = sm;                          // [kDC][ds]
-  float* Qs = Ks + kDC * ds;               // [kDC][ds]
-  float* Am = Qs + kDC * ds;               // [kDC][as]  beta_t exp(L_t - L_j) (k_t . k_j), j < t
-  float* Pm = Am + kDC * as;               // [kDC][as]  exp(L_t - L_j) (q_t . k_j), j <= t
-  float* Us = Pm + kDC * as;               // [kDC][32]  v_t, then u_t
-  float* W1 = Us + kDC * 32;               // [kDC][32]  S0^T k_t
-  float* W2 = W1 + kDC * 32;               // [kDC][32]  S0^T q_t
-  float* Wp = W2 + kDC * 32;               // [kDW][kDC][32] partial sums of the row groups
-  float* Ls = Wp + kDW * kDC * 32;         // [kDC]
-  float* Bs = Ls + kDC;                    // [kDC]
-  float* Gs = Bs + kDC;                    // [kDC][ds] (CH) running sums of the log decays, channel by channel
+  const int dim = p.dim, dz = delta_row(dim), ds = dz + 4;
+  float* Ks = sm;                          // [16][ds]
+  float* Qs = Ks + kDT * ds;               // [16][ds]
+  float* Gs = Qs + kDT * ds;               // [16][ds] (CH) running sums of the log2 decays, later exp(L_t) k_t
+  float* AT = Gs + (CH ? kDT * ds : 0);    // [16][20] AT[j][t] = beta_t (k_t . exp(L_t - L_j) k_j), t > j, else 0
+  float* Pm = AT + kDT * kDA;              // [16][20] Pm[t][j] = q_t . exp(L_t - L_j) k_j, j <= t, else 0
+  float* Us = Pm + kDT * kDA;              // [16][COLS] right sides, then u_t
+  float* Ss = Us + kDT * COLS;             // [dz][COLS] the state's columns
+  float* En = Ss + (size_t)dz * COLS;      // [dz] (CH) log2 decays over the whole chunk
+  float* Ls = En + dz;                     // [16] running sums of the head's log2 decays (zeros: CH)
+  float* Bs = Ls + kDT;                    // [16]
   pdl_wait();
   const int r0 = p.cu_seqlens ? p.cu_seqlens[b] : b;
   const int r1 = p.cu_seqlens ? p.cu_seqlens[b + 1] : b + 1;
   const bool fresh = p.positions[r0] == 0;
   const int slot = p.state_slots[b];
   advance_conv_state(p, r0, r1, fresh, slot);
-  const int d0 = w * DPT;
-  float S[DPT];                            // rows behind `dim` stay zero: the staged rows are zero there
   float* sp = a.state + (((int64_t)slot * p.heads + h) * dim) * p.vdim;
-#pragma unroll
-  for (int i = 0; i < DPT; ++i) S[i] = (!fresh && vok && d0 + i < dim) ? sp[(int64_t)(d0 + i) * p.vdim + v] : 0.f;
-  for (int c0 = r0; c0 < r1; c0 += kDC) {
-    const int n = min(kDC, r1 - c0);
-    // ---- stage the chunk (a row per warp and pass: no division, coalesced)
-    for (int t = w; t < kDC; t += kDW) {
-      const float* kg = p.k_out + (int64_t)(c0 + t) * p.ldk + hk * dim;
-      const float* qg = p.q_out + (int64_t)(c0 + t) * p.ldq + hk * dim;
-      for (int c = lane; c < dz; c += 32) {
-        const bool in = t < n && c < dim;
-        Ks[t * ds + c] = in ? kg[c] : 0.f;
-        Qs[t * ds + c] = in ? qg[c] : 0.f;
-        if (CH) Gs[t * ds + c] = in ? p.channel_g[((int64_t)(c0 + t) * p.heads + h) * dim + c] : 0.f;
+  for (int i = threadIdx.x; i < dz * COLS; i += THREADS) {
+    const int d = i / COLS, c = i % COLS;
+    Ss[i] = (!fresh && d < dim && v0 + c < p.vdim) ? sp[(int64_t)d * p.vdim + v0 + c] : 0.f;
+  }
+  for (int i = threadIdx.x; i < 2 * kDT * kDA; i += THREADS) AT[i] = 0.f;      // what the products never write stays zero
+  const int cl = (w >> 2) * 32 * C + lane * C;             // this lane's first column of the slice
+  for (int c0 = r0; c0 < r1; c0 += kDT) {
+    const int n = min(kDT, r1 - c0);
+    // ---- copy
+    const float* kg = p.k_out + (int64_t)c0 * p.ldk + hk * dim;
+    const float* qg = p.q_out + (int64_t)c0 * p.ldq + hk * dim;
+    const float* gg = CH ? p.channel_g + ((int64_t)c0 * p.heads + h) * dim : nullptr;
+    const int ldg = p.heads * dim;
+    for (int t = w; t < kDT; t += NW) {
+      if (a.vec && t < n) {
+        for (int c = 4 * lane; c < dz; c += 128) {
+          if (c < dim) {
+            copy_async16(Ks + t * ds + c, kg + (int64_t)t * p.ldk + c);
+            copy_async16(Qs + t * ds + c, qg + (int64_t)t * p.ldq + c);
+            if (CH) copy_async16(Gs + t * ds + c, gg + (int64_t)t * ldg + c);
+          } else {
+            const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+            *reinterpret_cast<float4*>(Ks + t * ds + c) = z;
+            *reinterpret_cast<float4*>(Qs + t * ds + c) = z;
+            if (CH) *reinterpret_cast<float4*>(Gs + t * ds + c) = z;
+          }
+        }
+      } else {
+        for (int c = lane; c < dz; c += 32) {
+          if (t < n && c < dim) {
+            copy_async4(Ks + t * ds + c, kg + (int64_t)t * p.ldk + c);
+            copy_async4(Qs + t * ds + c, qg + (int64_t)t * p.ldq + c);
+            if (CH) copy_async4(Gs + t * ds + c, gg + (int64_t)t * ldg + c);
+          } else {
+            Ks[t * ds + c] = 0.f;
+            Qs[t * ds + c] = 0.f;
+            if (CH) Gs[t * ds + c] = 0.f;
+          }
+        }
       }
-      Us[t * 32 + lane] = (t < n && vok) ? p.v_out[(int64_t)(c0 + t) * p.ldv + h * p.vdim + v] : 0.f;
     }
-    if (w == 0) {
-      float lg = (!CH && lane < n) ? p.gb_out[(int64_t)(c0 + lane) * 2 * p.heads + 2 * h] : 0.f;
+    // what this warp needs of v: the tokens of its key rows (rg 0 and 1)
+    float vt[8][C];
+    if (rg < 2) {
 #pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float up = __shfl_up_sync(0xffffffffu, lg, o);
+      for (int r = 0; r < 8; ++r) {
+        const int t = 8 * rg + r;
+        const float* vp = p.v_out + (int64_t)(c0 + t) * p.ldv + h * p.vdim + v0 + cl;
+#pragma unroll
+        for (int e = 0; e < C; ++e) vt[r][e] = (t < n && v0 + cl + e < p.vdim) ? vp[e] : 0.f;
+      }
+    }
+    if (w == 0 && lane < kDT) {
+      const float* gb = p.gb_out + ((int64_t)(c0 + lane) * p.heads + h) * 2;
+      float lg = (!CH && lane < n) ? gb[0] * kLog2e : 0.f;
+#pragma unroll
+      for (int o = 1; o < kDT; o <<= 1) {
+        const float up = __shfl_up_sync(0xffffu, lg, o);
         if (lane >= o) lg += up;
       }
       Ls[lane] = lg;
-      Bs[lane] = lane < n ? p.gb_out[(int64_t)(c0 + lane) * 2 * p.heads + 2 * h + 1] : 0.f;
+      Bs[lane] = lane < n ? gb[1] : 0.f;
     }
+    copy_async_wait();
     __syncthreads();
     if constexpr (CH) {
-      for (int c = threadIdx.x; c < dz; c += kDW * 32) {
-        float l = 0.f;
-        for (int t = 0; t < kDC; ++t) { l += Gs[t * ds + c]; Gs[t * ds + c] = l; }
+      for (int c = threadIdx.x; c < dz; c += THREADS) {
+        float x[kDT], l = 0.f;
+#pragma unroll
+        for (int t = 0; t < kDT; ++t) x[t] = Gs[t * ds + c];
+#pragma unroll
+        for (int t = 0; t < kDT; ++t) { l = fmaf(x[t], kLog2e, l); Gs[t * ds + c] = l; }
+        En[c] = l;
       }
       __syncthreads();
     }
-    // ---- products between the chunk's tokens: two rows t per warp and pass, column j per lane, 16-byte operands
+    // ---- products: a row t against four earlier tokens at a time, groups of GL lanes along the channels.  The eight sums of a group (k and
+    // q against four j) are added up by exchange: with every step a lane keeps half of its sums and one more bit of which ones.
     {
-      const int Z = kCluster ? (int)gridDim.z : 1, zr = kCluster ? (int)blockIdx.z : 0;
-      for (int t = 2 * (zr + Z * w); t < kDC; t += 2 * Z * kDW) {
-        float kk0 = 0.f, qk0 = 0.f, kk1 = 0.f, qk1 = 0.f;
-        if (lane <= t + 1) {
-          const float4* kt0 = reinterpret_cast<const float4*>(Ks + t * ds);
-          const float4* qt0 = reinterpret_cast<const float4*>(Qs + t * ds);
-          const float4* kt1 = reinterpret_cast<const float4*>(Ks + (t + 1) * ds);
-          const float4* qt1 = reinterpret_cast<const float4*>(Qs + (t + 1) * ds);
-          const float4* kj = reinterpret_cast<const float4*>(Ks + lane * ds);
-          if constexpr (CH) {
-            const float4* gt0 = reinterpret_cast<const float4*>(Gs + t * ds);
-            const float4* gt1 = reinterpret_cast<const float4*>(Gs + (t + 1) * ds);
-            const float4* gj = reinterpret_cast<const float4*>(Gs + lane * ds);
+      const int GL = dz > 64 ? 32 : (dz > 32 ? 16 : 8), gl = lane & (GL - 1), sub = lane / GL, subs = 32 / GL;
 #pragma unroll 1
-            for (int c = 0; c < dz / 4; ++c) {
-              const float4 x = kj[c], g = gj[c];
-              const float4 y0 = scaled_by_exp(x, gt0[c], g), y1 = scaled_by_exp(x, gt1[c], g);
-              kk0 = fma4(kt0[c], y0, kk0);
-              qk0 = fma4(qt0[c], y0, qk0);
-              kk1 = fma4(kt1[c], y1, kk1);
-              qk1 = fma4(qt1[c], y1, qk1);
+      for (int i = 0; i < kDT / NW; ++i) {                  // rows in pairs that add up to equal work
+        const int t = (i & 1) ? (i + 1) * NW - 1 - w : i * NW + w;
+        float4 kt[2], qt[2], gt[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int c = 4 * gl + 4 * GL * e;
+          kt[e] = qt[e] = gt[e] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (c < dz) {
+            kt[e] = *reinterpret_cast<const float4*>(Ks + t * ds + c);
+            qt[e] = *reinterpret_cast<const float4*>(Qs + t * ds + c);
+            if (CH) gt[e] = *reinterpret_cast<const float4*>(Gs + t * ds + c);
+          }
+        }
+        const float bt = Bs[t], lt = Ls[t];
+#pragma unroll 1
+        for (int j0 = 0; j0 <= t; j0 += 4 * subs) {
+          const int jb = min(j0 + 4 * sub, kDT - 4);        // groups behind the last row repeat it
+          float v[8];
+#pragma unroll
+          for (int y = 0; y < 8; ++y) v[y] = 0.f;
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int c = 4 * gl + 4 * GL * e;
+            if (c < dz) {
+#pragma unroll
+              for (int y = 0; y < 4; ++y) {
+                float4 x = *reinterpret_cast<const float4*>(Ks + (jb + y) * ds + c);
+                if (CH) {                                   // j > t: anything may come out, nothing is kept
+                  const float4 g = *reinterpret_cast<const float4*>(Gs + (jb + y) * ds + c);
+                  x.x *= ex2(gt[e].x - g.x); x.y *= ex2(gt[e].y - g.y); x.z *= ex2(gt[e].z - g.z); x.w *= ex2(gt[e].w - g.w);
+                }
+                v[y] = fma4(kt[e], x, v[y]);
+                v[4 + y] = fma4(qt[e], x, v[4 + y]);
+              }
             }
-          } else
-#pragma unroll 2
-          for (int c = 0; c < dz / 4; ++c) {
-            const float4 x = kj[c];
-            kk0 = fma4(kt0[c], x, kk0);
-            qk0 = fma4(qt0[c], x, qk0);
-            kk1 = fma4(kt1[c], x, kk1);
-            qk1 = fma4(qt1[c], x, qk1);
           }
-          const float e0 = expf(fminf(Ls[t] - Ls[lane], 0.f)), e1 = expf(fminf(Ls[t + 1] - Ls[lane], 0.f));
-          kk0 *= e0 * Bs[t];
-          qk0 *= e0;
-          kk1 *= e1 * Bs[t + 1];
-          qk1 *= e1;
-        }
-        const float a0 = lane < t ? kk0 : 0.f, p0 = lane <= t ? qk0 : 0.f, a1 = lane < t + 1 ? kk1 : 0.f, p1 = lane <= t + 1 ? qk1 : 0.f;
-        if constexpr (kCluster) {
-          cg::cluster_group cl = cg::this_cluster();
-          for (int r = 0; r < Z; ++r) {
-            float* am = cl.map_shared_rank(Am, r);
-            float* pm = cl.map_shared_rank(Pm, r);
-            am[t * as + lane] = a0;
-            pm[t * as + lane] = p0;
-            am[(t + 1) * as + lane] = a1;
-            pm[(t + 1) * as + lane] = p1;
+          int o = GL >> 1, which = 0;
+#pragma unroll
+          for (int half = 4; half > 0; half >>= 1, o >>= 1) {
+            const bool up = (gl & o) != 0;
+#pragma unroll
+            for (int y = 0; y < half; ++y) {
+              const float give = up ? v[y] : v[y + half], keep = up ? v[y + half] : v[y];
+              v[y] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+            }
+            which = 2 * which + (up ? 1 : 0);
           }
-        } else {
-          Am[t * as + lane] = a0;
-          Pm[t * as + lane] = p0;
-          Am[(t + 1) * as + lane] = a1;
-          Pm[(t + 1) * as + lane] = p1;
+          const bool writer = (gl & (GL / 8 - 1)) == 0;
+          for (; o > 0; o >>= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+          const int j = jb + (which & 3);
+          if (writer && j <= t) {
+            const float x = CH ? v[0] : ex2(lt - Ls[j]) * v[0];
+            if (which >= 4) Pm[t * kDA + j] = x;
+            else if (j < t) AT[j * kDA + t] = bt * x;
+          }
         }
       }
     }
-    // ---- what the state before the chunk says to every key and query: partial sums over this warp's rows, then over the warps
     if constexpr (CH) {
-      __syncthreads();                       // the products above have read the plain rows
-      for (int t = w; t < kDC; t += kDW)
-        for (int c = lane; c < dz; c += 32) Qs[t * ds + c] *= expf(Gs[t * ds + c]);
-      __syncthreads();
-    }
-#pragma unroll 1
-    for (int pass = 0; pass < 2; ++pass) {
-      // CH: the queries first; their rows then hold the keys, scaled for the second pass, and the keys are scaled for the state update
-      const float* X = CH || pass == 1 ? Qs : Ks;
-      float* Wd = (pass == 0) != CH ? W1 : W2;
-      if (CH && pass == 1) {
-        for (int t = w; t < kDC; t += kDW)
-          for (int c = lane; c < dz; c += 32) {
-            const float k = Ks[t * ds + c], l = Gs[t * ds + c];
-            Qs[t * ds + c] = k * expf(l);
-            Ks[t * ds + c] = k * expf(Gs[(kDC - 1) * ds + c] - l);
-          }
-        __syncthreads();
-      }
-#pragma unroll 1
-      for (int t0 = 0; t0 < kDC; t0 += 8) {
-        float acc[8];
-#pragma unroll
-        for (int u = 0; u < 8; ++u) acc[u] = 0.f;
-#pragma unroll
-        for (int i = 0; i < DPT; i += 4) {
-#pragma unroll
-          for (int u = 0; u < 8; ++u) {
-            const float4 x = *reinterpret_cast<const float4*>(X + (t0 + u) * ds + d0 + i);
-            acc[u] = fmaf(S[i], x.x, acc[u]);
-            acc[u] = fmaf(S[i + 1], x.y, acc[u]);
-            acc[u] = fmaf(S[i + 2], x.z, acc[u]);
-            acc[u] = fmaf(S[i + 3], x.w, acc[u]);
-          }
+      __syncthreads();                                      // the products have read the plain rows
+      for (int t = w; t < kDT; t += NW)
+        for (int c = 4 * lane; c < dz; c += 128) {
+          float4 k = *reinterpret_cast<float4*>(Ks + t * ds + c), q = *reinterpret_cast<float4*>(Qs + t * ds + c);
+          const float4 l = *reinterpret_cast<float4*>(Gs + t * ds + c), ln = *reinterpret_cast<float4*>(En + c);
+          const float4 f = make_float4(ex2(l.x), ex2(l.y), ex2(l.z), ex2(l.w));
+          *reinterpret_cast<float4*>(Qs + t * ds + c) = make_float4(q.x * f.x, q.y * f.y, q.z * f.z, q.w * f.w);
+          *reinterpret_cast<float4*>(Gs + t * ds + c) = make_float4(k.x * f.x, k.y * f.y, k.z * f.z, k.w * f.w);
+          *reinterpret_cast<float4*>(Ks + t * ds + c) =
+              make_float4(k.x * ex2(ln.x - l.x), k.y * ex2(ln.y - l.y), k.z * ex2(ln.z - l.z), k.w * ex2(ln.w - l.w));
         }
-#pragma unroll
-        for (int u = 0; u < 8; ++u) Wp[(w * kDC + t0 + u) * 32 + lane] = acc[u];
-      }
-      __syncthreads();
-      for (int t = w; t < kDC; t += kDW) {
-        float s = 0.f;
-#pragma unroll
-        for (int g = 0; g < kDW; ++g) s += Wp[(g * kDC + t) * 32 + lane];
-        Wd[t * 32 + lane] = s;
-      }
-      __syncthreads();
     }
-    if constexpr (kCluster) cg::this_cluster().sync();      // every slice's rows of the two matrices have arrived
-    // ---- the triangular system, one value column per lane of warp 0
-    if (w == 0) delta_chunk_solve(Am, Us, W1, Ls, Bs, lane);
     __syncthreads();
-    // ---- outputs and the state behind the chunk
+    // ---- state: rows 0 .. 15 are the keys', 16 .. 31 the queries'
+    float acc[8][C];
+#pragma unroll
+    for (int r = 0; r < 8; ++r)
+#pragma unroll
+      for (int e = 0; e < C; ++e) acc[r][e] = 0.f;
     {
-      float uu[kDC];
+      const float* X = (rg < 2 ? (CH ? Gs : Ks) : Qs) + (rg & 1) * 8 * ds;
+#pragma unroll 2
+      for (int d = 0; d < dz; d += 4) {
+        float s[4][C];
 #pragma unroll
-      for (int j = 0; j < kDC; ++j) uu[j] = Us[j * 32 + lane];
-      for (int t = w; t < n; t += kDW) {
-        float o = expf(Ls[t]) * W2[t * 32 + lane];
+        for (int i = 0; i < 4; ++i) ld_cols<C>(s[i], Ss + (d + i) * COLS + cl);
 #pragma unroll
-        for (int j4 = 0; j4 < kDC; j4 += 4) {     // entries behind the diagonal are zero
-          const float4 pm = *reinterpret_cast<const float4*>(Pm + t * as + j4);
-          o = fmaf(pm.x, uu[j4], o);
-          o = fmaf(pm.y, uu[j4 + 1], o);
-          o = fmaf(pm.z, uu[j4 + 2], o);
-          o = fmaf(pm.w, uu[j4 + 3], o);
-        }
-        if (vok) a.o[(int64_t)(c0 + t) * a.ldo + h * p.vdim + v] = o;
-      }
-      const float Ln = Ls[kDC - 1];
-      const float gn = expf(Ln);
+        for (int r = 0; r < 8; ++r) {
+          const float4 x = *reinterpret_cast<const float4*>(X + r * ds + d);
 #pragma unroll
-      for (int i = 0; i < DPT; ++i) S[i] *= CH ? expf(Gs[(kDC - 1) * ds + min(d0 + i, dz - 1)]) : gn;
-#pragma unroll 4
-      for (int j = 0; j < kDC; ++j) {             // a loop over the tokens around an unrolled pass over this thread's rows: short code
-        const float uj = Us[j * 32 + lane] * expf(Ln - Ls[j]);
-#pragma unroll
-        for (int i = 0; i < DPT; i += 4) {
-          const float4 x = *reinterpret_cast<const float4*>(Ks + j * ds + d0 + i);
-          S[i] = fmaf(x.x, uj, S[i]);
-          S[i + 1] = fmaf(x.y, uj, S[i + 1]);
-          S[i + 2] = fmaf(x.z, uj, S[i + 2]);
-          S[i + 3] = fmaf(x.w, uj, S[i + 3]);
+          for (int e = 0; e < C; ++e) {
+            acc[r][e] = fmaf(x.x, s[0][e], acc[r][e]);
+            acc[r][e] = fmaf(x.y, s[1][e], acc[r][e]);
+            acc[r][e] = fmaf(x.z, s[2][e], acc[r][e]);
+            acc[r][e] = fmaf(x.w, s[3][e], acc[r][e]);
+          }
         }
       }
     }
-    if constexpr (kCluster) cg::this_cluster().sync();      // no slice writes the next chunk's rows into a neighbour that still reads these
-    else __syncthreads();
-  }
-  if (vok)
+    if (rg < 2) {
 #pragma unroll
-    for (int i = 0; i < DPT; ++i)
-      if (d0 + i < dim) sp[(int64_t)(d0 + i) * p.vdim + v] = S[i];
+      for (int r = 0; r < 8; ++r) {
+        const int t = 8 * rg + r;
+        const float bt = Bs[t], f = CH ? 1.f : ex2(Ls[t]);
+        float x[C];
+#pragma unroll
+        for (int e = 0; e < C; ++e) x[e] = bt * (vt[r][e] - f * acc[r][e]);
+        st_cols<C>(Us + t * COLS + cl, x);
+      }
+    }
+    __syncthreads();
+    // ---- solve: one warp per group of columns
+    if (rg == 0) {
+      float x[kDT][C];
+#pragma unroll
+      for (int t = 0; t < kDT; ++t) ld_cols<C>(x[t], Us + t * COLS + cl);
+#pragma unroll
+      for (int j = 0; j + 1 < kDT; ++j) {
+#pragma unroll
+        for (int t4 = (j + 1) / 4 * 4; t4 < kDT; t4 += 4) {
+          const float4 m = *reinterpret_cast<const float4*>(AT + j * kDA + t4);
+#pragma unroll
+          for (int e = 0; e < C; ++e) {
+            if (t4 > j) x[t4][e] = fmaf(-m.x, x[j][e], x[t4][e]);
+            if (t4 + 1 > j) x[t4 + 1][e] = fmaf(-m.y, x[j][e], x[t4 + 1][e]);
+            if (t4 + 2 > j) x[t4 + 2][e] = fmaf(-m.z, x[j][e], x[t4 + 2][e]);
+            if (t4 + 3 > j) x[t4 + 3][e] = fmaf(-m.w, x[j][e], x[t4 + 3][e]);
+          }
+        }
+      }
+#pragma unroll
+      for (int t = 1; t < kDT; ++t) st_cols<C>(Us + t * COLS + cl, x[t]);
+    }
+    __syncthreads();
+    // ---- outputs
+    float u[kDT][C];
+#pragma unroll
+    for (int j = 0; j < kDT; ++j) ld_cols<C>(u[j], Us + j * COLS + cl);
+    if (rg >= 2) {
+#pragma unroll
+      for (int r = 0; r < 8; ++r) {
+        const int t = 8 * (rg - 2) + r;
+        float o[C];
+        const float f = CH ? 1.f : ex2(Ls[t]);
+#pragma unroll
+        for (int e = 0; e < C; ++e) o[e] = f * acc[r][e];
+#pragma unroll
+        for (int j4 = 0; j4 < kDT; j4 += 4) {               // entries behind the diagonal are zero
+          const float4 m = *reinterpret_cast<const float4*>(Pm + t * kDA + j4);
+#pragma unroll
+          for (int e = 0; e < C; ++e) {
+            o[e] = fmaf(m.x, u[j4][e], o[e]);
+            o[e] = fmaf(m.y, u[j4 + 1][e], o[e]);
+            o[e] = fmaf(m.z, u[j4 + 2][e], o[e]);
+            o[e] = fmaf(m.w, u[j4 + 3][e], o[e]);
+          }
+        }
+        float* op = a.o + (int64_t)(c0 + t) * a.ldo + h * p.vdim + v0 + cl;
+#pragma unroll
+        for (int e = 0; e < C; ++e)
+          if (t < n && v0 + cl + e < p.vdim) op[e] = o[e];
+      }
+    }
+    // ---- the state behind the chunk
+    if (!CH) {
+      const float ln = Ls[kDT - 1];
+#pragma unroll
+      for (int j = 0; j < kDT; ++j) {
+        const float f = ex2(ln - Ls[j]);
+#pragma unroll
+        for (int e = 0; e < C; ++e) u[j][e] *= f;
+      }
+    }
+    for (int d = 4 * rg; d < dz; d += 16) {
+      float s[4][C];
+      const float4 g = CH ? *reinterpret_cast<const float4*>(En + d) : make_float4(Ls[kDT - 1], Ls[kDT - 1], Ls[kDT - 1], Ls[kDT - 1]);
+      const float f[4] = {ex2(g.x), ex2(g.y), ex2(g.z), ex2(g.w)};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        ld_cols<C>(s[i], Ss + (d + i) * COLS + cl);
+#pragma unroll
+        for (int e = 0; e < C; ++e) s[i][e] *= f[i];
+      }
+#pragma unroll
+      for (int j = 0; j < kDT; ++j) {
+        const float4 k = *reinterpret_cast<const float4*>(Ks + j * ds + d);
+#pragma unroll
+        for (int e = 0; e < C; ++e) {
+          s[0][e] = fmaf(k.x, u[j][e], s[0][e]);
+          s[1][e] = fmaf(k.y, u[j][e], s[1][e]);
+          s[2][e] = fmaf(k.z, u[j][e], s[2][e]);
+          s[3][e] = fmaf(k.w, u[j][e], s[3][e]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) st_cols<C>(Ss + (d + i) * COLS + cl, s[i]);
+    }
+    __syncthreads();
+  }
+  for (int i = threadIdx.x; i < dim * COLS; i += THREADS) {
+    const int d = i / COLS, c = i % COLS;
+    if (v0 + c < p.vdim) sp[(int64_t)d * p.vdim + v0 + c] = Ss[i];
+  }
 }
 
-template <int DPT, bool CH>
-cudaError_t launch_delta_chunk(nvc_ctx* ctx, const DeltaArgs& a, dim3 grid, size_t smem, cudaStream_t st) {
+template <int C, int NW, bool CH>
+cudaError_t launch_delta_chunk(nvc_ctx* ctx, const DeltaArgs& a, cudaStream_t st) {
+  constexpr int COLS = 32 * C * (NW / 4);
+  const size_t smem = delta_chunk_smem_floats(a.p.dim, COLS, CH) * sizeof(float);
   static bool attr_set = false;
   if (!attr_set && smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(delta_chunk_kernel<DPT, false, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_kernel<DPT, true, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(delta_chunk_kernel<C, NW, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
     if (e != cudaSuccess) return e;
     attr_set = true;
   }
-  static const bool no_cluster = getenv("NVC_DELTA_CLUSTER") && atoi(getenv("NVC_DELTA_CLUSTER")) == 0;
-  if (grid.z >= 2 && grid.z <= 8 && !no_cluster)       // the value slices of a (sequence, head) as one cluster
-    return nvc_launch_cluster3(ctx, delta_chunk_kernel<DPT, true, CH>, grid, dim3(kDW * 32), smem, st, dim3(1, 1, grid.z), a);
-  return nvc_launch(ctx, delta_chunk_kernel<DPT, false, CH>, grid, dim3(kDW * 32), smem, st, a);
+  return nvc_launch(ctx, delta_chunk_kernel<C, NW, CH>, dim3(a.p.B, a.p.heads, (a.p.vdim + COLS - 1) / COLS), dim3(NW * 32), smem, st, a);
+}
+
+// The wider the slice, the less often the token-by-token products of a head are repeated; as long as the slices fill the GPU
+template <bool CH>
+cudaError_t launch_delta_chunk_sized(nvc_ctx* ctx, const DeltaArgs& a, cudaStream_t st) {
+  const int units = a.p.B * a.p.heads, sms = ctx->num_sms;
+  if (a.p.vdim > 64 && 4 * units * ((a.p.vdim + 127) / 128) >= 3 * sms) return launch_delta_chunk<2, 8, CH>(ctx, a, st);
+  return launch_delta_chunk<1, 8, CH>(ctx, a, st);
 }
 
 int check_prep(nvc_ctx* ctx, const nvc_delta_prep* p) {
@@ -585,21 +676,10 @@ extern "C" int nvc_delta_rule_scan(nvc_ctx* ctx, const nvc_delta_prep* p, float*
   DeltaArgs a{*p, 0, 0, o, ldo, state};
   const int dim = p->dim;
   if (p->cu_seqlens && max_qlen >= 8 && dim <= 256) {
-    // prompt portions: 32 tokens at a time (keys of more than 256 numbers stay token by token)
-    const int per = (dim + kDW - 1) / kDW;     // rows of the state per warp
-    const int cd = per <= 8 ? 8 : (per <= 16 ? 16 : (per <= 32 ? 32 : 64));
-    const dim3 grid(p->B, p->heads, (p->vdim + 31) / 32);
-    const size_t smem = delta_chunk_smem_floats(dim, cd, p->channel_a != nullptr) * sizeof(float);
-    cudaError_t ce;
-    auto go = [&](auto ch) {
-      constexpr bool CH = decltype(ch)::value;
-      if (cd == 8) ce = launch_delta_chunk<8, CH>(ctx, a, grid, smem, nvc_stream(stream));
-      else if (cd == 16) ce = launch_delta_chunk<16, CH>(ctx, a, grid, smem, nvc_stream(stream));
-      else if (cd == 32) ce = launch_delta_chunk<32, CH>(ctx, a, grid, smem, nvc_stream(stream));
-      else ce = launch_delta_chunk<64, CH>(ctx, a, grid, smem, nvc_stream(stream));
-    };
-    if (p->channel_a) go(std::true_type());
-    else go(std::false_type());
+    // prompt portions: 16 tokens at a time (keys of more than 256 numbers stay token by token)
+    auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+    a.vec = dim % 4 == 0 && p->ldq % 4 == 0 && p->ldk % 4 == 0 && al16(p->q_out) && al16(p->k_out) && al16(p->channel_g);
+    const cudaError_t ce = p->channel_a ? launch_delta_chunk_sized<true>(ctx, a, nvc_stream(stream)) : launch_delta_chunk_sized<false>(ctx, a, nvc_stream(stream));
     NVC_CUDA_CHECK(ctx, ce);
     ctx->launches++;
     return NVC_OK;
