@@ -19,7 +19,7 @@
 // Everything here is plain fp32 FMA code.
 #include <type_traits>
 
-#include "typed.cuh"
+#include "scan_common.cuh"
 
 namespace {
 
@@ -269,39 +269,9 @@ __global__ void delta_scan_kernel(const DeltaArgs a) {
 constexpr int kDT = 16;                  // tokens per chunk
 constexpr int kDA = kDT + 4;             // row stride of the token-by-token matrices (16-byte rows)
 
-__host__ __device__ inline int delta_row(int dim) { return (dim + 7) / 8 * 8; }       // staged numbers of a row (zeros behind dim)
 __host__ __device__ inline size_t delta_chunk_smem_floats(int dim, int cols, bool channels) {
-  const int dz = delta_row(dim);
+  const int dz = scan_row(dim);
   return (size_t)(channels ? 3 : 2) * kDT * (dz + 4) + 2 * kDT * kDA + (size_t)kDT * cols + (size_t)dz * cols + dz + 2 * kDT;
-}
-
-__device__ __forceinline__ float ex2(float x) {          // 2^x
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ void copy_async16(float* dst, const float* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void copy_async4(float* dst, const float* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
-
-__device__ __forceinline__ float fma4(const float4& x, const float4& y, float acc) {
-  acc = fmaf(x.x, y.x, acc);
-  acc = fmaf(x.y, y.y, acc);
-  acc = fmaf(x.z, y.z, acc);
-  return fmaf(x.w, y.w, acc);
-}
-
-template <int C> __device__ __forceinline__ void ld_cols(float (&x)[C], const float* p) {
-  if constexpr (C == 2) { const float2 v = *reinterpret_cast<const float2*>(p); x[0] = v.x; x[1] = v.y; }
-  else x[0] = *p;
-}
-template <int C> __device__ __forceinline__ void st_cols(float* p, const float (&x)[C]) {
-  if constexpr (C == 2) *reinterpret_cast<float2*>(p) = make_float2(x[0], x[1]);
-  else *p = x[0];
 }
 
 template <int C, int NW, bool CH>
@@ -314,7 +284,7 @@ __global__ void __launch_bounds__(NW * 32, NW == 8 ? 2 : 3) delta_chunk_kernel(c
   const int b = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * COLS;
   const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, rg = w & 3;
   const int hk = h / (p.heads / p.kv_heads);
-  const int dim = p.dim, dz = delta_row(dim), ds = dz + 4;
+  const int dim = p.dim, dz = scan_row(dim), ds = dz + 4;
   float* Ks = sm;                          // [16][ds]
   float* Qs = Ks + kDT * ds;               // [16][ds]
   float* Gs = Qs + kDT * ds;               // [16][ds] (CH) running sums of the log2 decays, later exp(L_t) k_t
@@ -346,32 +316,9 @@ __global__ void __launch_bounds__(NW * 32, NW == 8 ? 2 : 3) delta_chunk_kernel(c
     const float* gg = CH ? p.channel_g + ((int64_t)c0 * p.heads + h) * dim : nullptr;
     const int ldg = p.heads * dim;
     for (int t = w; t < kDT; t += NW) {
-      if (a.vec && t < n) {
-        for (int c = 4 * lane; c < dz; c += 128) {
-          if (c < dim) {
-            copy_async16(Ks + t * ds + c, kg + (int64_t)t * p.ldk + c);
-            copy_async16(Qs + t * ds + c, qg + (int64_t)t * p.ldq + c);
-            if (CH) copy_async16(Gs + t * ds + c, gg + (int64_t)t * ldg + c);
-          } else {
-            const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
-            *reinterpret_cast<float4*>(Ks + t * ds + c) = z;
-            *reinterpret_cast<float4*>(Qs + t * ds + c) = z;
-            if (CH) *reinterpret_cast<float4*>(Gs + t * ds + c) = z;
-          }
-        }
-      } else {
-        for (int c = lane; c < dz; c += 32) {
-          if (t < n && c < dim) {
-            copy_async4(Ks + t * ds + c, kg + (int64_t)t * p.ldk + c);
-            copy_async4(Qs + t * ds + c, qg + (int64_t)t * p.ldq + c);
-            if (CH) copy_async4(Gs + t * ds + c, gg + (int64_t)t * ldg + c);
-          } else {
-            Ks[t * ds + c] = 0.f;
-            Qs[t * ds + c] = 0.f;
-            if (CH) Gs[t * ds + c] = 0.f;
-          }
-        }
-      }
+      copy_row(Ks + t * ds, kg + (int64_t)t * p.ldk, dim, dz, t < n, a.vec, lane);
+      copy_row(Qs + t * ds, qg + (int64_t)t * p.ldq, dim, dz, t < n, a.vec, lane);
+      if (CH) copy_row(Gs + t * ds, gg + (int64_t)t * ldg, dim, dz, t < n, a.vec, lane);
     }
     // what this warp needs of v: the tokens of its key rows (rg 0 and 1)
     float vt[8][C];
@@ -408,8 +355,8 @@ __global__ void __launch_bounds__(NW * 32, NW == 8 ? 2 : 3) delta_chunk_kernel(c
       }
       __syncthreads();
     }
-    // ---- products: a row t against four earlier tokens at a time, groups of GL lanes along the channels.  The eight sums of a group (k and
-    // q against four j) are added up by exchange: with every step a lane keeps half of its sums and one more bit of which ones.
+    // ---- products: a row t against four earlier tokens at a time, groups of GL lanes along the channels.  The eight sums of a group: k and
+    // q against four j.
     {
       const int GL = dz > 64 ? 32 : (dz > 32 ? 16 : 8), gl = lane & (GL - 1), sub = lane / GL, subs = 32 / GL;
 #pragma unroll 1
@@ -449,22 +396,12 @@ __global__ void __launch_bounds__(NW * 32, NW == 8 ? 2 : 3) delta_chunk_kernel(c
               }
             }
           }
-          int o = GL >> 1, which = 0;
-#pragma unroll
-          for (int half = 4; half > 0; half >>= 1, o >>= 1) {
-            const bool up = (gl & o) != 0;
-#pragma unroll
-            for (int y = 0; y < half; ++y) {
-              const float give = up ? v[y] : v[y + half], keep = up ? v[y + half] : v[y];
-              v[y] = keep + __shfl_xor_sync(0xffffffffu, give, o);
-            }
-            which = 2 * which + (up ? 1 : 0);
-          }
-          const bool writer = (gl & (GL / 8 - 1)) == 0;
-          for (; o > 0; o >>= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+          int which;
+          bool writer;
+          const float sum = group_sum8(v, GL, gl, &which, &writer);
           const int j = jb + (which & 3);
           if (writer && j <= t) {
-            const float x = CH ? v[0] : ex2(lt - Ls[j]) * v[0];
+            const float x = CH ? sum : ex2(lt - Ls[j]) * sum;
             if (which >= 4) Pm[t * kDA + j] = x;
             else if (j < t) AT[j * kDA + t] = bt * x;
           }

@@ -140,9 +140,9 @@ __device__ __forceinline__ int prep_find_seq(const int32_t* cu, int B, int row) 
 // whole query and key projection - or none - then rotation and stores.  P: numbers per access (4: every width, offset and stride is a
 // multiple of 4 and the pointers are 16-byte aligned).
 template <typename TQ, typename TKV, int P>
-__global__ void __launch_bounds__(256) prep_token_kernel(const PrepArgs a, const nvc_short_conv cv) {
+__global__ void __launch_bounds__(1024) prep_token_kernel(const PrepArgs a, const nvc_short_conv cv) {
   extern __shared__ __align__(16) float row[];          // [qw + kw + vw]
-  __shared__ float part[2][8];
+  __shared__ float part[2][32];
   __shared__ int s_r0, s_fresh, s_slot;
   pdl_trigger();
   const nvc_qkv_prep& p = a.p;
@@ -426,8 +426,11 @@ int launch_prep_token(nvc_ctx* ctx, const nvc_qkv_prep* p, int N, void* stream) 
     NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(prep_token_kernel<TQ, TKV, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     attr_set = true;
   }
-  if (vec) NVC_CUDA_CHECK(ctx, nvc_launch(ctx, prep_token_kernel<TQ, TKV, 4>, dim3((unsigned)N), dim3(256), smem, nvc_stream(stream), a, cv));
-  else NVC_CUDA_CHECK(ctx, nvc_launch(ctx, prep_token_kernel<TQ, TKV, 1>, dim3((unsigned)N), dim3(256), smem, nvc_stream(stream), a, cv));
+  // few rows: one access per thread, so that a row's loads are all in flight at once
+  const int units = ((qw + kw + vw) / (vec ? 4 : 1) + 31) / 32 * 32;
+  const int threads = std::min(std::max(units, 64), N <= 2 * ctx->num_sms ? 1024 : 256);
+  if (vec) NVC_CUDA_CHECK(ctx, nvc_launch(ctx, prep_token_kernel<TQ, TKV, 4>, dim3((unsigned)N), dim3(threads), smem, nvc_stream(stream), a, cv));
+  else NVC_CUDA_CHECK(ctx, nvc_launch(ctx, prep_token_kernel<TQ, TKV, 1>, dim3((unsigned)N), dim3(threads), smem, nvc_stream(stream), a, cv));
   ctx->launches++;
   return NVC_OK;
 }

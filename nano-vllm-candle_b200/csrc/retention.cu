@@ -5,18 +5,20 @@
 // its slot holds, and the slot is written back after the last token.  q, k, v, o are fp32 rows (the caller has already rotated q and
 // k and scaled k).
 //
-// Two kernels, both with one CTA per (sequence, head, slice of 32 value columns) whose threads (column v, row group r) keep rows
-// [r DPT, (r + 1) DPT) of column v of the state in registers (token by token: 32 rows per warp, up to 32 warps):
-//   retention_scan_kernel    token by token (decode steps and very short portions): 2 DPT FMAs per thread and token and, when the
-//                            rows are split, one shared-memory reduction; the next token's q / k / v are fetched meanwhile.
-//   retention_chunk_kernel   32 tokens at a time (prompt portions), the same recurrence regrouped:
+// Two kernels, both with one CTA per (sequence, head, slice of value columns):
+//   retention_scan_kernel    token by token (decode steps and very short portions), slices of 32 columns: thread (column v, row group r)
+//                            keeps rows [r DPT, (r + 1) DPT) of column v of the state in registers (32 rows per warp, up to 32 warps);
+//                            2 DPT FMAs per thread and token and, when the rows are split, one shared-memory reduction; the next
+//                            token's q / k / v are fetched meanwhile.
+//   retention_chunk_kernel   32 tokens at a time (prompt portions), slices of 32, 64 or 128 columns whose state stays in shared memory
+//                            (every product is a tile of 8 rows or 4 rows x C columns per thread), the same recurrence regrouped:
 //                              A[t][j] = decay^(t - j) (q_t . k_j), j <= t            inside the chunk
 //                              o_t     = sum_j A[t][j] v_j + decay^(t + 1) S^T q_t     S: the state before the chunk
 //                              S      <- decay^n S + sum_j decay^(n - 1 - j) k_j v_j^T n: tokens of the chunk
 //                            Powers of the decay come from a table built by repeated multiplication (exact for 0 and 1).
 // Both are plain fp32 FMA code; they differ from one another by rounding only.
 //
-// nvc_decay_scan is the same pair of kernels with what other linear recurrences of this shape need (VAR = true):
+// nvc_decay_scan is the same pair of kernels with what other linear recurrences of this shape need (kVar):
 //   a decay per token and head, given as its logarithm: S_t = exp(l_t) S_(t-1) + k_t v_t^T.  Inside a chunk only differences of the
 //     running sums L_t = l_0 + .. + l_t are exponentiated (all <= 0): A[t][j] carries exp(L_t - L_j), the state's share exp(L_t), the
 //     state update exp(L_(n-1) - L_j); a decay that underflows stays a plain zero;
@@ -26,13 +28,13 @@
 // stabilised by a running maximum m_t = max(f_t + m_(t-1), i_t):
 //   S_t = exp(f_t + m_(t-1) - m_t) S_(t-1) + exp(i_t - m_t) k_t v_t^T,   n_t likewise with k_t alone,
 //   o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + eps)
-//   Every CTA (a slice of 32 value columns) carries n and m itself and keeps a copy of its own in the slot: no slice waits for another.
+//   Every CTA carries n and m itself; the slot holds a copy per 32 value columns, so that no slice waits for another.
 //   Inside a chunk, with F_t the running sum of f and b_j = i_j - F_j:  M_t = max(m, b_0 .. b_t), m_t = F_t + M_t, and the decay of the
 //   state up to token t is exp(m - M_t), the weight of token j at token t exp(b_j - M_t): every exponent is <= 0.  F, b and M are kept in
 //   double precision (32 numbers per chunk), so a long run of small forget gates costs no digits of the differences.
 //
 // A selective state space layer in its dual form is the decayed recurrence with q = C, k = B, v = dt x, l = -exp(A_log) dt, skip = x.
-#include "typed.cuh"
+#include "scan_common.cuh"
 
 namespace {
 
@@ -42,10 +44,10 @@ struct RetArgs {
   int ldq, ldk, ldv, ldo;
   float* state;                  // [slots, heads, dim, vdim]
   const int32_t *state_slots, *cu_seqlens, *positions;
-  const float* decay;            // [heads]                       (VAR = false)
+  const float* decay;            // [heads]                       (kFixed)
   int heads, dim, vdim;
   int qk_heads;                  // q / k heads (a divisor of heads)
-  const float* log_decay;        // [rows, ldl], one per head       (VAR = true)
+  const float* log_decay;        // [rows, ldl], one per head       (kVar)
   int ldl;
   const float* skip;             // [rows, lds] like v, or NULL
   const float* skip_w;           // [heads]
@@ -177,47 +179,41 @@ __global__ void retention_scan_kernel(const RetArgs a) {
 }
 
 constexpr int kChunk = 32;          // tokens per chunk
-constexpr int kChunkWarps = 8;         // a divisor of 8: the chunk's 8 groups of four keys are dealt out to the warps
-constexpr int kKeyGroups = 8 / kChunkWarps;
+constexpr int kChunkA = kChunk + 4; // row stride of A (16-byte rows)
 
-__device__ __forceinline__ float dot4(const float4& x, const float4& y, float acc) {
-  acc = fmaf(x.x, y.x, acc);
-  acc = fmaf(x.y, y.y, acc);
-  acc = fmaf(x.z, y.z, acc);
-  return fmaf(x.w, y.w, acc);
+// shared memory of a CTA: q and k of the chunk, A, the state's columns, the gate arrays of the chunk
+__host__ __device__ inline size_t chunk_smem_floats(int dim, int cols) {
+  const int dz = scan_row(dim);
+  return (size_t)2 * kChunk * (dz + 4) + kChunk * kChunkA + (size_t)dz * cols + dz + 4 * kChunk + 4 * kChunk + kChunk + 4;
 }
 
-// float4 units per staged q row: odd, so that the 8 lanes of a 128-bit shared-memory phase (lane = token) hit distinct banks
-__host__ __device__ inline int chunk_q_stride4(int dim) { const int q4 = (dim + 3) / 4; return (q4 & 1) ? q4 : q4 + 1; }
-
-// Shared-memory operands are read as float4 (one load per four FMAs) and reused across a register tile: the kernel is bound
-// by the FMA pipe, not by shared-memory loads.
-// The variant with per-token decays at up to 16 rows per warp is capped at 85 registers (a few spilled words) so that three CTAs -
-// what shared memory allows - fit an SM; the fixed-decay variant needs 80 as it is.
-template <int DPT, int MODE>
-__global__ void __launch_bounds__(kChunkWarps * 32, DPT <= 16 ? 3 : 0) retention_chunk_kernel(const RetArgs a) {
+// One CTA per (sequence, head, COLS = 32 C NW / 4 value columns); its slice of the state stays in shared memory.  Stages of a chunk:
+//   copy      q and k, asynchronously; the chunk's decays or gates by one warp
+//   products  A, rows t against eight earlier tokens at a time, lanes along the channels (scan_common.cuh)
+//   state     a warp takes 8 of the 32 queries against 32 C columns of the state: 8 C sums per thread
+//   outputs   A against the values (straight from global memory, 32 C numbers per thread), then the state update 4 rows at a time
+template <int C, int NW, int MODE>
+__global__ void __launch_bounds__(NW * 32, 2) retention_chunk_kernel(const RetArgs a, const int vec) {
   constexpr bool VAR = MODE == kVar, MEM = MODE == kMemory;
+  constexpr int COLS = 32 * C * (NW / 4), THREADS = NW * 32;
   extern __shared__ __align__(16) float sm[];
   pdl_trigger();
-  const int b = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * 32;
-  const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
-  const int v = v0 + lane;
-  const bool vok = v < a.vdim;
-  const int dim = a.dim, q4 = (dim + 3) / 4, dim4 = 4 * q4, RS = chunk_q_stride4(dim);
-  float4* q_s = reinterpret_cast<float4*>(sm);                 // [32][RS]   rows padded with zeros
-  float4* k_s = q_s + kChunk * RS;                             // [32][q4]   (read as broadcasts)
-  float* v_s = reinterpret_cast<float*>(k_s + kChunk * q4);    // [32][32]
-  float4* a_s = reinterpret_cast<float4*>(v_s + kChunk * 32);  // [32][9]    A[t][j], j in fours, zero above the diagonal
-  float* part = reinterpret_cast<float*>(a_s + kChunk * 9);    // [warps][32][32]
-  float* gp = part + kChunkWarps * kChunk * 32;                // decay^0 .. decay^32;  VAR: the running sums L_0 .. L_31 of the chunk
-  double* bD = reinterpret_cast<double*>(gp + kChunk + 4);     // MEM [32] b_j = i_j - F_j
-  double* MD = bD + kChunk;                                    // MEM [32] M_t
-  float* keep_s = reinterpret_cast<float*>(MD + kChunk);       // MEM [32] exp(m - M_t): the state's decay up to token t
-  float* em_s = keep_s + kChunk;                               // MEM [32] exp(-m_t)
-  float* wj_s = em_s + kChunk;                                 // MEM [32] exp(b_j - M_(n-1)): the weight of token j in the state behind the chunk
-  float* nq_s = wj_s + kChunk;                                 // MEM [warps][32] shares of n . q_t
-  float* n_s = nq_s + kChunkWarps * kChunk;                    // MEM [warps * DPT] n, zeros behind dim
-  double m0 = 0.0;                                             // MEM, warp 0: the running maximum in front of the chunk
+  const int b = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * COLS;
+  const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, rg = w & 3;
+  const int dim = a.dim, dz = scan_row(dim), ds = dz + 4;
+  float* Qs = sm;                          // [32][ds]
+  float* Ks = Qs + kChunk * ds;            // [32][ds]
+  float* As = Ks + kChunk * ds;            // [32][36]  A[t][j], zero above the diagonal
+  float* Ss = As + kChunk * kChunkA;       // [dz][COLS]
+  float* n_s = Ss + (size_t)dz * COLS;     // [dz] MEM: n, zeros behind dim
+  double* bD = reinterpret_cast<double*>(n_s + dz);        // [32] MEM: b_j = i_j - F_j
+  double* MD = bD + kChunk;                                // [32] MEM: M_t
+  float* keep_s = reinterpret_cast<float*>(MD + kChunk);   // [32] the state's decay up to token t
+  float* wj_s = keep_s + kChunk;                           // [32] the weight of token j in the state behind the chunk
+  float* em_s = wj_s + kChunk;                             // [32] MEM: exp(-m_t)
+  float* nq_s = em_s + kChunk;                             // [32] MEM: n . q_t
+  float* gp = nq_s + kChunk;                               // [33] decay^0 .. decay^32;  VAR: the running sums L_0 .. L_31
+  double m0 = 0.0;                                         // MEM, warp 0: the running maximum in front of the chunk
   const int hq = h / (a.heads / a.qk_heads);
   const float sw = a.skip ? __ldg(a.skip_w + h) : 0.f;
   const float qs = MEM ? a.mem.q_scale : 1.f;
@@ -229,226 +225,241 @@ __global__ void __launch_bounds__(kChunkWarps * 32, DPT <= 16 ? 3 : 0) retention
   pdl_wait();
   const int r0 = a.cu_seqlens ? a.cu_seqlens[b] : b;
   const int r1 = a.cu_seqlens ? a.cu_seqlens[b + 1] : b + 1;
-  const int d0 = w * DPT;                                      // this warp's rows of the state (DPT is a multiple of 4)
-  float S[DPT];
-  float* sp = a.state + (((int64_t)a.state_slots[b] * a.heads + h) * dim) * a.vdim;
+  const int slot = a.state_slots[b];
   const bool fresh = a.positions[r0] == 0;
-#pragma unroll
-  for (int i = 0; i < DPT; ++i) S[i] = (!fresh && vok && d0 + i < dim) ? sp[(int64_t)(d0 + i) * a.vdim + v] : 0.f;
-  float* np = MEM ? a.mem.nm_state + (((int64_t)a.state_slots[b] * a.heads + h) * gridDim.z + blockIdx.z) * (dim + 1) : nullptr;
+  float* sp = a.state + (((int64_t)slot * a.heads + h) * dim) * a.vdim;
+  for (int i = threadIdx.x; i < dz * COLS; i += THREADS) {
+    const int d = i / COLS, c = i % COLS;
+    Ss[i] = (!fresh && d < dim && v0 + c < a.vdim) ? sp[(int64_t)d * a.vdim + v0 + c] : 0.f;
+  }
+  for (int i = threadIdx.x; i < kChunk * kChunkA; i += THREADS) As[i] = 0.f;      // what the products never write stays zero
+  // MEM: n and m of this CTA's columns; a copy per 32 of them, all alike
+  const int copies = (a.vdim + 31) / 32;
+  float* np = MEM ? a.mem.nm_state + (((int64_t)slot * a.heads + h) * copies + v0 / 32) * (dim + 1) : nullptr;
   if (MEM) {
-    for (int d = threadIdx.x; d < kChunkWarps * DPT; d += blockDim.x) n_s[d] = (!fresh && d < dim) ? np[d] : 0.f;
+    for (int d = threadIdx.x; d < dz; d += THREADS) n_s[d] = (!fresh && d < dim) ? np[d] : 0.f;
     if (!fresh) m0 = (double)np[dim];
   }
-  float* q_sf = reinterpret_cast<float*>(q_s);
-  float* k_sf = reinterpret_cast<float*>(k_s);
-  const bool vec = (dim & 3) == 0 && (a.ldq & 3) == 0 && (a.ldk & 3) == 0 && ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k)) & 15) == 0;
+  const int cl = (w >> 2) * 32 * C + lane * C;             // this lane's first column of the slice
   for (int c0 = r0; c0 < r1; c0 += kChunk) {
     const int n = min(kChunk, r1 - c0);
-    __syncthreads();                                   // the previous chunk is done with the staged rows
-    // a warp stages whole rows (t = w, w + warps, ...), lanes along the row: no index division, 16-byte loads where the layout allows
-    for (int t = w; t < kChunk; t += kChunkWarps) {
-      const bool tin = t < n;
-      const float* qrow = a.q + (int64_t)(c0 + t) * a.ldq + hq * dim;
-      const float* krow = a.k + (int64_t)(c0 + t) * a.ldk + hq * dim;
-      if (vec) {
-        for (int d4 = lane; d4 < q4; d4 += 32) {
-          const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
-          float4 qv = tin ? *reinterpret_cast<const float4*>(qrow + 4 * d4) : z;
-          if (MEM) { qv.x *= qs; qv.y *= qs; qv.z *= qs; qv.w *= qs; }
-          q_s[t * RS + d4] = qv;
-          k_s[t * q4 + d4] = tin ? *reinterpret_cast<const float4*>(krow + 4 * d4) : z;
+    __syncthreads();                                       // the previous chunk is done with the staged rows
+    for (int t = w; t < kChunk; t += NW) {
+      copy_row(Qs + t * ds, a.q + (int64_t)(c0 + t) * a.ldq + hq * dim, dim, dz, t < n, vec, lane);
+      copy_row(Ks + t * ds, a.k + (int64_t)(c0 + t) * a.ldk + hq * dim, dim, dz, t < n, vec, lane);
+    }
+    if (w == 0) {
+      if (MODE == kFixed) {
+        keep_s[lane] = gp[min(lane, n - 1) + 1];
+        wj_s[lane] = lane < n ? gp[n - 1 - lane] : 0.f;
+      } else if (VAR) {       // inclusive running sums of the chunk's log decays (a fixed order: lane by lane)
+        float l = lane < n ? a.log_decay[(int64_t)(c0 + lane) * a.ldl + h] : 0.f;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+          const float up = __shfl_up_sync(0xffffffffu, l, o);
+          if (lane >= o) l += up;
         }
+        gp[lane] = l;
+        keep_s[lane] = expf(l);
+        wj_s[lane] = expf(__shfl_sync(0xffffffffu, l, n - 1) - l);
       } else {
-        for (int d = lane; d < dim4; d += 32) {
-          const bool in = tin && d < dim;
-          q_sf[t * 4 * RS + d] = in ? (MEM ? qs * qrow[d] : qrow[d]) : 0.f;
-          k_sf[t * dim4 + d] = in ? krow[d] : 0.f;
+        const bool in = lane < n;
+        const int64_t gr = (int64_t)(c0 + lane) * a.mem.ldg + h;
+        const float gi = in ? capped(a.mem.i_in[gr] + __ldg(a.mem.i_bias + h), a.mem.cap) : -INFINITY;      // no token: weight 0
+        double F = in ? (double)log_sigmoid(capped(a.mem.f_in[gr] + __ldg(a.mem.f_bias + h), a.mem.cap)) : 0.0;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+          const double up = __shfl_up_sync(0xffffffffu, F, o);
+          if (lane >= o) F += up;
         }
-      }
-    }
-    if (VAR && threadIdx.x < 32) {        // inclusive running sums of the chunk's log decays (a fixed order: lane by lane)
-      float l = lane < n ? a.log_decay[(int64_t)(c0 + lane) * a.ldl + h] : 0.f;
+        const double bj = (double)gi - F;
+        double M = fmax(bj, m0);
 #pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float up = __shfl_up_sync(0xffffffffu, l, o);
-        if (lane >= o) l += up;
+        for (int o = 1; o < 32; o <<= 1) {
+          const double up = __shfl_up_sync(0xffffffffu, M, o);
+          if (lane >= o) M = fmax(M, up);
+        }
+        const double Mn = __shfl_sync(0xffffffffu, M, n - 1), Fn = __shfl_sync(0xffffffffu, F, n - 1);
+        bD[lane] = bj;
+        MD[lane] = M;
+        keep_s[lane] = expf((float)(m0 - M));
+        em_s[lane] = expf((float)-(F + M));
+        wj_s[lane] = expf((float)(bj - Mn));
+        m0 = Fn + Mn;
       }
-      gp[lane] = l;
     }
-    if (MEM && threadIdx.x < 32) {
-      const bool in = lane < n;
-      const int64_t gr = (int64_t)(c0 + lane) * a.mem.ldg + h;
-      const float gi = in ? capped(a.mem.i_in[gr] + __ldg(a.mem.i_bias + h), a.mem.cap) : -INFINITY;      // no token: weight 0
-      double F = in ? (double)log_sigmoid(capped(a.mem.f_in[gr] + __ldg(a.mem.f_bias + h), a.mem.cap)) : 0.0;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const double up = __shfl_up_sync(0xffffffffu, F, o);
-        if (lane >= o) F += up;
-      }
-      const double bj = (double)gi - F;
-      double M = fmax(bj, m0);
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const double up = __shfl_up_sync(0xffffffffu, M, o);
-        if (lane >= o) M = fmax(M, up);
-      }
-      const double Mn = __shfl_sync(0xffffffffu, M, n - 1), Fn = __shfl_sync(0xffffffffu, F, n - 1);
-      bD[lane] = bj;
-      MD[lane] = M;
-      keep_s[lane] = expf((float)(m0 - M));
-      em_s[lane] = expf((float)-(F + M));
-      wj_s[lane] = expf((float)(bj - Mn));
-      m0 = Fn + Mn;
-    }
-    for (int idx = threadIdx.x; idx < kChunk * 32; idx += blockDim.x) {
-      const int t = idx >> 5, c = idx & 31;
-      v_s[idx] = (t < n && v0 + c < a.vdim) ? a.v[(int64_t)(c0 + t) * a.ldv + h * a.vdim + v0 + c] : 0.f;
-    }
+    copy_async_wait();
     __syncthreads();
-    // ---- A[t][j]: lane = t; warp w takes the groups of four keys jg = w, w + warps, ... (j = 4 jg + u)
+    // ---- A[t][j]: a row t against eight earlier tokens at a time, groups of GL lanes along the channels
     {
-      float acc[kKeyGroups][4];
-#pragma unroll
-      for (int g = 0; g < kKeyGroups; ++g) acc[g][0] = acc[g][1] = acc[g][2] = acc[g][3] = 0.f;
-      for (int d4 = 0; d4 < q4; ++d4) {
-        const float4 qv = q_s[lane * RS + d4];
-#pragma unroll
-        for (int g = 0; g < kKeyGroups; ++g)
-#pragma unroll
-          for (int u = 0; u < 4; ++u) acc[g][u] = dot4(qv, k_s[(4 * (w + kChunkWarps * g) + u) * q4 + d4], acc[g][u]);
-      }
-#pragma unroll
-      for (int g = 0; g < kKeyGroups; ++g) {
-        const int j0 = 4 * (w + kChunkWarps * g);
-        float4 r;
+      const int GL = dz > 64 ? 32 : (dz > 32 ? 16 : 8), gl = lane & (GL - 1), sub = lane / GL, subs = 32 / GL;
+#pragma unroll 1
+      for (int i = 0; i < kChunk / NW; ++i) {               // rows in pairs that add up to equal work
+        const int t = (i & 1) ? (i + 1) * NW - 1 - w : i * NW + w;
+        const float* qt = Qs + t * ds;
         if (MEM) {
-          const double Mt = MD[lane];
-          r.x = j0 <= lane ? acc[g][0] * expf((float)(bD[j0] - Mt)) : 0.f;
-          r.y = j0 + 1 <= lane ? acc[g][1] * expf((float)(bD[j0 + 1] - Mt)) : 0.f;
-          r.z = j0 + 2 <= lane ? acc[g][2] * expf((float)(bD[j0 + 2] - Mt)) : 0.f;
-          r.w = j0 + 3 <= lane ? acc[g][3] * expf((float)(bD[j0 + 3] - Mt)) : 0.f;
-        } else if (VAR) {
-          const float Lt = gp[lane];
-          r.x = j0 <= lane ? acc[g][0] * expf(Lt - gp[j0]) : 0.f;
-          r.y = j0 + 1 <= lane ? acc[g][1] * expf(Lt - gp[j0 + 1]) : 0.f;
-          r.z = j0 + 2 <= lane ? acc[g][2] * expf(Lt - gp[j0 + 2]) : 0.f;
-          r.w = j0 + 3 <= lane ? acc[g][3] * expf(Lt - gp[j0 + 3]) : 0.f;
-        } else {
-          r.x = j0 <= lane ? acc[g][0] * gp[lane - j0] : 0.f;
-          r.y = j0 + 1 <= lane ? acc[g][1] * gp[lane - j0 - 1] : 0.f;
-          r.z = j0 + 2 <= lane ? acc[g][2] * gp[lane - j0 - 2] : 0.f;
-          r.w = j0 + 3 <= lane ? acc[g][3] * gp[lane - j0 - 3] : 0.f;
+          float x = 0.f;
+          for (int c = 4 * lane; c < dz; c += 128)
+            x = fma4(*reinterpret_cast<const float4*>(qt + c), *reinterpret_cast<const float4*>(n_s + c), x);
+          x = warp_sum(x);
+          if (lane == 0) nq_s[t] = qs * x;
         }
-        a_s[lane * 9 + w + kChunkWarps * g] = r;
-      }
-    }
-    // ---- the state's share of every output: this warp's rows of S against q_t, lane = value column
-    for (int t = 0; t < n; ++t) {
-      float acc = 0.f;
+#pragma unroll 1
+        for (int j0 = 0; j0 <= t; j0 += 8 * subs) {
+          const int jb = min(j0 + 8 * sub, kChunk - 8);     // groups behind the last row repeat it
+          float v[8];
 #pragma unroll
-      for (int i4 = 0; i4 < DPT / 4; ++i4) {
-        if (d0 + 4 * i4 < dim4) {
-          const float4 qv = q_s[t * RS + (d0 >> 2) + i4];
-          acc = fmaf(S[4 * i4], qv.x, acc);
-          acc = fmaf(S[4 * i4 + 1], qv.y, acc);
-          acc = fmaf(S[4 * i4 + 2], qv.z, acc);
-          acc = fmaf(S[4 * i4 + 3], qv.w, acc);
-        }
-      }
-      part[(w * kChunk + t) * 32 + lane] = acc;
-    }
-    if (MEM) {       // this warp's rows of n against q_t, lane = t
-      float acc = 0.f;
-#pragma unroll 4
-      for (int i4 = 0; i4 < DPT / 4; ++i4)
-        if (d0 + 4 * i4 < dim4) acc = dot4(q_s[lane * RS + (d0 >> 2) + i4], *reinterpret_cast<const float4*>(n_s + d0 + 4 * i4), acc);
-      nq_s[w * kChunk + lane] = acc;
-    }
-    __syncthreads();
-    // ---- o_t for this warp's tokens t = w, w + warps, ... (a register tile of tokens against four value rows at a time)
-    {
-      float acc[kChunk / kChunkWarps];
+          for (int y = 0; y < 8; ++y) v[y] = 0.f;
+          for (int c = 4 * gl; c < dz; c += 4 * GL) {
+            const float4 x = *reinterpret_cast<const float4*>(qt + c);
 #pragma unroll
-      for (int tt = 0; tt < kChunk / kChunkWarps; ++tt) acc[tt] = 0.f;
-      const int j4n = (n + 3) >> 2;
-      for (int j4 = 0; j4 < j4n; ++j4) {
-        float4 vv;
-        vv.x = v_s[(4 * j4) * 32 + lane];
-        vv.y = v_s[(4 * j4 + 1) * 32 + lane];
-        vv.z = v_s[(4 * j4 + 2) * 32 + lane];
-        vv.w = v_s[(4 * j4 + 3) * 32 + lane];
-#pragma unroll
-        for (int tt = 0; tt < kChunk / kChunkWarps; ++tt) acc[tt] = dot4(a_s[(w + kChunkWarps * tt) * 9 + j4], vv, acc[tt]);
-      }
-#pragma unroll
-      for (int tt = 0; tt < kChunk / kChunkWarps; ++tt) {
-        const int t = w + kChunkWarps * tt;
-        if (t < n) {
-          float cross = 0.f;
-#pragma unroll
-          for (int g = 0; g < kChunkWarps; ++g) cross += part[(g * kChunk + t) * 32 + lane];
-          if (MEM) {
-            const float keep = keep_s[t];
-            float nq = 0.f;
-#pragma unroll
-            for (int g = 0; g < kChunkWarps; ++g) nq += nq_s[g * kChunk + t];
-            nq = fmaf(keep, nq, warp_sum(reinterpret_cast<const float*>(a_s)[t * 36 + lane]));
-            if (vok) a.o[(int64_t)(c0 + t) * a.ldo + h * a.vdim + v] = fmaf(keep, cross, acc[tt]) / (fmaxf(fabsf(nq), em_s[t]) + a.mem.den_eps);
-            continue;
+            for (int y = 0; y < 8; ++y) v[y] = fma4(x, *reinterpret_cast<const float4*>(Ks + (jb + y) * ds + c), v[y]);
           }
-          const float sk = (a.skip && vok) ? sw * a.skip[(int64_t)(c0 + t) * a.lds + h * a.vdim + v] : 0.f;
-          if (vok) a.o[(int64_t)(c0 + t) * a.ldo + h * a.vdim + v] = fmaf(VAR ? expf(gp[t]) : gp[t + 1], cross, acc[tt]) + sk;
+          int which;
+          bool writer;
+          const float sum = group_sum8(v, GL, gl, &which, &writer);
+          const int j = jb + which;
+          if (writer && j <= t) {
+            const float f = MEM ? qs * expf((float)(bD[j] - MD[t])) : (VAR ? expf(gp[t] - gp[j]) : gp[t - j]);
+            As[t * kChunkA + j] = f * sum;
+          }
         }
       }
     }
-    // ---- the state after the chunk
+    // ---- the state's share of every output: 8 queries per warp
+    float acc[8][C];
+#pragma unroll
+    for (int r = 0; r < 8; ++r)
+#pragma unroll
+      for (int e = 0; e < C; ++e) acc[r][e] = 0.f;
     {
-      const float gn = MEM ? keep_s[n - 1] : (VAR ? expf(gp[n - 1]) : gp[n]);
+      const float* X = Qs + 8 * rg * ds;
+#pragma unroll 2
+      for (int d = 0; d < dz; d += 4) {
+        float s[4][C];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) ld_cols<C>(s[i], Ss + (d + i) * COLS + cl);
+#pragma unroll
+        for (int r = 0; r < 8; ++r) {
+          const float4 x = *reinterpret_cast<const float4*>(X + r * ds + d);
+#pragma unroll
+          for (int e = 0; e < C; ++e) {
+            acc[r][e] = fmaf(x.x, s[0][e], acc[r][e]);
+            acc[r][e] = fmaf(x.y, s[1][e], acc[r][e]);
+            acc[r][e] = fmaf(x.z, s[2][e], acc[r][e]);
+            acc[r][e] = fmaf(x.w, s[3][e], acc[r][e]);
+          }
+        }
+      }
+    }
+    // the chunk's values of this lane's columns
+    float vv[kChunk][C];
+    {
+      const float* vp = a.v + (int64_t)c0 * a.ldv + h * a.vdim + v0 + cl;
+#pragma unroll
+      for (int j = 0; j < kChunk; ++j)
+#pragma unroll
+        for (int e = 0; e < C; ++e) vv[j][e] = (j < n && v0 + cl + e < a.vdim) ? vp[(int64_t)j * a.ldv + e] : 0.f;
+    }
+    __syncthreads();                                       // A is complete, the state has been read
+    // ---- outputs
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      const int t = 8 * rg + r;
+      const float keep = keep_s[t] * qs;
+      float o[C], den = 0.f;
+#pragma unroll
+      for (int e = 0; e < C; ++e) o[e] = keep * acc[r][e];
+#pragma unroll
+      for (int j4 = 0; j4 < kChunk; j4 += 4) {              // entries behind the diagonal are zero
+        const float4 m = *reinterpret_cast<const float4*>(As + t * kChunkA + j4);
+        if (MEM) den += (m.x + m.y) + (m.z + m.w);
+#pragma unroll
+        for (int e = 0; e < C; ++e) {
+          o[e] = fmaf(m.x, vv[j4][e], o[e]);
+          o[e] = fmaf(m.y, vv[j4 + 1][e], o[e]);
+          o[e] = fmaf(m.z, vv[j4 + 2][e], o[e]);
+          o[e] = fmaf(m.w, vv[j4 + 3][e], o[e]);
+        }
+      }
       if (MEM) {
-        for (int d = threadIdx.x; d < dim; d += blockDim.x) {
-          float x = gn * n_s[d];
-          for (int j = 0; j < n; ++j) x = fmaf(wj_s[j], k_sf[j * dim4 + d], x);
-          n_s[d] = x;                                  // read again behind the next chunk's first barrier
+        den = fmaxf(fabsf(fmaf(keep_s[t], nq_s[t], den)), em_s[t]) + a.mem.den_eps;
+#pragma unroll
+        for (int e = 0; e < C; ++e) o[e] /= den;
+      }
+      float* op = a.o + (int64_t)(c0 + t) * a.ldo + h * a.vdim + v0 + cl;
+#pragma unroll
+      for (int e = 0; e < C; ++e) {
+        if (t < n && v0 + cl + e < a.vdim) {
+          if (a.skip) o[e] += sw * a.skip[(int64_t)(c0 + t) * a.lds + h * a.vdim + v0 + cl + e];
+          op[e] = o[e];
+        }
+      }
+    }
+    // ---- the state behind the chunk
+    const float gn = keep_s[n - 1];
+#pragma unroll
+    for (int j = 0; j < kChunk; ++j) {
+      const float f = wj_s[j];
+#pragma unroll
+      for (int e = 0; e < C; ++e) vv[j][e] *= f;
+    }
+    for (int d = 4 * rg; d < dz; d += 16) {
+      float s[4][C];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        ld_cols<C>(s[i], Ss + (d + i) * COLS + cl);
+#pragma unroll
+        for (int e = 0; e < C; ++e) s[i][e] *= gn;
+      }
+#pragma unroll
+      for (int j = 0; j < kChunk; ++j) {
+        const float4 k = *reinterpret_cast<const float4*>(Ks + j * ds + d);
+#pragma unroll
+        for (int e = 0; e < C; ++e) {
+          s[0][e] = fmaf(k.x, vv[j][e], s[0][e]);
+          s[1][e] = fmaf(k.y, vv[j][e], s[1][e]);
+          s[2][e] = fmaf(k.z, vv[j][e], s[2][e]);
+          s[3][e] = fmaf(k.w, vv[j][e], s[3][e]);
         }
       }
 #pragma unroll
-      for (int i = 0; i < DPT; ++i) S[i] *= gn;
-      for (int j = 0; j < n; ++j) {
-        const float vv = v_s[j * 32 + lane] * (MEM ? wj_s[j] : (VAR ? expf(gp[n - 1] - gp[j]) : gp[n - 1 - j]));
-#pragma unroll
-        for (int i4 = 0; i4 < DPT / 4; ++i4) {
-          if (d0 + 4 * i4 < dim4) {
-            const float4 kv = k_s[j * q4 + (d0 >> 2) + i4];
-            S[4 * i4] = fmaf(kv.x, vv, S[4 * i4]);
-            S[4 * i4 + 1] = fmaf(kv.y, vv, S[4 * i4 + 1]);
-            S[4 * i4 + 2] = fmaf(kv.z, vv, S[4 * i4 + 2]);
-            S[4 * i4 + 3] = fmaf(kv.w, vv, S[4 * i4 + 3]);
-          }
-        }
+      for (int i = 0; i < 4; ++i) st_cols<C>(Ss + (d + i) * COLS + cl, s[i]);
+    }
+    if (MEM) {
+      for (int d = threadIdx.x; d < dim; d += THREADS) {
+        float x = gn * n_s[d];
+        for (int j = 0; j < n; ++j) x = fmaf(wj_s[j], Ks[j * ds + d], x);
+        n_s[d] = x;                                        // read again behind the next chunk's first barrier
       }
     }
   }
-  if (vok)
-#pragma unroll
-    for (int i = 0; i < DPT; ++i)
-      if (d0 + i < dim) sp[(int64_t)(d0 + i) * a.vdim + v] = S[i];
+  __syncthreads();
+  for (int i = threadIdx.x; i < dim * COLS; i += THREADS) {
+    const int d = i / COLS, c = i % COLS;
+    if (v0 + c < a.vdim) sp[(int64_t)d * a.vdim + v0 + c] = Ss[i];
+  }
   if (MEM) {
-    __syncthreads();
-    for (int d = threadIdx.x; d < dim; d += blockDim.x) np[d] = n_s[d];
-    if (threadIdx.x == 0) np[dim] = (float)m0;
+    const int mine = min(COLS, a.vdim - v0), groups = (mine + 31) / 32;
+    for (int g = 0; g < groups; ++g) {
+      for (int d = threadIdx.x; d < dim; d += THREADS) np[(int64_t)g * (dim + 1) + d] = n_s[d];
+      if (threadIdx.x == 0) np[(int64_t)g * (dim + 1) + dim] = (float)m0;
+    }
   }
 }
 
-template <int DPT, int MODE>
-cudaError_t launch_chunk(nvc_ctx* ctx, const RetArgs& a, dim3 grid, size_t smem, cudaStream_t st) {
+template <int C, int NW, int MODE>
+cudaError_t launch_chunk(nvc_ctx* ctx, const RetArgs& a, int B, cudaStream_t st) {
+  constexpr int COLS = 32 * C * (NW / 4);
+  const size_t smem = chunk_smem_floats(a.dim, COLS) * sizeof(float);
   static bool attr_set = false;
   if (!attr_set && smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(retention_chunk_kernel<DPT, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(retention_chunk_kernel<C, NW, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
     if (e != cudaSuccess) return e;
     attr_set = true;
   }
-  return nvc_launch(ctx, retention_chunk_kernel<DPT, MODE>, grid, dim3(kChunkWarps * 32), smem, st, a);
+  const int vec = (a.dim & 3) == 0 && (a.ldq & 3) == 0 && (a.ldk & 3) == 0 && ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k)) & 15) == 0;
+  return nvc_launch(ctx, retention_chunk_kernel<C, NW, MODE>, dim3(B, a.heads, (a.vdim + COLS - 1) / COLS), dim3(NW * 32), smem, st, a, vec);
 }
 
 template <int MODE>
@@ -456,16 +467,11 @@ int run_scan(nvc_ctx* ctx, const RetArgs& a, int B, int max_qlen, void* stream) 
   const int heads = a.heads, dim = a.dim, vdim = a.vdim;
   if (a.cu_seqlens && max_qlen > 4 && dim <= 512) {
     // prompt portions: 32 tokens at a time
-    const int per = ((dim + 3) / 4 * 4 + kChunkWarps - 1) / kChunkWarps;     // rows of the state per warp
-    const dim3 grid(B, heads, (vdim + 31) / 32);
-    const size_t mem = MODE == kMemory ? 7 * kChunk + kChunkWarps * kChunk + kChunkWarps * (per <= 8 ? 8 : (per <= 16 ? 16 : (per <= 32 ? 32 : 64))) : 0;
-    const size_t smem = ((size_t)kChunk * 4 * chunk_q_stride4(dim) + (size_t)kChunk * 4 * ((dim + 3) / 4) + kChunk * 32 + kChunk * 36 +
-                         kChunkWarps * kChunk * 32 + kChunk + 4 + mem) * sizeof(float);
+    // wide slices while they fill the GPU; keys of more than 256 numbers leave room for 32 columns only
     cudaError_t ce;
-    if (per <= 8) ce = launch_chunk<8, MODE>(ctx, a, grid, smem, nvc_stream(stream));
-    else if (per <= 16) ce = launch_chunk<16, MODE>(ctx, a, grid, smem, nvc_stream(stream));
-    else if (per <= 32) ce = launch_chunk<32, MODE>(ctx, a, grid, smem, nvc_stream(stream));
-    else ce = launch_chunk<64, MODE>(ctx, a, grid, smem, nvc_stream(stream));      // dim <= 512: at most 64 rows per warp
+    if (dim > 256) ce = launch_chunk<1, 4, MODE>(ctx, a, B, nvc_stream(stream));
+    else if (vdim > 64 && 4 * B * heads * ((vdim + 127) / 128) >= 3 * ctx->num_sms) ce = launch_chunk<2, 8, MODE>(ctx, a, B, nvc_stream(stream));
+    else ce = launch_chunk<1, 8, MODE>(ctx, a, B, nvc_stream(stream));
     NVC_CUDA_CHECK(ctx, ce);
     ctx->launches++;
     return NVC_OK;
