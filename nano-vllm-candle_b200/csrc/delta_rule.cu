@@ -36,6 +36,8 @@ __device__ __forceinline__ float softplus_f32(float x) { return x > 20.f ? x : l
 
 // grid (token tiles of the longest portion, units, sequences): the sequence comes from the block index, so a warp's first loads are
 // its sequence's bounds and nothing has to be searched; CTAs behind a sequence's last token leave at once
+// TAPS: the convolution's taps when they are 2 .. 4 (all inputs of a channel are in flight at once), 0: any number of them
+template <int TAPS>
 __global__ void __launch_bounds__(128, 8) delta_prep_kernel(const DeltaArgs a) {
   pdl_trigger();
   pdl_wait();
@@ -55,7 +57,15 @@ __global__ void __launch_bounds__(128, 8) delta_prep_kernel(const DeltaArgs a) {
     const float* bias = p.dt_bias + h * p.dim;
     float* g = p.channel_g + ((int64_t)n * p.heads + h) * p.dim;
     const float na = -expf(__ldg(p.A_log + h));
-    for (int j = lane; j < p.dim; j += 32) g[j] = na * softplus_f32(x[j] + __ldg(bias + j));
+    if (a.vec && (p.ldca & 3) == 0) {
+      for (int j = 4 * lane; j < p.dim; j += 128) {
+        const float4 v = *reinterpret_cast<const float4*>(x + j), u = __ldg(reinterpret_cast<const float4*>(bias + j));
+        *reinterpret_cast<float4*>(g + j) =
+            make_float4(na * softplus_f32(v.x + u.x), na * softplus_f32(v.y + u.y), na * softplus_f32(v.z + u.z), na * softplus_f32(v.w + u.w));
+      }
+    } else {
+      for (int j = lane; j < p.dim; j += 32) g[j] = na * softplus_f32(x[j] + __ldg(bias + j));
+    }
     return;
   }
   if (uu == units - 1) {
@@ -95,16 +105,27 @@ __global__ void __launch_bounds__(128, 8) delta_prep_kernel(const DeltaArgs a) {
       y[k] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (j < width) {
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int i = 0; i < p.taps; ++i) {
-          const int src = t - (p.taps - 1) + i;
-          float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (src >= 0) x = *reinterpret_cast<const float4*>(in + (int64_t)(src - t) * p.ldi + col + j);
-          else if (!fresh) x = *reinterpret_cast<const float4*>(cs + (int64_t)(p.taps - 1 + src) * C + ch + j);
+        const int taps = TAPS > 0 ? TAPS : p.taps;
+        auto input = [&](int i) {          // the input under tap i
+          const int src = t - (taps - 1) + i;
+          const float* xp = src >= 0 ? in + (int64_t)(src - t) * p.ldi + col + j : cs + (int64_t)(taps - 1 + src) * C + ch + j;
+          return (src < 0 && fresh) ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(xp);
+        };
+        auto apply = [&](int i, const float4& x) {
           const float4 w = __ldg(reinterpret_cast<const float4*>(p.conv_w + (int64_t)i * C + ch + j));      // tap-major: lanes read side by side
           acc.x = fmaf(w.x, x.x, acc.x);
           acc.y = fmaf(w.y, x.y, acc.y);
           acc.z = fmaf(w.z, x.z, acc.z);
           acc.w = fmaf(w.w, x.w, acc.w);
+        };
+        if constexpr (TAPS > 0) {
+          float4 x[TAPS];
+#pragma unroll
+          for (int i = 0; i < TAPS; ++i) x[i] = input(i);
+#pragma unroll
+          for (int i = 0; i < TAPS; ++i) apply(i, x[i]);
+        } else {
+          for (int i = 0; i < taps; ++i) apply(i, input(i));
         }
         y[k] = make_float4(acc.x * sigmoid_f32(acc.x), acc.y * sigmoid_f32(acc.y), acc.z * sigmoid_f32(acc.z), acc.w * sigmoid_f32(acc.w));
         ss4 += y[k].x * y[k].x + y[k].y * y[k].y + y[k].z * y[k].z + y[k].w * y[k].w;
@@ -594,14 +615,16 @@ extern "C" int nvc_delta_prep_run(nvc_ctx* ctx, const nvc_delta_prep* p, int N, 
   if (N == 0) return NVC_OK;
   auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
   const int vec = p->dim % 4 == 0 && p->vdim % 4 == 0 && p->ldi % 4 == 0 && p->q_off % 4 == 0 && p->k_off % 4 == 0 && p->v_off % 4 == 0 && p->ldq % 4 == 0 &&
-                  p->ldk % 4 == 0 && p->ldv % 4 == 0 && al16(p->in) && al16(p->conv_state) && al16(p->conv_w) && al16(p->q_out) && al16(p->k_out) && al16(p->v_out);
+                  p->ldk % 4 == 0 && p->ldv % 4 == 0 && al16(p->in) && al16(p->conv_state) && al16(p->conv_w) && al16(p->q_out) && al16(p->k_out) && al16(p->v_out) &&
+                  (!p->channel_a || (al16(p->channel_a) && al16(p->channel_g) && al16(p->dt_bias)));
   DeltaArgs a{*p, N, vec, nullptr, 0, nullptr};
   const int units = 2 * p->kv_heads + p->heads + 1 + (p->channel_a ? p->heads : 0);
   const int longest = p->cu_seqlens ? std::min(N, std::max(max_qlen, 1)) : 1;
   NVC_REQUIRE(ctx, units <= 65535 && p->B <= 65535, NVC_ESHAPE, "more than 65 535 heads or sequences");
   const int warps = longest >= 4 ? 4 : 1;
-  NVC_CUDA_CHECK(ctx, nvc_launch(ctx, delta_prep_kernel, dim3((unsigned)((longest + warps - 1) / warps), units, p->B), dim3(32 * warps), 0,
-                                 nvc_stream(stream), a));
+  const dim3 grid((unsigned)((longest + warps - 1) / warps), units, p->B);
+  auto* kernel = p->taps == 2 ? delta_prep_kernel<2> : (p->taps == 3 ? delta_prep_kernel<3> : (p->taps == 4 ? delta_prep_kernel<4> : delta_prep_kernel<0>));
+  NVC_CUDA_CHECK(ctx, nvc_launch(ctx, kernel, grid, dim3(32 * warps), 0, nvc_stream(stream), a));
   ctx->launches++;
   return NVC_OK;
 }

@@ -138,8 +138,9 @@ __device__ __forceinline__ int prep_find_seq(const int32_t* cu, int B, int row) 
 
 // One CTA per token: bias, short causal convolution, activation (the whole row [q | k | v] waits in shared memory), the norms over the
 // whole query and key projection - or none - then rotation and stores.  P: numbers per access (4: every width, offset and stride is a
-// multiple of 4 and the pointers are 16-byte aligned).
-template <typename TQ, typename TKV, int P>
+// multiple of 4 and the pointers are 16-byte aligned).  TAPS: the convolution's taps when they are 2 .. 4 (all inputs of a channel are in
+// flight at once), 0: any number of them, or no convolution.
+template <typename TQ, typename TKV, int P, int TAPS>
 __global__ void __launch_bounds__(1024) prep_token_kernel(const PrepArgs a, const nvc_short_conv cv) {
   extern __shared__ __align__(16) float row[];          // [qw + kw + vw]
   __shared__ float part[2][32];
@@ -165,43 +166,32 @@ __global__ void __launch_bounds__(1024) prep_token_kernel(const PrepArgs a, cons
   float sq = 0.f, sk = 0.f;
   for (int c = P * threadIdx.x; c < C; c += step) {
     const int col = c < qw ? p.q_off + c : (c < qw + kw ? p.k_off + c - qw : p.v_off + c - qw - kw);
-    float b[P], y[P];
+    float b[P], y[P] = {};
     if constexpr (P == 4) {
       const float4 t = p.bias ? *reinterpret_cast<const float4*>(p.bias + col) : make_float4(0.f, 0.f, 0.f, 0.f);
       b[0] = t.x; b[1] = t.y; b[2] = t.z; b[3] = t.w;
     } else {
       b[0] = p.bias ? __ldg(p.bias + col) : 0.f;
     }
-    if (cv.w) {
-      const int keep = cv.taps - 1, t = (int)n - s_r0;
+    if (TAPS > 0 || cv.w) {
+      const int taps = TAPS > 0 ? TAPS : cv.taps, keep = taps - 1, t = (int)n - s_r0;
       float* st = cv.state + (int64_t)s_slot * keep * C + c;
       const bool shift = cv.cu_seqlens == nullptr;      // one row per sequence: this CTA is the state's only reader
-#pragma unroll
-      for (int e = 0; e < P; ++e) y[e] = 0.f;
-      for (int i = 0; i < cv.taps; ++i) {
-        const int src = t - keep + i;                   // the input's index inside the portion; negative: in front of it
-        float x[P];
-        if (src >= 0) {
-          const float* xp = p.in + (s_r0 + src) * (int64_t)p.ldi + col;
-          if constexpr (P == 4) {
-            const float4 v = *reinterpret_cast<const float4*>(xp);
-            x[0] = v.x + b[0]; x[1] = v.y + b[1]; x[2] = v.z + b[2]; x[3] = v.w + b[3];
-          } else {
-            x[0] = *xp + b[0];
-          }
+      auto input = [&](int i, float (&x)[P]) {          // the input under tap i
+        const int src = t - keep + i;                   // its index inside the portion; negative: in front of it
+        const float* xp = src >= 0 ? p.in + (s_r0 + src) * (int64_t)p.ldi + col : st + (int64_t)(keep + src) * C;
+        const bool none = src < 0 && s_fresh;
+        if constexpr (P == 4) {
+          const float4 v = none ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(xp);
+          x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
         } else {
-          const float* sp = st + (int64_t)(keep + src) * C;
-#pragma unroll
-          for (int e = 0; e < P; ++e) x[e] = 0.f;
-          if (!s_fresh) {
-            if constexpr (P == 4) {
-              const float4 v = *reinterpret_cast<const float4*>(sp);
-              x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
-            } else {
-              x[0] = *sp;
-            }
-          }
+          x[0] = none ? 0.f : *xp;
         }
+        if (src >= 0)
+#pragma unroll
+          for (int e = 0; e < P; ++e) x[e] += b[e];
+      };
+      auto apply = [&](int i, const float (&x)[P]) {
         const float* wp = cv.w + (int64_t)i * C + c;
         if constexpr (P == 4) {
           const float4 w = __ldg(reinterpret_cast<const float4*>(wp));
@@ -214,6 +204,19 @@ __global__ void __launch_bounds__(1024) prep_token_kernel(const PrepArgs a, cons
           if constexpr (P == 4) *reinterpret_cast<float4*>(dp) = make_float4(x[0], x[1], x[2], x[3]);
           else *dp = x[0];
         }
+      };
+      if constexpr (TAPS > 0) {
+        float x[TAPS][P];
+#pragma unroll
+        for (int i = 0; i < TAPS; ++i) input(i, x[i]);
+#pragma unroll
+        for (int i = 0; i < TAPS; ++i) apply(i, x[i]);
+      } else {
+        for (int i = 0; i < taps; ++i) {
+          float x[P];
+          input(i, x);
+          apply(i, x);
+        }
       }
     } else {
 #pragma unroll
@@ -222,10 +225,11 @@ __global__ void __launch_bounds__(1024) prep_token_kernel(const PrepArgs a, cons
 #pragma unroll
     for (int e = 0; e < P; ++e) {
       if (p.act == NVC_PREP_ACT_SILU) y[e] *= sigmoid_f32(y[e]);
-      row[c + e] = y[e];
+      if (P == 1) row[c] = y[e];
       if (c + e < qw) sq += y[e] * y[e];
       else if (c + e < qw + kw) sk += y[e] * y[e];
     }
+    if constexpr (P == 4) *reinterpret_cast<float4*>(row + c) = make_float4(y[0], y[1], y[2], y[3]);
   }
   sq = warp_sum(sq);
   sk = warp_sum(sk);
@@ -253,6 +257,31 @@ __global__ void __launch_bounds__(1024) prep_token_kernel(const PrepArgs a, cons
     const float r = is_q ? rq : rk, post = is_q ? 1.f : p.k_scale;
     const float* nw = is_q ? p.q_norm : p.k_norm;
     const float* x = row + c0;
+    if constexpr (P == 4) {
+      if (p.rot_dims == 0 || (p.rot_half && (half & 3) == 0)) {      // four neighbours meet four neighbours
+        auto normed = [&](int k) {
+          float4 v = *reinterpret_cast<const float4*>(x + k);
+          const float4 w = nw ? __ldg(reinterpret_cast<const float4*>(nw + k)) : make_float4(1.f, 1.f, 1.f, 1.f);
+          v.x = v.x * r * w.x; v.y = v.y * r * w.y; v.z = v.z * r * w.z; v.w = v.w * r * w.w;
+          return v;
+        };
+        float4 z = normed(cc);
+        if (j0 < p.rot_dims) {
+          const bool lo = j0 < half;
+          const float4* cs = reinterpret_cast<const float4*>(tab + (lo ? j0 : j0 - half));
+          const float4 t0 = __ldg(cs), t1 = __ldg(cs + 1), q = normed(lo ? cc + half : cc - half);
+          const float sign = lo ? -1.f : 1.f;
+          z.x = z.x * t0.x + sign * q.x * t0.y;
+          z.y = z.y * t0.z + sign * q.y * t0.w;
+          z.z = z.z * t1.x + sign * q.z * t1.y;
+          z.w = z.w * t1.z + sign * q.w * t1.w;
+        }
+        z.x *= post; z.y *= post; z.z *= post; z.w *= post;
+        if (is_q) store4(reinterpret_cast<TQ*>(p.q_out) + n * p.ldq + cc, z);
+        else store4(reinterpret_cast<TKV*>(p.k_out) + orow * p.ldk + cc, z);
+        continue;
+      }
+    }
 #pragma unroll
     for (int e = 0; e < P; ++e) {
       const int j = j0 + e, k = cc + e;                 // number inside its head, number inside the projection
@@ -410,29 +439,40 @@ int launch_prep(nvc_ctx* ctx, const nvc_qkv_prep* p, int N, void* stream) {
   return NVC_OK;
 }
 
+template <typename TQ, typename TKV, int P, int TAPS>
+int launch_prep_token_as(nvc_ctx* ctx, const PrepArgs& a, const nvc_short_conv& cv, void* stream) {
+  const nvc_qkv_prep& p = a.p;
+  const int C = p.q_heads * p.dim + p.kv_heads * (p.dim + p.vdim);
+  const size_t smem = (size_t)C * sizeof(float);
+  static bool attr_set = false;
+  if (!attr_set && smem > 48 * 1024) {
+    NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(prep_token_kernel<TQ, TKV, P, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    attr_set = true;
+  }
+  // few rows: one access per thread, so that a row's loads are all in flight at once
+  const int units = (C / P + 31) / 32 * 32;
+  const int threads = std::min(std::max(units, 64), a.N <= 2 * ctx->num_sms ? 1024 : 256);
+  NVC_CUDA_CHECK(ctx, nvc_launch(ctx, prep_token_kernel<TQ, TKV, P, TAPS>, dim3((unsigned)a.N), dim3(threads), smem, nvc_stream(stream), a, cv));
+  ctx->launches++;
+  return NVC_OK;
+}
+
 template <typename TQ, typename TKV>
 int launch_prep_token(nvc_ctx* ctx, const nvc_qkv_prep* p, int N, void* stream) {
   PrepArgs a{*p, N};
   nvc_short_conv cv{};
   if (p->conv) cv = *p->conv;
-  const int qw = p->q_heads * p->dim, kw = p->kv_heads * p->dim, vw = p->kv_heads * p->vdim;
+  const int kw = p->kv_heads * p->dim, vw = p->kv_heads * p->vdim;
   auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
   const bool vec = ((p->dim | kw | vw | p->q_off | p->k_off | p->v_off | p->ldi | p->ldq | p->ldk | p->ldv) & 3) == 0 && al16(p->in) && al16(p->bias) &&
-                   al16(cv.w) && al16(cv.state) && al16(p->q_out) && al16(p->k_out) && al16(p->v_out);
-  const size_t smem = (size_t)(qw + kw + vw) * sizeof(float);
-  static bool attr_set = false;
-  if (!attr_set && smem > 48 * 1024) {
-    NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(prep_token_kernel<TQ, TKV, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(prep_token_kernel<TQ, TKV, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    attr_set = true;
+                   al16(cv.w) && al16(cv.state) && al16(p->q_norm) && al16(p->k_norm) && al16(p->rot_table) && al16(p->q_out) && al16(p->k_out) && al16(p->v_out);
+  if (!vec) return launch_prep_token_as<TQ, TKV, 1, 0>(ctx, a, cv, stream);
+  switch (cv.w ? cv.taps : 0) {
+    case 2: return launch_prep_token_as<TQ, TKV, 4, 2>(ctx, a, cv, stream);
+    case 3: return launch_prep_token_as<TQ, TKV, 4, 3>(ctx, a, cv, stream);
+    case 4: return launch_prep_token_as<TQ, TKV, 4, 4>(ctx, a, cv, stream);
+    default: return launch_prep_token_as<TQ, TKV, 4, 0>(ctx, a, cv, stream);
   }
-  // few rows: one access per thread, so that a row's loads are all in flight at once
-  const int units = ((qw + kw + vw) / (vec ? 4 : 1) + 31) / 32 * 32;
-  const int threads = std::min(std::max(units, 64), N <= 2 * ctx->num_sms ? 1024 : 256);
-  if (vec) NVC_CUDA_CHECK(ctx, nvc_launch(ctx, prep_token_kernel<TQ, TKV, 4>, dim3((unsigned)N), dim3(threads), smem, nvc_stream(stream), a, cv));
-  else NVC_CUDA_CHECK(ctx, nvc_launch(ctx, prep_token_kernel<TQ, TKV, 1>, dim3((unsigned)N), dim3(threads), smem, nvc_stream(stream), a, cv));
-  ctx->launches++;
-  return NVC_OK;
 }
 
 }  // namespace
