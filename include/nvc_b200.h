@@ -692,6 +692,10 @@ typedef struct nvc_memory_scan_args {
   int heads, dim, vdim;
 } nvc_memory_scan_args;
 int nvc_memory_scan(nvc_ctx* ctx, const nvc_memory_scan_args* p, int B, int max_qlen, void* stream);
+/* nvc_gemm_bf16_silu_mul with the clamped gated unit in its epilogue (NVC_ACT_GLU_CLAMP with p1 = 1.702):
+ *   g = min(A Wgate^T, limit), u = clamp(A Wup^T, -limit, limit):  act = g sigmoid(1.702 g) (u + 1);  W_gu16 interleaved as there. */
+int nvc_gemm_bf16_glu_clamp_mul(nvc_ctx* ctx, const nvc_bf16* A, int lda, const nvc_bf16* W_gu16, nvc_bf16* act, int ldc, int M, int I, int K,
+                                float limit, void* stream);
 
 /* K8. Replaces Qwen3ModelRunner::argmax (src/engine/llm_engine.rs:135-142) on device:
  * idx[b] = LAST index of the maximum of logits[b, :] (Iterator::max_by tie rule);

@@ -144,6 +144,7 @@ def _declare(l: C.CDLL) -> None:
         "nvc_streams_norm": [_vp, _vp, _vp, _i, _i, _i, _vp],
         "nvc_short_conv_advance": [_vp, _vp, _vp, _i, _i, _vp, _i, _vp, _vp],
         "nvc_memory_scan": [_vp, _vp, _i, _i, _vp],
+        "nvc_gemm_bf16_glu_clamp_mul": [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _f, _vp],
         "nvc_debug_set": [_i, _i],
     }
     for name, args in sigs.items():

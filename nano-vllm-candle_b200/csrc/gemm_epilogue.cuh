@@ -18,16 +18,34 @@ enum { NVC_EPI_NONE = 0, NVC_EPI_SILU_MUL = 1, NVC_EPI_TRANSPOSE = 2, NVC_EPI_QK
 // the element-wise epilogues
 __host__ __device__ __forceinline__ bool nvc_epi_unary(int epi) { return epi == NVC_EPI_RELU2 || epi == NVC_EPI_GELU_TANH; }
 
+// A negative value is the clamped gated unit and carries its limit: the bits of -limit.
+//   g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(1.702 g) (u + 1)
+__host__ __device__ __forceinline__ bool nvc_epi_glu_clamp(int epi) { return epi < 0; }
+static inline int nvc_epi_glu_clamp_of(float limit) {
+  union { float f; int i; } bits;
+  bits.f = -limit;
+  return bits.i;
+}
+
 // the gated epilogues write half as many columns as the accumulator has
-__host__ __device__ __forceinline__ bool nvc_epi_gated(int epi) { return epi == NVC_EPI_SILU_MUL || epi == NVC_EPI_GELU_TANH_MUL; }
+__host__ __device__ __forceinline__ bool nvc_epi_gated(int epi) {
+  return epi == NVC_EPI_SILU_MUL || epi == NVC_EPI_GELU_TANH_MUL || nvc_epi_glu_clamp(epi);
+}
 
 #ifdef __CUDACC__
-// act(gate) * up for 16 features; silu with the fast reciprocal, tanh-gelu with the hardware tanh (both far inside the
+// act(gate) * up for 16 features; silu and the clamped unit with the fast reciprocal, tanh-gelu with the hardware tanh (far inside the
 // bf16 rounding of the result)
 __device__ __forceinline__ void nvc_gated16(int epi, const float* f, float* o) {
   if (epi == NVC_EPI_SILU_MUL) {
 #pragma unroll
     for (int j = 0; j < 16; ++j) o[j] = __fdividef(f[j], 1.0f + __expf(-f[j])) * f[16 + j];
+  } else if (nvc_epi_glu_clamp(epi)) {
+    const float limit = -__int_as_float(epi);
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      const float g = fminf(f[j], limit), u = fminf(fmaxf(f[16 + j], -limit), limit);
+      o[j] = __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+    }
   } else {
 #pragma unroll
     for (int j = 0; j < 16; ++j) {

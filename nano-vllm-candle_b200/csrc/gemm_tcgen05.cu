@@ -651,6 +651,13 @@ extern "C" int nvc_gemm_bf16_gelu_mul(nvc_ctx* ctx, const nvc_bf16* A, int lda, 
   return gemm_impl(ctx, A, lda, W_gu16, act, ldc, NVC_DT_BF16, M, 2 * I, K, 0, 0, NVC_EPI_GELU_TANH_MUL, stream, nullptr);
 }
 
+// The same fused kernel with the clamped gated unit: g = min(A Wg^T, limit), u = clamp(A Wu^T, -limit, limit): g sigmoid(1.702 g) (u + 1).
+extern "C" int nvc_gemm_bf16_glu_clamp_mul(nvc_ctx* ctx, const nvc_bf16* A, int lda, const nvc_bf16* W_gu16, nvc_bf16* act, int ldc, int M,
+                                           int I, int K, float limit, void* stream) {
+  NVC_REQUIRE(ctx, I > 0 && I % 16 == 0 && limit >= 0.f, NVC_ESHAPE, "I must be a multiple of 16, the limit not negative");
+  return gemm_impl(ctx, A, lda, W_gu16, act, ldc, NVC_DT_BF16, M, 2 * I, K, 0, 0, nvc_epi_glu_clamp_of(limit), stream, nullptr);
+}
+
 // C = act(A W^T) with the plain activations of nvc_linear (NVC_ACT_NONE, NVC_ACT_RELU2) in the epilogue.
 extern "C" int nvc_gemm_bf16_act(nvc_ctx* ctx, const nvc_bf16* A, int lda, const nvc_bf16* W, void* C, int ldc, int out_dtype, int M,
                                  int Nout, int K, int act, void* stream) {

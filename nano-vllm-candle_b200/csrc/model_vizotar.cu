@@ -18,7 +18,7 @@
 //                             and gate in one product (block-diagonal weights)
 //     nvc_delta_prep_run      short convolutions + silu, unit q / k, log decays per channel, beta;  nvc_delta_rule_scan;
 //     nvc_head_gate_w         per-head root mean square, weight, sigmoid gate;  linear o
-//   dense ff:  linear [gate; up] -> clamped gated unit -> linear down (fp32)
+//   dense ff:  linear [gate; up] with the clamped gated unit in its epilogue -> linear down (fp32)
 //   moe ff:    routed_experts.h: biased logits, softmax over the chosen
 // A layer with `weights_of` runs another layer's weights with pools and state of its own.
 //
@@ -71,7 +71,7 @@ struct VLayerW {
   void* w_o = nullptr;                  // [Wp, owp]
   int owp = 0;
   // dense ff
-  void *w_gu = nullptr, *w_down = nullptr;          // [2 ffp, Wp] (gate rows, then up rows at ffp), [Wp, ffp]
+  void *w_gu = nullptr, *w_down = nullptr;          // [2 ffp, Wp] (16 gate rows, 16 up rows, ...; without tcgen05: all gate rows, all up rows), [Wp, ffp]
   int ffp = 0;
   nvc_experts_weights moe;
 };
@@ -243,7 +243,7 @@ struct VizotarBody : nvc_body_base {
     if (m_dqk && ((rc = zalloc(r, &rq, T * m_dqk * 4)) || (rc = zalloc(r, &rk, T * m_dqk * 4)) || (rc = zalloc(r, &rv, T * m_dv * 4)) ||
                   (rc = zalloc(r, &gb, T * m_gb * 4)) || (rc = zalloc(r, &gch, T * m_g * 4))))
       return rc;
-    if (m_ff && ((rc = zalloc(r, &gu, T * 2 * m_ff * esz)) || (rc = zalloc(r, &act, T * m_ff * esz)))) return rc;
+    if (m_ff && ((!use_tc && (rc = zalloc(r, &gu, T * 2 * m_ff * esz))) || (rc = zalloc(r, &act, T * m_ff * esz)))) return rc;
     return experts.alloc(*this, r, Wp, T);
   }
 
@@ -358,7 +358,11 @@ struct VizotarBody : nvc_body_base {
         }
       } else if (f.kind == nvc_routed_mlp_spec::Dense) {
         if (sub == "mlp.down") rc = out_matrix(w.w_down, w.ffp, f.ff);
-        else rc = shape_is(f.ff, W) ? put_matrix(r, w.w_gu, Wp, sub == "mlp.up" ? w.ffp : 0, 0, v.data(), f.ff, W, W, 1) : bad();
+        else if (!shape_is(f.ff, W)) return bad();
+        else if (!use_tc) rc = put_matrix(r, w.w_gu, Wp, sub == "mlp.up" ? w.ffp : 0, 0, v.data(), f.ff, W, W, 1);
+        else
+          for (int j = 0; j < f.ff && rc == NVC_OK; j += 16)
+            rc = put_matrix(r, w.w_gu, Wp, 2 * j + (sub == "mlp.up" ? 16 : 0), 0, v.data() + (size_t)j * W, std::min(16, f.ff - j), W, W, 1);
       }
     }
     if (rc == NVC_OK) it->second = true;
@@ -573,10 +577,17 @@ struct VizotarBody : nvc_body_base {
         if ((rc = land(r, pd, &w.sub[1], nullptr, nullptr, dt, nullptr, N))) return rc;
         mark(r, "streams_norm");
         if (f.kind == nvc_routed_mlp_spec::Dense) {
-          if ((rc = linear(r, h, Wp, w.w_gu, gu, 2 * w.ffp, dt, N, 2 * w.ffp, Wp))) return rc;
-          mark(r, "gemm_gate_up");
-          if ((rc = nvc_act_mul_p(ctx, gu, 2 * w.ffp, act, w.ffp, dt, N, f.ff, w.ffp, NVC_ACT_GLU_CLAMP, f.limit, kGluAlpha, st))) return rc;
-          mark(r, "glu");
+          if (use_tc) {        // the gated unit in the epilogue of the product
+            if ((rc = nvc_gemm_bf16_glu_clamp_mul(ctx, reinterpret_cast<const nvc_bf16*>(h), Wp, reinterpret_cast<const nvc_bf16*>(w.w_gu),
+                                                  reinterpret_cast<nvc_bf16*>(act), w.ffp, N, w.ffp, Wp, f.limit, st)))
+              return rc;
+            mark(r, "gemm_gate_up");
+          } else {
+            if ((rc = linear(r, h, Wp, w.w_gu, gu, 2 * w.ffp, dt, N, 2 * w.ffp, Wp))) return rc;
+            mark(r, "gemm_gate_up");
+            if ((rc = nvc_act_mul_p(ctx, gu, 2 * w.ffp, act, w.ffp, dt, N, f.ff, w.ffp, NVC_ACT_GLU_CLAMP, f.limit, kGluAlpha, st))) return rc;
+            mark(r, "glu");
+          }
           if ((rc = linear(r, act, w.ffp, w.w_down, ffo, Wp, NVC_DT_F32, N, Wp, w.ffp))) return rc;
           mark(r, "gemm_down");
         } else if ((rc = experts.run(*this, r, f, w.moe, h, ffo, N, W))) {

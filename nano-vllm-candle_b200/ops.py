@@ -898,3 +898,14 @@ def memory_scan(ctx, q, k, v, i_in, f_in, i_bias, f_bias, cap: float, state, nm_
                     _a(cu_seqlens), _a(positions), heads, dim, vdim)
     check(ctx.l.nvc_memory_scan(ctx.h, C.byref(p), state_slots.numel(), max_qlen, _stream()), "nvc_memory_scan", ctx.h)
     return o
+
+
+def gemm_glu_clamp_mul(ctx, A, Wg, Wu, limit: float):
+    """bf16 A [M, K], Wg and Wu [I, K]: the clamped gated unit in the product's epilogue."""
+    M, K = A.shape
+    n = Wg.shape[0]
+    W = torch.stack([Wg.view(n // 16, 16, K), Wu.view(n // 16, 16, K)], 1).reshape(2 * n, K).contiguous()
+    act = torch.empty(M, n, dtype=torch.bfloat16, device=A.device)
+    check(ctx.l.nvc_gemm_bf16_glu_clamp_mul(ctx.h, _ptr(A), A.stride(0), _ptr(W), _ptr(act), n, M, n, K, limit, _stream()),
+          "nvc_gemm_bf16_glu_clamp_mul", ctx.h)
+    return act

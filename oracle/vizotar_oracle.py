@@ -348,7 +348,9 @@ def make_config(vocab=200, width=96, layers=None, eps=1e-5, streams=2) -> dict:
 
 def make_weights(cfg: dict, seed: int = 0, bf16_values: bool = True, rank_a: int = 12, rank_g: int = 20, sink: float = 0.5) -> Dict[str, torch.Tensor]:
     """Random weights under the checkpoint's names; values bf16-representable by default so that the bf16 and fp32 paths load
-    identical numbers.  rank_a / rank_g: the inner sizes of the low-rank decay and gate projections (a tensor's shape, not config)."""
+    identical numbers.  rank_a / rank_g: the inner sizes of the low-rank decay and gate projections (a tensor's shape, not config).
+    The recurrences' keys lean towards their queries: a first output is sign(k . q) v / rms(v), and independent keys and queries put
+    some token of every prompt so close to the jump that bf16 rounding decides it."""
     gen = torch.Generator().manual_seed(seed)
     W, n = cfg["width"], cfg["streams"]
 
@@ -363,6 +365,9 @@ def make_weights(cfg: dict, seed: int = 0, bf16_values: bool = True, rank_a: int
 
     def lin(o, i):
         return rnd(o, i, s=i ** -0.5)
+
+    def lean(w, k, q):
+        w[k] = fix(0.6 * w[k] + 0.8 * w[q])
 
     w = {"embed": rnd(cfg["vocab"], W), "final.norm": one(W)}
     for i, ly in enumerate(cfg["layers"]):
@@ -379,6 +384,8 @@ def make_weights(cfg: dict, seed: int = 0, bf16_values: bool = True, rank_a: int
             for t, c in (("q", G * d), ("k", G * d), ("v", H * vd)):
                 w[p + f"mix.{t}"] = lin(c, W)
                 w[p + f"mix.{t}.conv"] = rnd(c, taps, s=0.6)
+            lean(w, p + "mix.k", p + "mix.q")
+            lean(w, p + "mix.k.conv", p + "mix.q.conv")
             w[p + "mix.b"] = lin(H, W)
             w[p + "mix.A_log"] = rnd(H, s=0.7)
             w[p + "mix.dt_bias"] = fix(-2.0 + torch.randn(H * d, generator=gen))
@@ -400,6 +407,7 @@ def make_weights(cfg: dict, seed: int = 0, bf16_values: bool = True, rank_a: int
             H, d, vd = r["heads"], r["dim"], r["vdim"]
             for t, c in (("q", H * d), ("k", H * d), ("v", H * vd), ("g", H * vd), ("i", H), ("f", H)):
                 w[p + f"mix.right.{t}"] = lin(c, W)
+            lean(w, p + "mix.right.k", p + "mix.right.q")
             w[p + "mix.right.i.b"] = rnd(H, s=1.0)
             w[p + "mix.right.f.b"] = fix(3.0 + torch.randn(H, generator=gen))
             w[p + "mix.right.norm"] = one(H * vd)

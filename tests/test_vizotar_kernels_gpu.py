@@ -401,3 +401,15 @@ def test_router_by_biased_logits_with_a_softmax_over_the_chosen(ctx, ops, E, top
     if 1 < top < E:                                       # neither a softmax over all experts nor weights without the bias
         assert (torch.gather(torch.softmax(z[:, :E] + b, -1), 1, wi) - torch.softmax(v, -1)).abs().max() > 0.05
         assert (torch.softmax(torch.gather(z[:, :E], 1, wi), -1) - torch.softmax(v, -1)).abs().max() > 0.05
+
+
+@pytest.mark.parametrize("M", [1, 5, 64, 130, 700])
+@pytest.mark.parametrize("ff,W,limit", [(64, 64, 0.6), (192, 128, 7.0), (1024, 512, 1.0), (64, 64, 0.0)])
+def test_clamped_gated_unit_in_the_epilogue_of_a_product(ctx, ops, M, ff, W, limit):
+    g = gen(61)
+    h, wg, wu = (torch.randn(*s, generator=g).bfloat16() for s in ((M, W), (ff, W), (ff, W)))
+    wg, wu = (wg * 2 * W ** -0.5).bfloat16(), (wu * 2 * W ** -0.5).bfloat16()
+    gate, up = torch.clamp(h.float() @ wg.float().T, max=limit), torch.clamp(h.float() @ wu.float().T, -limit, limit)
+    want = gate * torch.sigmoid(1.702 * gate) * (up + 1.0)
+    got = ops.gemm_glu_clamp_mul(ctx, h.to(DEV), wg.to(DEV), wu.to(DEV), limit).float().cpu()
+    assert torch.allclose(got, want, rtol=1e-2, atol=1e-2)
