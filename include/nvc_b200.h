@@ -277,6 +277,13 @@ int nvc_prefill_attn_paged_sink(nvc_ctx* ctx, const nvc_bf16* q, int ldq, const 
                                 int total_q_tokens, int max_seqlen_q, int nh, int kv, int hd, int block_size,
                                 int num_blocks, float scale, const float* sink, nvc_bf16* out, int ldo, void* stream);
 
+/* The same over a sliding window: window > 0: a row sees itself and the window - 1 tokens before it (0: every earlier token). */
+int nvc_prefill_attn_paged_window(nvc_ctx* ctx, const nvc_bf16* q, int ldq, const nvc_bf16* k_cache,
+                                  const nvc_bf16* v_cache, const int32_t* block_tables, int bt_stride,
+                                  const int32_t* context_lens, const int32_t* cu_seqlens_q, int B,
+                                  int total_q_tokens, int max_seqlen_q, int nh, int kv, int hd, int block_size,
+                                  int num_blocks, float scale, int window, const float* sink, nvc_bf16* out, int ldo, void* stream);
+
 /* K5. Decode: paged attention over block_tables (N2) with GQA head grouping.
  * q: [B, nh, hd] row stride ldq; caches [num_blocks, block_size, kv, hd];
  * block_tables: i32 [B, max_blocks] (-1 padded); context_lens: i32 [B] (tokens in the cache

@@ -58,6 +58,7 @@ struct nvc_body_base : nvc_model_body {
   int dt = NVC_DT_BF16;                // storage format of weights and activations
   size_t esz = 2;
   bool use_tc = true;                  // tcgen05 GEMMs for the plain products of the bf16 mode
+  bool use_flash = true;               // tcgen05 attention for long portions where a body has it
   bool prof_armed = false, prof_on = false;
   std::vector<std::pair<const char*, cudaEvent_t>> marks;
   std::string prof_json = "{}";
@@ -138,6 +139,13 @@ struct nvc_body_base : nvc_model_body {
       return nvc_gemm_bf16(r->ctx, reinterpret_cast<const nvc_bf16*>(A), lda, reinterpret_cast<const nvc_bf16*>(Wt), C, ldc, out_dt, M, N, K,
                            r->stream);
     return nvc_linear(r->ctx, A, lda, 0, Wt, K, 0, C, ldc, 0, dt, dt == NVC_DT_F32 ? NVC_DT_F32 : out_dt, M, N, K, 1, act, r->stream);
+  }
+
+  static constexpr int kFlashMinChunk = 64;
+  // a step whose prompt portions are long enough, with a block size the tcgen05 kernel's boxes take
+  bool flash_step(const nvc_runner* r, const nvc_step_shape& s) const {
+    const int bs = r->opt.kvcache_block_size;
+    return use_flash && !s.decode && s.num_decode < s.B && s.max_chunk >= kFlashMinChunk && (bs == 16 || bs == 32 || bs == 64 || bs % 128 == 0);
   }
 
   // (cos, sin) tables, one per rotation of the configuration

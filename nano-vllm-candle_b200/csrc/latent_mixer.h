@@ -37,7 +37,6 @@ struct nvc_latent_weights {
 };
 
 struct nvc_latent_body : nvc_body_base {
-  bool use_flash = true;
   float *lat_qf = nullptr, *lat_hv = nullptr;
   void *lat_cq = nullptr, *lat_qn = nullptr, *lat_qabs = nullptr, *lat_olat = nullptr;
   size_t lat_qrp = 0, lat_uqn = 0, lat_qn_cols = 0, lat_qa = 0, lat_ol = 0, lat_hv_cols = 0;
@@ -129,12 +128,6 @@ struct nvc_latent_body : nvc_body_base {
     return NVC_OK;
   }
 
-  static constexpr int kFlashMinChunk = 64;
-  // a step whose prompt portions are long enough, with a block size the tcgen05 kernel's boxes take
-  bool flash_step(const nvc_runner* r, const nvc_step_shape& s) const {
-    const int bs = r->opt.kvcache_block_size;
-    return use_flash && !s.decode && s.num_decode < s.B && s.max_chunk >= kFlashMinChunk && (bs == 16 || bs == 32 || bs == 64 || bs % 128 == 0);
-  }
 
   // attention over a pool of shared rows, keys and values at once: one-token sequences of a mixed step come first in the batch and keep
   // the decode path of the wide kernel, the portions behind them take the tcgen05 kernel when `flash`

@@ -9,7 +9,7 @@
 //                             [q | k | v | memory q | k | v | gate | i | f]
 //     nvc_qkv_prep_run        biases, short convolutions, norms over the whole query / key projection, rotary positions, k / v into this
 //                             layer's paged pools;  nvc_short_conv_advance (portions only): the convolution state
-//     nvc_attn_paged_wide     window and sink
+//     nvc_attn_paged_wide     window and sink (long portions of 128-wide heads: nvc_prefill_attn_paged_window)
 //     nvc_memory_scan         gates and the matrix memory, straight from the projection rows;  nvc_group_norm_gate: per-head norm,
 //                             weight, sigmoid gate
 //     linear o (left, its bias rides on the next nvc_streams_norm), linear o (right)
@@ -125,6 +125,7 @@ struct VizotarBody : nvc_body_base {
     esz = dt == NVC_DT_F32 ? 4 : 2;
     use_tc = dt == NVC_DT_BF16 && !(getenv("NVC_VIZOTAR_TC") && atoi(getenv("NVC_VIZOTAR_TC")) == 0);
     experts.use_tc = use_tc && !(getenv("NVC_VIZOTAR_MOE_TC") && atoi(getenv("NVC_VIZOTAR_MOE_TC")) == 0);
+    use_flash = use_tc && !(getenv("NVC_VIZOTAR_FLASH") && atoi(getenv("NVC_VIZOTAR_FLASH")) == 0);
     Wp = pad64(cfg.width);
     Vp = pad64(cfg.vocab);
     ldx = cfg.streams * Wp;
@@ -443,8 +444,22 @@ struct VizotarBody : nvc_body_base {
     sp.window = a.window;
     sp.sink = w.sink;
     sp.out_scale = 1.f;
-    rc = nvc_attn_paged_wide(ctx, q, p.ldq, rs.k_cache, p.ldk, rs.v_cache, p.ldv, r->d_bt, r->max_blocks_cap, r->d_ctx, s.decode ? nullptr : r->d_cu,
-                             s.B, s.N, s.decode ? 1 : s.max_seqlen, r->opt.kvcache_block_size, &sp, ao, w.owp, dt, st);
+    const int bs = r->opt.kvcache_block_size, cap = r->max_blocks_cap;
+    if (a.dim == 128 && a.vdim == 128 && a.scale > 0.f && flash_step(r, s)) {
+      // portions with 128-wide keys and values take the tcgen05 kernel; the one-token sequences of a mixed step come first in the batch and
+      // keep the decode path of the wide kernel
+      const int nd = s.num_decode;
+      if (nd > 0 && (rc = nvc_attn_paged_wide(ctx, q, p.ldq, rs.k_cache, p.ldk, rs.v_cache, p.ldv, r->d_bt, cap, r->d_ctx, nullptr, nd, nd, 1, bs, &sp, ao,
+                                              w.owp, dt, st)))
+        return rc;
+      rc = nvc_prefill_attn_paged_window(ctx, reinterpret_cast<const nvc_bf16*>(q) + (size_t)nd * p.ldq, p.ldq, reinterpret_cast<const nvc_bf16*>(rs.k_cache),
+                                         reinterpret_cast<const nvc_bf16*>(rs.v_cache), r->d_bt + (size_t)nd * cap, cap, r->d_ctx + nd,
+                                         nd ? r->d_cu2 : r->d_cu, s.B - nd, s.N - nd, s.max_chunk, a.heads, a.kv_heads, 128, bs,
+                                         r->opt.num_kvcache_blocks, a.scale, a.window, w.sink, reinterpret_cast<nvc_bf16*>(ao) + (size_t)nd * w.owp, w.owp, st);
+    } else {
+      rc = nvc_attn_paged_wide(ctx, q, p.ldq, rs.k_cache, p.ldk, rs.v_cache, p.ldv, r->d_bt, cap, r->d_ctx, s.decode ? nullptr : r->d_cu, s.B, s.N,
+                               s.decode ? 1 : s.max_seqlen, bs, &sp, ao, w.owp, dt, st);
+    }
     mark(r, "attention");
     return rc;
   }

@@ -48,8 +48,8 @@ struct PagedKV {                              // kPaged only
   int block_size;
   int box_rows;                               // token rows per K / V TMA box = min(64, block_size)
   const float* sink;                          // optional [nh]: one more term exp(sink_h) in every row's denominator, no value
+  int window;                                 // > 0: a row sees itself and the window - 1 keys before it (not in the plain mode)
   // shared key / value rows only
-  int window;                                 // > 0: a row sees itself and the window - 1 keys before it
   const float* bias;                          // sigmoid weights: [nh], added to the scores
   const float* key_scale;                     // sigmoid weights: [slots], a factor on the scores of a cached key
   const float* gate;                          // sigmoid weights: fp32 [rows, ldg], a sigmoid gate on every output number
@@ -90,7 +90,7 @@ cudaError_t launch_v2(nvc_ctx* ctx, int QT, int nh, int kv, int B, cudaStream_t 
 
 extern "C" int nvc_prefill_attn_init(nvc_ctx* ctx) {
   for (auto k : {v2::prefill_attn_v2_kernel<false, v2::kPlain>, v2::prefill_attn_v2_kernel<true, v2::kPlain>,
-                 v2::prefill_attn_v2_kernel<true, v2::kShared>, v2::prefill_attn_v2_kernel<true, v2::kSigmoid>})
+                 v2::prefill_attn_v2_kernel<true, v2::kWindow>, v2::prefill_attn_v2_kernel<true, v2::kShared>, v2::prefill_attn_v2_kernel<true, v2::kSigmoid>})
     NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, v2::kSmemBytes));
   return NVC_OK;
 }
@@ -147,6 +147,16 @@ extern "C" int nvc_prefill_attn_paged_sink(nvc_ctx* ctx, const nvc_bf16* q, int 
                                            const int32_t* context_lens, const int32_t* cu_seqlens_q, int B,
                                            int total_q_tokens, int max_seqlen_q, int nh, int kv, int hd, int block_size,
                                            int num_blocks, float scale, const float* sink, nvc_bf16* out, int ldo, void* stream) {
+  return nvc_prefill_attn_paged_window(ctx, q, ldq, k_cache, v_cache, block_tables, bt_stride, context_lens, cu_seqlens_q, B, total_q_tokens,
+                                       max_seqlen_q, nh, kv, hd, block_size, num_blocks, scale, 0, sink, out, ldo, stream);
+}
+
+extern "C" int nvc_prefill_attn_paged_window(nvc_ctx* ctx, const nvc_bf16* q, int ldq, const nvc_bf16* k_cache,
+                                             const nvc_bf16* v_cache, const int32_t* block_tables, int bt_stride,
+                                             const int32_t* context_lens, const int32_t* cu_seqlens_q, int B,
+                                             int total_q_tokens, int max_seqlen_q, int nh, int kv, int hd, int block_size,
+                                             int num_blocks, float scale, int window, const float* sink, nvc_bf16* out, int ldo, void* stream) {
+  NVC_REQUIRE(ctx, window >= 0, NVC_EINVAL, "bad window");
   NVC_REQUIRE(ctx, ctx && ldo >= nh * hd && ldo % 8 == 0 && ((uintptr_t)out % 16) == 0, NVC_ESHAPE,
               "output rows must cover the heads, with a stride that is a multiple of 8 and a 16-byte aligned start");
   NVC_REQUIRE(ctx, ctx && q && k_cache && v_cache && block_tables && context_lens && cu_seqlens_q && out, NVC_EINVAL,
@@ -173,9 +183,13 @@ extern "C" int nvc_prefill_attn_paged_sink(nvc_ctx* ctx, const nvc_bf16* q, int 
   PagedKV pk{};
   pk.block_tables = block_tables; pk.context_lens = context_lens; pk.bt_stride = bt_stride; pk.block_size = block_size; pk.box_rows = box_rows;
   pk.sink = sink;
+  pk.window = window;
   const int QT = (max_seqlen_q + 127) / 128;
-  NVC_CUDA_CHECK(ctx, launch_v2<true>(ctx, QT, nh, kv, B, nvc_stream(stream), tq, tk, tv, cu_seqlens_q,
-                                      scale * 1.4426950408889634f, out, ldo, pk));
+  const float scale_log2e = scale * 1.4426950408889634f;
+  if (window > 0)
+    NVC_CUDA_CHECK(ctx, (launch_v2<true, v2::kWindow>(ctx, QT, nh, kv, B, nvc_stream(stream), tq, tk, tv, cu_seqlens_q, scale_log2e, out, ldo, pk)));
+  else
+    NVC_CUDA_CHECK(ctx, launch_v2<true>(ctx, QT, nh, kv, B, nvc_stream(stream), tq, tk, tv, cu_seqlens_q, scale_log2e, out, ldo, pk));
   NVC_CUDA_CHECK(ctx, cudaGetLastError());
   ctx->launches++;
   return NVC_OK;

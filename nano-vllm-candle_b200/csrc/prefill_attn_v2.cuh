@@ -20,7 +20,8 @@
 //   * barrier init / TMEM allocation / descriptor prefetch run before the PDL dependency wait.
 // A share of the exponentials on the FMA pipe (degree-3 polynomial) was measured and is not used: no gain at 1/4,
 // a loss at 1/2 (same profile file) - the kernel is bound by dependent latency per tile, not by the MUFU unit.
-// kMode: kPlain = separate key and value tensors, causal softmax.  kShared = the cache rows are keys AND values (latent attention in its
+// kMode: kPlain = separate key and value tensors, causal softmax.  kWindow = kPlain over a sliding window: kv tiles in front of the q tile's
+// first visible key are never loaded (a mode of its own, so that the plain one keeps its code).  kShared = the cache rows are keys AND values (latent attention in its
 // absorbed form): one ring of four tiles serves both products - S reads a tile K-major, P V reads the same bytes MN-major - with an
 // optional sliding window (kv tiles in front of the q tile's first visible key are never loaded).  kSigmoid = the same shared tiles
 // with sigmoid(scale key_scale_j s + bias_h) weights: no maximum, no sum and no rescaling of O, so P V runs without any wait on the
@@ -49,7 +50,7 @@ constexpr int kNumBars = 2 + 2 * kKStages + 2 * kVStages + 2 + 4;
 constexpr int kSmemBytes = 115712;
 static_assert(kOffBar + kNumBars * 8 + 16 + 768 <= kSmemBytes, "shared memory budget for two CTAs per SM");
 constexpr int kTmemCols = 256;                 // S / P (double-buffered): columns [0, 64) and [64, 128); O: [128, 256)
-enum { kPlain = 0, kShared = 1, kSigmoid = 2 };
+enum { kPlain = 0, kShared = 1, kSigmoid = 2, kWindow = 3 };
 // shared tiles: stages of the one ring; the key factors of a stage take the place of a fourth tile
 template <int kMode> struct SharedRing { static constexpr int kStages = kMode == kSigmoid ? 3 : 4; };
 constexpr int kOffScale = kOffK + 3 * kKBytes;
@@ -90,6 +91,7 @@ __global__ void __launch_bounds__(192, 2)
 prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                        const __grid_constant__ CUtensorMap tma_v, const int32_t* __restrict__ cu_seqlens, const Sched sc,
                        float scale_log2e, nvc_bf16* __restrict__ out, int ldo, const PagedKV pk) {
+  constexpr bool kSep = kMode == kPlain || kMode == kWindow;       // keys and values are separate tensors
   pdl_trigger();
   const int num_items = sc.num_items, nh = sc.nh.d;
   extern __shared__ __align__(1024) uint8_t smem_v2[];
@@ -138,7 +140,7 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     if (lane == 0) {
       ptx::tma_prefetch_desc(&tma_q);
       ptx::tma_prefetch_desc(&tma_k);
-      if (kMode == kPlain) ptx::tma_prefetch_desc(&tma_v);
+      if (kSep) ptx::tma_prefetch_desc(&tma_v);
       ptx::mbar_init(q_full, 1);
       ptx::mbar_init(q_empty, 1);
       for (int s = 0; s < 2 * (kKStages + kVStages); ++s) ptx::mbar_init(bar0 + 8u * (2 + s), 1);     // the tiles' full / empty pairs
@@ -177,7 +179,7 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         if constexpr (kPaged) {
           // boxes of box_rows tokens; only those that start inside the context are loaded (the rest of
           // the slot keeps stale bytes: masked in S, zeroed in V by the softmax warps)
-          const int rows = pk.box_rows, tok0 = j * kKT;
+          const int rows = pk.box_rows, tok0 = (ge.j0 + j) * kKT;
           const int nbox = min(kKT / rows, (ge.kv_len - tok0 + rows - 1) / rows);
           ptx::mbar_arrive_expect_tx(bar, (uint32_t)(nbox * rows * 256));   // two 64-wide halves
           const int32_t* bt = pk.block_tables + (int64_t)x.b * pk.bt_stride;
@@ -238,7 +240,7 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         ptx::tma_load_3d(base + kOffQ + 16384, &tma_q, q_full, 64, x.h, ge.seq_start + x.qt * 128);
       }
       __syncwarp();
-      if constexpr (kMode == kPlain) {
+      if constexpr (kSep) {
         load_kv(x, ge, 0, g, false);
         for (int j = 0; j < ge.n_tiles; ++j) {
           if (j + 1 < ge.n_tiles) load_kv(x, ge, j + 1, g + j + 1, false);   // K runs one tile ahead of V, as S runs ahead of P V
@@ -259,9 +261,9 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     // S(g) = Q K^T into S buffer g & 1 : 8 k-steps of 16 over head_dim (two 64-wide swizzled halves).  The buffer last
     // held S / P of tile g - 2, whose P V MMA was issued earlier by this thread: tcgen05.mma executes in issue order.
     auto issue_s = [&](uint32_t g, bool last_of_item) {
-      constexpr int kStagesS = kMode == kPlain ? kKStages : kKV;
+      constexpr int kStagesS = kSep ? kKStages : kKV;
       const int s = (int)(g % kStagesS);
-      ptx::mbar_wait(kMode == kPlain ? k_full(s) : kv_full(s), (g / kStagesS) & 1);
+      ptx::mbar_wait(kSep ? k_full(s) : kv_full(s), (g / kStagesS) & 1);
       ptx::tcgen05_fence_after();
       if (ptx::elect_one()) {
         const uint32_t k_lo = ptx::umma_desc_lo(base + kOffK + s * kKBytes, 16);
@@ -273,7 +275,7 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
                             ks != 0);
         }
         ptx::umma_commit(s_full(g & 1));
-        if (kMode == kPlain) ptx::umma_commit(k_empty(s));          // the K slot is free as soon as these MMAs have read it
+        if (kSep) ptx::umma_commit(k_empty(s));          // the K slot is free as soon as these MMAs have read it
         if (last_of_item) ptx::umma_commit(q_empty);   // ... and so is Q after the item's last S
       }
       __syncwarp();
@@ -297,22 +299,22 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         if (j + 1 < n) issue_s(g + j + 1, j + 2 == n);
         // P(j) is in tensor memory, O has been rescaled for tile j (both by the softmax threads)
         ptx::mbar_wait(p_full(g + j), p_phase(g + j));
-        const int vs = (int)((g + j) % (kMode == kPlain ? kVStages : kKV));
-        if (kMode == kPlain) ptx::mbar_wait(v_full(vs), ((g + j) / kVStages) & 1);     // shared: S has read the same tile
+        const int vs = (int)((g + j) % (kSep ? kVStages : kKV));
+        if (kSep) ptx::mbar_wait(v_full(vs), ((g + j) / kVStages) & 1);     // shared: S has read the same tile
         // the first P V of an item overwrites O: the previous item's output rows have been read out of it
         if (j == 0 && n_done > 0) ptx::mbar_wait(o_free, (n_done - 1) & 1);
         ptx::tcgen05_fence_after();
         if (ptx::elect_one()) {
           // O += P V_j: A = P from tensor memory (8 columns per 16 kv tokens); B = V (MN-major: LBO = 8 KB between the
           // two 64-wide head-dim halves, SBO = 1 KB between groups of 8 token rows, 16 token rows = 2048 bytes per step)
-          const uint32_t v_lo = ptx::umma_desc_lo(base + (kMode == kPlain ? kOffV : kOffK) + vs * kKBytes, (uint32_t)kHalfKV);
+          const uint32_t v_lo = ptx::umma_desc_lo(base + (kSep ? kOffV : kOffK) + vs * kKBytes, (uint32_t)kHalfKV);
 #pragma unroll
           for (int ks = 0; ks < kKT / 16; ++ks)
             ptx::umma_bf16_ts(tmem_o, tmem_s + ((g + j) & 1) * kKT + ks * 8, ptx::umma_desc(v_lo + ks * (2048 >> 4), hi_k),
                               idesc_pv, (j | ks) != 0);
           // sigmoid: nobody looks at O before the item's last tile, whose barrier phase counts items
           if (kMode != kSigmoid || j + 1 == n) ptx::umma_commit(o_full);
-          ptx::umma_commit(kMode == kPlain ? v_empty(vs) : kv_empty(vs));
+          ptx::umma_commit(kSep ? v_empty(vs) : kv_empty(vs));
         }
         __syncwarp();
       }
@@ -345,7 +347,7 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         for (int c = 0; c < 4; ++c) asm volatile("prefetch.global.L2 [%0];" ::"l"(grow + c * 32));
       }
       // with a window a row's first tiles may hold none of its keys: a finite floor keeps every difference of maxima defined
-      float m = kMode == kShared ? -1e30f : -INFINITY, l = 0.f;                 // m: the maximum the exponentials are taken against (may lag the true one)
+      float m = kMode == kShared || kMode == kWindow ? -1e30f : -INFINITY, l = 0.f;                 // m: the maximum the exponentials are taken against (may lag the true one)
       for (int j = 0; j < n; ++j) {
         const uint32_t gi = g + j;
         const uint32_t s_addr = tmem_s + (gi & 1) * kKT + lane_addr;
@@ -408,7 +410,7 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
             for (int i = 0; i < kKT; ++i)
               if (i > lim) sv[i] = 0xff800000u;
           }
-          if (kMode == kShared && pk.window > 0 && t0 <= ge.q0 + 127 - pk.window) {
+          if ((kMode == kShared || kMode == kWindow) && pk.window > 0 && t0 <= ge.q0 + 127 - pk.window) {
             const int first = ge.q0 + r - pk.window + 1 - t0;      // first visible column of this row
 #pragma unroll
             for (int i = 0; i < kKT; ++i)
@@ -476,11 +478,11 @@ prefill_attn_v2_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
           // but the cache bytes may be NaN) once the slot's TMA has landed; the proxy fence orders these
           // generic stores before the P V MMA.
           if (t0 + kKT > ge.kv_len) {
-            constexpr int kStagesV = kMode == kPlain ? kVStages : kKV;
+            constexpr int kStagesV = kSep ? kVStages : kKV;
             const int vs = (int)(gi % kStagesV);
-            ptx::mbar_wait(kMode == kPlain ? v_full(vs) : kv_full(vs), (gi / kStagesV) & 1);
+            ptx::mbar_wait(kSep ? v_full(vs) : kv_full(vs), (gi / kStagesV) & 1);
             if (r < kKT && t0 + r >= ge.kv_len) {
-              uint8_t* v_row = gen + (kMode == kPlain ? kOffV : kOffK) + vs * kKBytes + r * 128;
+              uint8_t* v_row = gen + (kSep ? kOffV : kOffK) + vs * kKBytes + r * 128;
 #pragma unroll
               for (int k16 = 0; k16 < 8; ++k16) {
                 *reinterpret_cast<uint4*>(v_row + (k16 << 4)) = make_uint4(0, 0, 0, 0);

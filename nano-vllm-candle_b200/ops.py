@@ -909,3 +909,14 @@ def gemm_glu_clamp_mul(ctx, A, Wg, Wu, limit: float):
     check(ctx.l.nvc_gemm_bf16_glu_clamp_mul(ctx.h, _ptr(A), A.stride(0), _ptr(W), _ptr(act), n, M, n, K, limit, _stream()),
           "nvc_gemm_bf16_glu_clamp_mul", ctx.h)
     return act
+
+
+def prefill_attn_window(ctx, q, k_cache, v_cache, block_tables, context_lens, cu_seqlens, max_qlen: int, block_size: int, heads: int, kv_heads: int,
+                        scale: float, window: int, sink=None):
+    """Prompt portions on tcgen05 over a sliding window; q: bf16 [rows, heads * 128]; caches [slots, kv_heads * 128]."""
+    out = torch.empty_like(q)
+    check(ctx.l.nvc_prefill_attn_paged_window(ctx.h, _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(block_tables), block_tables.stride(0),
+                                              _ptr(context_lens), _ptr(cu_seqlens), context_lens.numel(), q.shape[0], max_qlen, heads, kv_heads, 128,
+                                              block_size, k_cache.shape[0] // block_size, scale, window, _ptr(sink), _ptr(out), out.stride(0),
+                                              _stream()), "nvc_prefill_attn_paged_window", ctx.h)
+    return out

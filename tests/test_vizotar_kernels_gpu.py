@@ -202,6 +202,53 @@ def test_window_attention_with_a_sink_over_a_mixed_batch(ctx, ops, dt, H, G, d, 
     assert torch.allclose(got.float().cpu(), torch.cat(want), **tol(dt))
 
 
+@pytest.mark.parametrize("bs", [16, 64])
+@pytest.mark.parametrize("window", [1, 39, 64, 65, 128, 200, 1000])
+def test_long_portions_over_a_window_on_the_tensor_memory_kernel(ctx, ops, bs, window):
+    """Heads of 128 numbers on tcgen05: whole prompts, portions behind a prefix that ends inside a page, short portions beside long ones; one
+    key of huge score just inside the window of a row and just outside that of the next."""
+    g = gen(32)
+    H, G, d, scale = 4, 2, 128, 128 ** -0.5
+    lens, qlens = [300, 131, 517, 70], [300, 64, 260, 3]
+    sink = torch.randn(H, generator=g) + 1.0
+    nb = sum((n + bs - 1) // bs for n in lens) + 2
+    order = torch.randperm(nb, generator=g).tolist()
+    kc = torch.full((nb * bs, G * d), float("nan"))                  # rows nobody wrote may hold anything
+    vc = kc.clone()
+    tables, want, qs, moved = [], [], [], []
+    for n, m in zip(lens, qlens):
+        k, v, q = torch.randn(n, G, d, generator=g), torch.randn(n, G, d, generator=g), torch.randn(m, H, d, generator=g)
+        edge = n - m // 2                                            # row at position edge: its window starts at edge - window + 1
+        j = max(edge - window + 1, 0)
+        q[edge - (n - m), :] = q[edge - (n - m), 0]
+        k[j] = q[edge - (n - m), 0] * 2.0
+        if edge + 1 < n:
+            q[edge + 1 - (n - m), :] = q[edge - (n - m), 0]
+        k, v, q = (t.bfloat16().float() for t in (k, v, q))
+        bl, order = order[:(n + bs - 1) // bs], order[(n + bs - 1) // bs:]
+        for t in range(n):
+            kc[bl[t // bs] * bs + t % bs], vc[bl[t // bs] * bs + t % bs] = k[t].reshape(-1), v[t].reshape(-1)
+        tables.append(bl)
+        pos = torch.arange(n - m, n)
+        o, wide = torch.zeros(m, H, d), torch.zeros(m, H, d)
+        for h in range(H):
+            s = q[:, h] @ k[:, h // (H // G)].T * scale
+            o[:, h] = Z.softmax_with_sink(s, Z.window_mask(pos, n, window), sink[h]) @ v[:, h // (H // G)]
+            wide[:, h] = Z.softmax_with_sink(s, Z.window_mask(pos, n, window + 1), sink[h]) @ v[:, h // (H // G)]
+        if j > 0 and edge + 1 < n:
+            moved.append((o - wide)[edge + 1 - (n - m)].abs().max())
+        want.append(o.reshape(m, H * d))
+        qs.append(q.reshape(m, H * d))
+    assert all(x > 0.3 for x in moved)                               # a window one token too wide would show
+    width = max(len(t) for t in tables)
+    cu = [0]
+    for m in qlens:
+        cu.append(cu[-1] + m)
+    got = ops.prefill_attn_window(ctx, torch.cat(qs).bfloat16().to(DEV), kc.bfloat16().to(DEV), vc.bfloat16().to(DEV),
+                                  i32([t + [-1] * (width - len(t)) for t in tables]), i32(lens), i32(cu), max(qlens), bs, H, G, scale, window, sink.to(DEV))
+    assert torch.allclose(got.float().cpu(), torch.cat(want), rtol=2e-2, atol=2e-2)
+
+
 # ------------------------------------------------------------------------------------------ matrix memory
 def memory_want(data, H, d, vd, cap, bi, bf):
     q, k, v, zi, zf = data

@@ -46,14 +46,15 @@ def cfg_b(all_experts=False):
 
 
 def cfg_c(all_experts=False):
-    """Sizes of the tensor-pipe routes of the bf16 mode: attention heads of 64 and 128 numbers, experts of 128 hidden units (grouped
-    tcgen05 products); two streams; a delta state of 128 x 64."""
+    """Sizes of the tensor-pipe routes of the bf16 mode: attention heads of 64 and 128 numbers (128-wide keys and values: the tensor-memory
+    attention), experts of 128 hidden units (grouped tcgen05 products); two streams; a delta state of 128 x 64."""
     layers = [
         Z.with_moe(Z.parallel_cfg(heads=4, kv_heads=1, dim=64, vdim=128, conv=3, window=48, rot_dims=32, scaling=YARN, scale=0.12, mheads=2, mdim=64,
                                   mvdim=64, cap=15.0), 4, 4 if all_experts else 2, 128),
         Z.with_dense(Z.delta_cfg(heads=2, kv_heads=1, dim=128, vdim=64, conv=4), 192, 1.5),
         Z.with_moe(Z.parallel_cfg(heads=2, kv_heads=2, dim=128, vdim=64, conv=2, window=200, rot_dims=128, scale=0.09, mheads=1, mdim=128, mvdim=128,
                                   cap=15.0), 3, 3 if all_experts else 1, 160),
+        Z.with_none(Z.parallel_cfg(heads=2, kv_heads=1, dim=128, vdim=128, conv=4, window=100, rot_dims=64, scale=0.09, mheads=2, mdim=32, mvdim=160)),
     ]
     return Z.make_config(vocab=160, width=128, streams=2, layers=layers)
 
@@ -274,13 +275,13 @@ def test_sizes_of_the_tensor_pipe_routes(monkeypatch, dtype, tc):
         r.close()
 
 
-def sharp_window_model(window, seed=30, special=50):
+def sharp_window_model(window, seed=30, special=50, dim=16, vdim=32):
     """One parallel layer whose attention head 0 scores the token `special` far above every other key, and whose memory half is switched
     off (its closing norm weight is zero), so that the token reaches later positions through attention ONLY: the embedding gives that
     token alone a component along width 0 and every token the same component along width 1; key number 0 reads the first, query number 0
     of head 0 the second; the convolutions pass the current token alone."""
     cfg = Z.make_config(vocab=60, width=64, streams=2, layers=[
-        Z.with_none(Z.parallel_cfg(heads=2, kv_heads=1, dim=16, vdim=32, scale=0.6, window=window, conv=3, rot_dims=None))])
+        Z.with_none(Z.parallel_cfg(heads=2, kv_heads=1, dim=dim, vdim=vdim, scale=0.6, window=window, conv=3, rot_dims=None))])
     w = Z.make_weights(cfg, seed)
     w["embed"][:, 0] = 0.0
     w["embed"][special, 0] = 8.0
@@ -301,12 +302,12 @@ def sharp_window_model(window, seed=30, special=50):
     return cfg, {k: v.bfloat16().float() for k, v in w.items()}
 
 
-@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("dtype,dim,vdim", [("float32", 16, 32), ("bfloat16", 16, 32), ("bfloat16", 128, 128)])
 @pytest.mark.parametrize("back,seen", [(0, True), (1, True), (38, True), (39, False), (40, False), (200, False)])
-def test_a_key_just_inside_and_just_outside_the_window(dtype, back, seen):
+def test_a_key_just_inside_and_just_outside_the_window(dtype, dim, vdim, back, seen):
     """A window of 39 tokens (pages hold 16): a token that occurs once, `back` positions before the end, moves the last logits if and only
     if back < 39 - for a whole prompt, for portions cut inside the window and for decoding while the window passes over it."""
-    cfg, w = sharp_window_model(39)
+    cfg, w = sharp_window_model(39, dim=dim, vdim=vdim)
     r = Rig(cfg, dtype, blocks=24, weights=w)
     try:
         n = 312
