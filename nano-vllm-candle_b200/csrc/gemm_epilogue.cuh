@@ -20,6 +20,7 @@ __host__ __device__ __forceinline__ bool nvc_epi_unary(int epi) { return epi == 
 
 // A negative value is the clamped gated unit and carries its limit: the bits of -limit.
 //   g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(1.702 g) (u + 1)
+// Kernels know it only as variants of their own (kClamp): one more branch in the shared epilogues costs the dense models 2 - 3 %.
 __host__ __device__ __forceinline__ bool nvc_epi_glu_clamp(int epi) { return epi < 0; }
 static inline int nvc_epi_glu_clamp_of(float limit) {
   union { float f; int i; } bits;
@@ -28,18 +29,20 @@ static inline int nvc_epi_glu_clamp_of(float limit) {
 }
 
 // the gated epilogues write half as many columns as the accumulator has
+template <bool kClamp>
 __host__ __device__ __forceinline__ bool nvc_epi_gated(int epi) {
-  return epi == NVC_EPI_SILU_MUL || epi == NVC_EPI_GELU_TANH_MUL || nvc_epi_glu_clamp(epi);
+  return epi == NVC_EPI_SILU_MUL || epi == NVC_EPI_GELU_TANH_MUL || (kClamp && nvc_epi_glu_clamp(epi));
 }
 
 #ifdef __CUDACC__
 // act(gate) * up for 16 features; silu and the clamped unit with the fast reciprocal, tanh-gelu with the hardware tanh (far inside the
 // bf16 rounding of the result)
+template <bool kClamp>
 __device__ __forceinline__ void nvc_gated16(int epi, const float* f, float* o) {
   if (epi == NVC_EPI_SILU_MUL) {
 #pragma unroll
     for (int j = 0; j < 16; ++j) o[j] = __fdividef(f[j], 1.0f + __expf(-f[j])) * f[16 + j];
-  } else if (nvc_epi_glu_clamp(epi)) {
+  } else if (kClamp && nvc_epi_glu_clamp(epi)) {
     const float limit = -__int_as_float(epi);
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
@@ -108,14 +111,14 @@ __device__ __forceinline__ void store16(void* C, int out_f32, int64_t off, const
 //                    C[row, n0/2 .. n0/2+16) = silu(gate) * up   (src/layers/activation.rs:13-18,
 //                    silu(x) = x / (1 + exp(-x)) in f32), bf16.  row_off = row * ldc in elements of C.
 // kUnary = false compiles the element-wise epilogues (NVC_EPI_RELU2, NVC_EPI_GELU_TANH) out: the decode GEMMs of the dense models keep their code.
-template <bool kUnary = true>
+template <bool kUnary = true, bool kClamp = false>
 __device__ __forceinline__ void emit32(void* C, int out_f32, int epi, int64_t row_off, int n0, int N, const float* f) {
-  if (nvc_epi_gated(epi)) {
+  if (nvc_epi_gated<kClamp>(epi)) {
     if (n0 < N) {
       float o[16];
       // fast reciprocal (MUFU.RCP, 2 ulp): an IEEE division per element makes the epilogue of a K = 1024
       // prefill tile (128 of them per thread) as long as its main loop
-      nvc_gated16(epi, f, o);
+      nvc_gated16<kClamp>(epi, f, o);
       store16(C, 0, row_off + (n0 >> 1), o);
     }
   } else {
@@ -169,10 +172,11 @@ struct RowStage {
     filled = 0;
   }
   // 32 consecutive accumulator columns of this thread's row (same semantics as emit32); flushes every 128 bytes
+  template <bool kClamp = false>
   __device__ __forceinline__ void emit32(int lane, int out_f32, int epi, const float* f) {
-    if (nvc_epi_gated(epi)) {
+    if (nvc_epi_gated<kClamp>(epi)) {
       float o[16];
-      nvc_gated16(epi, f, o);
+      nvc_gated16<kClamp>(epi, f, o);
       put(lane, pack8(o));
       put(lane, pack8(o + 8));
       if (filled == 128) flush(lane);
@@ -203,13 +207,14 @@ struct RowStage {
 };
 
 // Output geometry of a tile for RowStage: bytes per accumulator column and the tile's byte window.
+template <bool kClamp = false>
 __device__ __forceinline__ RowStage make_row_stage(uint8_t* buf, void* C, int out_f32, int epi, int64_t ldc, int row0, int M,
                                                    int n_base, int n_tile_cols, int N) {
   // SiLU-mul: 32 accumulator columns -> 16 bf16; plain: bf16 or f32 per column
   const int esz = out_f32 ? 4 : 2;
-  const int col0 = nvc_epi_gated(epi) ? (n_base >> 1) : n_base;
-  const int n_out = nvc_epi_gated(epi) ? (N >> 1) : N;
-  const int tile_out = nvc_epi_gated(epi) ? (n_tile_cols >> 1) : n_tile_cols;
+  const int col0 = nvc_epi_gated<kClamp>(epi) ? (n_base >> 1) : n_base;
+  const int n_out = nvc_epi_gated<kClamp>(epi) ? (N >> 1) : N;
+  const int tile_out = nvc_epi_gated<kClamp>(epi) ? (n_tile_cols >> 1) : n_tile_cols;
   RowStage s;
   s.buf = buf;
   s.g_row0 = reinterpret_cast<uint8_t*>(C) + ((int64_t)row0 * ldc + col0) * esz;

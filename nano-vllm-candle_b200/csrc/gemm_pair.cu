@@ -127,7 +127,7 @@ __device__ __forceinline__ void pair_publish(float4* __restrict__ my_ws, uint32_
   }
 }
 
-template <int NT, int S>
+template <int NT, int S, bool kClamp>
 __device__ __forceinline__ void pair_reduce(const float4* __restrict__ ws_cluster, uint32_t taddr, int p, int h, int r,
                                             void* __restrict__ C, int out_f32, int epi, int64_t ldc, int row0, int M,
                                             int n_base, int N, uint8_t* stage_buf) {
@@ -178,13 +178,14 @@ __device__ __forceinline__ void pair_reduce(const float4* __restrict__ ws_cluste
         }
         // direct stores: a unit is only 32-128 bytes per row, staging it measured slower (16.0 vs 14.5 us on 8B o_proj)
         const int grow = row0 + (r & 31);
-        if (grow < M) emit32(C, out_f32, epi, (int64_t)grow * ldc, n_base + u * 32, N, f);
+        if (grow < M) emit32<true, kClamp>(C, out_f32, epi, (int64_t)grow * ldc, n_base + u * 32, N, f);
       }
     }
   }
 }
 
-template <int NT>
+// kClamp: the variant with the clamped gated epilogue
+template <int NT, bool kClamp = false>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant__ CUtensorMap tma_b,
                  void* __restrict__ C, int ldc, int out_f32, int M, int N, int k_blocks_total, int kb_per_split,
@@ -452,7 +453,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
         if (lane == 0) mbar_arrive_cluster(leader_tmem_empty0 + 8u * acc);
         continue;
       }
-      RowStage st = make_row_stage(smem_gen + cfg::kOffStage + q * cfg::kStageBuf, C, out_f32, epi, ldc,
+      RowStage st = make_row_stage<kClamp>(smem_gen + cfg::kOffStage + q * cfg::kStageBuf, C, out_f32, epi, ldc,
                                    m_tile * kTileM + h * kHalf + q * 32, M, n_tile * NT, NT, N);
 #pragma unroll 1
       for (int c = 0; c < cfg::kChunks; c += 2) {       // two 16-column chunks per tensor-memory round trip
@@ -463,7 +464,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
         float f[32];
 #pragma unroll
         for (int j = 0; j < 32; ++j) f[j] = __uint_as_float(v[j]);
-        st.emit32(lane, out_f32, epi, f);
+        st.template emit32<kClamp>(lane, out_f32, epi, f);
       }
       st.finish(lane);
       ptx::tcgen05_fence_before();
@@ -497,9 +498,9 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
     if (warp >= 2) {
       const int row0 = m_tile * kTileM + h * kHalf + q * 32;          // first row of this warp
       uint8_t* stage_buf = smem_gen + cfg::kOffStage + q * cfg::kStageBuf;
-      if (S == 2) pair_reduce<NT, 2>(ws_cluster, taddr, p, h, r, C, out_f32, epi, ldc, row0, M, n_tile * NT, N, stage_buf);
-      else if (S == 3) pair_reduce<NT, 3>(ws_cluster, taddr, p, h, r, C, out_f32, epi, ldc, row0, M, n_tile * NT, N, stage_buf);
-      else pair_reduce<NT, 4>(ws_cluster, taddr, p, h, r, C, out_f32, epi, ldc, row0, M, n_tile * NT, N, stage_buf);
+      if (S == 2) pair_reduce<NT, 2, kClamp>(ws_cluster, taddr, p, h, r, C, out_f32, epi, ldc, row0, M, n_tile * NT, N, stage_buf);
+      else if (S == 3) pair_reduce<NT, 3, kClamp>(ws_cluster, taddr, p, h, r, C, out_f32, epi, ldc, row0, M, n_tile * NT, N, stage_buf);
+      else pair_reduce<NT, 4, kClamp>(ws_cluster, taddr, p, h, r, C, out_f32, epi, ldc, row0, M, n_tile * NT, N, stage_buf);
       if (tr && threadIdx.x == 64) trace[83] = clock64();
     }
   }
@@ -559,7 +560,8 @@ int launch_pair(nvc_ctx* ctx, const nvc_bf16* A, int lda, const nvc_bf16* W, voi
   // qkv 18.4 -> 16.8 us, o_proj 14.6 -> 13.9, gate_up 49.6 -> 47.4, down 30.3 -> 28.4 without it) - the prefetches compete
   // with the ring's own TMA loads for the same L2 / HBM queues (profiles/r02_pair_prefetch_ab.txt)
   const int prefetch_w = (M <= kTileM && kb_total <= 48) ? 1 : 0;
-  NVC_CUDA_CHECK(ctx, nvc_launch_cluster(ctx, gemm_pair_kernel<NT>, grid, dim3(kThreads), cfg::kSmemBytes, stream, 2 * S,
+  auto* kernel = nvc_epi_glu_clamp(epi) ? gemm_pair_kernel<NT, true> : gemm_pair_kernel<NT>;
+  NVC_CUDA_CHECK(ctx, nvc_launch_cluster(ctx, kernel, grid, dim3(kThreads), cfg::kSmemBytes, stream, 2 * S,
                                          ta, tb, C, ldc, out_f32, M, N, kb_total, kb_per, tiles, n_tiles,
                                          prefetch_w, epi, reinterpret_cast<float4*>(ctx->gemm_ws), trace,
                                          qk));
@@ -574,7 +576,8 @@ int launch_pair(nvc_ctx* ctx, const nvc_bf16* A, int lda, const nvc_bf16* W, voi
 // them (cluster placement is per GPC: B200 holds 74 / 33 / 22 / 15 clusters of 2 / 4 / 6 / 8 CTAs).
 extern "C" int nvc_gemm_pair_init(nvc_ctx* ctx) {
 #define X(NT) \
-  NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(gemm_pair_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, PairCfg<NT>::kSmemBytes));
+  NVC_CUDA_CHECK(ctx, cudaFuncSetAttribute(gemm_pair_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, PairCfg<NT>::kSmemBytes)); \
+  NVC_CUDA_CHECK(ctx, (cudaFuncSetAttribute(gemm_pair_kernel<NT, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, PairCfg<NT>::kSmemBytes)));
   NVC_PAIR_WIDTHS(X)
 #undef X
   for (int S = 1; S <= 4; ++S) {

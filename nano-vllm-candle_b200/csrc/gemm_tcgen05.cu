@@ -248,7 +248,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid
           float f[32];
 #pragma unroll
           for (int j = 0; j < 32; ++j) f[j] = __uint_as_float(v[j]);
-          if (row_ok) emit32<kExt>(C, out_f32, epi, (int64_t)grow * ldc, n_tile * BN + c * 16, N, f);
+          if (row_ok) emit32<kExt, kExt>(C, out_f32, epi, (int64_t)grow * ldc, n_tile * BN + c * 16, N, f);
         }
       } else {
         uint32_t v[16];
@@ -435,9 +435,9 @@ int launch(nvc_ctx* ctx, const nvc_bf16* A, int lda, const nvc_bf16* W, void* C,
   // ks_cluster: the eff_splits CTAs of one output tile form a cluster (1,1,S) and reduce over DSMEM
   const int ks = (ks_cluster && CL == 1 && eff_splits > 1 && eff_splits <= 8) ? 1 : 0;
   NVC_REQUIRE(ctx, !ks || (size_t)BN * BM * 4 <= (size_t)cfg::kStages * cfg::kStageBytes, NVC_EINVAL, "ring too small for the partial tile");
-  // the extended variant exists for CL = 1 (the grouped products and the element-wise epilogues never use clusters)
+  // the extended variant exists for CL = 1 (the grouped products, the element-wise and the clamped epilogues never use clusters)
   constexpr bool kHasExt = CL == 1;
-  const bool ext = tile_group != nullptr || nvc_epi_unary(epi);
+  const bool ext = tile_group != nullptr || nvc_epi_unary(epi) || nvc_epi_glu_clamp(epi);
   NVC_REQUIRE(ctx, !ext || kHasExt, NVC_EINVAL, "grouped / element-wise epilogue products need a cluster size of 1");
   auto kernel = gemm_bf16_tcgen05_kernel<BN, KPS, CL, false>;
   if constexpr (kHasExt) { if (ext) kernel = gemm_bf16_tcgen05_kernel<BN, KPS, CL, true>; }
@@ -551,9 +551,9 @@ static int gemm_impl(nvc_ctx* ctx, const nvc_bf16* A, int lda, const nvc_bf16* W
   NVC_REQUIRE(ctx, K % 64 == 0, NVC_ESHAPE, "K must be a multiple of 64");
   NVC_REQUIRE(ctx, Nout % 16 == 0, NVC_ESHAPE, "Nout must be a multiple of 16");
   NVC_REQUIRE(ctx, lda % 8 == 0 && lda >= K, NVC_ESHAPE, "lda must be >= K and a multiple of 8");
-  NVC_REQUIRE(ctx, ldc >= (nvc_epi_gated(epi) ? Nout / 2 : Nout) && ldc % 8 == 0, NVC_ESHAPE,
+  NVC_REQUIRE(ctx, ldc >= (nvc_epi_gated<true>(epi) ? Nout / 2 : Nout) && ldc % 8 == 0, NVC_ESHAPE,
               "ldc must be >= the output width and a multiple of 8");
-  NVC_REQUIRE(ctx, epi == NVC_EPI_NONE || nvc_epi_unary(epi) || (nvc_epi_gated(epi) && Nout % 32 == 0 && out_dtype == NVC_DT_BF16),
+  NVC_REQUIRE(ctx, epi == NVC_EPI_NONE || nvc_epi_unary(epi) || (nvc_epi_gated<true>(epi) && Nout % 32 == 0 && out_dtype == NVC_DT_BF16),
               NVC_ESHAPE, "fused SiLU-mul epilogue needs Nout % 32 == 0 and bf16 output");
   NVC_REQUIRE(ctx, out_dtype == NVC_DT_BF16 || out_dtype == NVC_DT_F32, NVC_EINVAL, "bad out_dtype");
   NVC_REQUIRE(ctx, ((uintptr_t)A % 16) == 0 && ((uintptr_t)W % 16) == 0 && ((uintptr_t)C % 16) == 0, NVC_EINVAL,
@@ -599,7 +599,7 @@ static int gemm_impl(nvc_ctx* ctx, const nvc_bf16* A, int lda, const nvc_bf16* W
     splits = 1;
     ks = 0;
     if (bn < 32) { bn = 32; kps = 4; cl = 1; }
-    if (nvc_epi_unary(epi)) cl = 1;          // (every (bn, kps) the choice returns has a CL = 1 instantiation)
+    if (nvc_epi_unary(epi) || nvc_epi_glu_clamp(epi)) cl = 1;          // (every (bn, kps) the choice returns has a CL = 1 instantiation)
   }
   if (splits > K / BK) splits = K / BK;
   const int tiles = ((M + BM - 1) / BM) * ((Nout + bn - 1) / bn);
